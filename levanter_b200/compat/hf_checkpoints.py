@@ -40,6 +40,7 @@ DEFAULT_MAX_SHARD_SIZE = int(10e9)
 class HFCompatConfig(LmConfig):
     hf_model_type = None
     hf_architecture = None
+    hf_vocab_key = "vocab_size"  # where the checkpoint's config keeps the vocabulary size
 
     def hf_checkpoint_converter(self, ref_checkpoint: Optional[str] = None) -> "HFCheckpointConverter":
         raise NotImplementedError
@@ -111,6 +112,10 @@ def to_hf_state_dict(model: nn.Module, dtype: Optional[torch.dtype] = None, para
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)
         t = t.cpu()
+        if hasattr(model, "hf_tensor_names"):  # a model that names its checkpoint tensors itself
+            names = model.hf_tensor_names(name)
+            out.update({names: t.contiguous()} if isinstance(names, str) else {n: t[j].contiguous() for j, n in enumerate(names)})
+            continue
         leaf = name.rsplit(".", 1)[-1]
         if ".experts." in name and leaf in ("w1", "w2", "w3") and t.dim() == 3:
             base = _hf_name(name.rsplit(".", 1)[0], key_map)
@@ -138,6 +143,18 @@ def load_hf_state_dict(model: nn.Module, state_dict: Dict[str, torch.Tensor], *,
     missing: List[str] = []
     with torch.no_grad():
         for name, p in model.named_parameters():
+            if hasattr(model, "hf_tensor_names"):
+                names = model.hf_tensor_names(name)
+                parts = [(p.data, names)] if isinstance(names, str) else [(p.data[j], n) for j, n in enumerate(names)]
+                found = [(dst, lookup(n), n) for dst, n in parts]
+                if any(t is None for _, t, _ in found):
+                    missing.append(name)
+                    continue
+                for dst, t, n in found:
+                    if t.shape != dst.shape:
+                        raise ValueError(f"shape mismatch for {n}: checkpoint {tuple(t.shape)} vs model {tuple(dst.shape)}")
+                    dst.copy_(t.to(dst.dtype))
+                continue
             leaf = name.rsplit(".", 1)[-1]
             if ".experts." in name and leaf in ("w1", "w2", "w3") and p.dim() == 3:
                 base = _hf_name(name.rsplit(".", 1)[0], key_map)
@@ -247,18 +264,19 @@ class HFCheckpointConverter:
 
     @staticmethod
     def from_hf(model_name_or_path, trust_remote_code: bool = False) -> "HFCheckpointConverter":
-        """Infer the config class from the checkpoint's ``model_type``."""
+        """Infer the config class from the checkpoint's ``model_type`` (or, where the config has none, its ``architecture``)."""
         ref = _coerce_ref(model_name_or_path)
         cfg = _read_hf_config(ref)
         mt = cfg.get("model_type")
         for name, cls in LmConfig.get_known_choices().items():
-            if getattr(cls, "hf_model_type", None) == mt:
+            if (getattr(cls, "hf_model_type", None) == mt) if mt is not None else \
+                    (cfg.get("architecture") is not None and getattr(cls, "hf_architecture", None) == cfg["architecture"]):
                 try:
                     conv = cls().hf_checkpoint_converter(str(ref))  # picks up per-family settings (ignore_prefix, ...)
                     return conv.replaced(reference_checkpoint=ref)
                 except Exception:  # noqa: BLE001
                     return HFCheckpointConverter(cls, ref, trust_remote_code=trust_remote_code)
-        raise ValueError(f"no model config class handles HF model_type {mt!r}")
+        raise ValueError(f"no model config class handles HF model_type {mt!r} / architecture {cfg.get('architecture')!r}")
 
     # -- tokenizer / vocab ---------------------------------------------------------------------------------------
     @property
@@ -345,7 +363,7 @@ class HFCheckpointConverter:
             config = self.config_from_hf_config(hf_config)
         elif isinstance(config, dict):
             config = self.config_from_hf_config(hf_config, config)
-        ckpt_vocab = hf_config.get("vocab_size")
+        ckpt_vocab = hf_config.get(getattr(config, "hf_vocab_key", "vocab_size"))
         sd = self.load_state_dict(ref, dtype=dtype)
         if ckpt_vocab is None:
             for k, v in sd.items():

@@ -108,7 +108,7 @@ class _DecodeGraph:
         # warm-up and capture run on tables that address nothing: no sequences, every token destination invalid
         self.binfo = PageBatchInfo(z(example.slot_ids), z(example.page_indices), z(example.seq_lens), z(example.cu_q_lens),
                                    z(example.num_seqs), torch.full(example.new_token_dests.shape, INVALID, dtype=example.new_token_dests.dtype, device=dev),
-                                   example.page_size)
+                                   example.page_size, num_pages=example.num_pages)
         self._shapes = self._shape_key(example)
         if lib.available():
             lib.status_buffer()
@@ -332,9 +332,55 @@ class InferenceEngine:
             raise RuntimeError(f"slot {slot} was on the free list but the page table refused it")
         return slot
 
+    def _release_slots(self, mask: np.ndarray) -> None:
+        """Give back the pages of the slots in ``mask`` and put the slots on the free list."""
+        ds = self.gen_state.decode_state
+        ds.page_table = ds.page_table.free_pages_for_finished(mask)
+        self.free_slots = sorted(set(self.free_slots) | set(np.nonzero(mask)[0].tolist()))
+
+    def forward_packed(self, chunks: Sequence[Tuple[int, Sequence[int]]], rows: Sequence[int]) -> Optional[torch.Tensor]:
+        """One model step over the next tokens of several sequences: ``chunks`` holds ``(slot, tokens)``, each sequence's tokens
+        following what its slot already holds.  Pages are allocated as needed.  Returns the logits of the given rows of the
+        packed tokens (None when ``rows`` is empty; the tokens still enter the cache).
+
+        When every sequence starts here, attention runs densely over the packed tokens with one segment per sequence, and the
+        packed length is padded to the attention kernel's tile.  Otherwise tokens attend through the cache, and a step of at most
+        ``max_seqs`` tokens has the shape of a decode round."""
+        ds = self.gen_state.decode_state
+        starts = [int(ds.page_table.seq_lens[s]) for s, _ in chunks]
+        toks = [int(t) for _, ts in chunks for t in ts]
+        slots = [s for s, ts in chunks for _ in ts]
+        pos = [p0 + i for p0, (_, ts) in zip(starts, chunks) for i in range(len(ts))]
+        prefill = all(p == 0 for p in starts)
+        pad = (-len(toks)) % PREFILL_PAD if prefill else max(0, self.config.max_seqs - len(toks))
+        # padding: no slot, no page, segment -1, position 0
+        ds.page_table, binfo = ds.page_table.allocate_for_seq(np.asarray(slots + [INVALID] * pad, np.int32),
+                                                              np.asarray(pos + [INVALID] * pad, np.int32))
+        if prefill:
+            seg = [i for i, (_, ts) in enumerate(chunks) for _ in ts]
+            binfo = dataclasses.replace(binfo, prefill_segment_ids=torch.tensor(seg + [-1] * pad, dtype=torch.int32))
+        dev = self.device
+        logits = self._forward(torch.tensor(toks + [0] * pad, dtype=torch.int32, device=dev), binfo.to(dev),
+                               torch.tensor(pos + [0] * pad, dtype=torch.int32, device=dev),
+                               torch.tensor(list(rows) or [0], dtype=torch.long, device=dev))
+        return logits if len(rows) else None
+
+    # -- sequences fed by the caller ------------------------------------------------------------------------------
+    def open_sequence(self) -> int:
+        """Reserve a slot for a sequence whose tokens the caller feeds through :meth:`forward_packed`."""
+        if not self.free_slots:
+            raise RuntimeError(f"all {self.config.max_seqs} slots are in use")
+        return self._take_slot()
+
+    def close_sequences(self, slots: Sequence[int]) -> None:
+        """Give back the pages and slots of caller-fed sequences."""
+        mask = np.zeros(self.config.max_seqs, dtype=bool)
+        mask[list(slots)] = True
+        self._release_slots(mask)
+
     def _prefill_prompts(self, batch: List[Request]) -> None:
         ds = self.gen_state.decode_state
-        toks, slots, pos = [], [], []
+        chunks: List[Tuple[int, List[int]]] = []
         primary: List[Tuple[Request, int]] = []
         for r in batch:
             s = self._take_slot()
@@ -343,19 +389,8 @@ class InferenceEngine:
                                                                                  ds.page_table.max_len_per_seq)))
             ds.assign_seq(s, np.asarray(prompt, np.int32), len(prompt), seq_params=params)
             self.local_map[s] = (r.request_id, 0)
-            toks += prompt
-            slots += [s] * len(prompt)
-            pos += list(range(len(prompt)))
+            chunks.append((s, prompt))
             primary.append((r, s))
-        # every sequence of a prefill starts at position 0: attention runs densely over the packed tokens, one segment per
-        # prompt; pad the packed length to the attention kernel's tile (padding: no slot, no page, segment -1)
-        seg = [i for i, r in enumerate(batch) for _ in range(max(len(r.prompt_tokens), 1))]
-        pad = (-len(toks)) % PREFILL_PAD
-        slots_np = np.asarray(slots + [INVALID] * pad, np.int32)
-        pos_alloc = np.asarray(pos + [INVALID] * pad, np.int32)
-        ds.page_table, binfo = ds.page_table.allocate_for_seq(slots_np, pos_alloc)
-        binfo = dataclasses.replace(binfo, prefill_segment_ids=torch.tensor(seg + [-1] * pad, dtype=torch.int32))
-        dev = self.device
         # the last prompt token of each sequence predicts its first new token; clones sample the same row with their own key
         last_index, cursor = {}, 0
         for r, s in primary:
@@ -363,8 +398,7 @@ class InferenceEngine:
             last_index[s] = cursor - 1
         # one logits row per generation: the primary and each of its clones read the row of the prompt's last token
         rows = [last_index[s] for r, s in primary for _ in range(r.n_generations)]
-        logits = self._forward(torch.tensor(toks + [0] * pad, dtype=torch.int32, device=dev), binfo.to(dev),
-                               torch.tensor(pos + [0] * pad, dtype=torch.int32, device=dev), torch.tensor(rows, dtype=torch.long, device=dev))
+        logits = self.forward_packed(chunks, rows)
         # clones are made after the forward pass: they copy pages that the pass has just filled
         row_slots = []
         for r, s in primary:
@@ -531,7 +565,6 @@ class InferenceEngine:
             rid, choice = self.local_map.pop(s)
             self.results[rid][choice].done = True
         ds.purge_queue_of_slot(np.asarray(slots, np.int32))
-        ds.page_table = ds.page_table.free_pages_for_finished(fin)
+        self._release_slots(fin)
         ds.invalidate_finished()
         ds.seq_lens[fin] = 0
-        self.free_slots = sorted(set(self.free_slots) | set(slots))

@@ -72,6 +72,14 @@ class PageBatchInfo:
     token belongs to, -1 for padding.  Attention then needs no cached context and can run as dense causal attention over the
     packed tokens with these segment ids."""
 
+    num_pages: int = 0
+    """pages of the cache the destinations point into"""
+
+    @property
+    def num_slots(self) -> int:
+        """Destinations outside ``[0, num_slots)`` are padding."""
+        return min(self.num_pages * self.page_size, INVALID)
+
     def pages_and_slots(self) -> Tuple[torch.Tensor, torch.Tensor]:
         d = self.new_token_dests
         ok = is_valid(d)
@@ -82,7 +90,7 @@ class PageBatchInfo:
         mv = lambda t: t.to(device, non_blocking=non_blocking)  # noqa: E731
         return PageBatchInfo(mv(self.slot_ids), mv(self.page_indices), mv(self.seq_lens), mv(self.cu_q_lens), mv(self.num_seqs),
                              mv(self.new_token_dests), self.page_size,
-                             None if self.prefill_segment_ids is None else mv(self.prefill_segment_ids))
+                             None if self.prefill_segment_ids is None else mv(self.prefill_segment_ids), self.num_pages)
 
 
 @dataclass
@@ -169,7 +177,8 @@ class PageTable:
         else:
             num = _allocate_numpy(new, slots, pos, o_slot, o_pages, o_lens, o_cu, o_dest)
         info = PageBatchInfo(torch.from_numpy(o_slot), torch.from_numpy(o_pages), torch.from_numpy(o_lens), torch.from_numpy(o_cu),
-                             torch.tensor(num, dtype=torch.int32), torch.from_numpy(o_dest), self.page_size)
+                             torch.tensor(num, dtype=torch.int32), torch.from_numpy(o_dest), self.page_size,
+                             num_pages=self.num_pages)
         return new, info
 
     # -- release ----------------------------------------------------------------------------------------------

@@ -55,9 +55,21 @@ def causal_mask(q_len: int, k_len: int, q_start=0, k_start=0, device=None) -> to
     return qp[:, None] >= kp[None, :]
 
 
+def chunk_segments(segment_ids: torch.Tensor, chunk_size: int) -> torch.Tensor:
+    """Segment ids ``[..., S]`` cut further into chunks of ``chunk_size`` positions, counted from the start of each run of equal
+    ids: non-decreasing ids, one per (run, chunk).  Negative ids (padding) stay as they are."""
+    S = segment_ids.shape[-1]
+    idx = torch.arange(S, device=segment_ids.device).expand(segment_ids.shape)
+    new_run = torch.ones_like(segment_ids, dtype=torch.bool)
+    new_run[..., 1:] = segment_ids[..., 1:] != segment_ids[..., :-1]
+    start = torch.where(new_run, idx, torch.zeros_like(idx)).cummax(dim=-1).values
+    out = torch.cumsum((idx - start) % chunk_size == 0, dim=-1) - 1
+    return torch.where(segment_ids < 0, segment_ids.to(out.dtype), out)
+
+
 @dataclass(frozen=True)
 class AttentionMask:
-    """Conjunction of structured masks: causal (with an optional offset), explicit, sliding window, segment ids.
+    """Conjunction of structured masks: causal (with an optional offset), explicit, sliding window, segment ids, chunks.
 
     ``materialize(q_len, k_len, q_slice, k_slice)`` returns the boolean mask of a block so block-wise kernels
     can skip or specialise blocks (src/levanter/layers/attention.py:795-846)."""
@@ -70,6 +82,9 @@ class AttentionMask:
     segments_sorted: bool = False
     """the segment ids are non-decreasing along the sequence with negative ids (padding) only at the end, as in packed
     batches: kernels may then skip every key block that lies before a query block's first sequence"""
+    chunk_size: Optional[int] = None
+    """positions are cut into chunks of this size, counted from the start of the sequence (of the segment, with segment ids), and a
+    query sees the keys of its own chunk only; queries and keys must be the same positions"""
 
     def __post_init__(self):
         if self.segment_ids is not None and not isinstance(self.segment_ids, tuple):
@@ -86,6 +101,16 @@ class AttentionMask:
     def with_segment_ids(self, segment_ids, kv_segment_ids=None, *, sorted: bool = False) -> "AttentionMask":
         return replace(self, segment_ids=(segment_ids, segment_ids if kv_segment_ids is None else kv_segment_ids),
                        segments_sorted=bool(sorted))
+
+    def with_chunk_size(self, chunk_size: Optional[int]) -> "AttentionMask":
+        return replace(self, chunk_size=chunk_size)
+
+    def chunks_as_segments(self) -> "AttentionMask":
+        """The same mask without a chunk size: chunks expressed as segment ids (needs segment ids to start from)."""
+        if self.chunk_size is None:
+            return self
+        seg = chunk_segments(self.segment_ids[0], self.chunk_size)
+        return replace(self, segment_ids=(seg, seg), chunk_size=None)
 
     def with_sliding_window(self, sliding_window: Optional[int]) -> "AttentionMask":
         return replace(self, sliding_window=sliding_window)
@@ -116,11 +141,15 @@ class AttentionMask:
             diff = qp[:, None] - kp[None, :]
             mask = _and(mask, (diff >= 0) & (diff < self.sliding_window))
         if self.segment_ids is not None:
-            qseg, kseg = self.segment_ids
+            qseg, kseg = self.segment_ids if self.chunk_size is None else self.chunks_as_segments().segment_ids
             sm = qseg[..., qs:qs + qn, None] == kseg[..., None, ks:ks + kn]
             if sm.dim() == 3:
                 sm = sm.unsqueeze(1)
             mask = _and(mask, sm)
+        elif self.chunk_size is not None:
+            qp = torch.arange(qn, device=device) + qs
+            kp = torch.arange(kn, device=device) + ks
+            mask = _and(mask, (qp // self.chunk_size)[:, None] == (kp // self.chunk_size)[None, :])
         return mask
 
     def __and__(self, other: "AttentionMask") -> "AttentionMask":
@@ -147,9 +176,15 @@ class AttentionMask:
             sw = self.sliding_window
         else:
             sw = min(self.sliding_window, other.sliding_window)
-        return AttentionMask(is_causal, offset, _and(self.explicit_mask, other.explicit_mask), self._same_segments(other), sw)
+        if self.chunk_size is not None and other.chunk_size is not None and self.chunk_size != other.chunk_size:
+            raise ValueError("Different chunk sizes cannot be combined with &")
+        chunk = self.chunk_size if self.chunk_size is not None else other.chunk_size
+        return AttentionMask(is_causal, offset, _and(self.explicit_mask, other.explicit_mask), self._same_segments(other), sw, chunk_size=chunk)
 
     def __or__(self, other: "AttentionMask") -> "AttentionMask":
+        if self.chunk_size != other.chunk_size:
+            raise ValueError("Different chunk sizes cannot be combined with |")
+
         def same_off():
             if self.causal_offset is None and other.causal_offset is None:
                 return True
@@ -166,7 +201,8 @@ class AttentionMask:
             sw = None
         else:
             sw = max(self.sliding_window, other.sliding_window)
-        return AttentionMask(is_causal, offset, _or(self.explicit_mask, other.explicit_mask), self._same_segments(other), sw)
+        return AttentionMask(is_causal, offset, _or(self.explicit_mask, other.explicit_mask), self._same_segments(other), sw,
+                             chunk_size=self.chunk_size)
 
     def _same_segments(self, other):
         a, b = self.segment_ids, other.segment_ids
@@ -272,7 +308,8 @@ def dot_product_attention(q, k, v, mask: Union[None, torch.Tensor, AttentionMask
         if backend == AttentionBackend.B200:
             raise ValueError("the B200 flash-attention kernel does not support this call (bias, dropout, explicit mask, dtype or head size)")
         plain = mask is None or (isinstance(mask, AttentionMask) and mask.explicit_mask is None and mask.segment_ids is None
-                                 and mask.sliding_window is None and _structured_only(mask))
+                                 and mask.sliding_window is None and mask.chunk_size is None and _structured_only(mask)) \
+            and v.shape[-1] == q.shape[-1]
         if q.is_cuda and plain and bias is None and no_drop and logits_soft_cap is None and q.dtype in (torch.bfloat16, torch.float16) \
                 and q.shape[1] == k.shape[1]:
             # shapes the tcgen05 kernels do not cover (head sizes other than 64 and 128, cross attention): the library's fused
@@ -285,13 +322,13 @@ def dot_product_attention(q, k, v, mask: Union[None, torch.Tensor, AttentionMask
         B, Sq, H, D = q.shape
         m = materialize_mask(mask, Sq, k.shape[1], device=q.device)
         is_causal = isinstance(mask, AttentionMask) and mask.is_causal and mask.explicit_mask is None and \
-            mask.segment_ids is None and mask.sliding_window is None and _structured_only(mask)
+            mask.segment_ids is None and mask.sliding_window is None and mask.chunk_size is None and _structured_only(mask)
         out = F.scaled_dot_product_attention(
             q.transpose(1, 2), _expand_kv(k, H).transpose(1, 2), _expand_kv(v, H).transpose(1, 2),
             attn_mask=None if is_causal else m, is_causal=is_causal, scale=scaling_factor)
         return out.transpose(1, 2)
 
-    if backend == AttentionBackend.TORCH_FLASH and bias is None:
+    if backend == AttentionBackend.TORCH_FLASH and bias is None and v.shape[-1] == q.shape[-1]:
         block = flash_block_size or FA.BLOCK_SIZE
         if q.shape[1] >= block and k.shape[1] >= block and q.shape[1] % block == 0 and k.shape[1] % block == 0:
             return FA.flash_attention(q, k, v, mask, dropout=dropout, inference=inference, block_size=block,
@@ -350,6 +387,9 @@ class AttentionConfig:
     logits_soft_cap: Optional[float] = None
     qk_norm: Optional[LayerNormConfigBase] = None
     sliding_window: Optional[int] = None
+    v_head_dim: Optional[int] = None          # value size per head where it differs from the query/key size
+    attention_chunk_size: Optional[int] = None  # a query sees its own chunk of that many positions only
+    output_gate: bool = False                 # the heads are multiplied by sigmoid(W_g x) before the output projection
 
     def __post_init__(self):
         assert self.num_heads % self.num_kv_heads == 0, "num_heads must be divisible by num_kv_heads"
@@ -357,6 +397,10 @@ class AttentionConfig:
     @property
     def head_size(self) -> int:
         return self.head_dim if self.head_dim is not None else self.hidden_dim // self.num_heads
+
+    @property
+    def v_head_size(self) -> int:
+        return self.v_head_dim if self.v_head_dim is not None else self.head_size
 
     @property
     def q_heads_per_group(self) -> int:
@@ -379,7 +423,7 @@ class Attention(nn.Module):
         super().__init__()
         c = config
         self.config = c
-        D = c.head_size
+        D, Dv = c.head_size, c.v_head_size
         self.tp = tp
         tp_size = tp.size if tp is not None else 1
         assert c.num_kv_heads % tp_size == 0 or tp_size == 1, "kv heads must divide the tensor-parallel size"
@@ -390,10 +434,13 @@ class Attention(nn.Module):
                              lev_out=(self.local_kv, c.q_heads_per_group, D), lev_in=(c.hidden_dim,), parallel=("column", tp))
         self.k_proj = Linear(c.hidden_dim, self.local_kv * D, bias=c.use_bias, init_std=init_std,
                              lev_out=(self.local_kv, D), lev_in=(c.hidden_dim,), parallel=("column", tp))
-        self.v_proj = Linear(c.hidden_dim, self.local_kv * D, bias=c.use_bias, init_std=init_std,
-                             lev_out=(self.local_kv, D), lev_in=(c.hidden_dim,), parallel=("column", tp))
-        self.o_proj = Linear(self.local_heads * D, c.hidden_dim, bias=out_bias, init_std=init_std,
-                             lev_out=(c.hidden_dim,), lev_in=(self.local_heads, D), parallel=("row", tp))
+        self.v_proj = Linear(c.hidden_dim, self.local_kv * Dv, bias=c.use_bias, init_std=init_std,
+                             lev_out=(self.local_kv, Dv), lev_in=(c.hidden_dim,), parallel=("column", tp))
+        self.o_proj = Linear(self.local_heads * Dv, c.hidden_dim, bias=out_bias, init_std=init_std,
+                             lev_out=(c.hidden_dim,), lev_in=(self.local_heads, Dv), parallel=("row", tp))
+        if c.output_gate:
+            self.g_proj = Linear(c.hidden_dim, self.local_heads * Dv, bias=c.use_bias, init_std=init_std,
+                                 lev_out=(self.local_kv, c.q_heads_per_group, Dv), lev_in=(c.hidden_dim,), parallel=("column", tp))
         if c.qk_norm is not None:
             self.q_norm = c.qk_norm.build(D)
             self.k_norm = c.qk_norm.build(D)
@@ -409,7 +456,7 @@ class Attention(nn.Module):
         lead = x.shape[:-1]
         q = self.q_proj(x).view(*lead, self.local_heads, D)
         k = self.k_proj(x).view(*lead, self.local_kv, D)
-        v = self.v_proj(x).view(*lead, self.local_kv, D)
+        v = self.v_proj(x).view(*lead, self.local_kv, c.v_head_size)
         if self.q_norm is not None:
             q = self.q_norm(q)
             k = self.k_norm(k)
@@ -428,6 +475,9 @@ class Attention(nn.Module):
         q, k, v = self._compute_qkv(x, pos_ids)
         if c.sliding_window is not None and isinstance(mask, AttentionMask) and mask.is_causal:
             mask = mask & AttentionMask.causal(sliding_window=c.sliding_window)
+        if c.attention_chunk_size is not None:
+            mask = (mask if isinstance(mask, AttentionMask) else AttentionMask.explicit(mask) if mask is not None
+                    else AttentionMask.causal()).with_chunk_size(c.attention_chunk_size)
         squeeze = q.dim() == 3
         if squeeze:
             q, k, v = q.unsqueeze(0), k.unsqueeze(0), v.unsqueeze(0)
@@ -437,7 +487,9 @@ class Attention(nn.Module):
             scaling_factor=c.scaling_factor, inference=True)
         if squeeze:
             attn = attn.squeeze(0)
-        attn = attn.reshape(*x.shape[:-1], self.local_heads * c.head_size).to(x.dtype)
+        attn = attn.reshape(*x.shape[:-1], self.local_heads * c.v_head_size).to(x.dtype)
+        if c.output_gate:
+            attn = attn * torch.sigmoid(self.g_proj(x).float()).to(attn.dtype)
         if residual is not None:
             if type(self.o_proj) is Linear:
                 from ..ops.gemm import linear_residual
@@ -459,6 +511,9 @@ class Attention(nn.Module):
         from ..ops import paged_attention as PA
 
         c = self.config
+        if c.output_gate or c.attention_chunk_size is not None or c.v_head_size != c.head_size:
+            out = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+            return (self.o_proj(out) if residual is None else self.o_proj(out) + residual), kv_cache
         q, k, v = self._compute_qkv(x, pos_ids)
         kv_cache = kv_cache.update(batch_info, k, v)
         scale = c.scaling_factor if c.scaling_factor is not None else 1.0 / math.sqrt(c.head_size)
@@ -482,8 +537,79 @@ class Attention(nn.Module):
             return self.o_proj(out) + residual, kv_cache
         return self.o_proj(out), kv_cache
 
+    def _fused_projection(self) -> Optional[torch.Tensor]:
+        """One weight ``[q; k; v; gate]`` for serving: the four projections read the same rows, so a decode step streams one matrix
+        instead of launching four products.  The projections' own parameters become row slices of it (nothing is stored
+        twice).  None when a projection is wrapped (LoRA, fp8) or has a bias, and for a model in training, whose parameters
+        belong to the gradient engine's own flat buffers."""
+        mods = [self.q_proj, self.k_proj, self.v_proj] + ([self.g_proj] if self.config.output_gate else [])
+        if any(type(m) is not Linear or m.bias is not None for m in mods):
+            return None
+        ws = [m.weight for m in mods]
+        if self.training or any(getattr(w, "main_grad", None) is not None or getattr(w, "grad_sink", None) is not None for w in ws):
+            return None
+        fused = getattr(self, "_fused", None)
+        if fused is not None:
+            at = fused.data_ptr()
+            for w in ws:  # still aliases of the fused buffer?  (a model that was moved or converted since has new storage)
+                if w.data_ptr() != at or w.dtype != fused.dtype:
+                    fused = None
+                    break
+                at += w.numel() * w.element_size()
+        if fused is None:
+            fused = torch.cat([w.detach() for w in ws])
+            row = 0
+            for w in ws:
+                w.data = fused[row:row + w.shape[0]]
+                row += w.shape[0]
+            self._fused = fused
+        return fused
+
+    def _paged_heads(self, x, kv_cache: "KvPageCache", batch_info, pos_ids) -> torch.Tensor:
+        """The gated, concatenated heads ``[T, heads * v_head_size]`` of packed tokens, for the forms of attention that the plain
+        paged path does not have (chunks, a value size of its own, an output gate)."""
+        from ..ops import flash_attention as FA
+        from ..ops import paged_attention as PA
+        from ..ops.residual_stream import project
+
+        c = self.config
+        T, D, Dv = x.shape[0], c.head_size, c.v_head_size
+        nq, nk, nv = self.local_heads * D, self.local_kv * D, self.local_kv * Dv
+        fused = self._fused_projection() if (x.is_cuda and not torch.is_grad_enabled() and self.q_norm is None and self.rot is None) else None
+        gate = None
+        if fused is not None:
+            y = project(x, fused)
+            q, k, v = y[:, :nq].unflatten(1, (-1, D)), y[:, nq:nq + nk].unflatten(1, (-1, D)), y[:, nq + nk:nq + nk + nv].unflatten(1, (-1, Dv))
+            if c.output_gate:
+                gate = y[:, nq + nk + nv:]
+        else:
+            q, k, v = self._compute_qkv(x, pos_ids)
+            if c.output_gate:
+                gate = self.g_proj(x)
+        PA.kv_page_write_general(kv_cache.kv_pages, k, v, batch_info.new_token_dests)
+        scale = c.scaling_factor if c.scaling_factor is not None else 1.0 / math.sqrt(D)
+        seg = getattr(batch_info, "prefill_segment_ids", None)
+        if seg is not None and FA.packed_supported(q, k, v, scale):
+            # pure prefill: every sequence starts at position 0, nothing is read back from the cache
+            out = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=scale, chunk=c.attention_chunk_size, gate=gate,
+                                            logits_soft_cap=c.logits_soft_cap)
+        else:
+            out = PA.paged_attention_general(q, kv_cache.kv_pages, self.local_kv, Dv, batch_info, sm_scale=scale,
+                                             chunk=c.attention_chunk_size, gate=gate, soft_cap=c.logits_soft_cap)
+        return out.reshape(T, self.local_heads * Dv).to(x.dtype)
+
+    def paged_decode_stream(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor):
+        """:meth:`paged_decode` for an fp32 residual stream: ``stream + o_proj(heads)``, added in the projection's epilogue."""
+        from ..ops.residual_stream import add_linear
+
+        out = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        if type(self.o_proj) is Linear and self.o_proj.bias is None:
+            return add_linear(stream, out, self.o_proj.weight), kv_cache
+        return stream + self.o_proj(out).float(), kv_cache
+
     def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
-        return KvPageCache.init(max_pages, page_size, self.local_kv, self.config.head_size, dtype=dtype, device=device)
+        return KvPageCache.init(max_pages, page_size, self.local_kv, self.config.head_size, v_head_size=self.config.v_head_size, dtype=dtype,
+                                device=device)
 
 
 class AttentionWithSink(Attention):
@@ -588,12 +714,16 @@ class MultiHeadLatentAttention(nn.Module):
 @dataclass
 class KvPageCache:
     """Paged KV storage ``kv_pages[page, slot, 2 * kv_heads, head_size]`` with K at even and V at odd head index
-    (src/levanter/layers/attention.py:1638-1707)."""
+    (src/levanter/layers/attention.py:1638-1707); with a value size of its own ``kv_pages[page, slot, kv_heads, head_size + v_head_size]``,
+    the same order in memory: per KV head a key row, then a value row."""
 
     kv_pages: torch.Tensor
 
     @staticmethod
-    def init(max_pages: int, page_size: int, kv_heads: int, head_size: int, *, dtype=torch.bfloat16, device=None):
+    def init(max_pages: int, page_size: int, kv_heads: int, head_size: int, *, v_head_size: Optional[int] = None, dtype=torch.bfloat16,
+             device=None):
+        if v_head_size is not None and v_head_size != head_size:
+            return KvPageCache(torch.zeros(max_pages, page_size, kv_heads, head_size + v_head_size, dtype=dtype, device=device))
         return KvPageCache(torch.zeros(max_pages, page_size, 2 * kv_heads, head_size, dtype=dtype, device=device))
 
     @property

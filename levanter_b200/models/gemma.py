@@ -23,6 +23,7 @@ from ..layers.normalization import LayerNormConfigBase
 from ..layers.rotary import rope_config_from_hf, rope_to_hf_dict, DefaultRotaryEmbeddingsConfig, RotaryEmbeddingsConfig
 from ..nn import Linear
 from ..ops.norm import fused_norm
+from ..ops.residual_stream import rms_norm_stream
 from ..utils.activation import ActivationFunctionEnum, from_hf_name
 from ..utils.flop_utils import lm_flops_per_token
 from ..utils.remat import should_recompute
@@ -42,6 +43,10 @@ class GemmaRMSNorm(nn.Module):
 
     def forward(self, x):
         return fused_norm(x, self.weight, None, self.eps, w_offset=1.0)[0]
+
+    def from_stream(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The norm of an fp32 residual stream, in the weight's dtype (``rows``: of these rows only)."""
+        return rms_norm_stream(x, self.weight, self.eps, w_offset=1.0, rows=rows)
 
 
 @LayerNormConfigBase.register_subclass("gemma")

@@ -91,7 +91,7 @@ class LmExample:
             em = None
             if m0.explicit_mask is not None:
                 em = torch.stack([e.attn_mask.explicit_mask for e in examples])
-            mask = AttentionMask(m0.is_causal, m0.causal_offset, em, seg, m0.sliding_window)
+            mask = AttentionMask(m0.is_causal, m0.causal_offset, em, seg, m0.sliding_window, chunk_size=m0.chunk_size)
         else:
             mask = torch.stack([e.attn_mask for e in examples])
         return LmExample(tokens, lm, mask)
@@ -103,7 +103,7 @@ class LmExample:
         m = self.attn_mask
         if isinstance(m, AttentionMask):
             seg = None if m.segment_ids is None else (mv(m.segment_ids[0]), mv(m.segment_ids[1]))
-            m = AttentionMask(m.is_causal, mv(m.causal_offset), mv(m.explicit_mask), seg, m.sliding_window)
+            m = AttentionMask(m.is_causal, mv(m.causal_offset), mv(m.explicit_mask), seg, m.sliding_window, chunk_size=m.chunk_size)
         else:
             m = mv(m)
         return LmExample(mv(self.tokens), mv(self.loss_mask), m)
@@ -117,7 +117,7 @@ class LmExample:
             off = m.causal_offset
             if isinstance(off, torch.Tensor) and off.dim() > 0:
                 off = off[start:stop]
-            m = AttentionMask(m.is_causal, off, em, seg, m.sliding_window)
+            m = AttentionMask(m.is_causal, off, em, seg, m.sliding_window, chunk_size=m.chunk_size)
         else:
             m = m[start:stop] if m.dim() > 2 else m
         return LmExample(self.tokens[start:stop], self.loss_mask[start:stop], m)

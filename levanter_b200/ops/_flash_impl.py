@@ -179,6 +179,10 @@ def flash_attention_cuda(q, k, v, mask, *, logits_soft_cap: Optional[float] = No
     window = 0
     causal = False
     B, S, Sk = q.shape[0], q.shape[1], k.shape[1]
+    if mask is not None and mask.chunk_size is not None:
+        if mask.segment_ids is None:
+            mask = mask.with_segment_ids(torch.zeros(B, S, dtype=torch.int32, device=q.device), sorted=True)
+        mask = mask.chunks_as_segments()  # a chunk is a segment of its own
     if mask is not None:
         causal = bool(mask.is_causal)
         window = mask.sliding_window or 0

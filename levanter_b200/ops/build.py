@@ -21,6 +21,16 @@ CSRC = Path(__file__).resolve().parent / "csrc"
 LIBDIR = Path(__file__).resolve().parent / "_lib"
 LIBNAME = "liblevanter_b200.so"
 
+# What a process that only serves a model needs (``lib.use_serving_library``): a subset of the same objects in a library of its
+# own, so that the first run in a fresh checkout compiles these sources and no others.
+SERVING_LIBNAME = "liblevanter_b200_serving.so"
+SERVING_SOURCES = ("attention_any", "flash_attn_fwd2", "gemm_bf16", "gemm_pair", "gemm_skinny", "moe_experts", "page_table",
+                   "paged_attention", "residual_stream", "sampler")
+
+# Kernels whose results are 32-bit throughout (norms of an fp32 stream, router scores, fp32 attention): no approximate
+# exponentials, divisions or square roots.
+ACCURATE_SOURCES = ("attention_any", "moe_experts", "residual_stream")
+
 NVCC_FLAGS = [
     "-gencode",
     "arch=compute_100a,code=sm_100a",
@@ -42,8 +52,15 @@ def _nvcc() -> str:
     return cand
 
 
-def _sources() -> list[Path]:
-    return sorted(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cpp")))
+def _sources(serving: bool = False) -> list[Path]:
+    every = sorted(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cpp")))
+    return [p for p in every if p.stem in SERVING_SOURCES] if serving else every
+
+
+def _flags(src: Path) -> list[str]:
+    if src.suffix != ".cu":
+        return ["-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
+    return [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.stem not in ACCURATE_SOURCES]
 
 
 def _digest(paths: list[Path]) -> str:
@@ -51,26 +68,31 @@ def _digest(paths: list[Path]) -> str:
     for p in sorted(paths + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))):
         h.update(p.name.encode())
         h.update(p.read_bytes())
-    h.update(" ".join(NVCC_FLAGS).encode())
+    for p in sorted(paths):
+        h.update(" ".join(_flags(p)).encode())
     return h.hexdigest()
 
 
-def lib_path() -> Path:
-    return LIBDIR / LIBNAME
+def lib_path(serving: bool = False) -> Path:
+    return LIBDIR / (SERVING_LIBNAME if serving else LIBNAME)
 
 
-def is_current() -> bool:
-    stamp = LIBDIR / "build.stamp"
-    return lib_path().exists() and stamp.exists() and stamp.read_text().strip() == _digest(_sources())
+def _stamp(serving: bool) -> Path:
+    return LIBDIR / ("serving.stamp" if serving else "build.stamp")
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` and link the shared object.  Returns its path."""
-    srcs = _sources()
+def is_current(serving: bool = False) -> bool:
+    stamp = _stamp(serving)
+    return lib_path(serving).exists() and stamp.exists() and stamp.read_text().strip() == _digest(_sources(serving))
+
+
+def build(force: bool = False, verbose: bool = False, serving: bool = False) -> Path:
+    """Compile every ``csrc/*.cu`` (``serving``: the serving subset) and link the shared object.  Returns its path."""
+    srcs = _sources(serving)
     if not srcs:
         raise RuntimeError(f"no CUDA sources in {CSRC}")
-    if not force and is_current():
-        return lib_path()
+    if not force and is_current(serving):
+        return lib_path(serving)
     LIBDIR.mkdir(parents=True, exist_ok=True)
     nvcc = _nvcc()
     objs: list[Path] = []
@@ -78,8 +100,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 
     def compile_one(src: Path) -> Path:
         obj = LIBDIR / (src.stem + ".o")
-        flags = NVCC_FLAGS if src.suffix == ".cu" else ["-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
-        cmd = [nvcc, *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+        cmd = [nvcc, *_flags(src), "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         r = subprocess.run(cmd, capture_output=True, text=True)
         logs[src.name] = r.stderr + r.stdout
         if r.returncode != 0:
@@ -88,15 +109,17 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
-    out = lib_path()
-    cmd = [nvcc, "-shared", "-o", str(out), *[str(o) for o in objs], "-gencode", "arch=compute_100a,code=sm_100a", "-ldl", "-lpthread"]
+    out = lib_path(serving)
+    part = out.with_suffix(f".{os.getpid()}.part")  # linked beside its final name: another process never loads half a library
+    cmd = [nvcc, "-shared", "-o", str(part), *[str(o) for o in objs], "-gencode", "arch=compute_100a,code=sm_100a", "-ldl", "-lpthread"]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
         raise RuntimeError(f"link failed:\n{r.stderr}")
-    (LIBDIR / "ptxas.log").write_text("\n".join(f"==== {k}\n{v}" for k, v in sorted(logs.items())))
-    (LIBDIR / "build.stamp").write_text(_digest(srcs))
+    os.replace(part, out)
+    (LIBDIR / ("ptxas_serving.log" if serving else "ptxas.log")).write_text("\n".join(f"==== {k}\n{v}" for k, v in sorted(logs.items())))
+    _stamp(serving).write_text(_digest(srcs))
     if verbose:
-        print((LIBDIR / "ptxas.log").read_text())
+        print("\n".join(logs[k] for k in sorted(logs)))
     return out
 
 

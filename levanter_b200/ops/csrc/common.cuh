@@ -431,6 +431,24 @@ inline int make_tmap_2d_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, u
   return r == CUDA_SUCCESS ? kErrOk : kErrTensorMap;
 }
 
+// Rows of several heads, [rows, heads, size] bf16 with row stride ld (elements): a box is 64 columns of one head in box_rows rows;
+// columns past `size` are filled with zeros.
+inline int make_tmap_heads_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t heads, uint64_t size, uint64_t ld,
+                                uint32_t box_rows) {
+  ensure_context_for(ptr);
+  EncodeTiledFn enc = get_encode_tiled();
+  if (enc == nullptr) return kErrTensorMap;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) != 0 || (ld * 2) % 16 != 0 || (size * 2) % 16 != 0) return kErrBadArg;
+  cuuint64_t gdim[3] = {size, heads, rows};
+  cuuint64_t gstr[2] = {size * 2, ld * 2};
+  cuuint32_t box[3] = {64, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), gdim, gstr, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? kErrOk : kErrTensorMap;
+}
+
 // Row-major 2-D tensor of one-byte elements [rows, cols] with row stride ld (bytes); box = [box_rows, 128].
 inline int make_tmap_2d_u8(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows) {
   ensure_context_for(ptr);

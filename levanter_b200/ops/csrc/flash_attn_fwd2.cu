@@ -10,6 +10,13 @@
 // TMEM map (512 columns): S_A/P_A [0,128)  S_B/P_B [128,256)  O_A [256,384)  O_B [384,512).
 // Shared memory: Q_A, Q_B, two K stages, two V stages (6 x 32 KB).
 // Mask semantics, outputs and the lazy-rescale rule are those of flash_fwd_kernel.
+//
+// kPacked (lvb_flash_attn_fwd_packed) is the form the inference engine prefills with: packed sequences, each starting at
+// position 0.  What a row sees is one contiguous range of packed keys, so the mask is a lower bound per row computed from its
+// position (the start of its sequence, or of its chunk when attention is chunked) instead of a segment id per key: blocks
+// between the bound and the diagonal need no mask at all.  Key and value sizes may differ and need not be 64 or 128: the tensor
+// maps are three-dimensional (size, head, row), columns past the size arrive as zeros, and the MMAs stop at the next
+// multiple of 16.  An optional gate is applied to the output on its way out.
 #include "common.cuh"
 
 namespace lvb {
@@ -36,6 +43,12 @@ struct Params {
   int window;
   int causal;  // 0: every key is visible (subject to segment ids); window must be 0 and kblock_lo null then
   int* status;
+  // ---- kPacked
+  const int* pos;            // [S]: position of each packed row in its sequence
+  int chunk;                 // > 0: a row at position i sees positions >= i - i % chunk only
+  int dk, dv;                // query/key and value sizes (multiples of 8, at most HD)
+  const __nv_bfloat16* gate; // optional [S, Hq * dv] (row stride ldg): the output is multiplied by its sigmoid
+  long long ldg;
 };
 
 template <int HD>
@@ -55,7 +68,13 @@ __device__ __forceinline__ float to_log2(float s, float scale_log2, float scale,
   else return s * scale_log2;
 }
 
-template <int HD, bool kSeg, bool kCap>
+// kPacked: first packed key that row qi sees
+__device__ __forceinline__ int row_lower_bound(const Params& p, int qi) {
+  const int pos = p.pos[qi];
+  return qi - (p.chunk > 0 ? pos % p.chunk : pos);
+}
+
+template <int HD, bool kSeg, bool kCap, bool kPacked = false>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, Params p) {
@@ -97,6 +116,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int lo = p.kblock_lo[b * (p.S / BT) + jdiagA];
     jlo = max(jlo, min(lo, jdiagA));
   }
+  if constexpr (kPacked) jlo = row_lower_bound(p, q0) / BT;  // bounds do not decrease along the packed rows
   const int nB = (causal ? jdiagB : p.Sk / BT - 1) - jlo + 1;  // blocks processed by tile B
   const int nA = causal ? nB - 1 : nB;                        // causal: tile A stops one block earlier (its diagonal)
 
@@ -132,11 +152,15 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       const int row_q = b * p.S + q0;
-      mbar_expect_tx(q_full, 2 * kQKV);
+      const int ck = kPacked ? (p.dk + 63) / 64 : D / 64, cv = kPacked ? (p.dv + 63) / 64 : D / 64;  // 64-column chunks
+      mbar_expect_tx(q_full, 2 * ck * kChunkBytes);
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
         for (int c = 0; c < D / 64; ++c)
+          if constexpr (kPacked) {
+            if (c < ck) tma_load_3d(smem + Smem::kQ + t * kQKV + c * kChunkBytes, &tmQ, q_full, 64 * c, h, row_q + t * BT);
+          } else
           tma_load_2d(smem + Smem::kQ + t * kQKV + c * kChunkBytes, &tmQ, q_full, h * D + 64 * c, row_q + t * BT);
       bool ok = true;
       for (int it = 0; it < nB && ok; ++it) {
@@ -146,22 +170,32 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         ok = mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 1200, it);
         if (!ok) break;
         uint8_t* ks = smem + Smem::kK + st * kQKV;
-        mbar_expect_tx(&k_full[st], kQKV);
+        mbar_expect_tx(&k_full[st], ck * kChunkBytes);
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c) tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * D + 64 * c, row_k);
+        for (int c = 0; c < D / 64; ++c)
+          if constexpr (kPacked) {
+            if (c < ck) tma_load_3d(ks + c * kChunkBytes, &tmK, &k_full[st], 64 * c, hkv, row_k);
+          } else
+          tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * D + 64 * c, row_k);
         ok = mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, 1201, it);
         if (!ok) break;
         uint8_t* vs = smem + Smem::kV + st * kQKV;
-        mbar_expect_tx(&v_full[st], kQKV);
+        mbar_expect_tx(&v_full[st], cv * kChunkBytes);
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c) tma_load_2d(vs + c * kChunkBytes, &tmV, &v_full[st], hkv * D + 64 * c, row_k);
+        for (int c = 0; c < D / 64; ++c)
+          if constexpr (kPacked) {
+            if (c < cv) tma_load_3d(vs + c * kChunkBytes, &tmV, &v_full[st], 64 * c, hkv, row_k);
+          } else
+          tma_load_2d(vs + c * kChunkBytes, &tmV, &v_full[st], hkv * D + 64 * c, row_k);
       }
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc_bf16(BT, BT, false, false);
-      constexpr uint32_t idesc_pv = make_idesc_bf16(BT, D, false, true);  // A = P in TMEM, B = V MN-major
+      // A = P in TMEM, B = V MN-major
+      const uint32_t idesc_pv = make_idesc_bf16(BT, kPacked ? (p.dv + 15) / 16 * 16 : D, false, true);
+      const int qk_steps = kPacked ? (p.dk + 15) / 16 : D / 16;
       const uint32_t sq = smem_u32(smem + Smem::kQ);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1300, 0);
 
@@ -171,6 +205,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const uint32_t sqt = sq + tile * kQKV;
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
+          if (kPacked && kk >= qk_steps) break;
           const uint32_t off = (kk >> 2) * kChunkBytes + (kk & 3) * 32;
           umma_bf16_ss(tmem_base + tile * BT, make_smem_desc(sqt + off, 16, 1024), make_smem_desc(sk + off, 16, 1024),
                        idesc_qk, kk > 0 ? 1u : 0u);
@@ -243,6 +278,11 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int* kseg_row = kSeg ? p.k_seg + b * p.Sk : nullptr;
     float m_used = -INFINITY, l_sum = 0.f;
     bool ok = true;
+    int row_lo = 0, tile_lo = 0;  // kPacked: this row's first visible key, and the last row's (the largest of the tile)
+    if constexpr (kPacked) {
+      row_lo = row_lower_bound(p, qi);
+      tile_lo = row_lower_bound(p, q0 + tile * BT + BT - 1);
+    }
 
     for (int it = 0; it < nT && ok; ++it) {
       const int j = jlo + it;
@@ -251,7 +291,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const bool need_mask = (j == jdiag) || kSeg || (p.window > 0 && k0 <= q0 + tile * BT + BT - 1 - p.window);
+      const bool need_mask = (j == jdiag) || kSeg || (kPacked && k0 < tile_lo) || (p.window > 0 && k0 <= q0 + tile * BT + BT - 1 - p.window);
 
       // ---- pass 1: row maximum (raw logits; the scale is positive and the soft-cap monotonic)
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -267,6 +307,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             bool valid = !causal || kj <= qi;
             if (p.window > 0) valid = valid && (qi - kj < p.window);
             if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
+            if (kPacked) valid = valid && kj >= row_lo;
             if (!valid) v[t] = __float_as_uint(-INFINITY);
           }
         }
@@ -320,6 +361,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             bool valid = !causal || kj <= qi;
             if (p.window > 0) valid = valid && (qi - kj < p.window);
             if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
+            if (kPacked) valid = valid && kj >= row_lo;
             const float x = kCap ? to_log2<kCap>(__uint_as_float(v[t]), scale_log2, p.scale, p.soft_cap) + neg_m
                                  : fmaf(__uint_as_float(v[t]), scale_log2, neg_m);
             e[t] = valid ? exp2f(x) : 0.f;
@@ -369,6 +411,40 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         m_used = m_new;
       }
       const float inv = l_sum > 0.f ? o_scale / l_sum : 0.f;
+      if constexpr (kPacked) {
+        __nv_bfloat16* orow = p.O + static_cast<size_t>(qi) * (static_cast<size_t>(p.Hq) * p.dv) + static_cast<size_t>(h) * p.dv;
+        const __nv_bfloat16* grow = p.gate != nullptr ? p.gate + static_cast<size_t>(qi) * p.ldg + static_cast<size_t>(h) * p.dv : nullptr;
+#pragma unroll 1
+        for (int c = 0; c < p.dv; c += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32(tO + c, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int q4 = 0; q4 < 4; ++q4) {
+            if (c + 8 * q4 < p.dv) {
+              float e[8];
+#pragma unroll
+              for (int t = 0; t < 8; ++t) e[t] = __uint_as_float(v[q4 * 8 + t]) * inv;
+              if (grow != nullptr) {
+                const uint4 gw = __ldg(reinterpret_cast<const uint4*>(grow + c) + q4);
+                const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&gw);
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                  const float2 f = __bfloat1622float2(gh[t]);
+                  e[2 * t] *= 1.f / (1.f + __expf(-f.x));
+                  e[2 * t + 1] *= 1.f / (1.f + __expf(-f.y));
+                }
+              }
+              uint4 w;
+              w.x = pack_bf16x2(e[0], e[1]);
+              w.y = pack_bf16x2(e[2], e[3]);
+              w.z = pack_bf16x2(e[4], e[5]);
+              w.w = pack_bf16x2(e[6], e[7]);
+              reinterpret_cast<uint4*>(orow + c)[q4] = w;
+            }
+          }
+        }
+      } else {
       __nv_bfloat16* orow = p.O + (static_cast<size_t>(b) * p.S + qi) * (static_cast<size_t>(p.Hq) * D) + static_cast<size_t>(h) * D;
 #pragma unroll 1
       for (int c = 0; c < D; c += 32) {
@@ -386,6 +462,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         }
       }
       p.lse2[(static_cast<size_t>(b) * p.Hq + h) * p.S + qi] = (l_sum > 0.f) ? m_used + log2f(l_sum) : -INFINITY;
+      }
     }
   }
 
@@ -397,10 +474,10 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   }
 }
 
-template <int HD, bool kSeg, bool kCap>
+template <int HD, bool kSeg, bool kCap, bool kPacked = false>
 int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const Params& p, cudaStream_t st) {
   using Smem = SmemT<HD>;
-  auto kern = flash_fwd2_kernel<HD, kSeg, kCap>;
+  auto kern = flash_fwd2_kernel<HD, kSeg, kCap, kPacked>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem::kTotal) != cudaSuccess) return kErrCuda;
@@ -459,6 +536,7 @@ extern "C" int lvb_flash_attn_fwd2_hd(const void* q, const void* k, const void* 
   p.scale = scale; p.soft_cap = soft_cap; p.window = window;
   p.causal = causal ? 1 : 0;
   p.status = status;
+  p.pos = nullptr; p.chunk = 0; p.dk = p.dv = head_dim; p.gate = nullptr; p.ldg = 0;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (head_dim == 128) return launch_hd<128>(q, k, v, p, st);
   if (head_dim == 64) return launch_hd<64>(q, k, v, p, st);
@@ -470,4 +548,37 @@ extern "C" int lvb_flash_attn_fwd2(const void* q, const void* k, const void* v, 
                                    const int* k_seg, const int* kblock_lo, int B, int S, int Hq, int Hkv, float scale, float soft_cap,
                                    int window, int* status, void* stream) {
   return lvb_flash_attn_fwd2_hd(q, k, v, o, lse2, q_seg, k_seg, kblock_lo, nullptr, B, S, S, Hq, Hkv, 128, 1, scale, soft_cap, window, status, stream);
+}
+
+// Causal attention over T packed rows (T a multiple of 256) of sequences that each start at position 0:
+//   q: row t, head h at q + t * ldq + h * dk     k / v: row t, head g at k + t * ldk + g * dk, v + t * ldv + g * dv
+//   o[T, Hq, dv] = softmax(scale q k^T over the visible keys) v  (* sigmoid(gate[t, h, :]))
+// pos[t] is the row's position in its sequence (padding rows: 0).  chunk > 0: positions are cut into chunks of that many, counted
+// from the sequence's start, and a row sees its own chunk only.  dk, dv: multiples of 8, at most 128; ldq, ldk, ldv and ldg
+// multiples of 8 and the pointers 16-byte aligned.
+extern "C" int lvb_flash_attn_fwd_packed(const void* q, const void* k, const void* v, const void* gate, void* o, const int* pos, int T,
+                                         int Hq, int Hkv, int dk, int dv, int ldq, int ldk, int ldv, int ldg, int chunk, float scale,
+                                         float soft_cap, int* status, void* stream) {
+  using namespace lvb;
+  using namespace lvb::fa2;
+  if (T <= 0 || (T % (2 * BT)) != 0 || Hq <= 0 || Hkv <= 0 || (Hq % Hkv) != 0 || pos == nullptr || chunk < 0) return kErrBadArg;
+  if (dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || (dk & 7) || (dv & 7) || (ldg & 7) || !(scale > 0.f)) return kErrBadArg;
+  if ((reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(o) & 15)) return kErrBadArg;
+  Params p;
+  p.O = reinterpret_cast<__nv_bfloat16*>(o);
+  p.lse2 = nullptr; p.q_seg = nullptr; p.k_seg = nullptr; p.kblock_lo = nullptr; p.sink = nullptr;
+  p.B = 1; p.S = T; p.Sk = T; p.Hq = Hq; p.Hkv = Hkv;
+  p.scale = scale; p.soft_cap = soft_cap; p.window = 0; p.causal = 1; p.status = status;
+  p.pos = pos; p.chunk = chunk; p.dk = dk; p.dv = dv;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  CUtensorMap tmQ, tmK, tmV;
+  int rc = make_tmap_heads_bf16(&tmQ, q, T, Hq, dk, ldq, BT);
+  if (rc == kErrOk) rc = make_tmap_heads_bf16(&tmK, k, T, Hkv, dk, ldk, BT);
+  if (rc == kErrOk) rc = make_tmap_heads_bf16(&tmV, v, T, Hkv, dv, ldv, BT);
+  if (rc != kErrOk) return rc;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const bool small = dk <= 64 && dv <= 64;
+  if (soft_cap > 0.f)
+    return small ? launch<64, false, true, true>(tmQ, tmK, tmV, p, st) : launch<128, false, true, true>(tmQ, tmK, tmV, p, st);
+  return small ? launch<64, false, false, true>(tmQ, tmK, tmV, p, st) : launch<128, false, false, true>(tmQ, tmK, tmV, p, st);
 }

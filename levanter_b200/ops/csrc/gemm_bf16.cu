@@ -37,6 +37,7 @@ enum EpiFlags : int {
   kBias = 4,         // + bias[N] (bf16)
   kResidual = 8,     // + residual[M,N] (bf16, row stride ldr)
   kBiasF32 = 16,     // bias is float
+  kSquaredRelu = 32, // max(v, 0)^2 of the product (after the bias, before residual / accumulate)
 };
 
 struct Params {
@@ -432,6 +433,13 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA_maps, const CUt
 #pragma unroll
               for (int j = 0; j < 32; ++j)
                 if (full || col0 + j < p.N) v[j] += __bfloat162float(b[j]);
+            }
+          }
+          if (p.flags & kSquaredRelu) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              const float a = fmaxf(v[j], 0.f);
+              v[j] = a * a;
             }
           }
           if (p.flags & kResidual) {
@@ -1252,7 +1260,7 @@ int launch_grouped(const void* A, const void* B, Params p, int a_rows, int a_col
 // tile_group: int32[ceil(Tp / 128)], the group of every 128-row block of A, -1 beyond the last group (kinds 0 and 1).
 // offsets:    int32[groups + 1], padded row offsets (multiples of 128) of the groups (kind 2).
 // For kinds 0 and 1, Tp is the static capacity of the padded buffer; blocks marked -1 are neither read nor written.
-// flags as lvb_gemm_bf16 (kOutF32, kAccumulate); M, N multiples of 8; for kind 2 M must be a multiple of 128.
+// flags as lvb_gemm_bf16 (kOutF32, kAccumulate, kSquaredRelu); M, N multiples of 8; for kind 2 M must be a multiple of 128.
 extern "C" int lvb_gemm_grouped(int kind, const void* A, const void* B, void* C, int groups, int Tp, int M, int N, int K, int lda,
                                 int ldb, int ldc, int flags, float alpha, const int* tile_group, const int* offsets, int* status,
                                 void* stream) {
@@ -1262,7 +1270,7 @@ extern "C" int lvb_gemm_grouped(int kind, const void* A, const void* B, void* C,
   Params p;
   p.C = C; p.bias = nullptr; p.residual = nullptr;
   p.ldc = ldc; p.ldr = 0;
-  p.flags = flags & (kOutF32 | kAccumulate); p.alpha = alpha; p.status = status; p.alpha_dev = nullptr;
+  p.flags = flags & (kOutF32 | kAccumulate | kSquaredRelu); p.alpha = alpha; p.status = status; p.alpha_dev = nullptr;
   p.a_fmt = p.b_fmt = 0;
   p.rank = 0; p.world = 1; p.m_rot = 0;
   p.a_rows_per_map = 0; p.c_rows_per_rank = 0;

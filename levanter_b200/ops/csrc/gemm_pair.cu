@@ -40,7 +40,7 @@ constexpr int kNumThreads = 192;  // warp0 TMA, warp1 MMA (leader) / TMEM alloca
 constexpr uint32_t kLeaderMask = 0xFEFFFFFFu;  // clears the CTA-rank bit of a shared-memory address: the leader's copy
 constexpr int kMaxPeers = 8;
 
-enum EpiFlags : int { kOutF32 = 1, kAccumulate = 2, kBias = 4, kResidual = 8, kBiasF32 = 16 };
+enum EpiFlags : int { kOutF32 = 1, kAccumulate = 2, kBias = 4, kResidual = 8, kBiasF32 = 16, kSquaredRelu = 32 };
 
 struct Params {
   void* C;
@@ -395,6 +395,13 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap& tmA, const CUt
                 if (full || col0 + j < p.N) v[j] += __bfloat162float(b[j]);
             }
           }
+          if (p.flags & kSquaredRelu) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              const float a = fmaxf(v[j], 0.f);
+              v[j] = a * a;
+            }
+          }
           if (p.flags & kResidual) {
             const __nv_bfloat16* rr = p.residual + static_cast<size_t>(row) * p.ldr + col0;
             if (full && (p.ldr & 7) == 0) {
@@ -710,7 +717,7 @@ int launch(const void* A, const void* B, Params p, int lda, int ldb, cudaStream_
     if (sp > 8) sp = 8;
     p.splits = sp < 1 ? 1 : sp;
   }
-  if (p.ws == nullptr || (p.N & 3) || (p.flags & kAccumulate)) p.splits = 1;
+  if (p.ws == nullptr || (p.N & 3)) p.splits = 1;
   if (p.splits > k_blocks) p.splits = k_blocks;
   p.kb_per_split = (k_blocks + p.splits - 1) / p.splits;
   p.splits = (k_blocks + p.kb_per_split - 1) / p.kb_per_split;  // no empty split
@@ -752,7 +759,7 @@ extern "C" int lvb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, 
 
 // lvb_gemm_bf16_pair for K-major operands with K split over `splits` CTA pairs per tile (0: chosen by the launcher so that about
 // every SM pair gets a piece; at most 8).  `workspace`: lvb_gemm_skinny_workspace_bytes(M, N) bytes of device memory, contents
-// irrelevant.  N % 4 == 0 and no accumulate flag, else one split is used.  The partial tiles are summed in a fixed order.
+// irrelevant.  N % 4 == 0, else one split is used.  The partial tiles are summed in a fixed order.
 extern "C" int lvb_gemm_bf16_pair_splitk(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int flags,
                                          float alpha, const void* bias, const void* residual, int ldr, int splits, void* workspace,
                                          int* status, void* stream) {

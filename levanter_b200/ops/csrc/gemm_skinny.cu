@@ -35,7 +35,7 @@ constexpr int kThreads = 192;
 constexpr int kMaxStages = 24;
 constexpr int kSmemBudget = 200 * 1024;  // ring bytes; the rest of the 227 KB holds barriers, slack and alignment
 
-enum Flags : int { kOutF32 = 1, kBias = 4, kResidual = 8, kBiasF32 = 16 };
+enum Flags : int { kOutF32 = 1, kAccumulate = 2, kBias = 4, kResidual = 8, kBiasF32 = 16, kSquaredRelu = 32 };
 
 struct Params {
   void* C;
@@ -53,9 +53,13 @@ struct Params {
   int kb_per_split;  // k-blocks per split
   float* ws;         // splits > 1: fp32 partials [splits, M, N]
   int* status;
+  // grouped form: row block b (block_rows rows of A, at most 128) multiplies B's rows [g * N, (g + 1) * N) with g = tile_group[b];
+  // blocks with g < 0 are skipped
+  const int* tile_group;
+  int block_rows;
 };
 
-template <int BN, int kAcc>
+template <int BN, int kAcc, bool kGrouped>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, Params p) {
   constexpr int kBBytes = BN * BK * 2;
@@ -108,9 +112,14 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
       uint32_t phase = 0;
       bool ok = true;
       for (int t = blockIdx.x; t < num_work && ok; t += gridDim.x) {
-        const int m0 = (t % p.tiles_m) * BM;
+        const int m0 = (t % p.tiles_m) * (kGrouped ? p.block_rows : BM);
         const int u = t / p.tiles_m;
-        const int n0 = (u / p.splits) * BN;
+        int n0 = (u / p.splits) * BN;
+        if constexpr (kGrouped) {
+          const int g = p.tile_group[t % p.tiles_m];
+          if (g < 0) continue;
+          n0 += g * p.N;
+        }
         const int kb0 = (u % p.splits) * p.kb_per_split;
         const int kb1 = min(k_blocks, kb0 + p.kb_per_split);
         for (int kb = kb0; kb < kb1; ++kb) {
@@ -133,6 +142,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
       uint32_t tphase = 0;
       bool ok = true;
       for (int t = blockIdx.x; t < num_work && ok; t += gridDim.x) {
+        if (kGrouped && p.tile_group[t % p.tiles_m] < 0) continue;
         ok = mbar_wait(&tempty_bar[buf], tphase ^ 1, abort_flag, p.status, 200, buf);
         if (!ok) break;
         tc_fence_after();
@@ -164,11 +174,13 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
     bool ok = true;
     const bool out_f32 = (p.flags & kOutF32) != 0;
     for (int t = blockIdx.x; t < num_work && ok; t += gridDim.x) {
+      if (kGrouped && p.tile_group[t % p.tiles_m] < 0) continue;
       ok = mbar_wait(&tfull_bar[buf], tphase, abort_flag, p.status, 300, buf);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int m0 = (t % p.tiles_m) * BM;
+      const int m0 = (t % p.tiles_m) * (kGrouped ? p.block_rows : BM);
+      const int m_end = kGrouped ? m0 + p.block_rows : p.M;
       const int u = t / p.tiles_m;
       const int n0 = (u / p.splits) * BN;
       const int split = u % p.splits;
@@ -178,7 +190,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + buf * kAcc * BN;
       const int n_acc = n_kb < kAcc ? n_kb : kAcc;  // accumulators that were written for this piece of work
       // warps whose 32 rows are all beyond M still take part in the barrier protocol but skip the loads
-      const bool warp_has_rows = m0 + quad * 32 < p.M;
+      const bool warp_has_rows = m0 + quad * 32 < m_end;
 #pragma unroll 1
       for (int c = 0; c < BN && warp_has_rows; c += 32) {
         float v[32];
@@ -207,7 +219,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
           }
           continue;
         }
-        if (row < p.M && col0 < p.N) {
+        if (row < m_end && col0 < p.N) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] *= p.alpha;
           const bool full = (col0 + 32 <= p.N);
@@ -224,11 +236,31 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
                 if (full || col0 + j < p.N) v[j] += __bfloat162float(b[j]);
             }
           }
+          if (p.flags & kSquaredRelu) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              const float a = fmaxf(v[j], 0.f);
+              v[j] = a * a;
+            }
+          }
           if (p.flags & kResidual) {
             const __nv_bfloat16* rr = p.residual + static_cast<size_t>(row) * p.ldr + col0;
 #pragma unroll
             for (int j = 0; j < 32; ++j)
               if (full || col0 + j < p.N) v[j] += __bfloat162float(rr[j]);
+          }
+          if (p.flags & kAccumulate) {
+            if (out_f32) {
+              const float* cr = reinterpret_cast<const float*>(p.C) + static_cast<size_t>(row) * p.ldc + col0;
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (full || col0 + j < p.N) v[j] += cr[j];
+            } else {
+              const __nv_bfloat16* cr = reinterpret_cast<const __nv_bfloat16*>(p.C) + static_cast<size_t>(row) * p.ldc + col0;
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (full || col0 + j < p.N) v[j] += __bfloat162float(cr[j]);
+            }
           }
           if (out_f32) {
             float* cp = reinterpret_cast<float*>(p.C) + static_cast<size_t>(row) * p.ldc + col0;
@@ -297,6 +329,13 @@ __global__ void splitk_finalize_kernel(const float* __restrict__ ws, int splits,
       for (int j = 0; j < 4; ++j)
         o[j] += (flags & kBiasF32) ? reinterpret_cast<const float*>(bias)[n + j] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(bias)[n + j]);
     }
+    if (flags & kSquaredRelu) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float a = fmaxf(o[j], 0.f);
+        o[j] = a * a;
+      }
+    }
     if (flags & kResidual) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) o[j] += __bfloat162float(residual[static_cast<size_t>(m) * ldr + n + j]);
@@ -304,20 +343,20 @@ __global__ void splitk_finalize_kernel(const float* __restrict__ ws, int splits,
     if (flags & kOutF32) {
       float* cp = reinterpret_cast<float*>(C) + static_cast<size_t>(m) * ldc + n;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) cp[j] = o[j];
+      for (int j = 0; j < 4; ++j) cp[j] = (flags & kAccumulate) ? cp[j] + o[j] : o[j];
     } else {
       __nv_bfloat16* cp = reinterpret_cast<__nv_bfloat16*>(C) + static_cast<size_t>(m) * ldc + n;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) cp[j] = __float2bfloat16(o[j]);
+      for (int j = 0; j < 4; ++j) cp[j] = __float2bfloat16((flags & kAccumulate) ? __bfloat162float(cp[j]) + o[j] : o[j]);
     }
   }
 }
 
-template <int BN, int kAcc>
-int launch(const void* A, const void* B, Params p, int lda, int ldb, cudaStream_t stream) {
+template <int BN, int kAcc, bool kGrouped = false>
+int launch(const void* A, const void* B, Params p, int lda, int ldb, cudaStream_t stream, int groups = 1) {
   constexpr int kBBytes = BN * BK * 2;
-  p.tiles_m = (p.M + BM - 1) / BM;
-  const int a_rows = p.tiles_m > 1 ? BM : ((p.M + 7) / 8) * 8;  // rows past M in the last block are zero-filled by TMA
+  p.tiles_m = kGrouped ? p.M / p.block_rows : (p.M + BM - 1) / BM;
+  const int a_rows = kGrouped ? p.block_rows : p.tiles_m > 1 ? BM : ((p.M + 7) / 8) * 8;  // rows past M in the last block are zero-filled by TMA
   p.a_bytes = a_rows * BK * 2;
   const int stride = p.a_bytes + kBBytes;
   int stages = kSmemBudget / stride;
@@ -334,9 +373,9 @@ int launch(const void* A, const void* B, Params p, int lda, int ldb, cudaStream_
   CUtensorMap tmA, tmB;
   int rc = make_tmap_2d_bf16(&tmA, A, p.M, p.K, lda, a_rows, BK);
   if (rc != kErrOk) return rc;
-  rc = make_tmap_2d_bf16(&tmB, B, p.N, p.K, ldb, BN, BK);
+  rc = make_tmap_2d_bf16(&tmB, B, static_cast<uint64_t>(groups) * p.N, p.K, ldb, BN, BK);
   if (rc != kErrOk) return rc;
-  auto kern = gemm_skinny_kernel<BN, kAcc>;
+  auto kern = gemm_skinny_kernel<BN, kAcc, kGrouped>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448) != cudaSuccess) return kErrCuda;
@@ -371,7 +410,7 @@ int launch_splitk_finalize(const float* ws, int splits, int M, int N, float alph
 extern "C" long long lvb_gemm_skinny_workspace_bytes(int M, int N) { return 8LL * M * N * 4; }
 
 // C[M,N] = alpha * A[M,K] B[N,K]^T (+ bias) (+ residual) for M <= 512.  flags: 1 = fp32 output, 4 = bias, 16 = bias is fp32,
-// 8 = residual (bf16 [M, N], row stride ldr).  bn: tile width (32, 64 or 128), or 0 to let the launcher choose.
+// 8 = residual (bf16 [M, N], row stride ldr), 32 = squared relu of the product, 2 = add to what C holds.  bn: tile width (32, 64 or 128), or 0 to let the launcher choose.
 // splits: CTAs per column tile along K, or 0 to let the launcher choose; more than one needs `workspace`
 // (lvb_gemm_skinny_workspace_bytes(M, N) bytes of device memory, contents irrelevant) and N % 4 == 0, else 1 is used.
 extern "C" int lvb_gemm_skinny(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int flags,
@@ -399,8 +438,32 @@ extern "C" int lvb_gemm_skinny(const void* A, const void* B, void* C, int M, int
   }
   if (workspace == nullptr || (N & 3)) splits = 1;
   p.splits = splits;
+  p.tile_group = nullptr; p.block_rows = 0;
   if (bn == 128) return skinny::launch<128, 2>(A, B, p, lda, ldb, s);
   if (bn == 64) return skinny::launch<64, 4>(A, B, p, lda, ldb, s);
   if (bn == 32) return skinny::launch<32, 8>(A, B, p, lda, ldb, s);
   return kErrBadArg;
+}
+
+// The weight-streaming form of lvb_gemm_grouped (kind 0) for a few rows per group: C[Tp, N] = A[Tp, K] B[g][N, K]^T where the rows of
+// A are sorted by group and every group's segment is padded to a multiple of `block_rows` (a multiple of 8, at most 128).
+// tile_group: int32[Tp / block_rows], the group of every row block, -1 for blocks past the last group (neither read nor written).
+// flags: 1 = fp32 output, 2 = add to C, 32 = squared relu.  K and ldb multiples of 8.
+extern "C" int lvb_gemm_skinny_grouped(const void* A, const void* B, void* C, int groups, int Tp, int block_rows, int N, int K, int lda,
+                                       int ldb, int ldc, int flags, float alpha, const int* tile_group, int* status, void* stream) {
+  using namespace lvb;
+  using namespace lvb::skinny;
+  if (groups <= 0 || Tp <= 0 || block_rows <= 0 || block_rows > BM || (block_rows & 7) || Tp % block_rows != 0 || N <= 0 || K <= 0 ||
+      (lda & 7) || (ldb & 7) || tile_group == nullptr)
+    return kErrBadArg;
+  Params p;
+  p.C = C; p.bias = nullptr; p.residual = nullptr;
+  p.M = Tp; p.N = N; p.K = K; p.ldc = ldc; p.ldr = 0;
+  p.flags = flags & (kOutF32 | kAccumulate | kSquaredRelu); p.alpha = alpha; p.status = status;
+  p.ws = nullptr; p.splits = 1;
+  p.tile_group = tile_group; p.block_rows = block_rows;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (N >= 96) return skinny::launch<128, 2, true>(A, B, p, lda, ldb, s, groups);
+  if (N > 32) return skinny::launch<64, 4, true>(A, B, p, lda, ldb, s, groups);
+  return skinny::launch<32, 8, true>(A, B, p, lda, ldb, s, groups);
 }

@@ -76,7 +76,20 @@ struct Params {
   float* part_ml;                 // [T, H, parts, 2]
   int T, H, KV, S, pages_per_seq, page_size, num_pages, parts;
   float scale, soft_cap;
+  // ---- general form (lvb_paged_attention_general); the plain entry point sets dk = dv = D, chunk = 0, no gate
+  int dk, dv;                 // query/key and value sizes; a cache slot holds, per KV head, dk key and dv value elements
+  int chunk;                  // > 0: a query at position i sees positions >= i - i % chunk only
+  long long ldq, ldg;         // row strides of q and gate
+  const __nv_bfloat16* gate;  // optional [T, H * dv]: the output is multiplied by its sigmoid
 };
+
+// First visible key of a query whose context (its position + 1) is ctx.
+__device__ __forceinline__ int first_key(const Params& p, int ctx) { return p.chunk > 0 ? ctx - 1 - (ctx - 1) % p.chunk : 0; }
+
+__device__ __forceinline__ float gate_factor(const Params& p, int t, int h, int d) {
+  if (p.gate == nullptr) return 1.f;
+  return 1.f / (1.f + __expf(-__bfloat162float(p.gate[t * p.ldg + static_cast<long long>(h) * p.dv + d])));
+}
 
 // Which sequence owns packed token t, and how many keys it may attend to.  Returns false for padding tokens.
 __device__ __forceinline__ bool locate(const Params& p, int t, int& seq, int& ctx) {
@@ -437,7 +450,9 @@ __global__ void __launch_bounds__(kThreads) paged_attention_staged_kernel(Params
   }
 }
 
-// Tensor-core variant for D = 128 and at most 16 query heads per KV head.  The query heads that share a KV head are the M rows
+// Tensor-core variant for at most 16 query heads per KV head.  DKC / DVC: room for the query/key and the value size; kExact: the
+// sizes are exactly those (D = 128, the form Llama decodes with), otherwise they are p.dk <= DKC and p.dv <= DVC (multiples of 8)
+// and the loops stop at the next multiple of 16.  The query heads that share a KV head are the M rows
 // of warp-level MMAs (m16n8k16, bf16, fp32 accumulation; rows beyond G are zero), so one pass over a key's K and V rows
 // serves all of them at a sixteenth of the instruction count of the scalar kernels, which were bound by instruction issue
 // and shared-memory reads, not by the cache traffic.  Each of the four warps owns 64 keys of the partition and is its own
@@ -447,9 +462,14 @@ __global__ void __launch_bounds__(kThreads) paged_attention_staged_kernel(Params
 // P is re-packed in registers as the A operand of O += P V (V rows through ldmatrix.trans), and the four warps' (max, sum,
 // O) are merged through shared memory at the end.
 constexpr int kMmaStageKeys = 16;
-constexpr int kMmaRowBytes = 528;  // K (256 B) + V (256 B) + 16 B padding
 constexpr int kMmaWarpKeys = kPart / (kThreads / 32);  // 64
-constexpr int kMmaStageBytes = kMmaStageKeys * kMmaRowBytes;
+template <int DKC, int DVC>
+struct MmaLayout {
+  static_assert((DKC + DVC) % 64 == 0, "row stride modulo 128 bytes must be 16");
+  static constexpr int kRowBytes = (DKC + DVC) * 2 + 16;  // K, V, 16 B padding
+  static constexpr int kStageBytes = kMmaStageKeys * kRowBytes;
+  static constexpr int kSmem = 4 * 2 * kStageBytes + kPart * 4 + 4 * 16 * 2 * 4;
+};
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -463,23 +483,27 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4],
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+template <int DKC, int DVC, bool kExact>
 __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p) {
-  constexpr int D = 128;
+  using L = MmaLayout<DKC, DVC>;
+  constexpr int kMmaRowBytes = L::kRowBytes, kMmaStageBytes = L::kStageBytes;
+  const int dk = kExact ? DKC : p.dk, dv = kExact ? DVC : p.dv;
+  const int dk16 = (dk + 15) & ~15;
   const int t = blockIdx.x, kvh = blockIdx.y, part = blockIdx.z;
   const int G = p.H / p.KV;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   extern __shared__ __align__(16) uint8_t s_dyn[];
-  uint8_t* s_stage = s_dyn;                                   // [4 warps][2 stages][16 keys][528 B] = 67584 B; reused for the merge
+  uint8_t* s_stage = s_dyn;                                   // [4 warps][2 stages][16 keys][row]; reused for the merge
   int* s_rows = reinterpret_cast<int*>(s_dyn + 4 * 2 * kMmaStageBytes);  // [kPart]
   float* s_ml = reinterpret_cast<float*>(s_rows + kPart);     // [4 warps][16 rows][2]
 
   int seq = 0, ctx = 0;
   const bool live = locate(p, t, seq, ctx);
-  const int k0 = part * kPart;
+  const int k0 = (live ? first_key(p, ctx) : 0) + part * kPart;
   if (!live || k0 >= ctx) {
     if (part == 0 && !live) {
-      for (int i = threadIdx.x; i < G * D; i += kThreads)
-        p.out[(static_cast<long long>(t) * p.H + kvh * G) * D + i] = __float2bfloat16(0.f);
+      for (int i = threadIdx.x; i < G * dv; i += kThreads)
+        p.out[(static_cast<long long>(t) * p.H + kvh * G) * dv + i] = __float2bfloat16(0.f);
     }
     return;
   }
@@ -495,44 +519,54 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
   }
   __syncthreads();
 
-  // ---- Q as A fragments (rows = query heads of this KV head, zero beyond G): 8 k-steps of 16 dimensions
+  // ---- Q as A fragments (rows = query heads of this KV head, zero beyond G): k-steps of 16 dimensions
   const int row_lo = lane >> 2, row_hi = row_lo + 8, kq = (lane & 3) * 2;
-  uint32_t qa[8][4];
+  uint32_t qa[DKC / 16][4];
   {
-    const __nv_bfloat16* qbase = p.q + (static_cast<long long>(t) * p.H + kvh * G) * D;
+    const __nv_bfloat16* qbase = p.q + t * p.ldq + static_cast<long long>(kvh) * G * dk;
 #pragma unroll
-    for (int ks = 0; ks < 8; ++ks) {
+    for (int ks = 0; ks < DKC / 16; ++ks) {
       const int d0 = ks * 16 + kq;
-      qa[ks][0] = row_lo < G ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * D + d0) : 0u;
-      qa[ks][1] = row_hi < G ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * D + d0) : 0u;
-      qa[ks][2] = row_lo < G ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * D + d0 + 8) : 0u;
-      qa[ks][3] = row_hi < G ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * D + d0 + 8) : 0u;
+      const bool in0 = kExact || d0 < dk, in1 = kExact || d0 + 8 < dk;
+      qa[ks][0] = row_lo < G && in0 ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * dk + d0) : 0u;
+      qa[ks][1] = row_hi < G && in0 ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * dk + d0) : 0u;
+      qa[ks][2] = row_lo < G && in1 ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * dk + d0 + 8) : 0u;
+      qa[ks][3] = row_hi < G && in1 ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * dk + d0 + 8) : 0u;
     }
   }
 
-  const long long tok_stride = 2LL * p.KV * D;
+  const long long tok_stride = static_cast<long long>(p.KV) * (dk + dv);
   const int wk0 = warp * kMmaWarpKeys;                       // this warp's first key inside the partition
   const int wnk = max(0, min(kMmaWarpKeys, nk - wk0));       // and how many of its 64 are real
   const int stages = (wnk + kMmaStageKeys - 1) / kMmaStageKeys;
   uint8_t* my_stage = s_stage + warp * (2 * kMmaStageBytes);
-  // one stage: 16 rows x 32 chunks of 16 bytes, 16 per lane; rows without a key are zero-filled (0 * NaN would poison O)
+  // one stage: 16 rows of 16-byte pieces; rows without a key are zero-filled (0 * NaN would poison O), and so are the columns
+  // between a size and the next multiple of 16
   auto issue = [&](int st) {
     uint8_t* dst = my_stage + (st & 1) * kMmaStageBytes;
 #pragma unroll 4
-    for (int c = lane; c < kMmaStageKeys * 32; c += 32) {
-      const int r = c >> 5, ch = c & 31;
+    for (int c = lane; c < kMmaStageKeys * ((DKC + DVC) / 8); c += 32) {
+      const int r = c / ((DKC + DVC) / 8), ch = c % ((DKC + DVC) / 8);
       const int i = wk0 + st * kMmaStageKeys + r;
       const int slot = (st * kMmaStageKeys + r < wnk) ? s_rows[i] : -1;
       uint8_t* d = dst + r * kMmaRowBytes + ch * 16;
-      if (slot >= 0) cp_async_16(d, p.kv_pages + slot * tok_stride + (2LL * kvh) * D + ch * 8);
-      else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+      const __nv_bfloat16* src = p.kv_pages + slot * tok_stride + static_cast<long long>(kvh) * (dk + dv);
+      if constexpr (kExact) {
+        if (slot >= 0) cp_async_16(d, src + ch * 8);
+        else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+      } else {
+        const int col = ch < DKC / 8 ? ch * 8 : ch * 8 - DKC;  // column of the key or value row
+        const int size = ch < DKC / 8 ? dk : dv;
+        if (slot >= 0 && col < size) cp_async_16(d, src + (ch < DKC / 8 ? col : dk + col));
+        else if (col < ((size + 15) & ~15)) *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
 
-  float o[16][4];
+  float o[DVC / 8][4];
 #pragma unroll
-  for (int n = 0; n < 16; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+  for (int n = 0; n < DVC / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;  // running max / sum of rows row_lo and row_hi
   const float sc_log2 = p.scale * 1.4426950408889634f;
 
@@ -549,12 +583,13 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     for (int j = 0; j < 2; ++j) {
       sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f;
 #pragma unroll
-      for (int kp = 0; kp < 4; ++kp) {  // 32 dimensions per ldmatrix.x4: matrices (d 0-7), (8-15), (16-23), (24-31) of the 8 keys
+      for (int kp = 0; kp < DKC / 32; ++kp) {  // 32 dimensions per ldmatrix.x4: matrices (d 0-7), (8-15), (16-23), (24-31) of the 8 keys
+        if (!kExact && kp * 32 >= dk16) break;
         uint32_t b0, b1, b2, b3;
         const uint32_t addr = buf + (8 * j + (lane & 7)) * kMmaRowBytes + (kp * 32 + (lane >> 3) * 8) * 2;
         ldmatrix_x4(addr, b0, b1, b2, b3);
         mma_16816(sacc[j], qa[2 * kp], b0, b1);
-        mma_16816(sacc[j], qa[2 * kp + 1], b2, b3);
+        if (kExact || kp * 32 + 16 < dk16) mma_16816(sacc[j], qa[2 * kp + 1], b2, b3);
       }
     }
     // ---- online softmax on the fragments: this lane holds keys (lane % 4) * 2 + {0, 1} of each n-tile, rows row_lo / row_hi
@@ -606,13 +641,14 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     l_hi = l_hi * a_hi + sum_hi;
     m_lo = mn_lo;
     m_hi = mn_hi;
-    // ---- O[16 heads, 128 d] = O * alpha + P V: pairs of 8-wide d tiles per ldmatrix.x4.trans
+    // ---- O[16 heads, dv] = O * alpha + P V: pairs of 8-wide d tiles per ldmatrix.x4.trans
 #pragma unroll
-    for (int np = 0; np < 8; ++np) {
+    for (int np = 0; np < DVC / 16; ++np) {
+      if (!kExact && np * 16 >= dv) break;
       uint32_t b0, b1, b2, b3;
       // matrices: (keys 0-7, d 16 np .. +7), (keys 8-15, same d), (keys 0-7, d 16 np + 8 ..), (keys 8-15, same)
       const int mi = lane >> 3;
-      const uint32_t addr = buf + ((mi & 1) * 8 + (lane & 7)) * kMmaRowBytes + 256 + (np * 16 + (mi >> 1) * 8) * 2;
+      const uint32_t addr = buf + ((mi & 1) * 8 + (lane & 7)) * kMmaRowBytes + DKC * 2 + (np * 16 + (mi >> 1) * 8) * 2;
       ldmatrix_x4_trans(addr, b0, b1, b2, b3);
       float* oa = o[2 * np];
       float* ob = o[2 * np + 1];
@@ -633,16 +669,16 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     s_ml[(warp * 16 + row_hi) * 2 + 0] = m_hi;
     s_ml[(warp * 16 + row_hi) * 2 + 1] = l_hi;
   }
-  float* s_o = reinterpret_cast<float*>(s_stage);  // [4 warps][16 rows][128] fp32 = 32 KB
+  float* s_o = reinterpret_cast<float*>(s_stage);  // [4 warps][16 rows][DVC] fp32
 #pragma unroll
-  for (int n = 0; n < 16; ++n) {
+  for (int n = 0; n < DVC / 8; ++n) {
     const int d0 = n * 8 + kq;
-    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_lo) * D + d0) = make_float2(o[n][0], o[n][1]);
-    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_hi) * D + d0) = make_float2(o[n][2], o[n][3]);
+    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_lo) * DVC + d0) = make_float2(o[n][0], o[n][1]);
+    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_hi) * DVC + d0) = make_float2(o[n][2], o[n][3]);
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < G * D; idx += kThreads) {
-    const int g = idx / D, d = idx - g * D;
+  for (int idx = threadIdx.x; idx < G * dv; idx += kThreads) {
+    const int g = idx / dv, d = idx - g * dv;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, s_ml[(w * 16 + g) * 2]);
@@ -651,14 +687,14 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     for (int w = 0; w < 4; ++w) {
       const float mw = s_ml[(w * 16 + g) * 2];
       const float f = (mw == -INFINITY) ? 0.f : exp2f(mw - m);
-      acc = fmaf(s_o[(w * 16 + g) * D + d], f, acc);
+      acc = fmaf(s_o[(w * 16 + g) * DVC + d], f, acc);
       l = fmaf(s_ml[(w * 16 + g) * 2 + 1], f, l);
     }
     const long long hrow = static_cast<long long>(t) * p.H + kvh * G + g;
     if (p.parts == 1) {
-      p.out[hrow * D + d] = __float2bfloat16(l > 0.f ? acc / l : 0.f);
+      p.out[hrow * dv + d] = __float2bfloat16(l > 0.f ? acc / l * gate_factor(p, t, kvh * G + g, d) : 0.f);
     } else {
-      p.part_o[(hrow * p.parts + part) * D + d] = acc;
+      p.part_o[(hrow * p.parts + part) * dv + d] = acc;
       if (d == 0) {
         // the merge kernel works with natural-log maxima: this kernel's are in base 2
         p.part_ml[(hrow * p.parts + part) * 2 + 0] = (m == -INFINITY) ? -INFINITY : m * 0.6931471805599453f;
@@ -667,15 +703,16 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     }
   }
 }
-constexpr int kMmaSmem = 4 * 2 * kMmaStageBytes + kPart * 4 + 4 * 16 * 2 * 4;
 
 // One CTA per (token, head): merge the partials of the partitions that were live for this token.
-template <int D>
-__global__ void __launch_bounds__(D <= 128 ? 128 : 256) paged_merge_kernel(Params p) {
+// kThreadsM: threads per CTA, a stride over the p.dv output dimensions.
+template <int kThreadsM>
+__global__ void __launch_bounds__(kThreadsM) paged_merge_kernel(Params p) {
+  const int D = p.dv;
   const int t = blockIdx.x, h = blockIdx.y;
   int seq = 0, ctx = 0;
   if (!locate(p, t, seq, ctx)) return;  // zeros were written by the attention kernel
-  const int np = (ctx + kPart - 1) / kPart;
+  const int np = (ctx - first_key(p, ctx) + kPart - 1) / kPart;
   const long long hrow = static_cast<long long>(t) * p.H + h;
   float m = -INFINITY;
   for (int i = 0; i < np; ++i) m = fmaxf(m, p.part_ml[(hrow * p.parts + i) * 2]);
@@ -691,7 +728,7 @@ __global__ void __launch_bounds__(D <= 128 ? 128 : 256) paged_merge_kernel(Param
       if (mi == -INFINITY) continue;
       o = fmaf(p.part_o[(hrow * p.parts + i) * D + d], __expf(mi - m), o);
     }
-    p.out[hrow * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+    p.out[hrow * D + d] = __float2bfloat16(l > 0.f ? o / l * gate_factor(p, t, h, d) : 0.f);
   }
 }
 
@@ -707,24 +744,40 @@ inline int paged_variant() {
   return v;
 }
 
+template <int DKC, int DVC, bool kExact>
+int launch_mma(const Params& p, cudaStream_t s) {
+  constexpr int smem = MmaLayout<DKC, DVC>::kSmem;
+  auto kern = paged_attention_mma_kernel<DKC, DVC, kExact>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return kErrCuda;
+    attr_set = true;
+  }
+  kern<<<dim3(p.T, p.KV, p.parts), kThreads, smem, s>>>(p);
+  return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+}
+
+int launch_merge(const Params& p, cudaStream_t s) {
+  if (p.parts > 1) {
+    if (p.dv <= 128) paged_merge_kernel<128><<<dim3(p.T, p.H), 128, 0, s>>>(p);
+    else paged_merge_kernel<256><<<dim3(p.T, p.H), 256, 0, s>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+}
+
 template <int D>
 int launch(const Params& p, cudaStream_t s) {
   dim3 grid(p.T, p.KV, p.parts);
   const int variant = paged_variant();
   if (D == 128 && p.H / p.KV <= 16 && variant == 2) {
-    static bool attr_set = false;
-    if (!attr_set) {
-      if (cudaFuncSetAttribute(paged_attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaSmem) != cudaSuccess) return kErrCuda;
-      attr_set = true;
-    }
-    paged_attention_mma_kernel<<<grid, kThreads, kMmaSmem, s>>>(p);
+    const int rc = launch_mma<128, 128, true>(p, s);
+    if (rc != kErrOk) return rc;
   } else if (D == 128 && p.H / p.KV <= kStagedMaxG && variant >= 1) {
     paged_attention_staged_kernel<<<grid, kThreads, 0, s>>>(p);
   } else {
     paged_attention_kernel<D><<<grid, kThreads, 0, s>>>(p);
   }
-  if (p.parts > 1) paged_merge_kernel<D><<<dim3(p.T, p.H), D <= 128 ? 128 : 256, 0, s>>>(p);
-  return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+  return launch_merge(p, s);
 }
 
 }  // namespace paged
@@ -764,6 +817,7 @@ extern "C" int lvb_paged_attention(const void* q, const void* kv_pages, const in
   p.T = T; p.H = H; p.KV = KV; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;
   p.parts = lvb_paged_attention_parts(pages_per_seq * page_size);
   p.scale = scale; p.soft_cap = soft_cap;
+  p.dk = p.dv = D; p.chunk = 0; p.ldq = static_cast<long long>(H) * D; p.gate = nullptr; p.ldg = 0;
   if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (D) {
@@ -772,4 +826,47 @@ extern "C" int lvb_paged_attention(const void* q, const void* kv_pages, const in
     case 256: return launch<256>(p, s);
     default: return kErrBadArg;
   }
+}
+
+// Partitions of keys per query of lvb_paged_attention_general: sizes part_o fp32 [T, H, parts, dv] and part_ml fp32 [T, H, parts, 2].
+extern "C" int lvb_paged_attention_general_parts(int max_context, int chunk) {
+  const int keys = chunk > 0 && chunk < max_context ? chunk : max_context;
+  return (keys + lvb::paged::kPart - 1) / lvb::paged::kPart;
+}
+
+// lvb_paged_attention for any key and value size up to 256 (multiples of 8), with
+//   * kv_pages [num_pages, page_size, KV, dk + dv]: a key row followed by a value row per KV head,
+//   * chunk > 0: positions are cut into chunks of that many, counted from the sequence's start, and a query sees its own chunk,
+//   * gate (optional, [T, H * dv], row stride ldg): the output is multiplied by its sigmoid,
+//   * ldq: row stride of q.  At most 16 query heads per KV head.
+extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices,
+                                           const int* cu_q_lens, const int* num_seqs, const void* gate, void* out, float* part_o,
+                                           float* part_ml, int T, int H, int KV, int dk, int dv, int ldq, int ldg, int S,
+                                           int pages_per_seq, int page_size, int num_pages, int chunk, float scale, float soft_cap,
+                                           void* stream) {
+  using namespace lvb;
+  using namespace lvb::paged;
+  if (T <= 0) return kErrOk;
+  if (H <= 0 || KV <= 0 || H % KV != 0 || H / KV > kMaxG || S <= 0 || chunk < 0) return kErrBadArg;
+  if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || (dk & 7) || (dv & 7) || (ldq & 1)) return kErrBadArg;
+  Params p;
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  p.kv_pages = reinterpret_cast<const __nv_bfloat16*>(kv_pages);
+  p.kv_lens = kv_lens; p.page_indices = page_indices; p.cu_q_lens = cu_q_lens; p.num_seqs = num_seqs;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.part_o = part_o; p.part_ml = part_ml;
+  p.T = T; p.H = H; p.KV = KV; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;
+  p.parts = lvb_paged_attention_general_parts(pages_per_seq * page_size, chunk);
+  p.scale = scale; p.soft_cap = soft_cap;
+  p.dk = dk; p.dv = dv; p.chunk = chunk; p.ldq = ldq; p.ldg = ldg;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  int rc;
+  if (dk == 128 && dv == 128) rc = launch_mma<128, 128, true>(p, s);
+  else if (dk <= 64 && dv <= 64) rc = launch_mma<64, 64, false>(p, s);
+  else if (dk <= 128 && dv <= 128) rc = launch_mma<128, 128, false>(p, s);
+  else rc = launch_mma<256, 256, false>(p, s);
+  if (rc != kErrOk) return rc;
+  return launch_merge(p, s);
 }

@@ -39,7 +39,47 @@ def supported(q, k, v, mask, bias, no_dropout: bool, attention_dtype) -> bool:
         return False  # different query and key lengths: cross attention only (no causal part); single-token decode steps stay off
     if isinstance(mask, AttentionMask) and not mask.is_causal and mask.sliding_window:
         return False
+    if isinstance(mask, AttentionMask) and mask.chunk_size is not None and q.shape[1] != k.shape[1]:
+        return False
     return _structured_only(mask)
+
+
+_packed = {}
+
+
+def packed_supported(q, k, v, scale: float) -> bool:
+    """Shapes :func:`flash_attention_packed` takes: bf16 rows on a B200, sizes that are multiples of 8 up to 128, a positive scale
+    (the running maximum is taken over unscaled scores) and 16-byte aligned rows."""
+    if not (q.is_cuda and lib.available()) or any(t.dtype != torch.bfloat16 for t in (q, k, v)):
+        return False
+    ok = all(t.shape[2] % 8 == 0 and t.shape[2] <= 128 and t.stride(2) == 1 and t.stride(1) == t.shape[2] and t.stride(0) % 8 == 0
+             and t.data_ptr() % 16 == 0 for t in (q, k, v))
+    return ok and q.shape[0] % 256 == 0 and scale > 0.0
+
+
+def flash_attention_packed(q, k, v, pos, *, scaling_factor: float, chunk: Optional[int] = None, gate=None,
+                           logits_soft_cap: Optional[float] = None) -> torch.Tensor:
+    """Causal attention over packed rows of sequences that start at position 0: ``q [T, Hq, dk]``, ``k [T, Hkv, dk]``, ``v [T, Hkv, dv]``
+    (slices of one wider row are fine), ``pos [T]`` int32 positions with padding rows at 0, ``T`` a multiple of 256 ->
+    ``[T, Hq, dv]``.  ``chunk``: a row sees its own chunk of that many positions only.  ``gate [T, Hq * dv]``: the result is
+    multiplied by its sigmoid.  Forward only; shapes as in :func:`packed_supported`."""
+    c = lib
+    if "f" not in _packed:
+        _packed["f"] = lib.fn("lvb_flash_attn_fwd_packed", [c.c_void_p] * 6 + [c.c_int] * 10 + [c.c_float, c.c_float, c.c_void_p, c.c_void_p])
+    T, Hq, dk = q.shape
+    Hkv, dv = v.shape[1], v.shape[2]
+    pos = pos.to(torch.int32).contiguous()
+    ldg = 0
+    if gate is not None:
+        if gate.dtype != torch.bfloat16 or gate.stride(1) != 1 or gate.stride(0) % 8 != 0 or gate.data_ptr() % 16 != 0:
+            gate = gate.to(torch.bfloat16).contiguous()
+        ldg = gate.stride(0)
+    out = torch.empty(T, Hq, dv, dtype=torch.bfloat16, device=q.device)
+    rc = _packed["f"](q.data_ptr(), k.data_ptr(), v.data_ptr(), lib.ptr(gate), out.data_ptr(), pos.data_ptr(), T, Hq, Hkv, dk, dv, q.stride(0),
+                      k.stride(0), v.stride(0), ldg, int(chunk or 0), float(scaling_factor), float(logits_soft_cap or 0.0),
+                      lib.status_buffer().data_ptr(), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_flash_attn_fwd_packed")
+    return out
 
 
 def flash_attention(q, k, v, mask, *, logits_soft_cap: Optional[float] = None, scaling_factor: Optional[float] = None, sink=None):

@@ -16,6 +16,7 @@ F_ACCUMULATE = 2
 F_BIAS = 4
 F_RESIDUAL = 8
 F_BIAS_F32 = 16
+F_SQUARED_RELU = 32
 
 _gemm_fn = None
 
@@ -41,13 +42,15 @@ def _rowmajor_2d(t: torch.Tensor) -> torch.Tensor:
 
 
 def gemm_reference(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=torch.bfloat16, accumulate=False,
-                   bias=None, residual=None, alpha=1.0):
+                   bias=None, residual=None, alpha=1.0, squared_relu=False):
     """PyTorch fp32 statement of :func:`gemm` (used on CPU and as the test oracle)."""
     af = (a.t() if a_mn else a).float()
     bf = (b if b_mn else b.t()).float()
     c = alpha * (af @ bf)
     if bias is not None:
         c = c + bias.float()
+    if squared_relu:
+        c = torch.relu(c).square()
     if residual is not None:
         c = c + residual.float()
     if out is not None:
@@ -71,15 +74,17 @@ def gemm(
     residual: Optional[torch.Tensor] = None,
     alpha: float = 1.0,
     max_ctas: int = 0,
+    squared_relu: bool = False,
 ) -> torch.Tensor:
-    """``C[M,N] = alpha * op(A) @ op(B)^T (+bias) (+residual) (+C)``.
+    """``C[M,N] = alpha * op(A) @ op(B)^T (+bias) (+residual) (+C)``; ``squared_relu`` applies ``max(., 0)^2`` to the product
+    and bias before the residual and the old ``C`` are added.
 
     ``a`` is ``[M,K]`` (``a_mn=False``) or ``[K,M]`` (``a_mn=True``); ``b`` is ``[N,K]`` or ``[K,N]``.
     Inputs are bf16; the accumulator is fp32; ``out`` may be bf16 or fp32.
     """
     if not (a.is_cuda and lib.available()):
         return gemm_reference(a, b, a_mn=a_mn, b_mn=b_mn, out=out, out_dtype=out_dtype, accumulate=accumulate,
-                              bias=bias, residual=residual, alpha=alpha)
+                              bias=bias, residual=residual, alpha=alpha, squared_relu=squared_relu)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
         raise TypeError("gemm expects bf16 operands")
     a = _rowmajor_2d(a)
@@ -108,6 +113,8 @@ def gemm(
         raise TypeError("out must be bf16 or fp32")
     if accumulate:
         flags |= F_ACCUMULATE
+    if squared_relu:
+        flags |= F_SQUARED_RELU
     if bias is not None:
         flags |= F_BIAS
         if bias.dtype == torch.float32:
@@ -120,7 +127,7 @@ def gemm(
             residual = residual.to(torch.bfloat16).contiguous()
         residual = residual.view(M, N) if residual.dim() != 2 else residual
         ldr = residual.stride(0)
-    if _use_skinny(M, N) and not a_mn and not b_mn and not accumulate and max_ctas == 0:
+    if _use_skinny(M, N) and not a_mn and not b_mn and max_ctas == 0:
         # a few row blocks (decode steps, small batches): the weight-streaming kernel
         rc = _skinny_fn()(
             a.data_ptr(), b.data_ptr(), out.data_ptr(), M, N, K, a.stride(0), b.stride(0), out.stride(0), flags, float(alpha),
@@ -141,7 +148,7 @@ def gemm(
             lib.check_rc(rc, "lvb_gemm_bf16_copy_job")
             return out
     pair = PAIR_ENABLED and N > 128 and M > 128
-    if pair and not a_mn and not b_mn and not accumulate and max_ctas == 0 and _use_pair_splitk(M, N, K):
+    if pair and not a_mn and not b_mn and max_ctas == 0 and _use_pair_splitk(M, N, K):
         rc = _pair_splitk_fn()(
             a.data_ptr(), b.data_ptr(), out.data_ptr(), M, N, K, a.stride(0), b.stride(0), out.stride(0), flags, float(alpha),
             lib.ptr(bias), lib.ptr(residual), ldr, 0, _splitk_workspace(a.device), lib.status_buffer().data_ptr(), lib.stream_ptr(),

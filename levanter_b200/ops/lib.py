@@ -57,13 +57,23 @@ def available() -> bool:
     return major == 10
 
 
+_serving = False
+
+
+def use_serving_library() -> None:
+    """For processes that only serve a model: when the whole library has not been built from the present sources, compile and
+    load the serving subset of it instead (``build.SERVING_SOURCES``).  Call it before the first kernel is needed."""
+    global _serving
+    _serving = not _build.is_current()
+
+
 def load() -> ctypes.CDLL:
     global _lib
     if _lib is not None:
         return _lib
     with _lock:
         if _lib is None:
-            path = _build.lib_path()
+            path = _build.build(serving=True) if _serving else _build.lib_path()
             if not path.exists():
                 path = _build.build()
             _lib = ctypes.CDLL(str(path))

@@ -238,3 +238,129 @@ def moe_route(router_logits: torch.Tensor, k: int):
     if router_logits.is_cuda and lib.available() and E <= 64 and k <= 8:
         return _MoeRoute.apply(router_logits, k)
     return moe_route_reference(router_logits, k)
+
+
+# ------------------------------------------------------------------------------------------------ sigmoid routing within groups
+# Serving form of a mixture whose router scores experts by a sigmoid, chooses by score + correction within the best groups of
+# neighbouring experts, and whose experts are plain (ungated) two-matrix layers.  ``csrc/moe_experts.cu``.
+def route_sigmoid_reference(logits: torch.Tensor, correction, k: int, groups: int, keep: int, scale: float):
+    """``(idx[T, k], w[T, k])``: see :func:`route_sigmoid`.  Differentiable in the weights."""
+    T, E = logits.shape
+    s = torch.sigmoid(logits.float())
+    c = s.detach() if correction is None else s.detach() + correction.float()
+    if groups > 1 and keep < groups:
+        size = E // groups
+        gs = c.view(T, groups, size).topk(min(2, size), dim=-1).values.sum(-1)
+        kept = torch.zeros(T, groups, dtype=torch.bool, device=c.device)
+        kept.scatter_(1, gs.topk(keep, dim=-1).indices, True)
+        c = c.masked_fill(~kept.repeat_interleave(size, dim=1), float("-inf"))
+    idx = c.topk(k, dim=-1).indices
+    return idx, s.gather(1, idx) * scale
+
+
+class RoutedTokens:
+    """What :func:`route_sigmoid` leaves on the device for the expert products: choices, weights and tokens per expert."""
+
+    def __init__(self, idx, w, counts):
+        self.idx, self.w, self.counts = idx, w, counts
+
+
+def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, keep: int = 1, scale: float = 1.0, live=None,
+                  live_limit: int = 0) -> RoutedTokens:
+    """Routing of fp32 ``logits [T, E]``: the ``k`` experts with the largest ``sigmoid(logits) + correction`` among those of the
+    ``keep`` (of ``groups``) neighbour groups whose two best choice scores sum highest; weights ``scale * sigmoid(logits)``.
+    ``live [T]`` int32: tokens whose value lies outside ``[0, live_limit)`` are padding and are sent to no expert (index -1)."""
+    from . import lib
+
+    T, E = logits.shape
+    if not (logits.is_cuda and lib.available()):
+        idx, w = route_sigmoid_reference(logits, correction, k, groups, keep, scale)
+        idx = idx.to(torch.int32)
+        if live is not None:
+            dead = (live < 0) | (live >= live_limit)
+            idx, w = idx.masked_fill(dead[:, None], -1), w.masked_fill(dead[:, None], 0.0)
+        return RoutedTokens(idx, w, None)
+    c = lib
+    if "rs" not in _g:
+        _g["rs"] = lib.fn("lvb_moe_route_sigmoid", [c.c_void_p, c.c_longlong, c.c_void_p, c.c_int, c.c_void_p] + [c.c_int] * 6 +
+                          [c.c_float, c.c_void_p, c.c_void_p, c.c_void_p, c.c_void_p])
+    dev = logits.device
+    z = logits if logits.stride(1) == 1 else logits.contiguous()
+    if correction is not None and correction.dtype not in (torch.float32, torch.bfloat16):
+        correction = correction.float()
+    idx = torch.empty(T, k, dtype=torch.int32, device=dev)
+    w = torch.empty(T, k, dtype=torch.float32, device=dev)
+    counts = torch.empty(2 * E, dtype=torch.int32, device=dev)
+    rc = _g["rs"](z.data_ptr(), z.stride(0), lib.ptr(correction), int(correction is not None and correction.dtype == torch.float32), lib.ptr(live),
+                  int(live_limit), T, E, k, groups, keep, float(scale), idx.data_ptr(), w.data_ptr(), counts.data_ptr(), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_moe_route_sigmoid")
+    return RoutedTokens(idx, w, counts)
+
+
+def _block_rows(pairs: int, experts: int) -> int:
+    """Rows an expert's segment is padded to: the tensor core's 128 when experts get that many tokens, fewer in decode rounds,
+    where the expert products are streams over the weights and padding rows only cost launch width."""
+    mean = pairs / experts
+    for rows in (16, 32, 64):
+        if mean <= rows // 2:
+            return rows
+    return BLOCK
+
+
+def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedTokens, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
+    """``stream[t] += sum_j w[t, j] * down[e] relu(up[e] h[t])^2`` with ``e = idx[t, j]``, in place on the fp32 stream; ``up [E, ff, width]``,
+    ``down [E, width, ff]``.  Forward only, CUDA only: dispatch into the block-padded expert-sorted layout, two grouped products (the
+    activation in the epilogue of the first), combine."""
+    from . import lib
+
+    c = lib
+    T, k = routed.idx.shape
+    E, ff, width = up.shape
+    dev = h.device
+    tma = h.dtype == torch.bfloat16 and up.dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
+    rows = _block_rows(T * k, E) if tma else 64
+    blocks = (T * k + E * (rows - 1) + rows - 1) // rows
+    if "d" not in _g:
+        _g["d"] = lib.fn("lvb_moe_dispatch", [c.c_void_p, c.c_void_p] + [c.c_int] * 5 + [c.c_void_p, c.c_void_p, c.c_int] + [c.c_void_p] * 3)
+        _g["c"] = lib.fn("lvb_moe_combine", [c.c_void_p, c.c_int, c.c_void_p, c.c_void_p] + [c.c_int] * 3 + [c.c_void_p, c.c_void_p])
+        _g["fma"] = lib.fn("lvb_grouped_fma", [c.c_void_p] * 4 + [c.c_int] * 5 + [c.c_void_p])
+        _g["sk"] = lib.fn("lvb_gemm_skinny_grouped", [c.c_void_p] * 3 + [c.c_int] * 9 + [c.c_float, c.c_void_p, c.c_void_p, c.c_void_p])
+    x_pad = torch.empty(blocks * rows, width, dtype=h.dtype, device=dev)
+    dest = torch.empty(T, k, dtype=torch.int32, device=dev)
+    tile_group = torch.empty(blocks, dtype=torch.int32, device=dev)
+    h = h.contiguous()
+    rc = _g["d"](routed.idx.data_ptr(), routed.counts.data_ptr(), T, k, E, rows, blocks, h.data_ptr(), x_pad.data_ptr(), width * h.element_size(),
+                 dest.data_ptr(), tile_group.data_ptr(), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_moe_dispatch")
+
+    def product(a, w, sq_relu: bool):
+        n, kk = w.shape[1], w.shape[2]
+        y = torch.empty(a.shape[0], n, dtype=a.dtype, device=dev)
+        w = w if w.is_contiguous() else w.contiguous()
+        if not tma:
+            rc = _g["fma"](a.data_ptr(), w.data_ptr(), y.data_ptr(), tile_group.data_ptr(), a.shape[0], n, kk, int(sq_relu),
+                           int(a.dtype == torch.float32), lib.stream_ptr())
+        elif rows == BLOCK:
+            _grouped(0, a, w, y, E, a.shape[0], 0, n, kk, 32 if sq_relu else 0, tile_group, None)
+            return y
+        else:
+            rc = _g["sk"](a.data_ptr(), w.data_ptr(), y.data_ptr(), E, a.shape[0], rows, n, kk, kk, kk, n, 32 if sq_relu else 0, 1.0,
+                          tile_group.data_ptr(), lib.status_buffer().data_ptr(), lib.stream_ptr())
+        lib.check_rc(rc, "grouped expert product")
+        return y
+
+    y = product(product(x_pad, up.to(h.dtype), True), down.to(h.dtype), False)
+    rc = _g["c"](y.data_ptr(), int(y.dtype == torch.float32), dest.data_ptr(), routed.w.data_ptr(), T, k, width, stream.data_ptr(), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_moe_combine")
+    return stream
+
+
+def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
+    """The sum :func:`add_expert_outputs` adds, as differentiable framework ops (training, and the CPU path): ``[T, width]`` fp32."""
+    T, k = idx.shape
+    keep = idx >= 0
+    dest, offsets, tile_group, capacity = padded_layout(idx.clamp_min(0).reshape(-1), up.shape[0])
+    x_pad = h.new_zeros(capacity, h.shape[1]).index_copy(0, dest, h.repeat_interleave(k, dim=0))
+    a = torch.relu(grouped_linear(x_pad, up.to(h.dtype), tile_group, offsets)).square()
+    y = grouped_linear(a, down.to(h.dtype), tile_group, offsets).index_select(0, dest).view(T, k, -1)
+    return (y.float() * (w.float() * keep).unsqueeze(-1)).sum(1)

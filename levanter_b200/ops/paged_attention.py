@@ -88,6 +88,139 @@ def _paged_attention_cuda(q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seq
     return out
 
 
+# ------------------------------------------------------------------------------------------------ general form
+# Key and value sizes of their own, attention within chunks of positions, an output gate, fp32.  The cache of a layer is then viewed
+# as [page, slot, kv_head, k_size + v_size], which for equal sizes is the memory of [page, slot, 2 * kv_head, size].
+def _kv_view(kv_pages: torch.Tensor, kv_heads: int, k_size: int, v_size: int) -> torch.Tensor:
+    return kv_pages.view(kv_pages.shape[0], kv_pages.shape[1], kv_heads, k_size + v_size)
+
+
+def _strided_rows(t: torch.Tensor, n: int) -> torch.Tensor:
+    """``t [T, heads, size]`` with heads and sizes packed inside a row (a row stride is fine)."""
+    return t if t.stride(2) == 1 and t.stride(1) == t.shape[2] and (t.shape[0] <= 1 or t.stride(0) >= n) else t.contiguous()
+
+
+def kv_page_write_general(kv_pages: torch.Tensor, new_k: torch.Tensor, new_v: torch.Tensor, dests: torch.Tensor) -> None:
+    """:func:`kv_page_write` for ``new_k [T, KV, k_size]`` and ``new_v [T, KV, v_size]`` (rows may be strided) in bf16 or fp32."""
+    KV, dk, dv = new_k.shape[1], new_k.shape[2], new_v.shape[2]
+    kv = _kv_view(kv_pages, KV, dk, dv)
+    slots = kv.shape[0] * kv.shape[1]
+    if _use_kernel(kv_pages, new_k, new_v, dests):
+        c = lib
+        if "wg" not in _f:
+            _f["wg"] = lib.fn("lvb_kv_page_write_general", [c.c_void_p] * 4 + [c.c_int] * 4 + [c.c_longlong] * 3 + [c.c_int, c.c_void_p])
+        dt = kv.dtype
+        k, v = _strided_rows(new_k.to(dt), KV * dk), _strided_rows(new_v.to(dt), KV * dv)
+        d = dests.to(torch.int32).contiguous()
+        rc = _f["wg"](kv.data_ptr(), k.data_ptr(), v.data_ptr(), d.data_ptr(), k.shape[0], KV, dk, dv, k.stride(0), v.stride(0), slots,
+                      int(dt == torch.float32), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_kv_page_write_general")
+        return
+    sel = ((dests >= 0) & (dests < slots)).nonzero().squeeze(-1)
+    flat = kv.view(slots, KV, dk + dv)
+    flat[dests[sel].long()] = torch.cat([new_k[sel], new_v[sel]], dim=-1).to(kv.dtype)
+
+
+def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: int, v_size: int, batch_info, *, sm_scale: float,
+                            chunk: Optional[int] = None, gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None) -> torch.Tensor:
+    """:func:`ragged_paged_attention` of ``q [T, H, k_size]`` (rows may be strided) over pages of ``kv_heads * (k_size + v_size)``
+    elements per slot -> ``[T, H, v_size]``.
+
+    ``chunk``: positions are cut into chunks of that many, counted from the start of the sequence, and a query sees the keys of
+    its own chunk only.  ``gate [T, H * v_size]``: the result is multiplied by its sigmoid.  bf16 with sizes that are multiples of 8
+    up to 256 and at most 16 query heads per KV head runs on tensor cores; everything else in fp32 arithmetic."""
+    T, H, dk = q.shape
+    b = batch_info
+    if not _use_kernel(q, kv_pages):
+        return paged_attention_general_reference(q, kv_pages, kv_heads, v_size, b, sm_scale=sm_scale, chunk=chunk, gate=gate, soft_cap=soft_cap)
+    kv = _kv_view(kv_pages, kv_heads, dk, v_size)
+    if q.dtype != kv.dtype or q.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"query and cache must both be bf16 or both fp32, got {q.dtype} and {kv.dtype}")
+    c = lib
+    P, ps = kv.shape[:2]
+    S, PP = b.page_indices.shape
+    dev = q.device
+    i32 = lambda t: t.to(device=dev, dtype=torch.int32).contiguous()  # noqa: E731
+    lens, pages, cu = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens)
+    ns = i32(b.num_seqs.reshape(1))
+    q = _strided_rows(q, H * dk)
+    ldg = 0
+    if gate is not None:
+        gate = gate if gate.stride(1) == 1 and gate.dtype == q.dtype else gate.to(q.dtype).contiguous()
+        ldg = gate.stride(0)
+    out = torch.empty(T, H, v_size, dtype=q.dtype, device=dev)
+    tensor_cores = (q.dtype == torch.bfloat16 and dk % 8 == 0 and v_size % 8 == 0 and max(dk, v_size) <= 256 and H // kv_heads <= 16
+                    and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0)
+    if not tensor_cores:
+        if "any" not in _f:
+            _f["any"] = lib.fn("lvb_attention_any", [c.c_void_p] * 8 + [c.c_int] * 5 + [c.c_longlong] * 2 + [c.c_int] * 5 +
+                               [c.c_float, c.c_float, c.c_int, c.c_void_p])
+        rc = _f["any"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), T, H,
+                       kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), float(sm_scale), float(soft_cap or 0.0),
+                       int(q.dtype == torch.float32), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_attention_any")
+        return out
+    if "g" not in _f:
+        _f["g"] = lib.fn("lvb_paged_attention_general", [c.c_void_p] * 10 + [c.c_int] * 12 + [c.c_float, c.c_float, c.c_void_p], launches=2)
+        _f["gparts"] = lib.fn("lvb_paged_attention_general_parts", [c.c_int, c.c_int], launches=0)
+    parts = _f["gparts"](PP * ps, int(chunk or 0))
+    po = pml = None
+    if parts > 1:
+        po, pml = _part_scratch(dev, T * H * parts * v_size, T * H * parts * 2)
+    rc = _f["g"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), lib.ptr(po),
+                 lib.ptr(pml), T, H, kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), float(sm_scale),
+                 float(soft_cap or 0.0), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_paged_attention_general")
+    return out
+
+
+_part = {}
+
+
+def _part_scratch(dev, n_o: int, n_ml: int):
+    """Scratch for the partitions' partial results, grown as needed and shared by every layer: on one stream a layer's merge has
+    consumed it before the next layer's partitions are written.  A buffer that grew stays referenced, because a captured graph
+    may still write to the smaller one."""
+    bufs = _part.setdefault(dev, [])
+    for o, ml in bufs:
+        if o.numel() >= n_o and ml.numel() >= n_ml:
+            return o, ml
+    pair = (torch.empty(n_o, dtype=torch.float32, device=dev), torch.empty(n_ml, dtype=torch.float32, device=dev))
+    bufs.append(pair)
+    return pair
+
+
+def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, batch_info, *, sm_scale: float, chunk: Optional[int] = None,
+                                      gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None) -> torch.Tensor:
+    """PyTorch statement of :func:`paged_attention_general` (CPU path and test oracle)."""
+    T, H, dk = q.shape
+    b = batch_info
+    kv_all = _kv_view(kv_pages, kv_heads, dk, v_size)
+    ps = kv_all.shape[1]
+    G = H // kv_heads
+    out = torch.zeros(T, H, v_size, dtype=torch.float32, device=q.device)
+    cu, lens = b.cu_q_lens.tolist(), b.seq_lens.tolist()
+    for i in range(int(b.num_seqs)):
+        q0, q1, kl = cu[i], cu[i + 1], lens[i]
+        if q1 <= q0 or kl <= 0 or kl == INVALID:
+            continue
+        n = (kl + ps - 1) // ps
+        kv = kv_all[b.page_indices[i, :n].long()].reshape(n * ps, kv_heads, dk + v_size)[:kl].float()
+        s = torch.einsum("qkgd,skd->kgqs", q[q0:q1].float().view(q1 - q0, kv_heads, G, dk), kv[..., :dk]) * sm_scale
+        if soft_cap:
+            s = torch.tanh(s / soft_cap) * soft_cap
+        qpos = torch.arange(q1 - q0, device=q.device) + (kl - (q1 - q0))
+        kpos = torch.arange(kl, device=q.device)
+        see = kpos[None, :] <= qpos[:, None]
+        if chunk:
+            see = see & (kpos[None, :] // chunk == qpos[:, None] // chunk)
+        p = torch.softmax(s.masked_fill(~see, -float("inf")), dim=-1)
+        out[q0:q1] = torch.einsum("kgqs,skd->qkgd", p, kv[..., dk:]).reshape(q1 - q0, H, v_size)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float()).view(T, H, v_size)
+    return out.to(q.dtype)
+
+
 def ragged_paged_attention_reference(q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, sm_scale: float = 1.0,
                                      soft_cap: Optional[float] = None) -> torch.Tensor:
     T, H, D = q.shape

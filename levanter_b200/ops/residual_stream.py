@@ -1,0 +1,101 @@
+"""Pre-norm blocks around an fp32 residual stream (``csrc/residual_stream.cu`` and the GEMM epilogues).
+
+The stream ``x`` is an fp32 tensor whatever the model's compute dtype: the embedding starts it, RMS norms read it and hand the
+compute dtype to the projections, and the projections that end a block accumulate into it in their epilogue.  The kernels run
+when no gradient is being recorded; with autograd the same steps are PyTorch ops on an fp32 stream, and on the CPU they are the
+PyTorch statements only."""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from . import lib
+from .gemm import gemm, linear
+
+_f = {}
+
+
+def _kernels(*tensors) -> bool:
+    """The in-place / fused kernels may run: CUDA tensors and nothing to differentiate."""
+    return not torch.is_grad_enabled() and all(t.is_cuda for t in tensors) and lib.available()
+
+
+def embed_stream(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch.Tensor:
+    """``scale * weight[ids]`` in fp32."""
+    if _kernels(ids, weight) and weight.dtype in (torch.float32, torch.bfloat16) and weight.is_contiguous():
+        c = lib
+        if "e" not in _f:
+            _f["e"] = lib.fn("lvb_embed_stream", [c.c_void_p, c.c_void_p, c.c_int, c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_float,
+                                                  c.c_void_p, c.c_void_p])
+        flat = ids.reshape(-1).to(torch.int32).contiguous()
+        V, D = weight.shape
+        out = torch.empty(flat.numel(), D, dtype=torch.float32, device=weight.device)
+        rc = _f["e"](flat.data_ptr(), weight.data_ptr(), int(weight.dtype == torch.float32), out.data_ptr(), flat.numel(), D, V, float(scale),
+                     lib.status_buffer().data_ptr(), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_embed_stream")
+        return out.view(*ids.shape, D)
+    return torch.nn.functional.embedding(ids.long(), weight).float() * scale
+
+
+def rms_norm_stream(x: torch.Tensor, weight: torch.Tensor, eps: float, *, w_offset: float = 0.0, out_dtype: Optional[torch.dtype] = None,
+                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm of the fp32 stream in ``out_dtype`` (default: the weight's dtype).  ``rows``: normalise these rows only."""
+    dt = out_dtype or weight.dtype
+    if _kernels(x, weight) and x.dtype == torch.float32 and dt in (torch.float32, torch.bfloat16) and weight.dtype in (torch.float32, torch.bfloat16) \
+            and weight.is_contiguous():
+        c = lib
+        if "n" not in _f:
+            _f["n"] = lib.fn("lvb_rms_stream", [c.c_void_p, c.c_void_p, c.c_void_p, c.c_int, c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_float,
+                                                c.c_float, c.c_void_p])
+        D = x.shape[-1]
+        x2 = x.reshape(-1, D)
+        x2 = x2 if x2.is_contiguous() else x2.contiguous()
+        if rows is not None:
+            rows = rows.to(torch.int64).contiguous()
+        n = x2.shape[0] if rows is None else rows.numel()
+        y = torch.empty(n, D, dtype=dt, device=x.device)
+        rc = _f["n"](x2.data_ptr(), lib.ptr(rows), weight.data_ptr(), int(weight.dtype == torch.float32), y.data_ptr(), int(dt == torch.float32), n, D,
+                     float(eps), float(w_offset), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_rms_stream")
+        return y.view(*x.shape[:-1], D) if rows is None else y
+    if rows is not None:
+        x = x.index_select(0, rows.long())
+    xf = x.float()
+    y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (weight.float() + w_offset)
+    return y.to(dt)
+
+
+def _gemm_ok(h: torch.Tensor, w: torch.Tensor) -> bool:
+    """The tcgen05 GEMM takes the product (forward only: the output size is free, the inner size a multiple of 8)."""
+    return h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] % 8 == 0
+
+
+def add_linear(x: torch.Tensor, h: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x + h W^T`` on the fp32 stream.  Without autograd ``x`` itself is updated and returned."""
+    if _kernels(x, h, weight):
+        x2, h2 = x.view(-1, x.shape[-1]), h.reshape(-1, h.shape[-1])
+        if _gemm_ok(h2, weight):
+            gemm(h2, weight, out=x2, accumulate=True)
+        elif h.dtype == torch.float32 and weight.dtype == torch.float32:
+            x2.addmm_(h2, weight.t())
+        else:
+            x2.add_(torch.nn.functional.linear(h2, weight))
+        return x
+    return x + linear(h, weight).float()
+
+
+def project(h: torch.Tensor, weight: torch.Tensor, *, squared_relu: bool = False, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``h W^T`` (``max(., 0)^2`` of it), in ``h``'s dtype or in fp32 straight from the accumulator."""
+    if _kernels(h, weight) and _gemm_ok(h, weight):
+        h2 = h.reshape(-1, h.shape[-1])
+        y = gemm(h2, weight, out_dtype=out_dtype or h.dtype, squared_relu=squared_relu)
+        return y.view(*h.shape[:-1], weight.shape[0])
+    if out_dtype == torch.float32 and h.dtype != torch.float32:
+        # sizes the GEMM does not take (or with autograd, or on the CPU): the product itself in fp32
+        y = torch.nn.functional.linear(h.float(), weight.float())
+    else:
+        y = linear(h, weight)
+        if out_dtype is not None:
+            y = y.to(out_dtype)
+    return torch.relu(y).square() if squared_relu else y
