@@ -21,8 +21,30 @@ MODELS = {
     "llama3_8b": dict(hidden_dim=4096, intermediate_dim=14336, num_layers=32, num_heads=32, num_kv_heads=8, vocab=128256),
     "llama2_7b": dict(hidden_dim=4096, intermediate_dim=11008, num_layers=32, num_heads=32, num_kv_heads=32, vocab=32000),
     "llama_1b": dict(hidden_dim=2048, intermediate_dim=8192, num_layers=16, num_heads=32, num_kv_heads=8, vocab=128256),
+    # Fedolorn at the size of llama3_8b: the same width, heads, layers and vocabulary; with an attention gate and two feed-forward
+    # matrices instead of a gated three, ff = 19456 gives a layer the same number of parameters.  The second one has 64 experts
+    "fedolorn_8b": dict(family="fedolorn", hidden_dim=4096, num_layers=32, intermediate_dim=19456, vocab=128256),
+    "fedolorn_moe": dict(family="fedolorn", hidden_dim=4096, num_layers=16, intermediate_dim=1536, vocab=128256,
+                         moe=dict(num_experts=64, num_experts_per_tok=8, expert_groups=8, expert_groups_kept=4, router_scale=2.5)),
+    "tiny_fedolorn": dict(family="fedolorn", hidden_dim=256, num_layers=2, intermediate_dim=64, vocab=1024,
+                          heads=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, chunk_size=96),
+                          moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=2, expert_groups_kept=1)),
     "tiny": dict(hidden_dim=256, intermediate_dim=512, num_layers=2, num_heads=4, num_kv_heads=2, vocab=1024),
 }
+
+
+def model_config(m: dict, seq_len: int):
+    """The model config of a ``MODELS`` entry (without its ``vocab``)."""
+    m = dict(m)
+    if m.pop("family", "llama") == "llama":
+        from ..models.llama import LlamaConfig
+
+        return LlamaConfig(seq_len=seq_len, gradient_checkpointing=False, **m)
+    from ..models.fedolorn import FedolornConfig, FedolornLayerConfig
+
+    layer = FedolornLayerConfig(intermediate_dim=m["intermediate_dim"], **m.get("heads", {}), **m.get("moe", {}))
+    return FedolornConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], embedding_scale=12.0, gradient_checkpointing=False,
+                          layers=(layer,) * m["num_layers"])
 
 
 def main(argv=None):
@@ -48,7 +70,6 @@ def run(a):
     import os
 
     from ..data.passthrough_tokenizer import PassthroughTokenizer
-    from ..models.llama import LlamaConfig
     from .engine import InferenceEngine, InferenceEngineConfig, Request
     from .jit_scheduler import SeqDecodingParams
 
@@ -59,7 +80,7 @@ def run(a):
     prompt_max = a.prompt_max or a.prompt_len
     prompt_min = a.prompt_min or prompt_max
     total_len = prompt_max + a.new_tokens
-    cfg = LlamaConfig(seq_len=max(total_len, 128), gradient_checkpointing=False, **m)
+    cfg = model_config(m, max(total_len, 128))
     rank, local_rank = int(os.environ.get("RANK", "0")), int(os.environ.get("LOCAL_RANK", "0"))
     if torch.cuda.is_available():
         torch.cuda.set_device(local_rank)

@@ -262,7 +262,7 @@ extern "C" int lvb_moe_route_sigmoid(const float* z, long long ldz, const void* 
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
-// Places the pairs of idx [T, k] in a buffer of `blocks` blocks of block_rows rows (at least T * k + E * (block_rows - 1) rows) and copies
+// Places the pairs of idx [T, k] in a buffer of `blocks` blocks of block_rows rows (at least T * k + min(E, T * k) * (block_rows - 1) rows) and copies
 // the rows x [T, row_bytes] there.  dest [T, k]: row of every pair (-1: none); tile_group [blocks]: expert of every block (-1: unused).
 // Rows of the buffer that no pair owns keep what they held.
 extern "C" int lvb_moe_dispatch(const int* idx, int* counts, int T, int k, int E, int block_rows, int blocks, const void* x, void* x_pad,
@@ -270,7 +270,8 @@ extern "C" int lvb_moe_dispatch(const int* idx, int* counts, int T, int k, int E
   using namespace lvb;
   using namespace lvb::experts;
   if (T <= 0 || k <= 0 || E <= 0 || E > kMaxExperts || block_rows <= 0 || row_bytes <= 0 || (row_bytes & 1)) return kErrBadArg;
-  if (static_cast<long long>(blocks) * block_rows < static_cast<long long>(T) * k + static_cast<long long>(E) * (block_rows - 1)) return kErrBadArg;
+  if (static_cast<long long>(blocks) * block_rows < static_cast<long long>(T) * k + static_cast<long long>(E < T * k ? E : T * k) * (block_rows - 1))
+    return kErrBadArg;
   const int pairs = T * k;
   const int vec = (row_bytes & 15) == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(x_pad)) & 15) == 0;
   int grid = (pairs + 7) / 8;

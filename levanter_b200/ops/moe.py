@@ -307,6 +307,31 @@ def _block_rows(pairs: int, experts: int) -> int:
     return BLOCK
 
 
+def grouped_product(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, rows: int, sq_relu: bool) -> torch.Tensor:
+    """``a[rows of block b] w[tile_group[b]]^T`` (``max(., 0)^2`` of it) over blocks of ``rows`` rows, forward only; ``w [E, out, in]``.
+    bf16 with sizes that are multiples of 8 on tensor cores, otherwise fp32 arithmetic on blocks of 64."""
+    from . import lib
+
+    c = lib
+    if "fma" not in _g:
+        _g["fma"] = lib.fn("lvb_grouped_fma", [c.c_void_p] * 4 + [c.c_int] * 5 + [c.c_void_p])
+        _g["sk"] = lib.fn("lvb_gemm_skinny_grouped", [c.c_void_p] * 3 + [c.c_int] * 9 + [c.c_float, c.c_void_p, c.c_void_p, c.c_void_p])
+    E, n, k = w.shape
+    w = w if w.is_contiguous() else w.contiguous()
+    y = torch.empty(a.shape[0], n, dtype=a.dtype, device=a.device)
+    if a.dtype != torch.bfloat16 or n % 8 or k % 8:
+        assert rows == 64
+        rc = _g["fma"](a.data_ptr(), w.data_ptr(), y.data_ptr(), tile_group.data_ptr(), a.shape[0], n, k, int(sq_relu),
+                       int(a.dtype == torch.float32), lib.stream_ptr())
+    elif rows == BLOCK:
+        return _grouped(0, a, w, y, E, a.shape[0], 0, n, k, 32 if sq_relu else 0, tile_group, None)
+    else:
+        rc = _g["sk"](a.data_ptr(), w.data_ptr(), y.data_ptr(), E, a.shape[0], rows, n, k, k, k, n, 32 if sq_relu else 0, 1.0,
+                      tile_group.data_ptr(), lib.status_buffer().data_ptr(), lib.stream_ptr())
+    lib.check_rc(rc, "grouped expert product")
+    return y
+
+
 def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedTokens, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
     """``stream[t] += sum_j w[t, j] * down[e] relu(up[e] h[t])^2`` with ``e = idx[t, j]``, in place on the fp32 stream; ``up [E, ff, width]``,
     ``down [E, width, ff]``.  Forward only, CUDA only: dispatch into the block-padded expert-sorted layout, two grouped products (the
@@ -318,13 +343,11 @@ def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedToke
     E, ff, width = up.shape
     dev = h.device
     tma = h.dtype == torch.bfloat16 and up.dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
-    rows = _block_rows(T * k, E) if tma else 64
-    blocks = (T * k + E * (rows - 1) + rows - 1) // rows
+    rows = _block_rows(T * k, E) if tma else 64  # 64: the tile of the fp32 product
+    blocks = (T * k + min(E, T * k) * (rows - 1) + rows - 1) // rows
     if "d" not in _g:
         _g["d"] = lib.fn("lvb_moe_dispatch", [c.c_void_p, c.c_void_p] + [c.c_int] * 5 + [c.c_void_p, c.c_void_p, c.c_int] + [c.c_void_p] * 3)
         _g["c"] = lib.fn("lvb_moe_combine", [c.c_void_p, c.c_int, c.c_void_p, c.c_void_p] + [c.c_int] * 3 + [c.c_void_p, c.c_void_p])
-        _g["fma"] = lib.fn("lvb_grouped_fma", [c.c_void_p] * 4 + [c.c_int] * 5 + [c.c_void_p])
-        _g["sk"] = lib.fn("lvb_gemm_skinny_grouped", [c.c_void_p] * 3 + [c.c_int] * 9 + [c.c_float, c.c_void_p, c.c_void_p, c.c_void_p])
     x_pad = torch.empty(blocks * rows, width, dtype=h.dtype, device=dev)
     dest = torch.empty(T, k, dtype=torch.int32, device=dev)
     tile_group = torch.empty(blocks, dtype=torch.int32, device=dev)
@@ -333,23 +356,8 @@ def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedToke
                  dest.data_ptr(), tile_group.data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_moe_dispatch")
 
-    def product(a, w, sq_relu: bool):
-        n, kk = w.shape[1], w.shape[2]
-        y = torch.empty(a.shape[0], n, dtype=a.dtype, device=dev)
-        w = w if w.is_contiguous() else w.contiguous()
-        if not tma:
-            rc = _g["fma"](a.data_ptr(), w.data_ptr(), y.data_ptr(), tile_group.data_ptr(), a.shape[0], n, kk, int(sq_relu),
-                           int(a.dtype == torch.float32), lib.stream_ptr())
-        elif rows == BLOCK:
-            _grouped(0, a, w, y, E, a.shape[0], 0, n, kk, 32 if sq_relu else 0, tile_group, None)
-            return y
-        else:
-            rc = _g["sk"](a.data_ptr(), w.data_ptr(), y.data_ptr(), E, a.shape[0], rows, n, kk, kk, kk, n, 32 if sq_relu else 0, 1.0,
-                          tile_group.data_ptr(), lib.status_buffer().data_ptr(), lib.stream_ptr())
-        lib.check_rc(rc, "grouped expert product")
-        return y
-
-    y = product(product(x_pad, up.to(h.dtype), True), down.to(h.dtype), False)
+    a = grouped_product(x_pad, up.to(h.dtype), tile_group, rows, True)
+    y = grouped_product(a, down.to(h.dtype), tile_group, rows, False)
     rc = _g["c"](y.data_ptr(), int(y.dtype == torch.float32), dest.data_ptr(), routed.w.data_ptr(), T, k, width, stream.data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_moe_combine")
     return stream
