@@ -463,13 +463,11 @@ __global__ void __launch_bounds__(kThreads) paged_attention_staged_kernel(Params
 // O) are merged through shared memory at the end.
 constexpr int kMmaStageKeys = 16;
 constexpr int kMmaWarpKeys = kPart / (kThreads / 32);  // 64
-template <int DKC, int DVC>
-struct MmaLayout {
-  static_assert((DKC + DVC) % 64 == 0, "row stride modulo 128 bytes must be 16");
-  static constexpr int kRowBytes = (DKC + DVC) * 2 + 16;  // K, V, 16 B padding
-  static constexpr int kStageBytes = kMmaStageKeys * kRowBytes;
-  static constexpr int kSmem = 4 * 2 * kStageBytes + kPart * 4 + 4 * 16 * 2 * 4;
-};
+// A staged row: K, V (each rounded up to 16 columns) and 16 bytes of padding, which makes the stride an odd multiple of 16 bytes, so
+// that the eight rows of an ldmatrix fall into different banks.
+__host__ __device__ constexpr int mma_row_bytes(int dk16, int dv16) { return (dk16 + dv16) * 2 + 16; }
+// The stage memory is reused for the warps' outputs, [4 warps][16 rows][dv16] fp32, which is never larger.
+constexpr int mma_smem(int dk16, int dv16) { return 4 * 2 * kMmaStageKeys * mma_row_bytes(dk16, dv16) + kPart * 4 + 4 * 16 * 2 * 4; }
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -485,10 +483,9 @@ __device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4],
 
 template <int DKC, int DVC, bool kExact>
 __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p) {
-  using L = MmaLayout<DKC, DVC>;
-  constexpr int kMmaRowBytes = L::kRowBytes, kMmaStageBytes = L::kStageBytes;
   const int dk = kExact ? DKC : p.dk, dv = kExact ? DVC : p.dv;
-  const int dk16 = (dk + 15) & ~15;
+  const int dk16 = (dk + 15) & ~15, dv16 = (dv + 15) & ~15;
+  const int kMmaRowBytes = mma_row_bytes(dk16, dv16), kMmaStageBytes = kMmaStageKeys * kMmaRowBytes;
   const int t = blockIdx.x, kvh = blockIdx.y, part = blockIdx.z;
   const int G = p.H / p.KV;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -542,11 +539,19 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
   uint8_t* my_stage = s_stage + warp * (2 * kMmaStageBytes);
   // one stage: 16 rows of 16-byte pieces; rows without a key are zero-filled (0 * NaN would poison O), and so are the columns
   // between a size and the next multiple of 16
+  const int per_row = (dk16 + dv16) / 8;
+  const int lane_row = lane / per_row, lane_piece = lane % per_row, step_row = 32 / per_row, step_piece = 32 % per_row;
   auto issue = [&](int st) {
     uint8_t* dst = my_stage + (st & 1) * kMmaStageBytes;
+    int r = lane_row, ch = lane_piece;  // row and piece of the lane's next copy
 #pragma unroll 4
-    for (int c = lane; c < kMmaStageKeys * ((DKC + DVC) / 8); c += 32) {
-      const int r = c / ((DKC + DVC) / 8), ch = c % ((DKC + DVC) / 8);
+    for (int c = lane; c < kMmaStageKeys * per_row; c += 32) {
+      if constexpr (kExact) {
+        r = c / ((DKC + DVC) / 8);
+        ch = c % ((DKC + DVC) / 8);
+      } else {
+        if (ch >= per_row) { ch -= per_row; ++r; }
+      }
       const int i = wk0 + st * kMmaStageKeys + r;
       const int slot = (st * kMmaStageKeys + r < wnk) ? s_rows[i] : -1;
       uint8_t* d = dst + r * kMmaRowBytes + ch * 16;
@@ -555,10 +560,12 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
         if (slot >= 0) cp_async_16(d, src + ch * 8);
         else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
       } else {
-        const int col = ch < DKC / 8 ? ch * 8 : ch * 8 - DKC;  // column of the key or value row
-        const int size = ch < DKC / 8 ? dk : dv;
-        if (slot >= 0 && col < size) cp_async_16(d, src + (ch < DKC / 8 ? col : dk + col));
-        else if (col < ((size + 15) & ~15)) *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+        const bool is_k = ch * 8 < dk16;
+        const int col = is_k ? ch * 8 : ch * 8 - dk16;  // column of the key or value row
+        if (slot >= 0 && col < (is_k ? dk : dv)) cp_async_16(d, src + (is_k ? col : dk + col));
+        else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+        r += step_row;
+        ch += step_piece;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -648,7 +655,7 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
       uint32_t b0, b1, b2, b3;
       // matrices: (keys 0-7, d 16 np .. +7), (keys 8-15, same d), (keys 0-7, d 16 np + 8 ..), (keys 8-15, same)
       const int mi = lane >> 3;
-      const uint32_t addr = buf + ((mi & 1) * 8 + (lane & 7)) * kMmaRowBytes + DKC * 2 + (np * 16 + (mi >> 1) * 8) * 2;
+      const uint32_t addr = buf + ((mi & 1) * 8 + (lane & 7)) * kMmaRowBytes + dk16 * 2 + (np * 16 + (mi >> 1) * 8) * 2;
       ldmatrix_x4_trans(addr, b0, b1, b2, b3);
       float* oa = o[2 * np];
       float* ob = o[2 * np + 1];
@@ -669,12 +676,13 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     s_ml[(warp * 16 + row_hi) * 2 + 0] = m_hi;
     s_ml[(warp * 16 + row_hi) * 2 + 1] = l_hi;
   }
-  float* s_o = reinterpret_cast<float*>(s_stage);  // [4 warps][16 rows][DVC] fp32
+  float* s_o = reinterpret_cast<float*>(s_stage);  // [4 warps][16 rows][dv16] fp32
 #pragma unroll
   for (int n = 0; n < DVC / 8; ++n) {
     const int d0 = n * 8 + kq;
-    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_lo) * DVC + d0) = make_float2(o[n][0], o[n][1]);
-    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_hi) * DVC + d0) = make_float2(o[n][2], o[n][3]);
+    if (!kExact && n * 8 >= dv16) break;
+    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_lo) * dv16 + d0) = make_float2(o[n][0], o[n][1]);
+    *reinterpret_cast<float2*>(s_o + (warp * 16 + row_hi) * dv16 + d0) = make_float2(o[n][2], o[n][3]);
   }
   __syncthreads();
   for (int idx = threadIdx.x; idx < G * dv; idx += kThreads) {
@@ -687,7 +695,7 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     for (int w = 0; w < 4; ++w) {
       const float mw = s_ml[(w * 16 + g) * 2];
       const float f = (mw == -INFINITY) ? 0.f : exp2f(mw - m);
-      acc = fmaf(s_o[(w * 16 + g) * DVC + d], f, acc);
+      acc = fmaf(s_o[(w * 16 + g) * dv16 + d], f, acc);
       l = fmaf(s_ml[(w * 16 + g) * 2 + 1], f, l);
     }
     const long long hrow = static_cast<long long>(t) * p.H + kvh * G + g;
@@ -746,11 +754,11 @@ inline int paged_variant() {
 
 template <int DKC, int DVC, bool kExact>
 int launch_mma(const Params& p, cudaStream_t s) {
-  constexpr int smem = MmaLayout<DKC, DVC>::kSmem;
+  const int smem = kExact ? mma_smem(DKC, DVC) : mma_smem((p.dk + 15) & ~15, (p.dv + 15) & ~15);
   auto kern = paged_attention_mma_kernel<DKC, DVC, kExact>;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return kErrCuda;
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mma_smem(DKC, DVC)) != cudaSuccess) return kErrCuda;
     attr_set = true;
   }
   kern<<<dim3(p.T, p.KV, p.parts), kThreads, smem, s>>>(p);
@@ -866,6 +874,8 @@ extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, 
   if (dk == 128 && dv == 128) rc = launch_mma<128, 128, true>(p, s);
   else if (dk <= 64 && dv <= 64) rc = launch_mma<64, 64, false>(p, s);
   else if (dk <= 128 && dv <= 128) rc = launch_mma<128, 128, false>(p, s);
+  else if (dk <= 192 && dv <= 128) rc = launch_mma<192, 128, false>(p, s);
+  else if (dv <= 128) rc = launch_mma<256, 128, false>(p, s);
   else rc = launch_mma<256, 256, false>(p, s);
   if (rc != kErrOk) return rc;
   return launch_merge(p, s);

@@ -163,7 +163,7 @@ def _check_rows(got, want, dtype):
 
 
 PAGED = [(BF, 4, 2, 96, 96, 200), (BF, 6, 2, 64, 64, 48), (BF, 8, 1, 128, 128, 300), (BF, 4, 4, 40, 72, 7), (BF, 8, 2, 128, 64, 520),
-         (BF, 3, 1, 256, 192, 64), (BF, 2, 2, 20, 12, 33), (BF, 20, 1, 64, 64, 50), (F32, 4, 2, 96, 80, 200), (F32, 6, 3, 33, 17, 10),
+         (BF, 3, 1, 256, 192, 64), (BF, 4, 1, 192, 128, 90), (BF, 4, 2, 200, 88, 40), (BF, 2, 2, 20, 12, 33), (BF, 20, 1, 64, 64, 50), (F32, 4, 2, 96, 80, 200), (F32, 6, 3, 33, 17, 10),
          (BF, 4, 2, 64, 64, 5000), (BF, 16, 1, 24, 128, 257)]
 
 
