@@ -134,8 +134,9 @@ def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: i
     if not _use_kernel(q, kv_pages):
         return paged_attention_general_reference(q, kv_pages, kv_heads, v_size, b, sm_scale=sm_scale, chunk=chunk, gate=gate, soft_cap=soft_cap)
     kv = _kv_view(kv_pages, kv_heads, dk, v_size)
-    if q.dtype != kv.dtype or q.dtype not in (torch.bfloat16, torch.float32):
-        raise TypeError(f"query and cache must both be bf16 or both fp32, got {q.dtype} and {kv.dtype}")
+    if kv.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"the cache must be bf16 or fp32, got {kv.dtype}")
+    q = q.to(kv.dtype)  # attention runs in the cache's type
     c = lib
     P, ps = kv.shape[:2]
     S, PP = b.page_indices.shape

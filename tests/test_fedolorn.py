@@ -297,3 +297,26 @@ def test_chunk_masks():
     assert torch.equal(m[:9, :9], O.visible(9, 4)) and torch.equal(m[9:19, 9:19], O.visible(10, 4)) and not m[9:19, :9].any()
     with pytest.raises(ValueError):
         AttentionMask.causal().with_chunk_size(4) & AttentionMask.causal().with_chunk_size(5)
+
+
+def test_sample_lm_command(checkpoint, tmp_path, monkeypatch, capsys):
+    """The sampling command line on a checkpoint directory: greedy tokens are the oracle's."""
+    from levanter_b200 import config as lev_config
+    from levanter_b200.data.passthrough_tokenizer import PassthroughTokenizer
+    from levanter_b200.main import sample_lm
+
+    cfg, W, path = checkpoint("odd")
+    monkeypatch.setattr(sample_lm, "load_tokenizer", lambda name: PassthroughTokenizer(cfg["vocab"]))
+    monkeypatch.setattr(sample_lm, "local_device", lambda: torch.device("cpu"))
+    prompt = _tokens(21, cfg["vocab"], 3)
+    sample_lm.main(lev_config.decode(sample_lm.SampleLmConfig, {
+        "hf_checkpoint": path, "tokenizer": "ids", "model": {"type": "fedolorn"}, "prompts": [" ".join(map(str, prompt))], "max_new_tokens": 12,
+        "n_rounds": 1, "stop_sequence": None, "temperature": 0.0, "engine": {"max_seqs": 2, "page_size": 8, "max_pages_per_seq": 6, "compute_dtype": "float32"},
+        "trainer": {"require_accelerator": False, "tracker": {"type": "noop"}, "log_dir": str(tmp_path), "mp": "f32"}}))
+    out = capsys.readouterr().out
+    toks = list(prompt)
+    for _ in range(12):
+        toks.append(int(O.logits(cfg, W, toks)[-1].argmax()))
+    want = [t for t in toks[21:] if t != cfg["vocab"] - 1]  # the command drops the padding token
+    got = out.split("Generated text for 0", 1)[1].split(":", 1)[1].split("\n")[0].split()
+    assert [int(t) for t in got] == want
