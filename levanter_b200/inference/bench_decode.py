@@ -25,7 +25,7 @@ MODELS = {
     # matrices instead of a gated three, ff = 19456 gives a layer the same number of parameters.  The second one has 64 experts
     "fedolorn_8b": dict(family="fedolorn", hidden_dim=4096, num_layers=32, intermediate_dim=19456, vocab=128256),
     "fedolorn_moe": dict(family="fedolorn", hidden_dim=4096, num_layers=16, intermediate_dim=1536, vocab=128256,
-                         moe=dict(num_experts=64, num_experts_per_tok=8, expert_groups=8, expert_groups_kept=4, router_scale=2.5)),
+                         moe=dict(num_experts=64, num_experts_per_tok=8, expert_groups=8, expert_groups_kept=4, router_scale=1.5)),
     "tiny_fedolorn": dict(family="fedolorn", hidden_dim=256, num_layers=2, intermediate_dim=64, vocab=1024,
                           heads=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, chunk_size=96),
                           moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=2, expert_groups_kept=1)),
@@ -43,7 +43,7 @@ def model_config(m: dict, seq_len: int):
     from ..models.fedolorn import FedolornConfig, FedolornLayerConfig
 
     layer = FedolornLayerConfig(intermediate_dim=m["intermediate_dim"], **m.get("heads", {}), **m.get("moe", {}))
-    return FedolornConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], embedding_scale=12.0, gradient_checkpointing=False,
+    return FedolornConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], embedding_scale=8.0, gradient_checkpointing=False,
                           layers=(layer,) * m["num_layers"])
 
 

@@ -137,7 +137,7 @@ def projections(tb: Table, E=4096, H=32, KV=8, D=128, ff=14336):
         ids = torch.randint(0, 32000, (T,), device="cuda", dtype=torch.int32)
         g = lambda n, k, out: dict(flops=2.0 * T * n * k, nbytes=2.0 * (T * k + n * k) + out)  # noqa: E731
         like = lambda n, k, out: dict(like_flops=2.0 * T * n * k, like_bytes=2.0 * (T * k + n * k) + out)  # noqa: E731
-        tb.pair(f"T={T}: embedding to the fp32 stream", lambda: embed_stream(ids, table, 12.0), "Llama embedding", lambda: embedding(ids, table),
+        tb.pair(f"T={T}: embedding to the fp32 stream", lambda: embed_stream(ids, table, 8.0), "Llama embedding", lambda: embedding(ids, table),
                 nbytes=6.0 * T * E, like_bytes=4.0 * T * E)
         tb.pair(f"T={T}: RMS norm of the fp32 stream", lambda: rms_norm_stream(x, wn, 1e-5, w_offset=1.0), "Llama RMS norm", lambda: rms_norm(xb, wn),
                 nbytes=6.0 * T * E, like_bytes=4.0 * T * E)
