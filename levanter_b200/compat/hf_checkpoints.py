@@ -112,6 +112,10 @@ def to_hf_state_dict(model: nn.Module, dtype: Optional[torch.dtype] = None, para
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)
         t = t.cpu()
+        if hasattr(model, "hf_tensor_parts"):  # a model that says which view of a parameter is which checkpoint tensor
+            for n, view, shape in model.hf_tensor_parts(name, t):
+                out[n] = view.reshape(shape).contiguous()
+            continue
         if hasattr(model, "hf_tensor_names"):  # a model that names its checkpoint tensors itself
             names = model.hf_tensor_names(name)
             out.update({names: t.contiguous()} if isinstance(names, str) else {n: t[j].contiguous() for j, n in enumerate(names)})
@@ -143,6 +147,16 @@ def load_hf_state_dict(model: nn.Module, state_dict: Dict[str, torch.Tensor], *,
     missing: List[str] = []
     with torch.no_grad():
         for name, p in model.named_parameters():
+            if hasattr(model, "hf_tensor_parts"):
+                found = [(n, view, shape, lookup(n)) for n, view, shape in model.hf_tensor_parts(name, p.data)]
+                if any(t is None for *_, t in found):
+                    missing.append(name)
+                    continue
+                for n, view, shape, t in found:
+                    if tuple(t.shape) != tuple(shape):
+                        raise ValueError(f"shape mismatch for {n}: checkpoint {tuple(t.shape)} vs model {tuple(shape)}")
+                    view.copy_(t.reshape(view.shape).to(view.dtype))
+                continue
             if hasattr(model, "hf_tensor_names"):
                 names = model.hf_tensor_names(name)
                 parts = [(p.data, names)] if isinstance(names, str) else [(p.data[j], n) for j, n in enumerate(names)]

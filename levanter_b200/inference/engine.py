@@ -78,7 +78,7 @@ class InferenceEngineConfig:
 
 @dataclass
 class GenState:
-    cache: object  # what ``model.initial_cache`` returned (a KvPageCache or a list of them, one per layer)
+    cache: object  # what ``model.initial_cache`` returned (a KvPageCache or SlotStateCache, or a list of them, one per layer)
     decode_state: DecodeState
 
 
@@ -144,8 +144,9 @@ class _DecodeGraph:
         self.seeds.copy_(seeds)
 
 
-def _caches(cache) -> List[KvPageCache]:
-    if isinstance(cache, KvPageCache):
+def _caches(cache) -> List[object]:
+    """The caches of the layers: key/value pages (:class:`KvPageCache`) or state by slot (:class:`SlotStateCache`)."""
+    if hasattr(cache, "copy_page"):
         return [cache]
     if isinstance(cache, (list, tuple)):
         return [c for x in cache for c in _caches(x)]
@@ -205,7 +206,8 @@ class InferenceEngine:
         return cls(model=model, tokenizer=tokenizer, cache=cache, decode_state=ds, sampler=Sampler(), config=config, device=device)
 
     def reset(self) -> None:
-        """Drop every sequence and request.  The KV cache contents are left as they are: pages are rewritten before use."""
+        """Drop every sequence and request.  The cache contents are left as they are: pages are rewritten before use, and a recurrent
+        state starts from zero at position 0."""
         cfg = self.config
         table = PageTable.init(cfg.imputed_max_pages, cfg.max_seqs, cfg.page_size, cfg.max_pages_per_seq)
         self.gen_state.decode_state = DecodeState.init(table, max_stop_seqs=cfg.max_stop_seqs, max_stop_tokens=cfg.max_stop_tokens,
@@ -415,7 +417,7 @@ class InferenceEngine:
 
     def _clone(self, src: int, dst: int, r: Request, choice: int) -> None:
         """Slot ``dst`` becomes a copy of ``src`` (same prompt, own sampling key); full pages are shared, a partial last page
-        is duplicated in every layer's cache."""
+        is duplicated in every layer's cache, and so is recurrent state."""
         ds = self.gen_state.decode_state
         before = ds.page_table.page_indices[src].copy()
         ds.page_table = ds.page_table.clone_pages_from(src, dst)
@@ -426,6 +428,8 @@ class InferenceEngine:
             if before[last] != after[last]:
                 for c in _caches(self.gen_state.cache):
                     c.copy_page(int(before[last]), int(after[last]))
+        for c in _caches(self.gen_state.cache):
+            c.copy_slot(src, dst)
         params = dataclasses.replace(r.decode_params, key=int(r.decode_params.key) * 1000003 + choice,
                                      max_num_tokens=int(min(int(r.decode_params.max_num_tokens), ds.page_table.max_len_per_seq)))
         n = int(ds.seq_lens[src])

@@ -366,7 +366,7 @@ def dot_product_attention_with_sink(q, k, v, sink: torch.Tensor, mask=None, bias
 
 
 # --------------------------------------------------------------------------------------------- module
-from ..nn import Linear, RmsNorm  # noqa: E402  (after function definitions to keep the file readable)
+from ..nn import FusedRows, Linear, RmsNorm  # noqa: E402  (after function definitions to keep the file readable)
 
 
 @dataclass(frozen=True)
@@ -390,6 +390,8 @@ class AttentionConfig:
     v_head_dim: Optional[int] = None          # value size per head where it differs from the query/key size
     attention_chunk_size: Optional[int] = None  # a query sees its own chunk of that many positions only
     output_gate: bool = False                 # the heads are multiplied by sigmoid(W_g x) before the output projection
+    head_temperature: bool = False            # a learned number per query head multiplies its scores
+    value_mixing: bool = False                # v <- (1 - m) v + m v_first with a learned m and the first such layer's values
 
     def __post_init__(self):
         assert self.num_heads % self.num_kv_heads == 0, "num_heads must be divisible by num_kv_heads"
@@ -448,9 +450,16 @@ class Attention(nn.Module):
             self.q_norm = None
             self.k_norm = None
         self.rot: Optional[RotaryEmbeddings] = c.rope.build(D) if c.rope is not None else None
+        if c.head_temperature:
+            self.temperature = nn.Parameter(torch.ones(self.local_heads))
+            self.temperature.lev_shape = (self.local_heads,)
+        if c.value_mixing:
+            self.value_mix = nn.Parameter(torch.tensor(0.5))
+            self.value_mix.lev_shape = ()
+        self._rows, self._bias_rows = FusedRows(), FusedRows()
 
     # -- projections shared by training and paged decode (src/levanter/layers/attention.py:1606-1635)
-    def _compute_qkv(self, x: torch.Tensor, pos_ids: Optional[torch.Tensor]):
+    def _compute_qkv(self, x: torch.Tensor, pos_ids: Optional[torch.Tensor], rotate: bool = True):
         c = self.config
         D = c.head_size
         lead = x.shape[:-1]
@@ -460,19 +469,39 @@ class Attention(nn.Module):
         if self.q_norm is not None:
             q = self.q_norm(q)
             k = self.k_norm(k)
-        if self.rot is not None:
+        if self.rot is not None and rotate:
             from ..ops import rope as rope_op
 
             q, k = rope_op.apply_rope(q, k, self.rot, pos_ids)
         return q, k, v
 
+    def _temper_and_mix(self, q, v, v_first):
+        """Differentiable forms of the head temperatures and of value mixing."""
+        if self.config.head_temperature:
+            q = (q.float() * self.temperature.float()[:, None]).to(q.dtype)
+        if self.config.value_mixing and v_first is not None:
+            from ..ops.qkv_prep import mix_values
+
+            v = mix_values(v, v_first, self.value_mix)
+        return q, v
+
     def forward(self, x: torch.Tensor, mask: Union[None, AttentionMask, torch.Tensor] = None,
                 pos_ids: Optional[torch.Tensor] = None, *, skip_out_bias: bool = False,
-                residual: Optional[torch.Tensor] = None, row_parallel=None) -> torch.Tensor:
+                residual: Optional[torch.Tensor] = None, row_parallel=None, v_first: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``row_parallel``: a ``TensorParallel`` whose ``row_linear`` applies the output projection and sums it over the model
-        axis (the caller then adds the bias once)."""
+        axis (the caller then adds the bias once).  ``v_first``: see :meth:`forward_mixing_values`."""
+        return self._forward(x, mask, pos_ids, skip_out_bias, residual, row_parallel, v_first)[0]
+
+    def forward_mixing_values(self, x, mask=None, pos_ids=None, v_first: Optional[torch.Tensor] = None):
+        """``(attention(x), v_first)`` for layers whose values are mixed with those of the first such layer: that layer is given None and
+        returns its own values, the others return what they were given."""
+        return self._forward(x, mask, pos_ids, False, None, None, v_first)
+
+    def _forward(self, x, mask, pos_ids, skip_out_bias, residual, row_parallel, v_first):
         c = self.config
         q, k, v = self._compute_qkv(x, pos_ids)
+        q, v = self._temper_and_mix(q, v, v_first)
+        first = v if v_first is None and c.value_mixing else v_first
         if c.sliding_window is not None and isinstance(mask, AttentionMask) and mask.is_causal:
             mask = mask & AttentionMask.causal(sliding_window=c.sliding_window)
         if c.attention_chunk_size is not None:
@@ -494,11 +523,11 @@ class Attention(nn.Module):
             if type(self.o_proj) is Linear:
                 from ..ops.gemm import linear_residual
 
-                return linear_residual(attn, self.o_proj.weight, None if skip_out_bias else self.o_proj.bias, residual)
-            return self.o_proj(attn, skip_bias=skip_out_bias) + residual  # wrapped projections (LoRA, fp8) add it themselves
+                return linear_residual(attn, self.o_proj.weight, None if skip_out_bias else self.o_proj.bias, residual), first
+            return self.o_proj(attn, skip_bias=skip_out_bias) + residual, first  # wrapped projections (LoRA, fp8) add it themselves
         if row_parallel is not None:
-            return row_parallel.row_linear(attn, self.o_proj)
-        return self.o_proj(attn, skip_bias=skip_out_bias)
+            return row_parallel.row_linear(attn, self.o_proj), first
+        return self.o_proj(attn, skip_bias=skip_out_bias), first
 
     def forward_with_residual(self, x, mask, pos_ids, residual):
         """``residual + attention(x)`` with the add done in the output-projection GEMM epilogue."""
@@ -511,8 +540,9 @@ class Attention(nn.Module):
         from ..ops import paged_attention as PA
 
         c = self.config
-        if c.output_gate or c.attention_chunk_size is not None or c.v_head_size != c.head_size:
-            out = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        if c.output_gate or c.attention_chunk_size is not None or c.v_head_size != c.head_size or c.sliding_window is not None \
+                or c.head_temperature or c.value_mixing or (self.rot is not None and not self.rot.is_plain):
+            out, _ = self._paged_heads(x, kv_cache, batch_info, pos_ids)
             return (self.o_proj(out) if residual is None else self.o_proj(out) + residual), kv_cache
         q, k, v = self._compute_qkv(x, pos_ids)
         kv_cache = kv_cache.update(batch_info, k, v)
@@ -537,75 +567,78 @@ class Attention(nn.Module):
             return self.o_proj(out) + residual, kv_cache
         return self.o_proj(out), kv_cache
 
-    def _fused_projection(self) -> Optional[torch.Tensor]:
-        """One weight ``[q; k; v; gate]`` for serving: the four projections read the same rows, so a decode step streams one matrix
-        instead of launching four products.  The projections' own parameters become row slices of it (nothing is stored
-        twice).  None when a projection is wrapped (LoRA, fp8) or has a bias, and for a model in training, whose parameters
-        belong to the gradient engine's own flat buffers."""
+    def _fused_projection(self):
+        """``(weight, bias or None)`` of the joint projection ``[q; k; v; gate]`` for serving: the projections read the same rows, so a
+        decode step streams one matrix instead of launching four products.  None when a projection is wrapped (LoRA, fp8) or only
+        some have a bias, and for a model in training."""
         mods = [self.q_proj, self.k_proj, self.v_proj] + ([self.g_proj] if self.config.output_gate else [])
-        if any(type(m) is not Linear or m.bias is not None for m in mods):
+        biased = [m.bias is not None for m in mods] if all(type(m) is Linear for m in mods) else [True, False]
+        if self.training or any(biased) != all(biased):
             return None
-        ws = [m.weight for m in mods]
-        if self.training or any(getattr(w, "main_grad", None) is not None or getattr(w, "grad_sink", None) is not None for w in ws):
-            return None
-        fused = getattr(self, "_fused", None)
-        if fused is not None:
-            at = fused.data_ptr()
-            for w in ws:  # still aliases of the fused buffer?  (a model that was moved or converted since has new storage)
-                if w.data_ptr() != at or w.dtype != fused.dtype:
-                    fused = None
-                    break
-                at += w.numel() * w.element_size()
-        if fused is None:
-            fused = torch.cat([w.detach() for w in ws])
-            row = 0
-            for w in ws:
-                w.data = fused[row:row + w.shape[0]]
-                row += w.shape[0]
-            self._fused = fused
-        return fused
+        w = self._rows.get([m.weight for m in mods])
+        b = self._bias_rows.get([m.bias for m in mods]) if w is not None and biased[0] else None
+        return None if w is None or (biased[0] and b is None) else (w, b)
 
-    def _paged_heads(self, x, kv_cache: "KvPageCache", batch_info, pos_ids) -> torch.Tensor:
-        """The gated, concatenated heads ``[T, heads * v_head_size]`` of packed tokens, for the forms of attention that the plain
-        paged path does not have (chunks, a value size of its own, an output gate)."""
+    def _paged_heads(self, x, kv_cache: "KvPageCache", batch_info, pos_ids, v_first: Optional[torch.Tensor] = None):
+        """``(heads, v_first)``: the (gated) concatenated heads ``[T, heads * v_head_size]`` of packed tokens, for the forms of attention
+        that the plain paged path does not have (chunks, windows, a value size of its own, an output gate, temperatures, mixed values,
+        partial rotations), and the values that later layers mix with."""
         from ..ops import flash_attention as FA
         from ..ops import paged_attention as PA
+        from ..ops.qkv_prep import prepare_qkv
         from ..ops.residual_stream import project
 
         c = self.config
         T, D, Dv = x.shape[0], c.head_size, c.v_head_size
         nq, nk, nv = self.local_heads * D, self.local_kv * D, self.local_kv * Dv
-        fused = self._fused_projection() if (x.is_cuda and not torch.is_grad_enabled() and self.q_norm is None and self.rot is None) else None
+        fused = self._fused_projection() if (x.is_cuda and not torch.is_grad_enabled() and self.q_norm is None) else None
         gate = None
         if fused is not None:
-            y = project(x, fused)
+            y = project(x, fused[0], bias=fused[1])
             q, k, v = y[:, :nq].unflatten(1, (-1, D)), y[:, nq:nq + nk].unflatten(1, (-1, D)), y[:, nq + nk:nq + nk + nv].unflatten(1, (-1, Dv))
             if c.output_gate:
                 gate = y[:, nq + nk + nv:]
         else:
-            q, k, v = self._compute_qkv(x, pos_ids)
+            q, k, v = self._compute_qkv(x, pos_ids, rotate=False)
             if c.output_gate:
                 gate = self.g_proj(x)
-        PA.kv_page_write_general(kv_cache.kv_pages, k, v, batch_info.new_token_dests)
+        if self.rot is not None or c.head_temperature or c.value_mixing:
+            q, k, v = prepare_qkv(q, k, v, kv_cache.kv_pages, batch_info.new_token_dests, pos_ids, rot=self.rot,
+                                  head_scale=self.temperature if c.head_temperature else None, v_first=v_first,
+                                  mix=self.value_mix if c.value_mixing else None)
+            if c.value_mixing and v_first is None:
+                v_first = v
+        else:
+            PA.kv_page_write_general(kv_cache.kv_pages, k, v, batch_info.new_token_dests)
         scale = c.scaling_factor if c.scaling_factor is not None else 1.0 / math.sqrt(D)
         seg = getattr(batch_info, "prefill_segment_ids", None)
         if seg is not None and FA.packed_supported(q, k, v, scale):
             # pure prefill: every sequence starts at position 0, nothing is read back from the cache
-            out = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=scale, chunk=c.attention_chunk_size, gate=gate,
+            out = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=scale, chunk=c.attention_chunk_size, window=c.sliding_window, gate=gate,
                                             logits_soft_cap=c.logits_soft_cap)
         else:
-            out = PA.paged_attention_general(q, kv_cache.kv_pages, self.local_kv, Dv, batch_info, sm_scale=scale,
-                                             chunk=c.attention_chunk_size, gate=gate, soft_cap=c.logits_soft_cap)
-        return out.reshape(T, self.local_heads * Dv).to(x.dtype)
+            out = PA.paged_attention_general(q, kv_cache.kv_pages, self.local_kv, Dv, batch_info, sm_scale=scale, chunk=c.attention_chunk_size,
+                                             window=c.sliding_window, gate=gate, soft_cap=c.logits_soft_cap)
+        return out.reshape(T, self.local_heads * Dv).to(x.dtype), v_first
 
     def paged_decode_stream(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor):
         """:meth:`paged_decode` for an fp32 residual stream: ``stream + o_proj(heads)``, added in the projection's epilogue."""
         from ..ops.residual_stream import add_linear
 
-        out = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        out, _ = self._paged_heads(x, kv_cache, batch_info, pos_ids)
         if type(self.o_proj) is Linear and self.o_proj.bias is None:
             return add_linear(stream, out, self.o_proj.weight), kv_cache
         return stream + self.o_proj(out).float(), kv_cache
+
+    def paged_decode_mixing_values(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, v_first: Optional[torch.Tensor] = None):
+        """:meth:`paged_decode` of a block whose output is normed before it joins the stream: ``(o_proj(heads) in fp32, v_first)``, with
+        ``v_first`` as in :meth:`forward_mixing_values`."""
+        from ..ops.residual_stream import project
+
+        out, v_first = self._paged_heads(x, kv_cache, batch_info, pos_ids, v_first)
+        if type(self.o_proj) is Linear:
+            return project(out, self.o_proj.weight, bias=self.o_proj.bias, out_dtype=torch.float32), v_first
+        return self.o_proj(out).float(), v_first
 
     def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
         return KvPageCache.init(max_pages, page_size, self.local_kv, self.config.head_size, v_head_size=self.config.v_head_size, dtype=dtype,
@@ -654,6 +687,12 @@ class MultiHeadLatentAttentionConfig:
     rope: Optional[RotaryEmbeddingsConfig] = None
     scaling_factor: Optional[float] = None
     logits_soft_cap: Optional[float] = None
+    norm_eps: float = 1e-6
+    sliding_window: Optional[int] = None  # a query sees itself and that many positions less one before it
+
+    @property
+    def softmax_scale(self) -> float:
+        return self.scaling_factor if self.scaling_factor is not None else 1.0 / math.sqrt(self.qk_head_dim)
 
     @property
     def qk_head_dim(self):
@@ -662,7 +701,12 @@ class MultiHeadLatentAttentionConfig:
 
 class MultiHeadLatentAttention(nn.Module):
     """K/V are reconstructed from a low-rank latent (``kv_lora_rank``) plus a decoupled RoPE key shared by all heads;
-    queries optionally pass through their own low-rank bottleneck (src/levanter/layers/attention.py:2063-2213)."""
+    queries optionally pass through their own low-rank bottleneck (src/levanter/layers/attention.py:2063-2213).
+
+    Serving (:meth:`paged_decode`) caches the normed latent and the rotated key part of a token, ``kv_lora_rank + qk_rope_head_dim``
+    numbers for all heads.  Prompts that start in a step are attended to with per-head keys and values: one product of the cache
+    rows with ``[[W_uk, 0], [0, 1]]`` yields whole keys, the identity block putting the shared part into every head.  Otherwise
+    (decoding, portions) ``W_uk`` is applied to the queries and ``W_uv`` to the result, and the heads read the cache rows as they are."""
 
     def __init__(self, config: MultiHeadLatentAttentionConfig, init_std: float = 0.02):
         super().__init__()
@@ -675,17 +719,101 @@ class MultiHeadLatentAttention(nn.Module):
         else:
             self.q_proj = None
             self.q_a_proj = Linear(c.hidden_dim, c.q_lora_rank, bias=c.use_bias, init_std=init_std)
-            self.q_a_norm = RmsNorm(c.q_lora_rank)
+            self.q_a_norm = RmsNorm(c.q_lora_rank, eps=c.norm_eps)
             self.q_b_proj = Linear(c.q_lora_rank, H * c.qk_head_dim, bias=c.use_bias, init_std=init_std)
         self.kv_a_proj = Linear(c.hidden_dim, c.kv_lora_rank + c.qk_rope_head_dim, bias=c.use_bias, init_std=init_std)
-        self.kv_a_norm = RmsNorm(c.kv_lora_rank)
+        self.kv_a_norm = RmsNorm(c.kv_lora_rank, eps=c.norm_eps)
         self.kv_b_proj = Linear(c.kv_lora_rank, H * (c.qk_nope_head_dim + c.v_head_dim), bias=c.use_bias, init_std=init_std)
         self.o_proj = Linear(H * c.v_head_dim, c.hidden_dim, bias=c.use_bias, init_std=init_std)
         rope = c.rope if c.rope is not None else DefaultRotaryEmbeddingsConfig()
         self.rot = rope.build(c.qk_rope_head_dim)
+        self._rows, self._whole_kv = FusedRows(), None
+
+    def up_projections(self, weight: torch.Tensor):
+        """``(W_uk [H, qk_nope_head_dim, rank], W_uv [H, v_head_dim, rank])``: views of ``kv_b_proj``'s weight (or of its gradient and the
+        like)."""
+        c = self.config
+        w = weight.view(c.num_heads, c.qk_nope_head_dim + c.v_head_dim, c.kv_lora_rank)
+        return w[:, :c.qk_nope_head_dim], w[:, c.qk_nope_head_dim:]
+
+    def _whole_kv_weight(self) -> torch.Tensor:
+        """``[H * qk_head_dim + H * v_head_dim, rank + rope]``: rows that turn ``[c, k_rot]`` into every head's key and then every head's
+        value.  Derived from ``kv_b_proj``, made again when its weight has changed."""
+        c = self.config
+        w = self.kv_b_proj.weight
+        key = (w.data_ptr(), w._version, w.dtype, w.device)
+        if self._whole_kv is None or self._whole_kv[0] != key:
+            H, r, rank = c.num_heads, c.qk_rope_head_dim, c.kv_lora_rank
+            uk, uv = self.up_projections(w.detach())
+            keys = w.new_zeros(H, c.qk_head_dim, rank + r)
+            keys[:, :c.qk_nope_head_dim, :rank] = uk
+            keys[:, c.qk_nope_head_dim:, rank:] = torch.eye(r, dtype=w.dtype, device=w.device)
+            values = w.new_zeros(H, c.v_head_dim, rank + r)
+            values[..., :rank] = uv
+            self._whole_kv = (key, torch.cat([keys.flatten(0, 1), values.flatten(0, 1)]))
+        return self._whole_kv[1]
+
+    def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
+        c = self.config
+        return KvPageCache.init(max_pages, page_size, 1, c.kv_lora_rank + c.qk_rope_head_dim, v_head_size=0, dtype=dtype, device=device)
+
+    def paged_decode(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids: torch.Tensor) -> torch.Tensor:
+        """Packed rows ``x [T, hidden]`` of a serving step -> ``[T, hidden]`` in fp32; their latents enter the cache."""
+        from ..ops import flash_attention as FA
+        from ..ops import paged_attention as PA
+        from ..ops.qkv_prep import prepare_latent
+        from ..ops.residual_stream import project
+
+        c = self.config
+        if c.logits_soft_cap is not None or c.use_bias:
+            raise NotImplementedError("serving latent attention takes neither a soft cap nor biases")
+        T, H, dn, dr, dv, rank = x.shape[0], c.num_heads, c.qk_nope_head_dim, c.qk_rope_head_dim, c.v_head_dim, c.kv_lora_rank
+        nq = H * c.qk_head_dim
+        w = None
+        if self.q_proj is not None and type(self.q_proj) is Linear and type(self.kv_a_proj) is Linear and x.is_cuda and not self.training \
+                and not torch.is_grad_enabled():
+            w = self._rows.get([self.q_proj.weight, self.kv_a_proj.weight])
+        if w is not None:
+            y = project(x, w)
+            q, down = y[:, :nq], y[:, nq:]
+        else:
+            q = self.q_proj(x) if self.q_proj is not None else self.q_b_proj(self.q_a_norm(self.q_a_proj(x)))
+            down = self.kv_a_proj(x)
+        q = q.unflatten(1, (H, c.qk_head_dim))
+        pages, dests = kv_cache.kv_pages, batch_info.new_token_dests
+        norm = (self.kv_a_norm.weight, self.kv_a_norm.eps)
+        weight = self.kv_b_proj.weight
+        if getattr(batch_info, "prefill_segment_ids", None) is not None and self._packed_prefill_fits(q):
+            latent, _ = prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:])
+            kv = project(latent, self._whole_kv_weight())
+            k, v = kv[:, :nq].unflatten(1, (H, c.qk_head_dim)), kv[:, nq:].unflatten(1, (H, dv))
+            heads = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=c.softmax_scale, window=c.sliding_window)
+        else:
+            uk, uv = self.up_projections(weight)
+            qa = q.new_empty(T, H, rank + dr)
+            prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:], qa[..., rank:])
+            PA.head_product(q[..., :dn], uk.to(q.dtype), qa[..., :rank], b_trans=False)
+            o = PA.paged_attention_latent(qa, pages, rank, batch_info, sm_scale=c.softmax_scale, window=c.sliding_window)
+            heads = PA.head_product(o.to(q.dtype), uv.to(q.dtype), q.new_empty(T, H, dv), b_trans=True)
+        heads = heads.reshape(T, H * dv).to(x.dtype)
+        if type(self.o_proj) is Linear:
+            return project(heads, self.o_proj.weight, out_dtype=torch.float32)
+        return self.o_proj(heads).float()
+
+    def _packed_prefill_fits(self, q: torch.Tensor) -> bool:
+        """Whether the packed flash kernel takes this layer's sizes (the joint product of keys and values has the strides of its columns)."""
+        from ..ops.flash_attention import packed_rows_ok
+
+        c = self.config
+        return (packed_rows_ok(q, 192) and q.shape[0] % 256 == 0 and c.softmax_scale > 0.0 and c.v_head_dim % 8 == 0 and c.v_head_dim <= 128
+                and (c.kv_lora_rank + c.qk_rope_head_dim) % 8 == 0 and type(self.kv_b_proj) is Linear and self.kv_b_proj.weight.dtype == q.dtype
+                and not torch.is_grad_enabled())
 
     def forward(self, x, mask=None, pos_ids=None):
         c = self.config
+        if c.sliding_window is not None:
+            mask = (mask if isinstance(mask, AttentionMask) else AttentionMask.explicit(mask) if mask is not None
+                    else AttentionMask.causal()) & AttentionMask.causal(sliding_window=c.sliding_window)
         B, S, _ = x.shape
         H = c.num_heads
         if pos_ids is None:
@@ -701,7 +829,7 @@ class MultiHeadLatentAttention(nn.Module):
         k_rope = self.rot(k_rope.unsqueeze(2), pos_ids).expand(B, S, H, c.qk_rope_head_dim)
         qf = torch.cat([q_nope, q_rope], dim=-1)
         kf = torch.cat([k_nope, k_rope], dim=-1)
-        scale = c.scaling_factor if c.scaling_factor is not None else 1.0 / math.sqrt(c.qk_head_dim)
+        scale = c.softmax_scale
         # value head size differs from the qk head size, so pad V for the shared kernel interface
         out = simple_attention_with_dropout(qf, kf, F.pad(v, (0, c.qk_head_dim - c.v_head_dim)) if c.v_head_dim < c.qk_head_dim else v,
                                             mask, attention_dtype=torch.float32 if c.upcast_attn else None,
@@ -715,7 +843,8 @@ class MultiHeadLatentAttention(nn.Module):
 class KvPageCache:
     """Paged KV storage ``kv_pages[page, slot, 2 * kv_heads, head_size]`` with K at even and V at odd head index
     (src/levanter/layers/attention.py:1638-1707); with a value size of its own ``kv_pages[page, slot, kv_heads, head_size + v_head_size]``,
-    the same order in memory: per KV head a key row, then a value row."""
+    the same order in memory: per KV head a key row, then a value row.  Latent attention keeps one row for all heads, whose first
+    part is also the value (``v_head_size`` 0)."""
 
     kv_pages: torch.Tensor
 
@@ -741,6 +870,9 @@ class KvPageCache:
     def copy_page(self, src_page: int, dst_page: int) -> "KvPageCache":
         self.kv_pages[dst_page].copy_(self.kv_pages[src_page])
         return self
+
+    def copy_slot(self, src: int, dst: int) -> "KvPageCache":
+        return self  # nothing is kept by slots
 
 
 def default_ragged_paged_attention(q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, sm_scale: float = 1.0, soft_cap=None):

@@ -22,17 +22,37 @@ def rotate_half(x: torch.Tensor) -> torch.Tensor:
 
 
 class RotaryEmbeddings:
-    """Callable that rotates ``q`` (``[..., pos, heads..., head_dim]`` with positions given explicitly)."""
+    """Callable that rotates ``q`` (``[..., pos, heads..., head_dim]`` with positions given explicitly).
 
-    def __init__(self, head_dim: int, inv_freq: torch.Tensor, position_scale: float = 1.0, temperature: float = 1.0):
+    The first ``rotary_dim = 2 * len(inv_freq)`` dimensions of a head turn, the rest pass.  Dimension ``i`` is paired with ``i +
+    rotary_dim / 2``, or, ``interleaved``, ``2i`` with ``2i + 1``."""
+
+    def __init__(self, head_dim: int, inv_freq: torch.Tensor, position_scale: float = 1.0, temperature: float = 1.0, interleaved: bool = False):
         self.head_dim = head_dim
-        self.inv_freq = inv_freq.float()  # [head_dim // 2]
+        self.inv_freq = inv_freq.float()  # [rotary_dim // 2]
         self.position_scale = position_scale
         self.temperature = temperature
+        self.interleaved = interleaved
         self._cache: dict = {}
 
+    @property
+    def rotary_dim(self) -> int:
+        return 2 * self.inv_freq.shape[0]
+
+    @property
+    def is_plain(self) -> bool:
+        """Whole heads in the half-split layout: what the tables of :meth:`cos_sin` and :meth:`table` describe."""
+        return self.rotary_dim == self.head_dim and not self.interleaved
+
+    def frequencies_on(self, device) -> torch.Tensor:
+        """``inv_freq`` on a device, kept: its address goes into captured graphs."""
+        key = ("inv_freq", str(device))
+        if key not in self._cache:
+            self._cache[key] = self.inv_freq.to(device).contiguous()
+        return self._cache[key]
+
     def cos_sin(self, position_ids: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
-        """cos, sin of shape ``position_ids.shape + [head_dim]`` in fp32."""
+        """cos, sin of shape ``position_ids.shape + [rotary_dim]`` in fp32 (half-split layout)."""
         inv = self.inv_freq.to(position_ids.device)
         freqs = (position_ids.float() * self.position_scale).unsqueeze(-1) * inv
         emb = torch.cat((freqs, freqs), dim=-1)
@@ -52,8 +72,17 @@ class RotaryEmbeddings:
         cos, sin = self.cos_sin(position_ids)
         cos = cos.unsqueeze(-2)
         sin = sin.unsqueeze(-2)
-        out = q.float() * cos + rotate_half(q.float()) * sin
-        return out.to(q.dtype)
+        r = self.rotary_dim
+        x = q[..., :r].float()
+        if self.interleaved:
+            half = r // 2
+            cos, sin = cos[..., :half], sin[..., :half]
+            u, v = x[..., 0::2], x[..., 1::2]
+            out = torch.stack((u * cos - v * sin, v * cos + u * sin), dim=-1).flatten(-2)
+        else:
+            out = x * cos + rotate_half(x) * sin
+        out = out.to(q.dtype)
+        return out if r == q.shape[-1] else torch.cat((out, q[..., r:]), dim=-1)
 
 
 def _base_inv_freq(theta: float, head_dim: int) -> torch.Tensor:
@@ -91,11 +120,18 @@ class RotaryEmbeddingsConfig(ChoiceRegistry):
 class DefaultRotaryEmbeddingsConfig(RotaryEmbeddingsConfig):
     theta: float = 10000
     factor: float = 1.0
+    rotary_dim: Optional[int] = None  # the first dimensions of a head that turn; None: all
+    interleaved: bool = False         # dimension 2i is paired with 2i + 1, not i with i + rotary_dim / 2
 
     def build(self, head_dim: int) -> RotaryEmbeddings:
-        return RotaryEmbeddings(head_dim, _base_inv_freq(self.theta, head_dim) / self.factor)
+        r = self.rotary_dim if self.rotary_dim is not None else head_dim
+        if r % 2 != 0 or not 0 < r <= head_dim:
+            raise ValueError(f"cannot rotate {r} of {head_dim} dimensions")
+        return RotaryEmbeddings(head_dim, _base_inv_freq(self.theta, r) / self.factor, interleaved=self.interleaved)
 
     def to_hf_config(self):
+        if self.rotary_dim is not None or self.interleaved:
+            raise ValueError("a partial or interleaved rotation has no Hugging Face rope config")
         if self.factor == 1.0:
             return self.theta, None
         return self.theta, {"rope_type": "linear", "factor": self.factor}

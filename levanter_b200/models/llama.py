@@ -21,9 +21,10 @@ from ..compat.hf_checkpoints import HFCheckpointConverter, HFCompatConfig
 from ..layers.attention import Attention, AttentionBackend, AttentionConfig, AttentionMask, KvPageCache
 from ..layers.normalization import LayerNormConfigBase, RmsNormConfig
 from ..layers.rotary import rope_config_from_hf, rope_to_hf_dict, DefaultRotaryEmbeddingsConfig, RotaryEmbeddingsConfig
-from ..nn import Embedding, Linear
+from ..nn import Embedding, FusedRows, Linear
 from ..ops.gemm import linear_residual
 from ..ops.glu import gated_activation
+from ..ops.residual_stream import glu_of_rows, project
 from ..utils.activation import ActivationFunctionEnum
 from ..utils.flop_utils import lm_flops_per_token
 from ..utils.remat import ScanCheckpointPolicy, checkpoint_layer, keeps_attention, should_recompute
@@ -161,6 +162,22 @@ class LlamaMlp(nn.Module):
         self.up_proj = Linear(hidden, local, bias=use_bias, init_std=init_std, parallel=("column", tp))
         self.down_proj = Linear(local, hidden, bias=use_bias, init_std=init_std, parallel=("row", tp))
         self.act = activation if isinstance(activation, ActivationFunctionEnum) else ActivationFunctionEnum(activation)
+        self._rows = FusedRows()
+
+    def forward_fp32(self, x: torch.Tensor) -> torch.Tensor:
+        """The MLP of packed rows ``x [T, hidden]`` in fp32 straight from the last product, for blocks whose output is normed before it
+        joins an fp32 stream; gate and up are one product when serving (no biases, tanh-gelu or any activation of ``ops.glu``)."""
+        mods = (self.gate_proj, self.up_proj)
+        w = None
+        if all(type(m) is Linear and m.bias is None for m in mods) and x.is_cuda and not self.training and not torch.is_grad_enabled():
+            w = self._rows.get([m.weight for m in mods])
+        if w is not None:
+            h = glu_of_rows(project(x, w), self.gate_proj.weight.shape[0], self.act)
+        else:
+            h = gated_activation(self.gate_proj(x), self.up_proj(x), self.act)
+        if type(self.down_proj) is Linear:
+            return project(h, self.down_proj.weight, bias=self.down_proj.bias, out_dtype=torch.float32)
+        return self.down_proj(h).float()
 
     def forward(self, x: torch.Tensor, residual: Optional[torch.Tensor] = None) -> torch.Tensor:
         if self.tp is not None and self.tp.size > 1:

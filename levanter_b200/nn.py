@@ -75,6 +75,40 @@ class Linear(nn.Module):
         return f"in={self.in_features}, out={self.out_features}, bias={self.bias is not None}"
 
 
+class FusedRows:
+    """One matrix (or vector) whose row slices are the given parameters: projections that read the same rows become one product when
+    a model serves, and nothing is stored twice.  :meth:`get` returns it, building it first when the parameters are not (or, after
+    a move or a conversion, no longer) its slices; None for parameters in training, which belong to the gradient engine's own
+    flat buffers.  ``pad``: zero rows at the end."""
+
+    def __init__(self, pad: int = 0):
+        self.pad = pad
+        self._fused: Optional[torch.Tensor] = None
+
+    def get(self, params: Sequence[torch.Tensor]) -> Optional[torch.Tensor]:
+        if any(getattr(p, "main_grad", None) is not None or getattr(p, "grad_sink", None) is not None for p in params):
+            return None
+        fused = self._fused
+        if fused is not None:
+            at = fused.data_ptr()
+            for p in params:
+                if p.data_ptr() != at or p.dtype != fused.dtype:
+                    fused = None
+                    break
+                at += p.numel() * p.element_size()
+        if fused is None:
+            rows = [p.detach() for p in params]
+            if self.pad:
+                rows.append(rows[0].new_zeros(self.pad, *rows[0].shape[1:]))
+            fused = torch.cat(rows)
+            at = 0
+            for p in params:
+                p.data = fused[at:at + p.shape[0]]
+                at += p.shape[0]
+            self._fused = fused
+        return fused
+
+
 class Embedding(nn.Module):
     """Token embedding ``weight[vocab, embed]`` with ``unembed`` for tied LM heads."""
 
@@ -133,6 +167,13 @@ class RmsNorm(nn.Module):
         from .ops.norm import rms_norm
 
         return rms_norm(x, self.weight, self.bias, self.eps)
+
+    def from_stream(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The norm of an fp32 residual stream, in the weight's dtype (``rows``: of these rows only)."""
+        from .ops.residual_stream import rms_norm_stream
+
+        assert self.weight is not None and self.bias is None
+        return rms_norm_stream(x, self.weight, self.eps, rows=rows)
 
 
 class LayerNorm(nn.Module):

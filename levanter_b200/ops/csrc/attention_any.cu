@@ -1,8 +1,8 @@
 // Paged attention and cache writes without restrictions on the element type or the sizes: fp32 serving, and bf16 models whose
 // head sizes the tensor-core kernels do not take (not a multiple of 8, above 256, more than 16 query heads per KV head).
 //
-// Same semantics as lvb_paged_attention_general (paged_attention.cu): packed query rows, pages, an optional chunk size and an
-// optional output gate.  Everything is fp32 arithmetic whatever the storage type (this file is built without fast-math).
+// Same semantics as lvb_paged_attention_general (paged_attention.cu): packed query rows, pages, an optional chunk size or window and
+// an optional output gate; and of lvb_paged_latent (paged_latent.cu), where a key's first columns are its value.  Everything is fp32 arithmetic whatever the storage type (this file is built without fast-math).
 // One CTA per (query row, query head) walks the visible keys in blocks: a key per thread for the scores, an online softmax over
 // the block, then an output column per thread for P V.
 #include "common.cuh"
@@ -50,14 +50,15 @@ __global__ void kv_write_vec_kernel(uint4* __restrict__ kv_pages, const uint4* _
 
 struct Params {
   const void* q;
-  const void* kv_pages;  // [num_pages, page_size, KV, dk + dv]
+  const void* kv_pages;  // [num_pages, page_size, KV, row]
   const int* kv_lens;
   const int* page_indices;
   const int* cu_q_lens;
   const int* num_seqs;
   const void* gate;
   void* out;
-  int T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages, chunk;
+  int T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages, chunk, window;
+  int row, v_at;         // elements of a KV head's row, and where in it the value starts
   long long ldq, ldg;
   float scale, soft_cap;
 };
@@ -100,8 +101,9 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
   const T* q = reinterpret_cast<const T*>(p.q) + t * p.ldq + static_cast<long long>(h) * p.dk;
   for (int d = threadIdx.x; d < p.dk; d += kThreads) s_q[d] = to_f<T>(q[d]);
   for (int d = threadIdx.x; d < p.dv; d += kThreads) s_o[d] = 0.f;
-  const int lo = p.chunk > 0 ? ctx - 1 - (ctx - 1) % p.chunk : 0;
-  const long long per = p.dk + p.dv;
+  int lo = p.chunk > 0 ? ctx - 1 - (ctx - 1) % p.chunk : 0;
+  if (p.window > 0) lo = max(lo, ctx - p.window);
+  const long long per = p.row;
   const T* pages = reinterpret_cast<const T*>(p.kv_pages);
   float m = -INFINITY, l = 0.f;
   for (int k0 = lo; k0 < ctx; k0 += kThreads) {
@@ -132,7 +134,7 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
       float acc = s_o[d] * alpha;
       for (int i = 0; i < nk; ++i) {
         const int sl = s_slot[i];
-        if (sl >= 0) acc = fmaf(s_p[i], to_f<T>(pages[(static_cast<long long>(sl) * p.KV + kvh) * per + p.dk + d]), acc);
+        if (sl >= 0) acc = fmaf(s_p[i], to_f<T>(pages[(static_cast<long long>(sl) * p.KV + kvh) * per + p.v_at + d]), acc);
       }
       s_o[d] = acc;
     }
@@ -172,18 +174,21 @@ extern "C" int lvb_kv_page_write_general(void* kv_pages, const void* k, const vo
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
+// window > 0: a query sees itself and the window - 1 positions before it.  shared: a KV head's row holds dk elements only and its first dv are
+// the value (dv <= dk).
 extern "C" int lvb_attention_any(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices, const int* cu_q_lens,
                                  const int* num_seqs, const void* gate, void* out, int T, int H, int KV, int dk, int dv, long long ldq,
-                                 long long ldg, int S, int pages_per_seq, int page_size, int num_pages, int chunk, float scale,
-                                 float soft_cap, int is_f32, void* stream) {
+                                 long long ldg, int S, int pages_per_seq, int page_size, int num_pages, int chunk, int window,
+                                 int shared, float scale, float soft_cap, int is_f32, void* stream) {
   using namespace lvb;
   using namespace lvb::any;
   if (T <= 0) return kErrOk;
-  if (H <= 0 || KV <= 0 || H % KV != 0 || dk <= 0 || dv <= 0 || S <= 0 || chunk < 0) return kErrBadArg;
+  if (H <= 0 || KV <= 0 || H % KV != 0 || dk <= 0 || dv <= 0 || S <= 0 || chunk < 0 || window < 0) return kErrBadArg;
+  if (shared && dv > dk) return kErrBadArg;
   const size_t smem = (static_cast<size_t>(dk) + dv + 2 * kThreads + kThreads / 32) * 4;
   if (smem > 48 * 1024) return kErrTooLarge;
   Params p{q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, gate, out, T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages,
-           chunk, ldq, ldg, scale, soft_cap};
+           chunk, window, shared ? dk : dk + dv, shared ? 0 : dk, ldq, ldg, scale, soft_cap};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (is_f32) attention_any_kernel<float><<<dim3(T, H), kThreads, smem, s>>>(p);
   else attention_any_kernel<__nv_bfloat16><<<dim3(T, H), kThreads, smem, s>>>(p);

@@ -13,10 +13,11 @@
 //
 // kPacked (lvb_flash_attn_fwd_packed) is the form the inference engine prefills with: packed sequences, each starting at
 // position 0.  What a row sees is one contiguous range of packed keys, so the mask is a lower bound per row computed from its
-// position (the start of its sequence, or of its chunk when attention is chunked) instead of a segment id per key: blocks
-// between the bound and the diagonal need no mask at all.  Key and value sizes may differ and need not be 64 or 128: the tensor
-// maps are three-dimensional (size, head, row), columns past the size arrive as zeros, and the MMAs stop at the next
-// multiple of 16.  An optional gate is applied to the output on its way out.
+// position (the start of its sequence, of its chunk when attention is chunked, or of its window) instead of a segment id per
+// key: blocks between the bound and the diagonal need no mask at all.  Key and value sizes may differ and need not be 64 or
+// 128: the tensor maps are three-dimensional (size, head, row), columns past the size arrive as zeros, and the MMAs stop at
+// the next multiple of 16.  Keys of up to 192 leave shared memory for one V stage only.  An optional gate is applied to the
+// output on its way out.
 #include "common.cuh"
 
 namespace lvb {
@@ -45,19 +46,22 @@ struct Params {
   int* status;
   // ---- kPacked
   const int* pos;            // [S]: position of each packed row in its sequence
-  int chunk;                 // > 0: a row at position i sees positions >= i - i % chunk only
+  int chunk;                 // > 0: a row at position i sees positions >= i - i % chunk only (window, above: positions > i - window)
   int dk, dv;                // query/key and value sizes (multiples of 8, at most HD)
   const __nv_bfloat16* gate; // optional [S, Hq * dv] (row stride ldg): the output is multiplied by its sigmoid
   long long ldg;
 };
 
-template <int HD>
+// HDK, HDV: room for the query/key and the value size
+template <int HDK, int HDV>
 struct SmemT {
-  static constexpr int kQKV = 128 * HD * 2;                   // a [128 rows, HD] tile: HD / 64 chunks of 64 columns
+  static constexpr int kQKTile = 128 * HDK * 2;               // a [128 rows, HDK] tile: HDK / 64 chunks of 64 columns
+  static constexpr int kVTile = 128 * HDV * 2;
+  static constexpr int kVStages = HDK > 128 ? 1 : kStages;
   static constexpr int kQ = 0;                                // 2 tiles
-  static constexpr int kK = kQ + 2 * kQKV;
-  static constexpr int kV = kK + kStages * kQKV;
-  static constexpr int kBars = kV + kStages * kQKV;
+  static constexpr int kK = kQ + 2 * kQKTile;
+  static constexpr int kV = kK + kStages * kQKTile;
+  static constexpr int kBars = kV + kVStages * kVTile;
   static constexpr int kNumBars = 1 + 4 * kStages + 2 + 2 + 2;
   static constexpr int kTotal = kBars + kNumBars * 8 + 16 + 1024;
 };
@@ -71,16 +75,16 @@ __device__ __forceinline__ float to_log2(float s, float scale_log2, float scale,
 // kPacked: first packed key that row qi sees
 __device__ __forceinline__ int row_lower_bound(const Params& p, int qi) {
   const int pos = p.pos[qi];
-  return qi - (p.chunk > 0 ? pos % p.chunk : pos);
+  const int back = p.chunk > 0 ? pos % p.chunk : pos;
+  return qi - (p.window > 0 ? min(back, p.window - 1) : back);
 }
 
-template <int HD, bool kSeg, bool kCap, bool kPacked = false>
+template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, Params p) {
-  using Smem = SmemT<HD>;
-  constexpr int D = HD;
-  constexpr int kQKV = Smem::kQKV;
+  using Smem = SmemT<HDK, HDV>;
+  constexpr int kQKTile = Smem::kQKTile, kVTile = Smem::kVTile, kVStages = Smem::kVStages;
   const bool causal = p.causal != 0;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -107,7 +111,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   // without the causal part there is no diagonal block (the mask test below never matches -1) and both tiles see every block
   const int jdiagA = causal ? 2 * cb : -1, jdiagB = causal ? 2 * cb + 1 : -1;
   int jlo = 0;
-  if (p.window > 0) {
+  if (!kPacked && p.window > 0) {
     const int first_key = q0 - p.window + 1;
     jlo = first_key > 0 ? first_key / BT : 0;
   }
@@ -152,16 +156,16 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       const int row_q = b * p.S + q0;
-      const int ck = kPacked ? (p.dk + 63) / 64 : D / 64, cv = kPacked ? (p.dv + 63) / 64 : D / 64;  // 64-column chunks
+      const int ck = kPacked ? (p.dk + 63) / 64 : HDK / 64, cv = kPacked ? (p.dv + 63) / 64 : HDV / 64;  // 64-column chunks
       mbar_expect_tx(q_full, 2 * ck * kChunkBytes);
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c)
+        for (int c = 0; c < HDK / 64; ++c)
           if constexpr (kPacked) {
-            if (c < ck) tma_load_3d(smem + Smem::kQ + t * kQKV + c * kChunkBytes, &tmQ, q_full, 64 * c, h, row_q + t * BT);
+            if (c < ck) tma_load_3d(smem + Smem::kQ + t * kQKTile + c * kChunkBytes, &tmQ, q_full, 64 * c, h, row_q + t * BT);
           } else
-          tma_load_2d(smem + Smem::kQ + t * kQKV + c * kChunkBytes, &tmQ, q_full, h * D + 64 * c, row_q + t * BT);
+          tma_load_2d(smem + Smem::kQ + t * kQKTile + c * kChunkBytes, &tmQ, q_full, h * HDK + 64 * c, row_q + t * BT);
       bool ok = true;
       for (int it = 0; it < nB && ok; ++it) {
         const int st = it % kStages;
@@ -169,24 +173,25 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int row_k = b * p.Sk + (jlo + it) * BT;
         ok = mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 1200, it);
         if (!ok) break;
-        uint8_t* ks = smem + Smem::kK + st * kQKV;
+        uint8_t* ks = smem + Smem::kK + st * kQKTile;
         mbar_expect_tx(&k_full[st], ck * kChunkBytes);
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c)
+        for (int c = 0; c < HDK / 64; ++c)
           if constexpr (kPacked) {
             if (c < ck) tma_load_3d(ks + c * kChunkBytes, &tmK, &k_full[st], 64 * c, hkv, row_k);
           } else
-          tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * D + 64 * c, row_k);
-        ok = mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, 1201, it);
+          tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * HDK + 64 * c, row_k);
+        const int sv = it % kVStages;
+        ok = mbar_wait(&v_empty[sv], ((it / kVStages) & 1) ^ 1, abort_flag, p.status, 1201, it);
         if (!ok) break;
-        uint8_t* vs = smem + Smem::kV + st * kQKV;
-        mbar_expect_tx(&v_full[st], cv * kChunkBytes);
+        uint8_t* vs = smem + Smem::kV + sv * kVTile;
+        mbar_expect_tx(&v_full[sv], cv * kChunkBytes);
 #pragma unroll
-        for (int c = 0; c < D / 64; ++c)
+        for (int c = 0; c < HDV / 64; ++c)
           if constexpr (kPacked) {
-            if (c < cv) tma_load_3d(vs + c * kChunkBytes, &tmV, &v_full[st], 64 * c, hkv, row_k);
+            if (c < cv) tma_load_3d(vs + c * kChunkBytes, &tmV, &v_full[sv], 64 * c, hkv, row_k);
           } else
-          tma_load_2d(vs + c * kChunkBytes, &tmV, &v_full[st], hkv * D + 64 * c, row_k);
+          tma_load_2d(vs + c * kChunkBytes, &tmV, &v_full[sv], hkv * HDV + 64 * c, row_k);
       }
     }
   } else if (warp == 1) {
@@ -194,17 +199,17 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc_bf16(BT, BT, false, false);
       // A = P in TMEM, B = V MN-major
-      const uint32_t idesc_pv = make_idesc_bf16(BT, kPacked ? (p.dv + 15) / 16 * 16 : D, false, true);
-      const int qk_steps = kPacked ? (p.dk + 15) / 16 : D / 16;
+      const uint32_t idesc_pv = make_idesc_bf16(BT, kPacked ? (p.dv + 15) / 16 * 16 : HDV, false, true);
+      const int qk_steps = kPacked ? (p.dk + 15) / 16 : HDK / 16;
       const uint32_t sq = smem_u32(smem + Smem::kQ);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1300, 0);
 
       auto qk = [&](int tile, int it) {
         const int st = it % kStages;
-        const uint32_t sk = smem_u32(smem + Smem::kK + st * kQKV);
-        const uint32_t sqt = sq + tile * kQKV;
+        const uint32_t sk = smem_u32(smem + Smem::kK + st * kQKTile);
+        const uint32_t sqt = sq + tile * kQKTile;
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < HDK / 16; ++kk) {
           if (kPacked && kk >= qk_steps) break;
           const uint32_t off = (kk >> 2) * kChunkBytes + (kk & 3) * 32;
           umma_bf16_ss(tmem_base + tile * BT, make_smem_desc(sqt + off, 16, 1024), make_smem_desc(sk + off, 16, 1024),
@@ -213,17 +218,16 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         umma_commit(&s_full[tile]);
       };
       auto pv = [&](int tile, int it) {
-        const int st = it % kStages;
-        const uint32_t sv = smem_u32(smem + Smem::kV + st * kQKV);
+        const uint32_t sv = smem_u32(smem + Smem::kV + (it % kVStages) * kVTile);
 #pragma unroll
         for (int kk = 0; kk < BT / 16; ++kk) {
           // 16 keys of P = 8 TMEM columns; 16 keys of V = two 8-row groups = 2048 B
-          umma_bf16_ts(tmem_base + 2 * BT + tile * D, tmem_base + tile * BT + kk * 8,
+          umma_bf16_ts(tmem_base + 2 * BT + tile * HDV, tmem_base + tile * BT + kk * 8,
                        make_smem_desc(sv + kk * 2048, kChunkBytes, 1024), idesc_pv, (it > 0 || kk > 0) ? 1u : 0u);
         }
       };
       auto wait_k = [&](int it) { return mbar_wait(&k_full[it % kStages], (it / kStages) & 1, abort_flag, p.status, 1301, it); };
-      auto wait_v = [&](int it) { return mbar_wait(&v_full[it % kStages], (it / kStages) & 1, abort_flag, p.status, 1302, it); };
+      auto wait_v = [&](int it) { return mbar_wait(&v_full[it % kVStages], (it / kVStages) & 1, abort_flag, p.status, 1302, it); };
 
       if (ok) ok = wait_k(0);
       if (ok) {
@@ -233,7 +237,6 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         umma_commit(&k_empty[0]);
       }
       for (int it = 0; it < nB && ok; ++it) {
-        const int st = it % kStages;
         ok = wait_v(it);
         if (!ok) break;
         if (it < nA) {
@@ -254,7 +257,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         if (!ok) break;
         tc_fence_after();
         pv(1, it);
-        umma_commit(&v_empty[st]);
+        umma_commit(&v_empty[it % kVStages]);
         if (it == nB - 1) umma_commit(&o_done[1]);
         if (more) {
           qk(1, it + 1);
@@ -272,7 +275,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int nT = tile == 0 ? nA : nB;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t tS = tmem_base + tile * BT + lane_addr;
-    const uint32_t tO = tmem_base + 2 * BT + tile * D + lane_addr;
+    const uint32_t tO = tmem_base + 2 * BT + tile * HDV + lane_addr;
     const float scale_log2 = p.scale * kLog2e;
     const int my_seg = kSeg ? p.q_seg[b * p.S + qi] : 0;
     const int* kseg_row = kSeg ? p.k_seg + b * p.Sk : nullptr;
@@ -291,7 +294,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const bool need_mask = (j == jdiag) || kSeg || (kPacked && k0 < tile_lo) || (p.window > 0 && k0 <= q0 + tile * BT + BT - 1 - p.window);
+      const bool need_mask = (j == jdiag) || kSeg || (kPacked && k0 < tile_lo) || (!kPacked && p.window > 0 && k0 <= q0 + tile * BT + BT - 1 - p.window);
 
       // ---- pass 1: row maximum (raw logits; the scale is positive and the soft-cap monotonic)
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -305,7 +308,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           for (int t = 0; t < 32; ++t) {
             const int kj = k0 + c + t;
             bool valid = !causal || kj <= qi;
-            if (p.window > 0) valid = valid && (qi - kj < p.window);
+            if (!kPacked && p.window > 0) valid = valid && (qi - kj < p.window);
             if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
             if (kPacked) valid = valid && kj >= row_lo;
             if (!valid) v[t] = __float_as_uint(-INFINITY);
@@ -333,7 +336,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           const float alpha = scale_row ? exp2f(m_used - m_new) : 1.f;
           l_sum *= alpha;
 #pragma unroll 1
-          for (int c = 0; c < D; c += 32) {
+          for (int c = 0; c < HDV; c += 32) {
             uint32_t v[32];
             tmem_ld_32x32(tO + c, v);
             tmem_ld_wait();
@@ -359,7 +362,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           for (int t = 0; t < 32; ++t) {
             const int kj = k0 + c + t;
             bool valid = !causal || kj <= qi;
-            if (p.window > 0) valid = valid && (qi - kj < p.window);
+            if (!kPacked && p.window > 0) valid = valid && (qi - kj < p.window);
             if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
             if (kPacked) valid = valid && kj >= row_lo;
             const float x = kCap ? to_log2<kCap>(__uint_as_float(v[t]), scale_log2, p.scale, p.soft_cap) + neg_m
@@ -445,9 +448,9 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           }
         }
       } else {
-      __nv_bfloat16* orow = p.O + (static_cast<size_t>(b) * p.S + qi) * (static_cast<size_t>(p.Hq) * D) + static_cast<size_t>(h) * D;
+      __nv_bfloat16* orow = p.O + (static_cast<size_t>(b) * p.S + qi) * (static_cast<size_t>(p.Hq) * HDV) + static_cast<size_t>(h) * HDV;
 #pragma unroll 1
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < HDV; c += 32) {
         uint32_t v[32];
         tmem_ld_32x32(tO + c, v);
         tmem_ld_wait();
@@ -474,10 +477,11 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   }
 }
 
-template <int HD, bool kSeg, bool kCap, bool kPacked = false>
+template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false>
 int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const Params& p, cudaStream_t st) {
-  using Smem = SmemT<HD>;
-  auto kern = flash_fwd2_kernel<HD, kSeg, kCap, kPacked>;
+  using Smem = SmemT<HDK, HDV>;
+  static_assert(Smem::kTotal <= 227 * 1024, "shared memory of one CTA");
+  auto kern = flash_fwd2_kernel<HDK, HDV, kSeg, kCap, kPacked>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem::kTotal) != cudaSuccess) return kErrCuda;
@@ -506,10 +510,10 @@ int launch_hd(const void* q, const void* k, const void* v, const Params& p, cuda
   if (rc != kErrOk) return rc;
   const bool seg = p.q_seg != nullptr;
   const bool cap = p.soft_cap > 0.f;
-  if (seg && cap) return launch<HD, true, true>(tmQ, tmK, tmV, p, st);
-  if (seg) return launch<HD, true, false>(tmQ, tmK, tmV, p, st);
-  if (cap) return launch<HD, false, true>(tmQ, tmK, tmV, p, st);
-  return launch<HD, false, false>(tmQ, tmK, tmV, p, st);
+  if (seg && cap) return launch<HD, HD, true, true>(tmQ, tmK, tmV, p, st);
+  if (seg) return launch<HD, HD, true, false>(tmQ, tmK, tmV, p, st);
+  if (cap) return launch<HD, HD, false, true>(tmQ, tmK, tmV, p, st);
+  return launch<HD, HD, false, false>(tmQ, tmK, tmV, p, st);
 }
 }  // namespace fa2
 }  // namespace lvb
@@ -554,21 +558,22 @@ extern "C" int lvb_flash_attn_fwd2(const void* q, const void* k, const void* v, 
 //   q: row t, head h at q + t * ldq + h * dk     k / v: row t, head g at k + t * ldk + g * dk, v + t * ldv + g * dv
 //   o[T, Hq, dv] = softmax(scale q k^T over the visible keys) v  (* sigmoid(gate[t, h, :]))
 // pos[t] is the row's position in its sequence (padding rows: 0).  chunk > 0: positions are cut into chunks of that many, counted
-// from the sequence's start, and a row sees its own chunk only.  dk, dv: multiples of 8, at most 128; ldq, ldk, ldv and ldg
+// from the sequence's start, and a row sees its own chunk only; window > 0: a row sees itself and the window - 1 positions before
+// it.  dk, dv: multiples of 8, at most 192 and 128; ldq, ldk, ldv and ldg
 // multiples of 8 and the pointers 16-byte aligned.
 extern "C" int lvb_flash_attn_fwd_packed(const void* q, const void* k, const void* v, const void* gate, void* o, const int* pos, int T,
-                                         int Hq, int Hkv, int dk, int dv, int ldq, int ldk, int ldv, int ldg, int chunk, float scale,
-                                         float soft_cap, int* status, void* stream) {
+                                         int Hq, int Hkv, int dk, int dv, int ldq, int ldk, int ldv, int ldg, int chunk, int window,
+                                         float scale, float soft_cap, int* status, void* stream) {
   using namespace lvb;
   using namespace lvb::fa2;
-  if (T <= 0 || (T % (2 * BT)) != 0 || Hq <= 0 || Hkv <= 0 || (Hq % Hkv) != 0 || pos == nullptr || chunk < 0) return kErrBadArg;
-  if (dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || (dk & 7) || (dv & 7) || (ldg & 7) || !(scale > 0.f)) return kErrBadArg;
+  if (T <= 0 || (T % (2 * BT)) != 0 || Hq <= 0 || Hkv <= 0 || (Hq % Hkv) != 0 || pos == nullptr || chunk < 0 || window < 0) return kErrBadArg;
+  if (dk <= 0 || dv <= 0 || dk > 192 || dv > 128 || (dk & 7) || (dv & 7) || (ldg & 7) || !(scale > 0.f)) return kErrBadArg;
   if ((reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(o) & 15)) return kErrBadArg;
   Params p;
   p.O = reinterpret_cast<__nv_bfloat16*>(o);
   p.lse2 = nullptr; p.q_seg = nullptr; p.k_seg = nullptr; p.kblock_lo = nullptr; p.sink = nullptr;
   p.B = 1; p.S = T; p.Sk = T; p.Hq = Hq; p.Hkv = Hkv;
-  p.scale = scale; p.soft_cap = soft_cap; p.window = 0; p.causal = 1; p.status = status;
+  p.scale = scale; p.soft_cap = soft_cap; p.window = window; p.causal = 1; p.status = status;
   p.pos = pos; p.chunk = chunk; p.dk = dk; p.dv = dv;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
   CUtensorMap tmQ, tmK, tmV;
@@ -578,7 +583,10 @@ extern "C" int lvb_flash_attn_fwd_packed(const void* q, const void* k, const voi
   if (rc != kErrOk) return rc;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool small = dk <= 64 && dv <= 64;
-  if (soft_cap > 0.f)
-    return small ? launch<64, false, true, true>(tmQ, tmK, tmV, p, st) : launch<128, false, true, true>(tmQ, tmK, tmV, p, st);
-  return small ? launch<64, false, false, true>(tmQ, tmK, tmV, p, st) : launch<128, false, false, true>(tmQ, tmK, tmV, p, st);
+  if (soft_cap > 0.f) {
+    if (dk > 128) return launch<192, 128, false, true, true>(tmQ, tmK, tmV, p, st);
+    return small ? launch<64, 64, false, true, true>(tmQ, tmK, tmV, p, st) : launch<128, 128, false, true, true>(tmQ, tmK, tmV, p, st);
+  }
+  if (dk > 128) return launch<192, 128, false, false, true>(tmQ, tmK, tmV, p, st);
+  return small ? launch<64, 64, false, false, true>(tmQ, tmK, tmV, p, st) : launch<128, 128, false, false, true>(tmQ, tmK, tmV, p, st);
 }

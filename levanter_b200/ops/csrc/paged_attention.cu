@@ -79,12 +79,16 @@ struct Params {
   // ---- general form (lvb_paged_attention_general); the plain entry point sets dk = dv = D, chunk = 0, no gate
   int dk, dv;                 // query/key and value sizes; a cache slot holds, per KV head, dk key and dv value elements
   int chunk;                  // > 0: a query at position i sees positions >= i - i % chunk only
+  int window;                 // > 0: a query at position i sees positions > i - window only
   long long ldq, ldg;         // row strides of q and gate
   const __nv_bfloat16* gate;  // optional [T, H * dv]: the output is multiplied by its sigmoid
 };
 
 // First visible key of a query whose context (its position + 1) is ctx.
-__device__ __forceinline__ int first_key(const Params& p, int ctx) { return p.chunk > 0 ? ctx - 1 - (ctx - 1) % p.chunk : 0; }
+__device__ __forceinline__ int first_key(const Params& p, int ctx) {
+  const int lo = p.chunk > 0 ? ctx - 1 - (ctx - 1) % p.chunk : 0;
+  return p.window > 0 ? max(lo, ctx - p.window) : lo;
+}
 
 __device__ __forceinline__ float gate_factor(const Params& p, int t, int h, int d) {
   if (p.gate == nullptr) return 1.f;
@@ -825,7 +829,7 @@ extern "C" int lvb_paged_attention(const void* q, const void* kv_pages, const in
   p.T = T; p.H = H; p.KV = KV; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;
   p.parts = lvb_paged_attention_parts(pages_per_seq * page_size);
   p.scale = scale; p.soft_cap = soft_cap;
-  p.dk = p.dv = D; p.chunk = 0; p.ldq = static_cast<long long>(H) * D; p.gate = nullptr; p.ldg = 0;
+  p.dk = p.dv = D; p.chunk = 0; p.window = 0; p.ldq = static_cast<long long>(H) * D; p.gate = nullptr; p.ldg = 0;
   if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (D) {
@@ -837,25 +841,27 @@ extern "C" int lvb_paged_attention(const void* q, const void* kv_pages, const in
 }
 
 // Partitions of keys per query of lvb_paged_attention_general: sizes part_o fp32 [T, H, parts, dv] and part_ml fp32 [T, H, parts, 2].
-extern "C" int lvb_paged_attention_general_parts(int max_context, int chunk) {
-  const int keys = chunk > 0 && chunk < max_context ? chunk : max_context;
+extern "C" int lvb_paged_attention_general_parts(int max_context, int chunk, int window) {
+  int keys = chunk > 0 && chunk < max_context ? chunk : max_context;
+  keys = window > 0 && window < keys ? window : keys;
   return (keys + lvb::paged::kPart - 1) / lvb::paged::kPart;
 }
 
 // lvb_paged_attention for any key and value size up to 256 (multiples of 8), with
 //   * kv_pages [num_pages, page_size, KV, dk + dv]: a key row followed by a value row per KV head,
 //   * chunk > 0: positions are cut into chunks of that many, counted from the sequence's start, and a query sees its own chunk,
+//   * window > 0: a query sees itself and the window - 1 positions before it,
 //   * gate (optional, [T, H * dv], row stride ldg): the output is multiplied by its sigmoid,
 //   * ldq: row stride of q.  At most 16 query heads per KV head.
 extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices,
                                            const int* cu_q_lens, const int* num_seqs, const void* gate, void* out, float* part_o,
                                            float* part_ml, int T, int H, int KV, int dk, int dv, int ldq, int ldg, int S,
-                                           int pages_per_seq, int page_size, int num_pages, int chunk, float scale, float soft_cap,
-                                           void* stream) {
+                                           int pages_per_seq, int page_size, int num_pages, int chunk, int window, float scale,
+                                           float soft_cap, void* stream) {
   using namespace lvb;
   using namespace lvb::paged;
   if (T <= 0) return kErrOk;
-  if (H <= 0 || KV <= 0 || H % KV != 0 || H / KV > kMaxG || S <= 0 || chunk < 0) return kErrBadArg;
+  if (H <= 0 || KV <= 0 || H % KV != 0 || H / KV > kMaxG || S <= 0 || chunk < 0 || window < 0) return kErrBadArg;
   if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || (dk & 7) || (dv & 7) || (ldq & 1)) return kErrBadArg;
   Params p;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
@@ -864,9 +870,9 @@ extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, 
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml;
   p.T = T; p.H = H; p.KV = KV; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;
-  p.parts = lvb_paged_attention_general_parts(pages_per_seq * page_size, chunk);
+  p.parts = lvb_paged_attention_general_parts(pages_per_seq * page_size, chunk, window);
   p.scale = scale; p.soft_cap = soft_cap;
-  p.dk = dk; p.dv = dv; p.chunk = chunk; p.ldq = ldq; p.ldg = ldg;
+  p.dk = dk; p.dv = dv; p.chunk = chunk; p.window = window; p.ldq = ldq; p.ldg = ldg;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);

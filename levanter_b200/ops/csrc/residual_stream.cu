@@ -1,6 +1,7 @@
 // The two ends of a pre-norm block whose residual stream is kept in fp32: the token embedding that starts it and the RMS norm that
-// reads it.  (The adds in between ride in the epilogues of the projections, which accumulate into the stream.)  Built without
-// fast-math: norms of a 32-bit stream are 32-bit arithmetic throughout.
+// reads it.  (The adds in between ride in the epilogues of the projections, which accumulate into the stream.)  Where a block's
+// output is normed before it is added, one kernel does both and the next block's norm.  Also here: the gated activation for fp32
+// and for sizes that are not multiples of 8.  Built without fast-math: norms of a 32-bit stream are 32-bit arithmetic throughout.
 #include "common.cuh"
 
 namespace lvb {
@@ -77,6 +78,86 @@ rms_kernel(const float* __restrict__ x, const long long* __restrict__ rows, cons
   }
 }
 
+// x[r, :] += rms(y[r, :]) * w_post, then h[d, :] = rms(x[r, :]) * w_next, for r = rows[d] (or d).  With `rows` the stream is read only:
+// the sum is what the last norm of a model sees.  The row stays in shared memory between the passes.
+__global__ void __launch_bounds__(256)
+add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const long long* __restrict__ rows, const void* __restrict__ w_post,
+                const void* __restrict__ w_next, int w_f32, void* __restrict__ h, int h_f32, int dim, float eps, int vec) {
+  extern __shared__ __align__(16) float s_row[];  // [dim]
+  __shared__ float s_red[2][8];
+  const size_t src = static_cast<size_t>(rows != nullptr ? rows[blockIdx.x] : blockIdx.x) * dim;
+  const size_t dst = static_cast<size_t>(blockIdx.x) * dim;
+  auto block_sum = [&](float v, int slot) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) s_red[slot][threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+    for (int i = 0; i < static_cast<int>(blockDim.x) / 32; ++i) t += s_red[slot][i];
+    return t;
+  };
+  const float n = static_cast<float>(dim);
+  float ss = 0.f;
+  if (vec) {
+    for (int c = threadIdx.x * 4; c < dim; c += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(y + src + c);
+      *reinterpret_cast<float4*>(s_row + c) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+      const float v = y[src + c];
+      s_row[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+  }
+  const float r1 = 1.f / sqrtf(block_sum(ss, 0) / n + eps);
+  ss = 0.f;
+  if (vec) {  // every thread reads back the columns that it wrote
+    for (int c = threadIdx.x * 4; c < dim; c += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(s_row + c), g = ld4(w_post, w_f32, c);
+      float4 o = *reinterpret_cast<const float4*>(x + src + c);
+      o.x += v.x * r1 * g.x; o.y += v.y * r1 * g.y; o.z += v.z * r1 * g.z; o.w += v.w * r1 * g.w;
+      *reinterpret_cast<float4*>(s_row + c) = o;
+      if (rows == nullptr) *reinterpret_cast<float4*>(x + src + c) = o;
+      ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, fmaf(o.w, o.w, ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+      const float o = x[src + c] + s_row[c] * r1 * ld1(w_post, w_f32, c);
+      s_row[c] = o;
+      if (rows == nullptr) x[src + c] = o;
+      ss = fmaf(o, o, ss);
+    }
+  }
+  const float r2 = 1.f / sqrtf(block_sum(ss, 1) / n + eps);
+  if (vec) {
+    for (int c = threadIdx.x * 4; c < dim; c += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(s_row + c), g = ld4(w_next, w_f32, c);
+      const float4 o = make_float4(v.x * r2 * g.x, v.y * r2 * g.y, v.z * r2 * g.z, v.w * r2 * g.w);
+      if (h_f32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(h) + dst + c) = o;
+      else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(h) + dst + c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    }
+  } else {
+    for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+      const float o = s_row[c] * r2 * ld1(w_next, w_f32, c);
+      if (h_f32) reinterpret_cast<float*>(h)[dst + c] = o;
+      else reinterpret_cast<__nv_bfloat16*>(h)[dst + c] = __float2bfloat16(o);
+    }
+  }
+}
+
+// out[r, c] = gelu(gate[r, c]) * up[r, c] with the tanh form of gelu, any size and either type
+__global__ void gelu_glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, void* __restrict__ out, int f32, long long total,
+                                int cols, long long ldg, long long ldu) {
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / cols, c = i - r * cols;
+    const float g = ld1(gate, f32, r * ldg + c), u = ld1(up, f32, r * ldu + c);
+    const float o = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    if (f32) reinterpret_cast<float*>(out)[i] = o;
+    else reinterpret_cast<__nv_bfloat16*>(out)[i] = __float2bfloat16(o);
+  }
+}
+
 inline int threads_for(int dim) {
   const int t = ((dim + 3) / 4 + 31) / 32 * 32;
   return t < 32 ? 32 : t > 256 ? 256 : t;
@@ -103,5 +184,35 @@ extern "C" int lvb_rms_stream(const float* x, const long long* rows, const void*
   const int vec = (dim & 3) == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
   stream32::rms_kernel<<<n_rows, stream32::threads_for(dim), 0, reinterpret_cast<cudaStream_t>(stream)>>>(x, rows, w, w_f32, y, y_f32, dim, eps,
                                                                                                        w_offset, vec);
+  return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+}
+
+// x[rows] += rms(y) * w_post; h = rms(x) * w_next.  x, y fp32 [.., dim]; w_f32: type of both weights; h [n_rows, dim] fp32 or bf16.  rows: null, or
+// int64 [n_rows] source rows (each in range), and then x is left as it is.
+extern "C" int lvb_add_norm_stream(float* x, const float* y, const long long* rows, const void* w_post, const void* w_next, int w_f32, void* h,
+                                   int h_f32, int n_rows, int dim, float eps, void* stream) {
+  using namespace lvb;
+  if (n_rows <= 0 || dim <= 0) return kErrBadArg;
+  const size_t smem = static_cast<size_t>(dim) * 4;
+  if (smem > 200 * 1024) return kErrTooLarge;
+  if (smem > 40 * 1024 &&
+      cudaFuncSetAttribute(stream32::add_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+    return kErrCuda;
+  const uintptr_t mis = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w_post) |
+                        reinterpret_cast<uintptr_t>(w_next) | reinterpret_cast<uintptr_t>(h);
+  const int vec = (dim & 3) == 0 && (mis & 15) == 0;
+  stream32::add_norm_kernel<<<n_rows, stream32::threads_for(dim), smem, reinterpret_cast<cudaStream_t>(stream)>>>(x, y, rows, w_post, w_next, w_f32,
+                                                                                                             h, h_f32, dim, eps, vec);
+  return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+}
+
+// out [rows, cols] = gelu_tanh(gate) * up; gate and up with row strides ldg and ldu; f32: type of all three.
+extern "C" int lvb_gelu_glu_any(const void* gate, const void* up, void* out, int f32, int rows, int cols, long long ldg, long long ldu, void* stream) {
+  using namespace lvb;
+  if (rows <= 0 || cols <= 0) return kErrBadArg;
+  const long long total = static_cast<long long>(rows) * cols, cap = static_cast<long long>(num_sms()) * 16;
+  long long blocks = (total + 255) / 256;
+  if (blocks > cap) blocks = cap;
+  stream32::gelu_glu_kernel<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, out, f32, total, cols, ldg, ldu);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }

@@ -48,24 +48,26 @@ _packed = {}
 
 
 def packed_supported(q, k, v, scale: float) -> bool:
-    """Shapes :func:`flash_attention_packed` takes: bf16 rows on a B200, sizes that are multiples of 8 up to 128, a positive scale
-    (the running maximum is taken over unscaled scores) and 16-byte aligned rows."""
-    if not (q.is_cuda and lib.available()) or any(t.dtype != torch.bfloat16 for t in (q, k, v)):
-        return False
-    ok = all(t.shape[2] % 8 == 0 and t.shape[2] <= 128 and t.stride(2) == 1 and t.stride(1) == t.shape[2] and t.stride(0) % 8 == 0
-             and t.data_ptr() % 16 == 0 for t in (q, k, v))
-    return ok and q.shape[0] % 256 == 0 and scale > 0.0
+    """Shapes :func:`flash_attention_packed` takes: bf16 rows on a B200, sizes that are multiples of 8 (keys up to 192, values up to 128), a
+    positive scale (the running maximum is taken over unscaled scores) and 16-byte aligned rows."""
+    return packed_rows_ok(q, 192) and packed_rows_ok(k, 192) and packed_rows_ok(v, 128) and q.shape[0] % 256 == 0 and scale > 0.0
 
 
-def flash_attention_packed(q, k, v, pos, *, scaling_factor: float, chunk: Optional[int] = None, gate=None,
+def packed_rows_ok(t: torch.Tensor, most: int) -> bool:
+    """Rows ``t [T, heads, size]`` that the packed kernel's tensor maps can describe, with a size of at most ``most``."""
+    return (t.is_cuda and lib.available() and t.dtype == torch.bfloat16 and t.shape[2] % 8 == 0 and t.shape[2] <= most and t.stride(2) == 1
+            and t.stride(1) == t.shape[2] and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0)
+
+
+def flash_attention_packed(q, k, v, pos, *, scaling_factor: float, chunk: Optional[int] = None, window: Optional[int] = None, gate=None,
                            logits_soft_cap: Optional[float] = None) -> torch.Tensor:
     """Causal attention over packed rows of sequences that start at position 0: ``q [T, Hq, dk]``, ``k [T, Hkv, dk]``, ``v [T, Hkv, dv]``
     (slices of one wider row are fine), ``pos [T]`` int32 positions with padding rows at 0, ``T`` a multiple of 256 ->
-    ``[T, Hq, dv]``.  ``chunk``: a row sees its own chunk of that many positions only.  ``gate [T, Hq * dv]``: the result is
-    multiplied by its sigmoid.  Forward only; shapes as in :func:`packed_supported`."""
+    ``[T, Hq, dv]``.  ``chunk``: a row sees its own chunk of that many positions only.  ``window``: a row sees itself and the
+    ``window - 1`` positions before it.  ``gate [T, Hq * dv]``: the result is multiplied by its sigmoid.  Forward only; shapes as in :func:`packed_supported`."""
     c = lib
     if "f" not in _packed:
-        _packed["f"] = lib.fn("lvb_flash_attn_fwd_packed", [c.c_void_p] * 6 + [c.c_int] * 10 + [c.c_float, c.c_float, c.c_void_p, c.c_void_p])
+        _packed["f"] = lib.fn("lvb_flash_attn_fwd_packed", [c.c_void_p] * 6 + [c.c_int] * 11 + [c.c_float, c.c_float, c.c_void_p, c.c_void_p])
     T, Hq, dk = q.shape
     Hkv, dv = v.shape[1], v.shape[2]
     pos = pos.to(torch.int32).contiguous()
@@ -76,7 +78,7 @@ def flash_attention_packed(q, k, v, pos, *, scaling_factor: float, chunk: Option
         ldg = gate.stride(0)
     out = torch.empty(T, Hq, dv, dtype=torch.bfloat16, device=q.device)
     rc = _packed["f"](q.data_ptr(), k.data_ptr(), v.data_ptr(), lib.ptr(gate), out.data_ptr(), pos.data_ptr(), T, Hq, Hkv, dk, dv, q.stride(0),
-                      k.stride(0), v.stride(0), ldg, int(chunk or 0), float(scaling_factor), float(logits_soft_cap or 0.0),
+                      k.stride(0), v.stride(0), ldg, int(chunk or 0), int(window or 0), float(scaling_factor), float(logits_soft_cap or 0.0),
                       lib.status_buffer().data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_flash_attn_fwd_packed")
     return out

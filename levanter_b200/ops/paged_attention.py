@@ -89,7 +89,7 @@ def _paged_attention_cuda(q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seq
 
 
 # ------------------------------------------------------------------------------------------------ general form
-# Key and value sizes of their own, attention within chunks of positions, an output gate, fp32.  The cache of a layer is then viewed
+# Key and value sizes of their own, attention within chunks of positions or a sliding window, an output gate, fp32.  The cache of a layer is then viewed
 # as [page, slot, kv_head, k_size + v_size], which for equal sizes is the memory of [page, slot, 2 * kv_head, size].
 def _kv_view(kv_pages: torch.Tensor, kv_heads: int, k_size: int, v_size: int) -> torch.Tensor:
     return kv_pages.view(kv_pages.shape[0], kv_pages.shape[1], kv_heads, k_size + v_size)
@@ -122,17 +122,19 @@ def kv_page_write_general(kv_pages: torch.Tensor, new_k: torch.Tensor, new_v: to
 
 
 def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: int, v_size: int, batch_info, *, sm_scale: float,
-                            chunk: Optional[int] = None, gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None) -> torch.Tensor:
+                            chunk: Optional[int] = None, window: Optional[int] = None, gate: Optional[torch.Tensor] = None,
+                            soft_cap: Optional[float] = None) -> torch.Tensor:
     """:func:`ragged_paged_attention` of ``q [T, H, k_size]`` (rows may be strided) over pages of ``kv_heads * (k_size + v_size)``
     elements per slot -> ``[T, H, v_size]``.
 
     ``chunk``: positions are cut into chunks of that many, counted from the start of the sequence, and a query sees the keys of
-    its own chunk only.  ``gate [T, H * v_size]``: the result is multiplied by its sigmoid.  bf16 with sizes that are multiples of 8
+    its own chunk only.  ``window``: a query sees itself and the ``window - 1`` positions before it.  ``gate [T, H * v_size]``: the result is multiplied by its sigmoid.  bf16 with sizes that are multiples of 8
     up to 256 and at most 16 query heads per KV head runs on tensor cores; everything else in fp32 arithmetic."""
     T, H, dk = q.shape
     b = batch_info
     if not _use_kernel(q, kv_pages):
-        return paged_attention_general_reference(q, kv_pages, kv_heads, v_size, b, sm_scale=sm_scale, chunk=chunk, gate=gate, soft_cap=soft_cap)
+        return paged_attention_general_reference(q, kv_pages, kv_heads, v_size, b, sm_scale=sm_scale, chunk=chunk, window=window, gate=gate,
+                                                 soft_cap=soft_cap)
     kv = _kv_view(kv_pages, kv_heads, dk, v_size)
     if kv.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"the cache must be bf16 or fp32, got {kv.dtype}")
@@ -153,26 +155,31 @@ def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: i
     tensor_cores = (q.dtype == torch.bfloat16 and dk % 8 == 0 and v_size % 8 == 0 and max(dk, v_size) <= 256 and H // kv_heads <= 16
                     and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0)
     if not tensor_cores:
-        if "any" not in _f:
-            _f["any"] = lib.fn("lvb_attention_any", [c.c_void_p] * 8 + [c.c_int] * 5 + [c.c_longlong] * 2 + [c.c_int] * 5 +
-                               [c.c_float, c.c_float, c.c_int, c.c_void_p])
-        rc = _f["any"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), T, H,
-                       kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), float(sm_scale), float(soft_cap or 0.0),
-                       int(q.dtype == torch.float32), lib.stream_ptr())
+        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), T, H,
+                       kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), int(window or 0), 0, float(sm_scale),
+                       float(soft_cap or 0.0), int(q.dtype == torch.float32), lib.stream_ptr())
         lib.check_rc(rc, "lvb_attention_any")
         return out
     if "g" not in _f:
-        _f["g"] = lib.fn("lvb_paged_attention_general", [c.c_void_p] * 10 + [c.c_int] * 12 + [c.c_float, c.c_float, c.c_void_p], launches=2)
-        _f["gparts"] = lib.fn("lvb_paged_attention_general_parts", [c.c_int, c.c_int], launches=0)
-    parts = _f["gparts"](PP * ps, int(chunk or 0))
+        _f["g"] = lib.fn("lvb_paged_attention_general", [c.c_void_p] * 10 + [c.c_int] * 13 + [c.c_float, c.c_float, c.c_void_p], launches=2)
+        _f["gparts"] = lib.fn("lvb_paged_attention_general_parts", [c.c_int] * 3, launches=0)
+    parts = _f["gparts"](PP * ps, int(chunk or 0), int(window or 0))
     po = pml = None
     if parts > 1:
         po, pml = _part_scratch(dev, T * H * parts * v_size, T * H * parts * 2)
     rc = _f["g"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), lib.ptr(po),
-                 lib.ptr(pml), T, H, kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), float(sm_scale),
-                 float(soft_cap or 0.0), lib.stream_ptr())
+                 lib.ptr(pml), T, H, kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), int(window or 0),
+                 float(sm_scale), float(soft_cap or 0.0), lib.stream_ptr())
     lib.check_rc(rc, "lvb_paged_attention_general")
     return out
+
+
+def _any_fn():
+    if "any" not in _f:
+        c = lib
+        _f["any"] = lib.fn("lvb_attention_any", [c.c_void_p] * 8 + [c.c_int] * 5 + [c.c_longlong] * 2 + [c.c_int] * 7 +
+                           [c.c_float, c.c_float, c.c_int, c.c_void_p])
+    return _f["any"]
 
 
 _part = {}
@@ -192,11 +199,14 @@ def _part_scratch(dev, n_o: int, n_ml: int):
 
 
 def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, batch_info, *, sm_scale: float, chunk: Optional[int] = None,
-                                      gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None) -> torch.Tensor:
-    """PyTorch statement of :func:`paged_attention_general` (CPU path and test oracle)."""
+                                      window: Optional[int] = None, gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None,
+                                      shared: bool = False) -> torch.Tensor:
+    """PyTorch statement of :func:`paged_attention_general` (CPU path and test oracle).  ``shared``: a KV head's row is its key, whose
+    first ``v_size`` elements are the value."""
     T, H, dk = q.shape
     b = batch_info
-    kv_all = _kv_view(kv_pages, kv_heads, dk, v_size)
+    kv_all = _kv_view(kv_pages, kv_heads, dk, 0 if shared else v_size)
+    v_at = 0 if shared else dk
     ps = kv_all.shape[1]
     G = H // kv_heads
     out = torch.zeros(T, H, v_size, dtype=torch.float32, device=q.device)
@@ -206,7 +216,7 @@ def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, b
         if q1 <= q0 or kl <= 0 or kl == INVALID:
             continue
         n = (kl + ps - 1) // ps
-        kv = kv_all[b.page_indices[i, :n].long()].reshape(n * ps, kv_heads, dk + v_size)[:kl].float()
+        kv = kv_all[b.page_indices[i, :n].long()].reshape(n * ps, kv_heads, -1)[:kl].float()
         s = torch.einsum("qkgd,skd->kgqs", q[q0:q1].float().view(q1 - q0, kv_heads, G, dk), kv[..., :dk]) * sm_scale
         if soft_cap:
             s = torch.tanh(s / soft_cap) * soft_cap
@@ -215,11 +225,72 @@ def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, b
         see = kpos[None, :] <= qpos[:, None]
         if chunk:
             see = see & (kpos[None, :] // chunk == qpos[:, None] // chunk)
+        if window:
+            see = see & (qpos[:, None] - kpos[None, :] < window)
         p = torch.softmax(s.masked_fill(~see, -float("inf")), dim=-1)
-        out[q0:q1] = torch.einsum("kgqs,skd->qkgd", p, kv[..., dk:]).reshape(q1 - q0, H, v_size)
+        out[q0:q1] = torch.einsum("kgqs,skd->qkgd", p, kv[..., v_at:v_at + v_size]).reshape(q1 - q0, H, v_size)
     if gate is not None:
         out = out * torch.sigmoid(gate.float()).view(T, H, v_size)
     return out.to(q.dtype)
+
+
+# ------------------------------------------------------------------------------------------------ latent form
+def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, batch_info, *, sm_scale: float,
+                           window: Optional[int] = None) -> torch.Tensor:
+    """Causal attention of ``q [T, H, width]`` over pages of ``width`` elements per slot whose first ``rank`` are the value: all heads read
+    the same row per key -> ``[T, H, rank]``.  ``window`` as in :func:`paged_attention_general`.  bf16 with sizes that are multiples of
+    8 (rank up to 512, width up to 640) runs on tensor cores; everything else in fp32 arithmetic."""
+    T, H, w = q.shape
+    b = batch_info
+    if not _use_kernel(q, kv_pages):
+        return paged_attention_general_reference(q, kv_pages, 1, rank, b, sm_scale=sm_scale, window=window, shared=True)
+    kv = kv_pages.view(kv_pages.shape[0], kv_pages.shape[1], w)
+    if kv.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"the cache must be bf16 or fp32, got {kv.dtype}")
+    q = q.to(kv.dtype).contiguous()
+    c = lib
+    P, ps = kv.shape[:2]
+    S, PP = b.page_indices.shape
+    dev = q.device
+    i32 = lambda t: t.to(device=dev, dtype=torch.int32).contiguous()  # noqa: E731
+    lens, pages, cu, ns = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
+    out = torch.empty(T, H, rank, dtype=q.dtype, device=dev)
+    if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 640:
+        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), 0, out.data_ptr(), T, H, 1, w, rank,
+                       H * w, 0, S, PP, ps, P, 0, int(window or 0), 1, float(sm_scale), 0.0, int(q.dtype == torch.float32), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_attention_any")
+        return out
+    if "l" not in _f:
+        _f["l"] = lib.fn("lvb_paged_latent", [c.c_void_p] * 9 + [c.c_int] * 10 + [c.c_float, c.c_void_p], launches=2)
+        _f["lparts"] = lib.fn("lvb_paged_latent_parts", [c.c_int] * 4, launches=0)
+    parts = _f["lparts"](T, H, PP * ps, int(window or 0))
+    po = pml = None
+    if parts > 1:
+        po, pml = _part_scratch(dev, T * H * parts * rank, T * H * parts * 2)
+    rc = _f["l"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), out.data_ptr(), lib.ptr(po), lib.ptr(pml), T,
+                 H, w, rank, S, PP, ps, P, int(window or 0), parts, float(sm_scale), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_paged_latent")
+    return out
+
+
+def head_product(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, *, b_trans: bool) -> torch.Tensor:
+    """``out[t, h] = a[t, h] b[h]`` (``b [H, K, N]``) or ``a[t, h] b[h]^T`` (``b_trans``, ``b [H, N, K]``) for ``a [T, H, K]``, written into
+    ``out [T, H, N]``; all three may be strided views with packed last dimensions."""
+    T, H, K = a.shape
+    N = out.shape[2]
+    kernel = (_use_kernel(a, b, out) and a.dtype == b.dtype == out.dtype == torch.bfloat16 and a.stride(2) == b.stride(2) == out.stride(2) == 1
+              and not any(v % 8 for v in (N, K, a.stride(0), a.stride(1), b.stride(0), b.stride(1), out.stride(0), out.stride(1)))
+              and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0)
+    if not kernel:
+        out.copy_(torch.matmul(a.transpose(0, 1), b.transpose(1, 2) if b_trans else b).transpose(0, 1))
+        return out
+    c = lib
+    if "hp" not in _f:
+        _f["hp"] = lib.fn("lvb_head_product", [c.c_void_p] * 3 + [c.c_int] * 4 + [c.c_longlong] * 6 + [c.c_int, c.c_void_p])
+    rc = _f["hp"](a.data_ptr(), b.data_ptr(), out.data_ptr(), T, H, N, K, a.stride(0), a.stride(1), b.stride(1), b.stride(0), out.stride(0), out.stride(1),
+                  int(b_trans), lib.stream_ptr())
+    lib.check_rc(rc, "lvb_head_product")
+    return out
 
 
 def ragged_paged_attention_reference(q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, sm_scale: float = 1.0,

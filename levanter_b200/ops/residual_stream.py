@@ -1,7 +1,8 @@
-"""Pre-norm blocks around an fp32 residual stream (``csrc/residual_stream.cu`` and the GEMM epilogues).
+"""Pre-norm (and pre- and post-normed) blocks around an fp32 residual stream (``csrc/residual_stream.cu`` and the GEMM epilogues).
 
 The stream ``x`` is an fp32 tensor whatever the model's compute dtype: the embedding starts it, RMS norms read it and hand the
-compute dtype to the projections, and the projections that end a block accumulate into it in their epilogue.  The kernels run
+compute dtype to the projections, and the projections that end a block accumulate into it in their epilogue.  Where a block's output is normed before it is added, the projection
+hands it over in fp32 and :func:`add_norm_stream` norms it, adds it and norms the sum for the next block.  The kernels run
 when no gradient is being recorded; with autograd the same steps are PyTorch ops on an fp32 stream, and on the CPU they are the
 PyTorch statements only."""
 from __future__ import annotations
@@ -10,8 +11,10 @@ from typing import Optional
 
 import torch
 
+from ..utils.activation import ActivationFunctionEnum
 from . import lib
 from .gemm import gemm, linear
+from .glu import gated_activation
 
 _f = {}
 
@@ -66,6 +69,47 @@ def rms_norm_stream(x: torch.Tensor, weight: torch.Tensor, eps: float, *, w_offs
     return y.to(dt)
 
 
+def add_norm_stream(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float, *,
+                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Adds ``rms_norm(y) * w_post`` to the fp32 stream ``x`` in place and returns ``rms_norm(x) * w_next`` in the weights' dtype.
+    ``rows``: the norm of these rows only; ``x`` is then left as it is (the last norm of a model)."""
+    if _kernels(x, y, w_post, w_next) and x.dtype == y.dtype == torch.float32 and w_post.dtype == w_next.dtype and x.is_contiguous() \
+            and w_post.dtype in (torch.float32, torch.bfloat16) and y.is_contiguous() and w_post.is_contiguous() and w_next.is_contiguous():
+        c = lib
+        if "an" not in _f:
+            _f["an"] = lib.fn("lvb_add_norm_stream", [c.c_void_p] * 5 + [c.c_int, c.c_void_p] + [c.c_int] * 3 + [c.c_float, c.c_void_p])
+        D = x.shape[-1]
+        if rows is not None:
+            rows = rows.to(torch.int64).contiguous()
+        n = x.numel() // D if rows is None else rows.numel()
+        h = torch.empty(n, D, dtype=w_next.dtype, device=x.device)
+        f32 = int(w_next.dtype == torch.float32)
+        rc = _f["an"](x.data_ptr(), y.data_ptr(), lib.ptr(rows), w_post.data_ptr(), w_next.data_ptr(), f32, h.data_ptr(), f32, n, D, float(eps),
+                      lib.stream_ptr())
+        lib.check_rc(rc, "lvb_add_norm_stream")
+        return h.view(*x.shape[:-1], D) if rows is None else h
+    if rows is not None:
+        x, y = x.index_select(0, rows.long()), y.index_select(0, rows.long())
+    x.add_(rms_norm_stream(y.float(), w_post, eps, out_dtype=torch.float32))
+    return rms_norm_stream(x, w_next, eps)
+
+
+def glu_of_rows(y: torch.Tensor, cols: int, act: ActivationFunctionEnum) -> torch.Tensor:
+    """``act(y[:, :cols]) * y[:, cols:]`` of the joint product of a gate and an up projection."""
+    gate, up = y[:, :cols], y[:, cols:]
+    if act == ActivationFunctionEnum.gelu_new and _kernels(y) and not (y.dtype == torch.bfloat16 and cols % 8 == 0) \
+            and y.dtype in (torch.float32, torch.bfloat16):
+        c = lib
+        if "g" not in _f:
+            _f["g"] = lib.fn("lvb_gelu_glu_any", [c.c_void_p] * 3 + [c.c_int] * 3 + [c.c_longlong] * 2 + [c.c_void_p])
+        out = torch.empty(y.shape[0], cols, dtype=y.dtype, device=y.device)
+        rc = _f["g"](gate.data_ptr(), up.data_ptr(), out.data_ptr(), int(y.dtype == torch.float32), y.shape[0], cols, y.stride(0), y.stride(0),
+                     lib.stream_ptr())
+        lib.check_rc(rc, "lvb_gelu_glu_any")
+        return out
+    return gated_activation(gate, up, act)
+
+
 def _gemm_ok(h: torch.Tensor, w: torch.Tensor) -> bool:
     """The tcgen05 GEMM takes the product (forward only: the output size is free, the inner size a multiple of 8)."""
     return h.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] % 8 == 0
@@ -85,17 +129,18 @@ def add_linear(x: torch.Tensor, h: torch.Tensor, weight: torch.Tensor) -> torch.
     return x + linear(h, weight).float()
 
 
-def project(h: torch.Tensor, weight: torch.Tensor, *, squared_relu: bool = False, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """``h W^T`` (``max(., 0)^2`` of it), in ``h``'s dtype or in fp32 straight from the accumulator."""
+def project(h: torch.Tensor, weight: torch.Tensor, *, bias: Optional[torch.Tensor] = None, squared_relu: bool = False,
+            out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``h W^T + b`` (``max(., 0)^2`` of it), in ``h``'s dtype or in fp32 straight from the accumulator."""
     if _kernels(h, weight) and _gemm_ok(h, weight):
         h2 = h.reshape(-1, h.shape[-1])
-        y = gemm(h2, weight, out_dtype=out_dtype or h.dtype, squared_relu=squared_relu)
+        y = gemm(h2, weight, out_dtype=out_dtype or h.dtype, bias=bias, squared_relu=squared_relu)
         return y.view(*h.shape[:-1], weight.shape[0])
     if out_dtype == torch.float32 and h.dtype != torch.float32:
         # sizes the GEMM does not take (or with autograd, or on the CPU): the product itself in fp32
-        y = torch.nn.functional.linear(h.float(), weight.float())
+        y = torch.nn.functional.linear(h.float(), weight.float(), None if bias is None else bias.float())
     else:
-        y = linear(h, weight)
+        y = linear(h, weight, bias)
         if out_dtype is not None:
             y = y.to(out_dtype)
     return torch.relu(y).square() if squared_relu else y

@@ -82,7 +82,7 @@ def apply_rope(q: torch.Tensor, k: torch.Tensor, rot: RotaryEmbeddings, pos_ids=
     position per token (``[B, S]`` / ``[T]``)."""
     D = q.shape[-1]
     S = q.shape[-3]
-    if q.is_cuda and lib.available() and q.dtype == torch.bfloat16 and D % 16 == 0:
+    if q.is_cuda and lib.available() and q.dtype == torch.bfloat16 and D % 16 == 0 and rot.is_plain:
         tokens = q.numel() // (q.shape[-2] * D)
         if pos_ids is None:
             cos, sin = rot.table(S, q.device)
