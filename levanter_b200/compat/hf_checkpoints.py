@@ -148,7 +148,7 @@ def load_hf_state_dict(model: nn.Module, state_dict: Dict[str, torch.Tensor], *,
     with torch.no_grad():
         for name, p in model.named_parameters():
             if hasattr(model, "hf_tensor_parts"):
-                found = [(n, view, shape, lookup(n)) for n, view, shape in model.hf_tensor_parts(name, p.data)]
+                found = [(n, view, shape, lookup(n)) for n, view, shape in model.hf_tensor_parts(name, p.detach())]
                 if any(t is None for *_, t in found):
                     missing.append(name)
                     continue

@@ -604,7 +604,7 @@ class Attention(nn.Module):
                 gate = self.g_proj(x)
         if self.rot is not None or c.head_temperature or c.value_mixing:
             q, k, v = prepare_qkv(q, k, v, kv_cache.kv_pages, batch_info.new_token_dests, pos_ids, rot=self.rot,
-                                  head_scale=self.temperature if c.head_temperature else None, v_first=v_first,
+                                  head_scale=self.temperature if c.head_temperature else None, v_first=v_first if c.value_mixing else None,
                                   mix=self.value_mix if c.value_mixing else None)
             if c.value_mixing and v_first is None:
                 v_first = v
@@ -738,7 +738,8 @@ class MultiHeadLatentAttention(nn.Module):
 
     def _whole_kv_weight(self) -> torch.Tensor:
         """``[H * qk_head_dim + H * v_head_dim, rank + rope]``: rows that turn ``[c, k_rot]`` into every head's key and then every head's
-        value.  Derived from ``kv_b_proj``, made again when its weight has changed."""
+        value.  Derived from ``kv_b_proj``; made again when its weight has moved or changed, and after every change of mode (an optimizer
+        writes into flat buffers behind the parameters)."""
         c = self.config
         w = self.kv_b_proj.weight
         key = (w.data_ptr(), w._version, w.dtype, w.device)
@@ -752,6 +753,10 @@ class MultiHeadLatentAttention(nn.Module):
             values[..., :rank] = uv
             self._whole_kv = (key, torch.cat([keys.flatten(0, 1), values.flatten(0, 1)]))
         return self._whole_kv[1]
+
+    def train(self, mode: bool = True):
+        self._whole_kv = None
+        return super().train(mode)
 
     def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
         c = self.config

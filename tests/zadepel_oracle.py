@@ -170,7 +170,7 @@ def random_weights(cfg, seed=0, dtype=torch.bfloat16):
         else:
             for n in ("z", "x", "g"):
                 W[x + n] = mat(m["width"], E, 1.5)
-            W[x + "z.b"], W[x + "x.b"], W[x + "o"] = vec(m["width"], 0.5, -1.0), vec(m["width"], 0.3), mat(E, m["width"])
+            W[x + "z.b"], W[x + "x.b"], W[x + "o"] = vec(m["width"], 1.5, -2.0), vec(m["width"], 0.3), mat(E, m["width"])
         if f is not None:
             for n in ("gate", "up"):
                 W[p + "mlp." + n] = mat(f["ff"], E)
