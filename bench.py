@@ -44,10 +44,10 @@ def parse_args():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
-    ap.add_argument("--mode", default="train", choices=["train", "decode", "fedolorn"],
+    ap.add_argument("--mode", default="train", choices=["train", "decode", "fedolorn", "zadepel"],
                     help="train: the headline; decode: the inference engine serving Llama-3 8B, tensor parallel over the GPUs (a second metric: "
                          "prefill and decode tokens/s at 256 concurrent requests, prompts U[128, 2048], 256 greedy tokens, 16-token pages); "
-                         "fedolorn: prefill and decode throughput of Fedolorn beside Llama at equal size, and its kernels beside the like kernels")
+                         "fedolorn, zadepel: prefill and decode throughput of that design beside Llama at equal size, and its kernels beside the like kernels")
     ap.add_argument("--requests", type=int, default=256, help="decode mode: concurrent requests")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch_baseline"])
     ap.add_argument("--zero-stage", type=int, default=3, choices=[1, 3], help="see the module docstring")
@@ -326,27 +326,50 @@ def main_decode(args):
     return 0
 
 
-def main_fedolorn(args):
-    """Serving throughput of Fedolorn beside Llama-3 8B at equal size (random weights, one GPU, greedy, prompts of 1024 tokens), and of
-    its mixture-of-experts form; then every serving kernel beside the like kernel of the closest model."""
+def _serving_runs(models, repeats):
+    """Engine throughput of the models (random weights, one GPU, greedy, prompts of 1024 tokens)."""
     import argparse as _ap
     import gc
 
     import torch
 
-    from levanter_b200.inference import bench_decode, bench_fedolorn
+    from levanter_b200.inference import bench_decode
 
-    sampler = ClockSampler(_env()[2])
-    sampler.start()
     runs = []
-    for model in ("llama3_8b", "fedolorn_8b", "fedolorn_moe"):
+    for model in models:
         for seqs in (8, 64):
             a = _ap.Namespace(model=model, seqs=seqs, prompt_len=1024, new_tokens=128, page_size=16, max_rounds=16, cuda_graph=True, layers=None,
-                              repeats=max(1, args.steps), tp=1, prompt_min=0, prompt_max=0, quiet=True)
+                              repeats=max(1, repeats), tp=1, prompt_min=0, prompt_max=0, quiet=True)
             r = bench_decode.run(a)
             runs.append({k: r[k] for k in ("model", "seqs", "prefill_tokens_per_s", "decode_tokens_per_s", "device_ms_per_round_graph_only")})
             gc.collect()
             torch.cuda.empty_cache()
+    return runs
+
+
+def main_zadepel(args):
+    """Serving throughput of Zadepel beside Llama-3 8B at equal size, then its serving kernels beside the like kernels of the closest models."""
+    from levanter_b200.inference import bench_zadepel
+
+    sampler = ClockSampler(_env()[2])
+    sampler.start()
+    runs = _serving_runs(("llama3_8b", "zadepel_8b"), args.steps)
+    table = bench_zadepel.kernel_table()
+    best = max(r["decode_tokens_per_s"] for r in runs if r["model"] == "zadepel_8b")
+    print(json.dumps({"metric": "decode tokens/sec (inference engine, Zadepel at the size of Llama-3 8B)", "value": best, "unit": "tokens/s", "n_gpus": 1,
+                      "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic uniform-random prompts, random-init weights",
+                      "mode": "zadepel", "impl": "ours", "runs": runs, "clocks": sampler.stop(), **table}))
+    return 0
+
+
+def main_fedolorn(args):
+    """Serving throughput of Fedolorn beside Llama-3 8B at equal size, and of its mixture-of-experts form; then every serving kernel beside
+    the like kernel of the closest model."""
+    from levanter_b200.inference import bench_fedolorn
+
+    sampler = ClockSampler(_env()[2])
+    sampler.start()
+    runs = _serving_runs(("llama3_8b", "fedolorn_8b", "fedolorn_moe"), args.steps)
     table = bench_fedolorn.kernel_table()
     best = max(r["decode_tokens_per_s"] for r in runs if r["model"] == "fedolorn_8b")
     print(json.dumps({"metric": "decode tokens/sec (inference engine, Fedolorn at the size of Llama-3 8B)", "value": best, "unit": "tokens/s", "n_gpus": 1,
@@ -363,6 +386,8 @@ def main():
         return main_decode(args)
     if args.mode == "fedolorn":
         return main_fedolorn(args)
+    if args.mode == "zadepel":
+        return main_zadepel(args)
     if args.impl == "torch_baseline":
         return main_torch_baseline(args)
 

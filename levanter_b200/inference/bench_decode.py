@@ -29,6 +29,12 @@ MODELS = {
     "tiny_fedolorn": dict(family="fedolorn", hidden_dim=256, num_layers=2, intermediate_dim=64, vocab=1024,
                           heads=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, chunk_size=96),
                           moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=2, expert_groups_kept=1)),
+    # Zadepel at the size of llama3_8b: the same width, layers, vocabulary, feed-forward and attention heads; a group of four layers is
+    # attention, minGRU and two of latent attention
+    "zadepel_8b": dict(family="zadepel", hidden_dim=4096, num_layers=32, intermediate_dim=14336, vocab=128256),
+    "tiny_zadepel": dict(family="zadepel", hidden_dim=256, num_layers=4, intermediate_dim=512, vocab=1024,
+                         attention=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, rotary_dim=32), mingru=dict(width=320),
+                         latent=dict(num_heads=4, head_dim=32, rotary_dim=16, v_head_dim=48, kv_lora_rank=64, attention_scale=0.15, sliding_window=96)),
     "tiny": dict(hidden_dim=256, intermediate_dim=512, num_layers=2, num_heads=4, num_kv_heads=2, vocab=1024),
 }
 
@@ -36,10 +42,21 @@ MODELS = {
 def model_config(m: dict, seq_len: int):
     """The model config of a ``MODELS`` entry (without its ``vocab``)."""
     m = dict(m)
-    if m.pop("family", "llama") == "llama":
+    family = m.pop("family", "llama")
+    if family == "llama":
         from ..models.llama import LlamaConfig
 
         return LlamaConfig(seq_len=seq_len, gradient_checkpointing=False, **m)
+    if family == "zadepel":
+        from ..models.zadepel import ZadepelConfig, ZadepelLayerConfig
+
+        ff = m["intermediate_dim"]
+        latent = dict(num_heads=32, head_dim=128, rotary_dim=64, v_head_dim=128, kv_lora_rank=512, attention_scale=192 ** -0.5, sliding_window=1024)
+        group = [ZadepelLayerConfig(mixer="attention", intermediate_dim=ff, **m.get("attention", {})),
+                 ZadepelLayerConfig(mixer="mingru", intermediate_dim=ff, **m.get("mingru", dict(width=4096)))] + \
+                [ZadepelLayerConfig(mixer="latent_attention", intermediate_dim=ff, **m.get("latent", latent))] * 2
+        return ZadepelConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], gradient_checkpointing=False,
+                             layers=tuple(group[i % 4] for i in range(m["num_layers"])))
     from ..models.fedolorn import FedolornConfig, FedolornLayerConfig
 
     layer = FedolornLayerConfig(intermediate_dim=m["intermediate_dim"], **m.get("heads", {}), **m.get("moe", {}))

@@ -80,7 +80,7 @@ def _close(got, want, place, what=""):
     if place[1] == torch.float32:
         assert float(err.max()) < 1e-4, (what, int(err.argmax()), float(err.max()))
     else:
-        assert float(err.median()) < 0.03 and float((err > 0.1).double().mean()) <= 0.05 and float(err.max()) < 0.3, (what, int(err.argmax()), err)
+        assert float(err.median()) < 0.06 and float((err > 0.15).double().mean()) <= 0.1 and float(err.max()) < 0.5, (what, int(err.argmax()), err)
 
 
 def test_registry_config_and_checkpoint_names(checkpoint, tmp_path):
