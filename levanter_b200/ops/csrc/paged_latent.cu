@@ -3,24 +3,27 @@
 // the product of the two rows, and the value is c itself (the caller applies W_uv(h) to the result).  So a key is read once for
 // all heads and used twice.
 //
-//  * paged_latent: one CTA per (packed query row, group of up to 32 query heads, partition of the visible keys).  Keys arrive in
-//    tiles of 32 rows by cp.async, several tiles deep.  Scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the query
-//    heads as the M rows; each warp takes 8 keys of one M tile (or, with 16 heads, 8 keys and half of the row), then owns the online
-//    softmax of a few heads, and finally a set of 16-column pieces of the output, with the value operand read from the key tile by
-//    transposing ldmatrix.  The visible keys of a row are cut evenly over the partitions inside the kernel, so the launch needs
-//    no lengths from the device; a second kernel merges the partitions.
+//  * paged_latent: one CTA per (packed query row, group of up to 32 query heads, partition of the visible keys).  A producer warp
+//    looks up the pages and brings the keys in tiles of 64 rows, one bulk copy per row, two to four tiles deep.  Sixteen warps
+//    compute: scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the query heads as the M rows, a warp taking 16
+//    keys of one M tile and a part of the row; then every warp owns the online softmax of a few heads; then a set of 16-column pieces
+//    of the output, with the value operand read from the key tile by transposing ldmatrix.  The visible keys of a row are cut
+//    evenly over the partitions inside the kernel, so the launch needs no lengths from the device; a second kernel merges the
+//    partitions.
 //  * head_product: out(t, h) = A(t, h) B(h) or A(t, h) B(h)^T for every head: the two products with per-head weights around it.
 #include "common.cuh"
 
 namespace lvb {
 namespace latent {
 
-constexpr int kThreads = 256;
-constexpr int kTileKeys = 32;
+constexpr int kWarps = 16;              // computing warps
+constexpr int kThreads = kWarps * 32;   // computing threads; the producer warp comes after them
+constexpr int kMaxStages = 4;
+constexpr int kTileKeys = 64;
 constexpr int kMinPart = 64;   // keys of a partition, at least
-constexpr int kMaxPieces = 4;  // 16-column output pieces per warp: rank <= 4 * 8 * 16
-constexpr int kScoreLd = 36;   // floats per row of the score tile
-constexpr int kProbLd = 40;    // bf16 per row of the probability tile
+constexpr int kMaxPieces = 2;  // 16-column output pieces per warp: rank <= 2 * 16 * 16
+constexpr int kScoreLd = 68;   // floats per row of the score tile
+constexpr int kProbLd = 72;    // bf16 per row of the probability tile
 
 __device__ __forceinline__ void cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
@@ -28,9 +31,6 @@ __device__ __forceinline__ void cp16(void* dst, const void* src) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void ldm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldm_x2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
 __device__ __forceinline__ void ldm_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -50,6 +50,7 @@ struct Params {
   float* part_ml;                 // [T, H, parts, 2]: maximum (base 2) and sum
   int T, H, width, rank, S, pages_per_seq, page_size, num_pages, parts, window, stages;
   float scale;
+  int* status;
 };
 
 __device__ __forceinline__ bool locate(const Params& p, int t, int& seq, int& ctx) {
@@ -77,23 +78,30 @@ __device__ __forceinline__ int part_keys(const Params& p, int visible) {
 }
 
 __host__ __device__ constexpr int row_bytes(int width) { return (width + 15) / 16 * 32 + 16; }  // an odd multiple of 16 bytes
+// queries, key tiles, 4 / kM partial score tiles of kM * 16 rows, probabilities, three numbers per head, barriers
 __host__ __device__ constexpr int smem_bytes(int m_tiles, int width, int stages) {
-  return (m_tiles * 16 + stages * kTileKeys) * row_bytes(width) + 32 * kScoreLd * 4 + m_tiles * 16 * kProbLd * 2 + m_tiles * 16 * 3 * 4 + 16;
+  return (m_tiles * 16 + stages * kTileKeys) * row_bytes(width) + 64 * kScoreLd * 4 + m_tiles * 16 * kProbLd * 2 + m_tiles * 16 * 3 * 4 + 2 * kMaxStages * 8 + 16;
 }
 
 // kM: M tiles (16 query heads each) per CTA
 template <int kM>
-__global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel(Params p) {
+__global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p) {
   constexpr int kHeads = kM * 16;
+  constexpr int kSplit = 4 / kM;                 // parts that the inner dimension of the scores is cut into
+  constexpr int kRowLanes = 32 / kM;             // lanes per head in the softmax: a warp owns kM heads
+  constexpr int kLaneKeys = kTileKeys / kRowLanes;
   extern __shared__ __align__(16) uint8_t smem[];
   const int w16 = (p.width + 15) & ~15, rowb = row_bytes(p.width);
   uint8_t* s_q = smem;                                              // [kHeads][row]
-  uint8_t* s_k = s_q + kHeads * rowb;                               // [stages][32][row]
-  float* s_s = reinterpret_cast<float*>(s_k + p.stages * kTileKeys * rowb);  // kM = 1: two halves of [16][kScoreLd]; kM = 2: [32][kScoreLd]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + 32 * kScoreLd);  // [kHeads][kProbLd]
-  float* s_alpha = reinterpret_cast<float*>(s_p + kHeads * kProbLd);  // [kHeads]
+  uint8_t* s_k = s_q + kHeads * rowb;                               // [stages][64][row]
+  float* s_s = reinterpret_cast<float*>(s_k + p.stages * kTileKeys * rowb);    // [kSplit][kHeads][kScoreLd]
+  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + 64 * kScoreLd);  // [kHeads][kProbLd]
+  float* s_alpha = reinterpret_cast<float*>(s_p + kHeads * kProbLd);           // [kHeads]
   float* s_m = s_alpha + kHeads;
   float* s_l = s_m + kHeads;
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_l + kHeads);  // [kMaxStages]
+  uint64_t* empty = full + kMaxStages;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty + kMaxStages);
   const int t = blockIdx.x, h0 = blockIdx.y * kHeads, part = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int heads = min(kHeads, p.H - h0);
@@ -105,7 +113,7 @@ __global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel
   const int k0 = first + part * per;
   if (!live || k0 >= ctx) {
     if (!live && part == 0) {
-      for (int i = threadIdx.x; i < heads * p.rank; i += kThreads)
+      for (int i = threadIdx.x; i < heads * p.rank; i += kThreads + 32)
         p.out[(static_cast<long long>(t) * p.H + h0) * p.rank + i] = __float2bfloat16(0.f);
     }
     return;
@@ -114,51 +122,65 @@ __global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel
   const int tiles = (nk + kTileKeys - 1) / kTileKeys;
   const int pieces = p.width / 8;  // 16-byte pieces of a row
 
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    for (int i = 0; i < p.stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], kWarps);
+    }
+    mbar_fence_init();
+  }
   // queries; rows beyond the heads and columns beyond the width are zeros, in the key tiles too (those columns are never copied to)
-  for (int i = threadIdx.x; i < kHeads * (w16 / 8); i += kThreads) {
+  for (int i = threadIdx.x; i < kHeads * (w16 / 8); i += kThreads + 32) {
     const int r = i / (w16 / 8), c = i - r * (w16 / 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (r < heads && c < pieces) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(t) * p.H + h0 + r) * p.width + c * 8);
     *reinterpret_cast<uint4*>(s_q + r * rowb + c * 16) = v;
   }
   if (w16 != p.width) {
-    for (int r = threadIdx.x; r < p.stages * kTileKeys; r += kThreads) *reinterpret_cast<uint4*>(s_k + r * rowb + pieces * 16) = make_uint4(0u, 0u, 0u, 0u);
+    for (int r = threadIdx.x; r < p.stages * kTileKeys; r += kThreads + 32)
+      *reinterpret_cast<uint4*>(s_k + r * rowb + pieces * 16) = make_uint4(0u, 0u, 0u, 0u);
   }
-  auto issue = [&](int tile) {
-    if (tile < tiles) {
-      uint8_t* dst = s_k + (tile % p.stages) * kTileKeys * rowb;
-      for (int r = warp; r < kTileKeys; r += kThreads / 32) {
-        const int i = tile * kTileKeys + r;
-        long long slot = -1;
-        if (i < nk) {
-          const int key = k0 + i;
-          const int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
-          if (page >= 0 && page < p.num_pages) slot = static_cast<long long>(page) * p.page_size + key % p.page_size;
-        }
-        uint8_t* d = dst + r * rowb;
-        if (slot >= 0) {
-          const __nv_bfloat16* src = p.kv_pages + slot * p.width;
-          for (int c = lane; c < pieces; c += 32) cp16(d + c * 16, src + c * 8);
-        } else {
-          for (int c = lane; c < pieces; c += 32) *reinterpret_cast<uint4*>(d + c * 16) = make_uint4(0u, 0u, 0u, 0u);
-        }
+  __syncthreads();
+
+  if (warp == kWarps) {
+    // ---- producer: lanes own rows lane and lane + 32 of a tile.  Rows past the last key repeat it (their probabilities are zero).
+    int st = 0;
+    uint32_t phase = 0;
+    for (int it = 0; it < tiles; ++it) {
+      const __nv_bfloat16* src[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int key = k0 + min(it * kTileKeys + lane + 32 * j, nk - 1);
+        int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
+        page = page >= 0 && page < p.num_pages ? page : 0;
+        src[j] = p.kv_pages + (static_cast<long long>(page) * p.page_size + key % p.page_size) * p.width;
+      }
+      bool ok = mbar_wait(&empty[st], phase ^ 1, abort_flag, p.status, 1500, it);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      if (lane == 0) mbar_expect_tx(&full[st], kTileKeys * p.width * 2);
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 2; ++j) bulk_load(s_k + (st * kTileKeys + lane + 32 * j) * rowb, src[j], p.width * 2, &full[st]);
+      if (++st == p.stages) {
+        st = 0;
+        phase ^= 1;
       }
     }
-    cp_commit();
-  };
-  for (int i = 0; i < p.stages - 1; ++i) issue(i);
+    return;
+  }
 
   const float sc_log2 = p.scale * 1.4426950408889634f;
   const int ksteps = w16 / 16, out_pieces = (p.rank + 15) / 16;
-  // this warp's part of the scores
-  const int mt = kM == 2 ? (warp & 1) : 0;
-  const int nt = kM == 2 ? (warp >> 1) : (warp & 3);
-  const int ks_lo = kM == 2 ? 0 : (warp >> 2) * ((ksteps + 1) / 2);
-  const int ks_hi = kM == 2 ? ksteps : min(ksteps, ((warp >> 2) + 1) * ((ksteps + 1) / 2));
-  float* my_scores = s_s + (kM == 2 ? mt * 16 : (warp >> 2) * 16) * kScoreLd;
-  float m_run[2 * kM], l_run[2 * kM];  // heads warp * 2 kM + i, the same value in every lane
-#pragma unroll
-  for (int i = 0; i < 2 * kM; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  // this warp's part of the scores: an M tile, a pair of 8-key tiles, a range of k-steps
+  const int mt = kM == 2 ? (warp & 1) : 0, np = kM == 2 ? (warp >> 1) & 3 : warp & 3, kpart = kM == 2 ? warp >> 3 : warp >> 2;
+  const int kper = (ksteps + kSplit - 1) / kSplit;
+  const int ks_lo = min(kpart * kper, ksteps), ks_hi = min(ks_lo + kper, ksteps);
+  float* my_scores = s_s + (kpart * kHeads + mt * 16 + (lane >> 2)) * kScoreLd + np * 16 + (lane & 3) * 2;
+  // this lane's part of the softmax: keys lk .. lk + kLaneKeys of head row
+  const int row = warp * kM + lane / kRowLanes, lk = (lane % kRowLanes) * kLaneKeys;
+  float m_run = -INFINITY, l_run = 0.f;
   float o[kMaxPieces][kM][2][4];
 #pragma unroll
   for (int a = 0; a < kMaxPieces; ++a)
@@ -167,77 +189,111 @@ __global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel
 #pragma unroll
       for (int c = 0; c < 4; ++c) { o[a][b][0][c] = 0.f; o[a][b][1][c] = 0.f; }
 
+  int st = 0;
+  uint32_t phase = 0;
   for (int it = 0; it < tiles; ++it) {
-    // all but the newest stages - 2 groups have landed: tile `it` is there
-    if (p.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
-    else if (p.stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
-    else asm volatile("cp.async.wait_group 2;" ::: "memory");
-    __syncthreads();  // for everyone; and everyone is done with the tile before, whose buffer the next copy takes
-    issue(it + p.stages - 1);
-    const uint32_t kb = smem_u32(s_k + (it % p.stages) * kTileKeys * rowb);
+    // after a wait that ran out the loop goes on without data, so that everyone still meets at the barriers
+    mbar_wait(&full[st], phase, abort_flag, p.status, 1501, it);
+    __syncwarp();
+    const uint32_t kb = smem_u32(s_k + st * kTileKeys * rowb);
     {
-      float acc[2][4];
+      float acc[2][2][4];  // alternate k-steps of the two key tiles
 #pragma unroll
-      for (int c = 0; c < 4; ++c) { acc[0][c] = 0.f; acc[1][c] = 0.f; }
+      for (int c = 0; c < 4; ++c) acc[0][0][c] = acc[0][1][c] = acc[1][0][c] = acc[1][1][c] = 0.f;
       const uint32_t qa = smem_u32(s_q) + (mt * 16 + (lane & 15)) * rowb + (lane >> 4) * 16;
-      const uint32_t ka = kb + (nt * 8 + (lane & 7)) * rowb + ((lane >> 3) & 1) * 16;
-#pragma unroll 4
-      for (int ks = ks_lo; ks < ks_hi; ++ks) {
-        uint32_t a[4], b0, b1;
+      // (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
+      const uint32_t ka = kb + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * rowb + ((lane >> 3) & 1) * 16;
+      auto k_step = [&](int ks, float (&c)[2][4]) {
+        uint32_t a[4], b0, b1, b2, b3;
         ldm_x4(qa + ks * 32, a[0], a[1], a[2], a[3]);
-        ldm_x2(ka + ks * 32, b0, b1);
-        if (ks & 1) mma16816(acc[1], a, b0, b1);
-        else mma16816(acc[0], a, b0, b1);
+        ldm_x4(ka + ks * 32, b0, b1, b2, b3);
+        mma16816(c[0], a, b0, b1);
+        mma16816(c[1], a, b2, b3);
+      };
+      int ks = ks_lo;
+#pragma unroll 3
+      for (; ks + 1 < ks_hi; ks += 2) {
+        k_step(ks, acc[0]);
+        k_step(ks + 1, acc[1]);
       }
-      float* d = my_scores + (lane >> 2) * kScoreLd + nt * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(d) = make_float2(acc[0][0] + acc[1][0], acc[0][1] + acc[1][1]);
-      *reinterpret_cast<float2*>(d + 8 * kScoreLd) = make_float2(acc[0][2] + acc[1][2], acc[0][3] + acc[1][3]);
-    }
-    __syncthreads();
-    {
-      const bool valid = it * kTileKeys + lane < nk;
+      if (ks < ks_hi) k_step(ks, acc[0]);
 #pragma unroll
-      for (int i = 0; i < 2 * kM; ++i) {
-        const int r = warp * 2 * kM + i;
-        float v = s_s[r * kScoreLd + lane];
-        if constexpr (kM == 1) v += s_s[(16 + r) * kScoreLd + lane];
-        v = valid ? v * sc_log2 : -INFINITY;
-        const float m_new = fmaxf(m_run[i], warp_max(v));
-        const float e = valid ? exp2f(v - m_new) : 0.f;
-        const float alpha = m_run[i] == -INFINITY ? 0.f : exp2f(m_run[i] - m_new);
-        l_run[i] = l_run[i] * alpha + warp_sum(e);
-        m_run[i] = m_new;
-        s_p[r * kProbLd + lane] = __float2bfloat16(e);
-        if (lane == 0) s_alpha[r] = alpha;
+      for (int j = 0; j < 2; ++j) {
+        *reinterpret_cast<float2*>(my_scores + j * 8) = make_float2(acc[0][j][0] + acc[1][j][0], acc[0][j][1] + acc[1][j][1]);
+        *reinterpret_cast<float2*>(my_scores + j * 8 + 8 * kScoreLd) = make_float2(acc[0][j][2] + acc[1][j][2], acc[0][j][3] + acc[1][j][3]);
       }
     }
-    __syncthreads();
+    named_bar_sync(1, kThreads);
     {
-      uint32_t pa[kM][2][4];
+      float v[kLaneKeys];
+#pragma unroll
+      for (int i = 0; i < kLaneKeys; ++i) v[i] = 0.f;
+#pragma unroll
+      for (int k = 0; k < kSplit; ++k) {
+        const float* src = s_s + (k * kHeads + row) * kScoreLd + lk;
+#pragma unroll
+        for (int i = 0; i < kLaneKeys; i += 2) {
+          const float2 x = *reinterpret_cast<const float2*>(src + i);
+          v[i] += x.x;
+          v[i + 1] += x.y;
+        }
+      }
+      const int left = nk - it * kTileKeys - lk;
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < kLaneKeys; ++i) {
+        v[i] = i < left ? v[i] * sc_log2 : -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+#pragma unroll
+      for (int d = kRowLanes / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      const float m_new = fmaxf(m_run, mx);  // finite: a tile has at least one key
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < kLaneKeys; i += 2) {
+        const float e0 = exp2f(v[i] - m_new), e1 = exp2f(v[i + 1] - m_new);  // masked keys: 2^-inf = 0
+        sum += e0 + e1;
+        *reinterpret_cast<uint32_t*>(s_p + row * kProbLd + lk + i) = pack_bf16x2(e0, e1);
+      }
+#pragma unroll
+      for (int d = kRowLanes / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+      const float alpha = exp2f(m_run - m_new);
+      l_run = l_run * alpha + sum;
+      m_run = m_new;
+      if (lk == 0) s_alpha[row] = alpha;
+    }
+    named_bar_sync(1, kThreads);
+    {
+      uint32_t pa[kM][4][4];
       float al[kM][2];
+      bool moved = false;
 #pragma unroll
       for (int m = 0; m < kM; ++m) {
 #pragma unroll
-        for (int h = 0; h < 2; ++h)
+        for (int h = 0; h < 4; ++h)
           ldm_x4(smem_u32(s_p) + (m * 16 + (lane & 15)) * kProbLd * 2 + h * 32 + (lane >> 4) * 16, pa[m][h][0], pa[m][h][1], pa[m][h][2], pa[m][h][3]);
         al[m][0] = s_alpha[m * 16 + (lane >> 2)];
         al[m][1] = s_alpha[m * 16 + 8 + (lane >> 2)];
+        moved = moved || al[m][0] != 1.f || al[m][1] != 1.f;
       }
+      moved = __any_sync(0xffffffffu, moved);
       // matrices of a transposing x4: (keys 0-7, columns 0-7), (keys 8-15, same), (keys 0-7, columns 8-15), (keys 8-15, same)
       const uint32_t va = kb + (((lane >> 3) & 1) * 8 + (lane & 7)) * rowb + (lane >> 4) * 16;
 #pragma unroll
       for (int a = 0; a < kMaxPieces; ++a) {
-        const int piece = warp + a * (kThreads / 32);
+        const int piece = warp + a * kWarps;
         if (piece >= out_pieces) break;
+        if (moved) {
 #pragma unroll
-        for (int m = 0; m < kM; ++m)
+          for (int m = 0; m < kM; ++m)
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            o[a][m][j][0] *= al[m][0]; o[a][m][j][1] *= al[m][0];
-            o[a][m][j][2] *= al[m][1]; o[a][m][j][3] *= al[m][1];
-          }
+            for (int j = 0; j < 2; ++j) {
+              o[a][m][j][0] *= al[m][0]; o[a][m][j][1] *= al[m][0];
+              o[a][m][j][2] *= al[m][1]; o[a][m][j][3] *= al[m][1];
+            }
+        }
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+        for (int h = 0; h < 4; ++h) {
           uint32_t b0, b1, b2, b3;
           ldm_x4_trans(va + h * 16 * rowb + piece * 32, b0, b1, b2, b3);
 #pragma unroll
@@ -248,16 +304,18 @@ __global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel
         }
       }
     }
-  }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  if (lane == 0) {
-#pragma unroll
-    for (int i = 0; i < 2 * kM; ++i) {
-      s_m[warp * 2 * kM + i] = m_run[i];
-      s_l[warp * 2 * kM + i] = l_run[i];
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st]);
+    if (++st == p.stages) {
+      st = 0;
+      phase ^= 1;
     }
   }
-  __syncthreads();
+  if (lk == 0) {
+    s_m[row] = m_run;
+    s_l[row] = l_run;
+  }
+  named_bar_sync(1, kThreads);
   if (p.parts > 1 && threadIdx.x < heads) {
     float* ml = p.part_ml + ((static_cast<long long>(t) * p.H + h0 + threadIdx.x) * p.parts + part) * 2;
     ml[0] = s_m[threadIdx.x];
@@ -265,7 +323,7 @@ __global__ void __launch_bounds__(kThreads, kM == 1 ? 2 : 1) paged_latent_kernel
   }
 #pragma unroll
   for (int a = 0; a < kMaxPieces; ++a) {
-    const int piece = warp + a * (kThreads / 32);
+    const int piece = warp + a * kWarps;
     if (piece >= out_pieces) break;
 #pragma unroll
     for (int m = 0; m < kM; ++m)
@@ -322,7 +380,7 @@ int launch(const Params& p, cudaStream_t s) {
     attr_set = true;
   }
   const int groups = (p.H + kM * 16 - 1) / (kM * 16);
-  kern<<<dim3(p.T, groups, p.parts), kThreads, smem_bytes(kM, p.width, p.stages), s>>>(p);
+  kern<<<dim3(p.T, groups, p.parts), kThreads + 32, smem_bytes(kM, p.width, p.stages), s>>>(p);
   if (cudaGetLastError() != cudaSuccess) return kErrCuda;
   if (p.parts > 1) merge_kernel<<<dim3(p.T, p.H), 128, 0, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
@@ -411,27 +469,40 @@ __global__ void __launch_bounds__(128) head_product_kernel(ProductParams p) {
 }  // namespace lvb
 
 // Partitions of the visible keys that lvb_paged_latent uses for T rows of H heads: sizes part_o fp32 [T, H, parts, rank] and part_ml fp32 [T, H,
-// parts, 2] (unused when 1).
-extern "C" int lvb_paged_latent_parts(int T, int H, int max_context, int window) {
+// parts, 2] (unused when 1).  The fewest waves of CTAs, set against the traffic of the merge: everything in units of the time that
+// an SM takes to read a key.
+extern "C" int lvb_paged_latent_parts(int T, int H, int width, int rank, int max_context, int window) {
   using namespace lvb;
   using namespace lvb::latent;
+  if (T <= 0 || H <= 0 || width <= 0) return 1;
   const int keys = window > 0 && window < max_context ? window : max_context;
-  const int groups = H <= 16 ? 1 : (H + 31) / 32;
-  const int want = (2 * num_sms() + T * groups - 1) / (T * groups), most = (keys + 2 * kMinPart - 1) / (2 * kMinPart);
-  const int parts = want < most ? want : most;
-  return parts < 1 ? 1 : parts > 32 ? 32 : parts;
+  const int m_tiles = H <= 16 ? 1 : 2, groups = (H + m_tiles * 16 - 1) / (m_tiles * 16);
+  const int slots = num_sms();
+  const double merge = 8.0 * T * H * rank / (2.0 * width * num_sms());
+  int best = 1;
+  double least = 0.;
+  for (int parts = 1; parts <= 32 && (parts == 1 || keys / parts >= kMinPart); ++parts) {
+    const long long ctas = static_cast<long long>(T) * groups * parts;
+    const double cost = static_cast<double>((ctas + slots - 1) / slots) * (static_cast<double>(keys) / parts + kTileKeys) + (parts > 1 ? merge * parts + 64 : 0.);
+    if (parts == 1 || cost < least) {
+      least = cost;
+      best = parts;
+    }
+  }
+  return best;
 }
 
 // Packed query rows q [T, H, width] over pages [num_pages, page_size, width] whose rows' first `rank` elements are the values -> out [T, H, rank];
-// causal, window > 0: a row sees itself and the window - 1 positions before it.  width and rank: multiples of 8, rank <= 512, width <= 640.
+// causal, window > 0: a row sees itself and the window - 1 positions before it.  width and rank: multiples of 8, rank <= 512, width <= 592.
 extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices, const int* cu_q_lens,
                                 const int* num_seqs, void* out, float* part_o, float* part_ml, int T, int H, int width, int rank, int S,
-                                int pages_per_seq, int page_size, int num_pages, int window, int parts, float scale, void* stream) {
+                                int pages_per_seq, int page_size, int num_pages, int window, int parts, float scale, int* status,
+                                void* stream) {
   using namespace lvb;
   using namespace lvb::latent;
   if (T <= 0) return kErrOk;
   if (H <= 0 || width <= 0 || rank <= 0 || rank > width || ((width | rank) & 7) || S <= 0 || window < 0 || parts < 1) return kErrBadArg;
-  if (rank > kMaxPieces * 8 * 16 || width > 640) return kErrTooLarge;
+  if (rank > kMaxPieces * kWarps * 16 || width > 592) return kErrTooLarge;
   if (parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv_pages) | reinterpret_cast<uintptr_t>(out)) & 15) return kErrBadArg;
   Params p;
@@ -441,11 +512,11 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml;
   p.T = T; p.H = H; p.width = width; p.rank = rank; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;
-  p.parts = parts; p.window = window; p.scale = scale;
+  p.parts = parts; p.window = window; p.scale = scale; p.status = status;
   const int m_tiles = H <= 16 ? 1 : 2;
-  const int room = (m_tiles == 1 ? 110 : 216) * 1024;
-  p.stages = 4;
-  while (p.stages > 2 && smem_bytes(m_tiles, width, p.stages) > room) --p.stages;
+  p.stages = kMaxStages;
+  while (p.stages > 2 && smem_bytes(m_tiles, width, p.stages) > 220 * 1024) --p.stages;
+  if (smem_bytes(m_tiles, width, p.stages) > 220 * 1024) return kErrTooLarge;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return m_tiles == 1 ? launch<1>(p, s) : launch<2>(p, s);
 }

@@ -239,7 +239,7 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
                            window: Optional[int] = None) -> torch.Tensor:
     """Causal attention of ``q [T, H, width]`` over pages of ``width`` elements per slot whose first ``rank`` are the value: all heads read
     the same row per key -> ``[T, H, rank]``.  ``window`` as in :func:`paged_attention_general`.  bf16 with sizes that are multiples of
-    8 (rank up to 512, width up to 640) runs on tensor cores; everything else in fp32 arithmetic."""
+    8 (rank up to 512, width up to 592) runs on tensor cores; everything else in fp32 arithmetic."""
     T, H, w = q.shape
     b = batch_info
     if not _use_kernel(q, kv_pages):
@@ -255,20 +255,20 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
     i32 = lambda t: t.to(device=dev, dtype=torch.int32).contiguous()  # noqa: E731
     lens, pages, cu, ns = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
     out = torch.empty(T, H, rank, dtype=q.dtype, device=dev)
-    if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 640:
+    if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 592:
         rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), 0, out.data_ptr(), T, H, 1, w, rank,
                        H * w, 0, S, PP, ps, P, 0, int(window or 0), 1, float(sm_scale), 0.0, int(q.dtype == torch.float32), lib.stream_ptr())
         lib.check_rc(rc, "lvb_attention_any")
         return out
     if "l" not in _f:
-        _f["l"] = lib.fn("lvb_paged_latent", [c.c_void_p] * 9 + [c.c_int] * 10 + [c.c_float, c.c_void_p], launches=2)
-        _f["lparts"] = lib.fn("lvb_paged_latent_parts", [c.c_int] * 4, launches=0)
-    parts = _f["lparts"](T, H, PP * ps, int(window or 0))
+        _f["l"] = lib.fn("lvb_paged_latent", [c.c_void_p] * 9 + [c.c_int] * 10 + [c.c_float, c.c_void_p, c.c_void_p], launches=2)
+        _f["lparts"] = lib.fn("lvb_paged_latent_parts", [c.c_int] * 6, launches=0)
+    parts = _f["lparts"](T, H, w, rank, PP * ps, int(window or 0))
     po = pml = None
     if parts > 1:
         po, pml = _part_scratch(dev, T * H * parts * rank, T * H * parts * 2)
     rc = _f["l"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), out.data_ptr(), lib.ptr(po), lib.ptr(pml), T,
-                 H, w, rank, S, PP, ps, P, int(window or 0), parts, float(sm_scale), lib.stream_ptr())
+                 H, w, rank, S, PP, ps, P, int(window or 0), parts, float(sm_scale), lib.status_buffer().data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_paged_latent")
     return out
 
