@@ -30,7 +30,7 @@ MODELS = {
                           heads=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, chunk_size=96),
                           moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=2, expert_groups_kept=1)),
     # Zadepel at the size of llama3_8b: the same width, layers, vocabulary, feed-forward and attention heads; a group of four layers is
-    # attention, minGRU and two of latent attention
+    # attention, latent attention, minGRU, latent attention
     "zadepel_8b": dict(family="zadepel", hidden_dim=4096, num_layers=32, intermediate_dim=14336, vocab=128256),
     "tiny_zadepel": dict(family="zadepel", hidden_dim=256, num_layers=4, intermediate_dim=512, vocab=1024,
                          attention=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, rotary_dim=32), mingru=dict(width=320),
@@ -52,9 +52,9 @@ def model_config(m: dict, seq_len: int):
 
         ff = m["intermediate_dim"]
         latent = dict(num_heads=32, head_dim=128, rotary_dim=64, v_head_dim=128, kv_lora_rank=512, attention_scale=192 ** -0.5, sliding_window=1024)
-        group = [ZadepelLayerConfig(mixer="attention", intermediate_dim=ff, **m.get("attention", {})),
-                 ZadepelLayerConfig(mixer="mingru", intermediate_dim=ff, **m.get("mingru", dict(width=4096)))] + \
-                [ZadepelLayerConfig(mixer="latent_attention", intermediate_dim=ff, **m.get("latent", latent))] * 2
+        latent = ZadepelLayerConfig(mixer="latent_attention", intermediate_dim=ff, **m.get("latent", latent))
+        group = [ZadepelLayerConfig(mixer="attention", intermediate_dim=ff, **m.get("attention", {})), latent,
+                 ZadepelLayerConfig(mixer="mingru", intermediate_dim=ff, **m.get("mingru", dict(width=4096))), latent]
         return ZadepelConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], gradient_checkpointing=False,
                              layers=tuple(group[i % 4] for i in range(m["num_layers"])))
     from ..models.fedolorn import FedolornConfig, FedolornLayerConfig

@@ -449,6 +449,23 @@ inline int make_tmap_heads_bf16(CUtensorMap* out, const void* ptr, uint64_t rows
   return r == CUDA_SUCCESS ? kErrOk : kErrTensorMap;
 }
 
+// Dense row-major bf16 [rows, cols], cols a multiple of 64, as [rows, cols / 64, 64]; box = box_rows whole rows, each cols / 64 lines of 128
+// bytes in shared memory, 128-byte swizzle.
+inline int make_tmap_chunked_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows) {
+  ensure_context_for(ptr);
+  EncodeTiledFn enc = get_encode_tiled();
+  if (enc == nullptr) return kErrTensorMap;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) != 0 || (cols & 63) != 0 || cols > 64 * 256) return kErrBadArg;
+  cuuint64_t gdim[3] = {64, cols / 64, rows};
+  cuuint64_t gstr[2] = {128, cols * 2};
+  cuuint32_t box[3] = {64, static_cast<cuuint32_t>(cols / 64), box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), gdim, gstr, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? kErrOk : kErrTensorMap;
+}
+
 // Row-major 2-D tensor of one-byte elements [rows, cols] with row stride ld (bytes); box = [box_rows, 128].
 inline int make_tmap_2d_u8(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows) {
   ensure_context_for(ptr);

@@ -4,24 +4,27 @@
 // all heads and used twice.
 //
 //  * paged_latent: one CTA per (packed query row, group of up to 32 query heads, partition of the visible keys).  A producer warp
-//    looks up the pages and brings the keys in tiles of 64 rows, one bulk copy per row, two to four tiles deep.  Sixteen warps
-//    compute: scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the query heads as the M rows, a warp taking 16
-//    keys of one M tile and a part of the row; then every warp owns the online softmax of a few heads; then a set of 16-column pieces
-//    of the output, with the value operand read from the key tile by transposing ldmatrix.  The visible keys of a row are cut
-//    evenly over the partitions inside the kernel, so the launch needs no lengths from the device; a second kernel merges the
-//    partitions.
+//    looks up the pages and brings the keys by TMA in tiles of 64 rows (128-byte swizzle; boxes of the rows of a page, at most
+//    64), two to four tiles deep.  Eight warps compute: scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the
+//    query heads as the M rows, a warp taking 32 keys and a quarter of the row; then every warp owns the online softmax of a few
+//    heads, which adds up the quarters; then a set of 16-column pieces of the output, with the value operand read from the key
+//    tile by transposing ldmatrix.  Shared-memory reads bound a tile as much as its transfer does, hence the large share per
+//    warp.  The visible keys of a row are cut evenly over the partitions inside the kernel, so the launch needs no lengths from
+//    the device; a second kernel merges the partitions.
 //  * head_product: out(t, h) = A(t, h) B(h) or A(t, h) B(h)^T for every head: the two products with per-head weights around it.
 #include "common.cuh"
 
 namespace lvb {
 namespace latent {
 
-constexpr int kWarps = 16;              // computing warps
-constexpr int kThreads = kWarps * 32;   // computing threads; the producer warp comes after them
+constexpr int kWarps = 8;              // computing warps
+constexpr int kThreads = kWarps * 32;  // computing threads; the producer warp comes after them
+constexpr int kSplit = 4;      // parts that the inner dimension of the scores is cut into
 constexpr int kMaxStages = 4;
+constexpr int kMaxSmem = 226 * 1024;
 constexpr int kTileKeys = 64;
 constexpr int kMinPart = 64;   // keys of a partition, at least
-constexpr int kMaxPieces = 2;  // 16-column output pieces per warp: rank <= 2 * 16 * 16
+constexpr int kMaxPieces = 4;  // 16-column output pieces per warp: rank <= 4 * 8 * 16
 constexpr int kScoreLd = 68;   // floats per row of the score tile
 constexpr int kProbLd = 72;    // bf16 per row of the probability tile
 
@@ -51,6 +54,9 @@ struct Params {
   int T, H, width, rank, S, pages_per_seq, page_size, num_pages, parts, window, stages;
   float scale;
   int* status;
+  int box;   // rows of a TMA box: a power of two that divides the page size and 64
+  int box_log;
+  int whole; // a box holds whole rows [box][chunks][128 bytes]; else one chunk of them [box][128 bytes]
 };
 
 __device__ __forceinline__ bool locate(const Params& p, int t, int& seq, int& ctx) {
@@ -77,25 +83,27 @@ __device__ __forceinline__ int part_keys(const Params& p, int visible) {
   return (n + kTileKeys - 1) / kTileKeys * kTileKeys;
 }
 
-__host__ __device__ constexpr int row_bytes(int width) { return (width + 15) / 16 * 32 + 16; }  // an odd multiple of 16 bytes
-// queries, key tiles, 4 / kM partial score tiles of kM * 16 rows, probabilities, three numbers per head, barriers
+// Key tiles are cut into chunks of 64 columns (128 bytes); columns past the width are zeros.
+__host__ __device__ constexpr int chunks_of(int width) { return (width + 63) / 64; }
+__host__ __device__ constexpr int stage_bytes(int width) { return chunks_of(width) * kTileKeys * 128; }
+__host__ __device__ constexpr int row_bytes(int width) { return chunks_of(width) * 128 + 16; }  // of a staged query: an odd multiple of 16
+// key tiles (1024-byte aligned), queries, partial score tiles, probabilities, three numbers per head, barriers
 __host__ __device__ constexpr int smem_bytes(int m_tiles, int width, int stages) {
-  return (m_tiles * 16 + stages * kTileKeys) * row_bytes(width) + 64 * kScoreLd * 4 + m_tiles * 16 * kProbLd * 2 + m_tiles * 16 * 3 * 4 + 2 * kMaxStages * 8 + 16;
+  return 1024 + stages * stage_bytes(width) + m_tiles * 16 * (row_bytes(width) + kSplit * kScoreLd * 4 + kProbLd * 2 + 3 * 4) + 2 * kMaxStages * 8 + 16;
 }
 
 // kM: M tiles (16 query heads each) per CTA
 template <int kM>
-__global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p) {
+__global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __grid_constant__ CUtensorMap tm, Params p) {
   constexpr int kHeads = kM * 16;
-  constexpr int kSplit = 4 / kM;                 // parts that the inner dimension of the scores is cut into
-  constexpr int kRowLanes = 32 / kM;             // lanes per head in the softmax: a warp owns kM heads
+  constexpr int kRowLanes = 16 / kM;             // lanes per head in the softmax: a warp owns 2 kM heads
   constexpr int kLaneKeys = kTileKeys / kRowLanes;
-  extern __shared__ __align__(16) uint8_t smem[];
-  const int w16 = (p.width + 15) & ~15, rowb = row_bytes(p.width);
-  uint8_t* s_q = smem;                                              // [kHeads][row]
-  uint8_t* s_k = s_q + kHeads * rowb;                               // [stages][64][row]
-  float* s_s = reinterpret_cast<float*>(s_k + p.stages * kTileKeys * rowb);    // [kSplit][kHeads][kScoreLd]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + 64 * kScoreLd);  // [kHeads][kProbLd]
+  extern __shared__ uint8_t smem_raw[];
+  const int chunks = chunks_of(p.width), rowb = row_bytes(p.width), stageb = stage_bytes(p.width);
+  uint8_t* s_k = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));  // [stages][64 / box][chunks][box][128]
+  uint8_t* s_q = s_k + p.stages * stageb;                                      // [kHeads][row]
+  float* s_s = reinterpret_cast<float*>(s_q + kHeads * rowb);                  // [kSplit][kHeads][kScoreLd]
+  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + kSplit * kHeads * kScoreLd);  // [kHeads][kProbLd]
   float* s_alpha = reinterpret_cast<float*>(s_p + kHeads * kProbLd);           // [kHeads]
   float* s_m = s_alpha + kHeads;
   float* s_l = s_m + kHeads;
@@ -109,8 +117,9 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
   int seq = 0, ctx = 0;
   const bool live = locate(p, t, seq, ctx);
   const int first = live ? first_key(p, ctx) : 0;
-  const int per = live ? part_keys(p, ctx - first) : 0;
-  const int k0 = first + part * per;
+  const int base = first & ~(p.box - 1);  // whole boxes: the keys before `first` are masked
+  const int per = live ? part_keys(p, ctx - base) : 0;
+  const int k0 = base + part * per;
   if (!live || k0 >= ctx) {
     if (!live && part == 0) {
       for (int i = threadIdx.x; i < heads * p.rank; i += kThreads + 32)
@@ -120,7 +129,7 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
   }
   const int nk = min(per, ctx - k0);
   const int tiles = (nk + kTileKeys - 1) / kTileKeys;
-  const int pieces = p.width / 8;  // 16-byte pieces of a row
+  const int below = first - k0;  // keys of the partition that come before the window (or <= 0)
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -129,40 +138,39 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
       mbar_init(&empty[i], kWarps);
     }
     mbar_fence_init();
+    tma_prefetch_desc(&tm);
   }
-  // queries; rows beyond the heads and columns beyond the width are zeros, in the key tiles too (those columns are never copied to)
-  for (int i = threadIdx.x; i < kHeads * (w16 / 8); i += kThreads + 32) {
-    const int r = i / (w16 / 8), c = i - r * (w16 / 8);
+  // queries; rows beyond the heads and columns beyond the width are zeros
+  for (int i = threadIdx.x; i < kHeads * chunks * 8; i += kThreads + 32) {
+    const int r = i / (chunks * 8), c = i - r * (chunks * 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < heads && c < pieces) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(t) * p.H + h0 + r) * p.width + c * 8);
+    if (r < heads && c * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(t) * p.H + h0 + r) * p.width + c * 8);
     *reinterpret_cast<uint4*>(s_q + r * rowb + c * 16) = v;
-  }
-  if (w16 != p.width) {
-    for (int r = threadIdx.x; r < p.stages * kTileKeys; r += kThreads + 32)
-      *reinterpret_cast<uint4*>(s_k + r * rowb + pieces * 16) = make_uint4(0u, 0u, 0u, 0u);
   }
   __syncthreads();
 
   if (warp == kWarps) {
-    // ---- producer: lanes own rows lane and lane + 32 of a tile.  Rows past the last key repeat it (their probabilities are zero).
+    // ---- producer: a lane per box
+    const int per_group = p.whole ? 1 : chunks, boxes = kTileKeys / p.box * per_group, boxb = p.box * 128 * (p.whole ? chunks : 1);
     int st = 0;
     uint32_t phase = 0;
     for (int it = 0; it < tiles; ++it) {
-      const __nv_bfloat16* src[2];
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int key = k0 + min(it * kTileKeys + lane + 32 * j, nk - 1);
-        int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
-        page = page >= 0 && page < p.num_pages ? page : 0;
-        src[j] = p.kv_pages + (static_cast<long long>(page) * p.page_size + key % p.page_size) * p.width;
-      }
       bool ok = mbar_wait(&empty[st], phase ^ 1, abort_flag, p.status, 1500, it);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
-      if (lane == 0) mbar_expect_tx(&full[st], kTileKeys * p.width * 2);
+      if (lane == 0) mbar_expect_tx(&full[st], stageb);
       __syncwarp();
-#pragma unroll
-      for (int j = 0; j < 2; ++j) bulk_load(s_k + (st * kTileKeys + lane + 32 * j) * rowb, src[j], p.width * 2, &full[st]);
+      for (int i = lane; i < boxes; i += 32) {
+        const int group = i / per_group, chunk = i - group * per_group;
+        const int key = k0 + it * kTileKeys + group * p.box;
+        int row = 0;  // past the last key: any rows will do, they are masked
+        if (key < ctx) {
+          const int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
+          if (page >= 0 && page < p.num_pages) row = page * p.page_size + key % p.page_size;
+        }
+        if (p.whole) tma_load_3d(s_k + st * stageb + i * boxb, &tm, &full[st], 0, 0, row);
+        else tma_load_2d(s_k + st * stageb + i * boxb, &tm, &full[st], chunk * 64, row);
+      }
       if (++st == p.stages) {
         st = 0;
         phase ^= 1;
@@ -172,14 +180,21 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
   }
 
   const float sc_log2 = p.scale * 1.4426950408889634f;
-  const int ksteps = w16 / 16, out_pieces = (p.rank + 15) / 16;
-  // this warp's part of the scores: an M tile, a pair of 8-key tiles, a range of k-steps
-  const int mt = kM == 2 ? (warp & 1) : 0, np = kM == 2 ? (warp >> 1) & 3 : warp & 3, kpart = kM == 2 ? warp >> 3 : warp >> 2;
-  const int kper = (ksteps + kSplit - 1) / kSplit;
-  const int ks_lo = min(kpart * kper, ksteps), ks_hi = min(ks_lo + kper, ksteps);
-  float* my_scores = s_s + (kpart * kHeads + mt * 16 + (lane >> 2)) * kScoreLd + np * 16 + (lane & 3) * 2;
+  const int out_pieces = (p.rank + 15) / 16;
+  // this warp's part of the scores: 32 keys and a range of k-steps, for all heads
+  const int keys_at = (warp & 1) * 32, kpart = warp >> 1;
+  const int ks_lo = chunks * 4 * kpart / kSplit, ks_hi = chunks * 4 * (kpart + 1) / kSplit;
+  // A 16-byte unit u of row r and chunk c of a tile lies at row_at(r) + c * chunkb, its place in the 128 bytes xor'ed with the
+  // number of that 128-byte line (the TMA swizzle).
+  const int chunkb = p.whole ? 128 : p.box * 128;
+  auto row_at = [&](int r) { return p.whole ? r * chunks * 128 : (r >> p.box_log) * chunks * chunkb + (r & (p.box - 1)) * 128; };
+  float* my_scores = s_s + (kpart * kHeads + (lane >> 2)) * kScoreLd + keys_at + (lane & 3) * 2;
+  int key_at[2];
+#pragma unroll
+  for (int j = 0; j < 2; ++j) key_at[j] = row_at(keys_at + j * 16 + (lane >> 4) * 8 + (lane & 7));
+  const int val_row = ((lane >> 3) & 1) * 8 + (lane & 7);
   // this lane's part of the softmax: keys lk .. lk + kLaneKeys of head row
-  const int row = warp * kM + lane / kRowLanes, lk = (lane % kRowLanes) * kLaneKeys;
+  const int row = warp * 2 * kM + lane / kRowLanes, lk = (lane % kRowLanes) * kLaneKeys;
   float m_run = -INFINITY, l_run = 0.f;
   float o[kMaxPieces][kM][2][4];
 #pragma unroll
@@ -195,35 +210,90 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
     // after a wait that ran out the loop goes on without data, so that everyone still meets at the barriers
     mbar_wait(&full[st], phase, abort_flag, p.status, 1501, it);
     __syncwarp();
-    const uint32_t kb = smem_u32(s_k + st * kTileKeys * rowb);
+    const uint32_t kb = smem_u32(s_k + st * stageb);
+    if (it == tiles - 1 && (nk & (kTileKeys - 1)) != 0) {
+      // what lies past the last key was never a key of this sequence: 0 * NaN would poison the output
+      const int r0 = nk & (kTileKeys - 1);
+      for (int i = threadIdx.x; i < (kTileKeys - r0) * chunks * 8; i += kThreads) {
+        const int r = r0 + i / (chunks * 8), c = i % (chunks * 8);
+        *reinterpret_cast<uint4*>(s_k + st * stageb + row_at(r) + (c >> 3) * chunkb + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+      }
+      named_bar_sync(1, kThreads);
+    }
     {
-      float acc[2][2][4];  // alternate k-steps of the two key tiles
+      float acc[kM][4][4];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) acc[0][0][c] = acc[0][1][c] = acc[1][0][c] = acc[1][1][c] = 0.f;
-      const uint32_t qa = smem_u32(s_q) + (mt * 16 + (lane & 15)) * rowb + (lane >> 4) * 16;
-      // (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
-      const uint32_t ka = kb + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * rowb + ((lane >> 3) & 1) * 16;
-      auto k_step = [&](int ks, float (&c)[2][4]) {
-        uint32_t a[4], b0, b1, b2, b3;
-        ldm_x4(qa + ks * 32, a[0], a[1], a[2], a[3]);
-        ldm_x4(ka + ks * 32, b0, b1, b2, b3);
-        mma16816(c[0], a, b0, b1);
-        mma16816(c[1], a, b2, b3);
+      for (int m = 0; m < kM; ++m)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) acc[m][j][c] = 0.f;
+      const uint32_t qa = smem_u32(s_q) + (lane & 15) * rowb + (lane >> 4) * 16;
+      const int unit = (lane >> 3) & 1;
+      struct Frags {
+        uint32_t a[kM][4], b[2][4];
+      } f0, f1;
+      auto load = [&](int ks, Frags& f) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int line = key_at[j] + (ks >> 2) * chunkb;
+          // (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
+          ldm_x4(kb + line + ((((ks & 3) * 2 + unit) ^ ((line >> 7) & 7)) << 4), f.b[j][0], f.b[j][1], f.b[j][2], f.b[j][3]);
+        }
+#pragma unroll
+        for (int m = 0; m < kM; ++m) ldm_x4(qa + m * 16 * rowb + ks * 32, f.a[m][0], f.a[m][1], f.a[m][2], f.a[m][3]);
       };
-      int ks = ks_lo;
-#pragma unroll 3
-      for (; ks + 1 < ks_hi; ks += 2) {
-        k_step(ks, acc[0]);
-        k_step(ks + 1, acc[1]);
-      }
-      if (ks < ks_hi) k_step(ks, acc[0]);
+      auto mul = [&](Frags& f) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        *reinterpret_cast<float2*>(my_scores + j * 8) = make_float2(acc[0][j][0] + acc[1][j][0], acc[0][j][1] + acc[1][j][1]);
-        *reinterpret_cast<float2*>(my_scores + j * 8 + 8 * kScoreLd) = make_float2(acc[0][j][2] + acc[1][j][2], acc[0][j][3] + acc[1][j][3]);
+        for (int m = 0; m < kM; ++m)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            mma16816(acc[m][2 * j], f.a[m], f.b[j][0], f.b[j][1]);
+            mma16816(acc[m][2 * j + 1], f.a[m], f.b[j][2], f.b[j][3]);
+          }
+      };
+      if constexpr (kM == 1) {  // the next step's fragments are read ahead; with two M tiles that would spill, and eight MMAs hide the reads
+        load(ks_lo, f0);
+        int ks = ks_lo;
+#pragma unroll 1
+        for (; ks + 1 < ks_hi; ks += 2) {
+          load(ks + 1, f1);
+          mul(f0);
+          if (ks + 2 < ks_hi) load(ks + 2, f0);
+          mul(f1);
+        }
+        if (ks < ks_hi) mul(f0);
+      } else {
+#pragma unroll 1
+        for (int ks = ks_lo; ks < ks_hi; ++ks) {
+          load(ks, f0);
+          mul(f0);
+        }
       }
+#pragma unroll
+      for (int m = 0; m < kM; ++m)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          *reinterpret_cast<float2*>(my_scores + m * 16 * kScoreLd + j * 8) = make_float2(acc[m][j][0], acc[m][j][1]);
+          *reinterpret_cast<float2*>(my_scores + (m * 16 + 8) * kScoreLd + j * 8) = make_float2(acc[m][j][2], acc[m][j][3]);
+        }
     }
     named_bar_sync(1, kThreads);
+    // the value operand of 16 keys for the warp's output pieces: (keys 0-7, columns 0-7), (keys 8-15, same), (keys 0-7, columns 8-15),
+    // (keys 8-15, same)
+    uint32_t vb[kMaxPieces][4];
+    auto load_values = [&](int h) {
+      const int at = row_at(h * 16 + val_row);
+#pragma unroll
+      for (int a = 0; a < kMaxPieces; ++a) {
+        const int piece = warp + a * kWarps;
+        if (piece < out_pieces) {
+          const int line = at + (piece >> 2) * chunkb, unit = (piece & 3) * 2 + (lane >> 4);
+          ldm_x4_trans(kb + line + ((unit ^ ((line >> 7) & 7)) << 4), vb[a][0], vb[a][1], vb[a][2], vb[a][3]);
+        }
+      }
+    };
+    load_values(0);
     {
       float v[kLaneKeys];
 #pragma unroll
@@ -238,16 +308,16 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
           v[i + 1] += x.y;
         }
       }
-      const int left = nk - it * kTileKeys - lk;
+      const int left = nk - it * kTileKeys - lk, hidden = below - it * kTileKeys - lk;
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < kLaneKeys; ++i) {
-        v[i] = i < left ? v[i] * sc_log2 : -INFINITY;
+        v[i] = i < left && i >= hidden ? v[i] * sc_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
       for (int d = kRowLanes / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-      const float m_new = fmaxf(m_run, mx);  // finite: a tile has at least one key
+      const float m_new = fmaxf(m_run, mx);  // finite: a tile has at least one visible key
       float sum = 0.f;
 #pragma unroll
       for (int i = 0; i < kLaneKeys; i += 2) {
@@ -264,26 +334,17 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
     }
     named_bar_sync(1, kThreads);
     {
-      uint32_t pa[kM][4][4];
       float al[kM][2];
       bool moved = false;
 #pragma unroll
       for (int m = 0; m < kM; ++m) {
-#pragma unroll
-        for (int h = 0; h < 4; ++h)
-          ldm_x4(smem_u32(s_p) + (m * 16 + (lane & 15)) * kProbLd * 2 + h * 32 + (lane >> 4) * 16, pa[m][h][0], pa[m][h][1], pa[m][h][2], pa[m][h][3]);
         al[m][0] = s_alpha[m * 16 + (lane >> 2)];
         al[m][1] = s_alpha[m * 16 + 8 + (lane >> 2)];
         moved = moved || al[m][0] != 1.f || al[m][1] != 1.f;
       }
-      moved = __any_sync(0xffffffffu, moved);
-      // matrices of a transposing x4: (keys 0-7, columns 0-7), (keys 8-15, same), (keys 0-7, columns 8-15), (keys 8-15, same)
-      const uint32_t va = kb + (((lane >> 3) & 1) * 8 + (lane & 7)) * rowb + (lane >> 4) * 16;
+      if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-      for (int a = 0; a < kMaxPieces; ++a) {
-        const int piece = warp + a * kWarps;
-        if (piece >= out_pieces) break;
-        if (moved) {
+        for (int a = 0; a < kMaxPieces; ++a)
 #pragma unroll
           for (int m = 0; m < kM; ++m)
 #pragma unroll
@@ -291,15 +352,22 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(Params p
               o[a][m][j][0] *= al[m][0]; o[a][m][j][1] *= al[m][0];
               o[a][m][j][2] *= al[m][1]; o[a][m][j][3] *= al[m][1];
             }
-        }
+      }
+      const uint32_t probs = smem_u32(s_p) + (lane & 15) * kProbLd * 2 + (lane >> 4) * 16;
+#pragma unroll 1
+      for (int h = 0; h < 4; ++h) {
+        uint32_t pa[kM][4];
 #pragma unroll
-        for (int h = 0; h < 4; ++h) {
-          uint32_t b0, b1, b2, b3;
-          ldm_x4_trans(va + h * 16 * rowb + piece * 32, b0, b1, b2, b3);
+        for (int m = 0; m < kM; ++m) ldm_x4(probs + m * 16 * kProbLd * 2 + h * 32, pa[m][0], pa[m][1], pa[m][2], pa[m][3]);
+        if (h > 0) load_values(h);
 #pragma unroll
-          for (int m = 0; m < kM; ++m) {
-            mma16816(o[a][m][0], pa[m][h], b0, b1);
-            mma16816(o[a][m][1], pa[m][h], b2, b3);
+        for (int a = 0; a < kMaxPieces; ++a) {
+          if (warp + a * kWarps < out_pieces) {
+#pragma unroll
+            for (int m = 0; m < kM; ++m) {
+              mma16816(o[a][m][0], pa[m], vb[a][0], vb[a][1]);
+              mma16816(o[a][m][1], pa[m], vb[a][2], vb[a][3]);
+            }
           }
         }
       }
@@ -352,7 +420,7 @@ __global__ void __launch_bounds__(128) merge_kernel(Params p) {
   const int t = blockIdx.x, h = blockIdx.y;
   int seq = 0, ctx = 0;
   if (!locate(p, t, seq, ctx)) return;  // zeros are in place
-  const int visible = ctx - first_key(p, ctx), per = part_keys(p, visible);
+  const int visible = ctx - (first_key(p, ctx) & ~(p.box - 1)), per = part_keys(p, visible);
   const int np = (visible + per - 1) / per;
   const long long hrow = static_cast<long long>(t) * p.H + h;
   const float* ml = p.part_ml + hrow * p.parts * 2;
@@ -372,15 +440,15 @@ __global__ void __launch_bounds__(128) merge_kernel(Params p) {
 }
 
 template <int kM>
-int launch(const Params& p, cudaStream_t s) {
+int launch(const CUtensorMap& tm, const Params& p, cudaStream_t s) {
   static bool attr_set = false;
   auto kern = paged_latent_kernel<kM>;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return kErrCuda;
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem) != cudaSuccess) return kErrCuda;
     attr_set = true;
   }
   const int groups = (p.H + kM * 16 - 1) / (kM * 16);
-  kern<<<dim3(p.T, groups, p.parts), kThreads + 32, smem_bytes(kM, p.width, p.stages), s>>>(p);
+  kern<<<dim3(p.T, groups, p.parts), kThreads + 32, smem_bytes(kM, p.width, p.stages), s>>>(tm, p);
   if (cudaGetLastError() != cudaSuccess) return kErrCuda;
   if (p.parts > 1) merge_kernel<<<dim3(p.T, p.H), 128, 0, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
@@ -493,7 +561,7 @@ extern "C" int lvb_paged_latent_parts(int T, int H, int width, int rank, int max
 }
 
 // Packed query rows q [T, H, width] over pages [num_pages, page_size, width] whose rows' first `rank` elements are the values -> out [T, H, rank];
-// causal, window > 0: a row sees itself and the window - 1 positions before it.  width and rank: multiples of 8, rank <= 512, width <= 592.
+// causal, window > 0: a row sees itself and the window - 1 positions before it.  width and rank: multiples of 8, rank <= 512, width <= 576.
 extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices, const int* cu_q_lens,
                                 const int* num_seqs, void* out, float* part_o, float* part_ml, int T, int H, int width, int rank, int S,
                                 int pages_per_seq, int page_size, int num_pages, int window, int parts, float scale, int* status,
@@ -502,7 +570,7 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   using namespace lvb::latent;
   if (T <= 0) return kErrOk;
   if (H <= 0 || width <= 0 || rank <= 0 || rank > width || ((width | rank) & 7) || S <= 0 || window < 0 || parts < 1) return kErrBadArg;
-  if (rank > kMaxPieces * kWarps * 16 || width > 592) return kErrTooLarge;
+  if (rank > kMaxPieces * kWarps * 16 || width > 576) return kErrTooLarge;
   if (parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv_pages) | reinterpret_cast<uintptr_t>(out)) & 15) return kErrBadArg;
   Params p;
@@ -515,10 +583,18 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   p.parts = parts; p.window = window; p.scale = scale; p.status = status;
   const int m_tiles = H <= 16 ? 1 : 2;
   p.stages = kMaxStages;
-  while (p.stages > 2 && smem_bytes(m_tiles, width, p.stages) > 220 * 1024) --p.stages;
-  if (smem_bytes(m_tiles, width, p.stages) > 220 * 1024) return kErrTooLarge;
+  while (p.stages > 2 && smem_bytes(m_tiles, width, p.stages) > kMaxSmem) --p.stages;
+  p.box = kTileKeys;
+  p.box_log = 6;
+  for (; page_size % p.box != 0; p.box /= 2) --p.box_log;
+  CUtensorMap tm;
+  // rows of an odd number of chunks are free of bank conflicts as they are; else the chunks are kept apart
+  p.whole = (width & 63) == 0 && (chunks_of(width) & 1) != 0;
+  const uint64_t rows = static_cast<uint64_t>(num_pages) * page_size;
+  const int rc = p.whole ? make_tmap_chunked_bf16(&tm, kv_pages, rows, width, p.box) : make_tmap_2d_bf16(&tm, kv_pages, rows, width, width, p.box, 64);
+  if (rc != kErrOk) return rc;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return m_tiles == 1 ? launch<1>(p, s) : launch<2>(p, s);
+  return m_tiles == 1 ? launch<1>(tm, p, s) : launch<2>(tm, p, s);
 }
 
 // out(t, h) [N] = A(t, h) [K] times B(h): [N, K] with b_trans, else [K, N].  A(t, h) starts at a + t * lda + h * a_head, B(h) at b + h * b_head (row

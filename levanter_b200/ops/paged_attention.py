@@ -239,7 +239,7 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
                            window: Optional[int] = None) -> torch.Tensor:
     """Causal attention of ``q [T, H, width]`` over pages of ``width`` elements per slot whose first ``rank`` are the value: all heads read
     the same row per key -> ``[T, H, rank]``.  ``window`` as in :func:`paged_attention_general`.  bf16 with sizes that are multiples of
-    8 (rank up to 512, width up to 592) runs on tensor cores; everything else in fp32 arithmetic."""
+    8 (rank up to 512, width up to 576) runs on tensor cores; everything else in fp32 arithmetic."""
     T, H, w = q.shape
     b = batch_info
     if not _use_kernel(q, kv_pages):
@@ -255,7 +255,7 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
     i32 = lambda t: t.to(device=dev, dtype=torch.int32).contiguous()  # noqa: E731
     lens, pages, cu, ns = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
     out = torch.empty(T, H, rank, dtype=q.dtype, device=dev)
-    if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 592:
+    if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 576:
         rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), 0, out.data_ptr(), T, H, 1, w, rank,
                        H * w, 0, S, PP, ps, P, 0, int(window or 0), 1, float(sm_scale), 0.0, int(q.dtype == torch.float32), lib.stream_ptr())
         lib.check_rc(rc, "lvb_attention_any")
