@@ -37,23 +37,28 @@ def attention(tb: Table, T=8192, n_seq=4, H=32, KV=8, S=64, ctx=4096):
         if what == "latent":
             tb.pair(name + " (again)", new, "Fedolorn prefill attention 128/128",
                     lambda: FA.flash_attention_packed(ql[0], kl[0], vl[0], pos, scaling_factor=128 ** -0.5), **base, **like)
-    kvl, bl = _pages(S, ctx - 1, 16, KV, 256)
-    kvl = kvl.view(kvl.shape[0], 16, 2 * KV, 128)
-    ql = _randn(S, H, 128)
-    like = lambda: PA.ragged_paged_attention(ql, kvl, bl.seq_lens, bl.page_indices, bl.cu_q_lens, bl.num_seqs, sm_scale=0.1)  # noqa: E731
-    like_bytes = 2.0 * S * (ctx * KV * 256 + 2 * H * 128)
+    def llama_decode(seqs, keys):
+        """Llama's decode attention over as many sequences and keys: the call, its name, its bytes."""
+        kvl, bl = _pages(seqs, keys - 1, 16, KV, 256)
+        kvl = kvl.view(kvl.shape[0], 16, 2 * KV, 128)
+        ql = _randn(seqs, H, 128)
+        call = lambda: PA.ragged_paged_attention(ql, kvl, bl.seq_lens, bl.page_indices, bl.cu_q_lens, bl.num_seqs, sm_scale=0.1)  # noqa: E731
+        return call, f"Llama decode attention 128, {seqs} x {keys} keys", 2.0 * seqs * (keys * KV * 256 + 2 * H * 128)
+
     for dk, dv in ((128, 128), (128, 64)):
         kv, b = _pages(S, ctx - 1, 16, KV, dk + dv)
         q = _randn(S, H, dk)
-        tb.pair(f"decode attention {dk}/{dv}, {ctx} keys", lambda: PA.paged_attention_general(q, kv, KV, dv, b, sm_scale=dk ** -0.5), "Llama decode attention 128",
+        like, like_name, like_bytes = llama_decode(S, ctx)
+        tb.pair(f"decode attention {dk}/{dv}, {S} x {ctx} keys", lambda: PA.paged_attention_general(q, kv, KV, dv, b, sm_scale=dk ** -0.5), like_name,
                 like, nbytes=2.0 * S * (ctx * KV * (dk + dv) + H * (dk + dv)), like_bytes=like_bytes)
     for heads, rank, r, window, seqs in ((32, 512, 64, None, S), (32, 512, 64, 1024, S), (16, 512, 64, None, S), (32, 256, 32, None, S), (32, 512, 64, None, 8),
                                          (128, 512, 64, None, S)):
         kv, b = _pages(seqs, ctx - 1, 16, 1, rank + r)
         q = _randn(seqs, heads, rank + r)
         seen = min(window or ctx, ctx)
+        like, like_name, like_bytes = llama_decode(seqs, seen)
         tb.pair(f"decode latent, {heads} heads, {rank}+{r}, {seqs} x {seen} keys", lambda: PA.paged_attention_latent(q, kv, rank, b, sm_scale=0.1, window=window),
-                "Llama decode attention 128, 64 x 4096 keys", like, flops=2.0 * seqs * seen * heads * (2 * rank + r),
+                like_name, like, flops=2.0 * seqs * seen * heads * (2 * rank + r),
                 nbytes=2.0 * seqs * (seen * (rank + r) + heads * (2 * rank + r)), like_bytes=like_bytes)
 
 
@@ -69,7 +74,6 @@ def around_attention(tb: Table, H=32, KV=8, D=128, rank=512, r=64, E=4096):
     rotl = DefaultRotaryEmbeddingsConfig().build(D)
     roti = DefaultRotaryEmbeddingsConfig(interleaved=True).build(r)
     temp, lam, wn = _randn(H), _randn(1)[0], _randn(rank)
-    wo, wq = _randn(E, H * D, scale=0.02), _randn((H + 2 * KV) * D, E, scale=0.02)
     w = _randn(H, 2 * D, rank, scale=0.05)
     whole = _randn(H * (2 * D + r), rank + r, scale=0.05)
     for T in (64, 8192):
@@ -95,26 +99,24 @@ def around_attention(tb: Table, H=32, KV=8, D=128, rank=512, r=64, E=4096):
         pl = _randn(pages, 16, 1, rank + r)
         tb.pair(f"T={T}: latent norm, rotations, cache write", lambda: prepare_latent(down, wn, 1e-6, pl, dest, pos, roti, lq[..., D:]),
                 "Llama rotation and cache write", llama, nbytes=2.0 * T * (3 * (rank + r) + 2 * H * r), like_bytes=llama_bytes)
-        h, a = _randn(T, E), _randn(T, H * D)
-        g = lambda n, kk, out: dict(flops=2.0 * T * n * kk, nbytes=2.0 * (T * kk + n * kk) + out)  # noqa: E731
         lk = lambda n, kk, out: dict(like_flops=2.0 * T * n * kk, like_bytes=2.0 * (T * kk + n * kk) + out)  # noqa: E731
-        n3 = (H + 2 * KV) * D
-        wide = lambda: linear(h, wq)  # noqa: E731
         if T == 64:
             qa = _randn(T, H, rank + r)
             o = _randn(T, H, rank)
             out = _randn(T, H, D)
             nb = 2.0 * (H * D * rank + T * H * (D + rank))
-            small = lambda: linear(a, wo)  # noqa: E731
-            tb.pair(f"T={T}: queries into the latent", lambda: PA.head_product(lq[..., :D], w[:, :D], qa[..., :rank], b_trans=False), "Llama output projection", small,
-                    flops=2.0 * T * H * D * rank, nbytes=nb, **lk(E, H * D, 2.0 * T * E))
-            tb.pair(f"T={T}: values out of the latent", lambda: PA.head_product(o, w[:, D:], out, b_trans=True), "Llama output projection", small,
-                    flops=2.0 * T * H * D * rank, nbytes=nb, **lk(E, H * D, 2.0 * T * E))
+            ws, as_ = _randn(E, rank, scale=0.02), _randn(T, rank)  # as many weights in one plain product
+            small = lambda: linear(as_, ws)  # noqa: E731
+            tb.pair(f"T={T}: queries into the latent", lambda: PA.head_product(lq[..., :D], w[:, :D], qa[..., :rank], b_trans=False), f"Llama product {rank} -> {E}",
+                    small, flops=2.0 * T * H * D * rank, nbytes=nb, **lk(E, rank, 2.0 * T * E))
+            tb.pair(f"T={T}: values out of the latent", lambda: PA.head_product(o, w[:, D:], out, b_trans=True), f"Llama product {rank} -> {E}", small,
+                    flops=2.0 * T * H * D * rank, nbytes=nb, **lk(E, rank, 2.0 * T * E))
         else:
             lat = _randn(T, rank + r)
             n = whole.shape[0]
-            tb.pair(f"T={T}: whole keys and values from the latent", lambda: project(lat, whole), "Llama q, k, v in one product", wide,
-                    flops=2.0 * T * H * 2 * D * rank, nbytes=2.0 * (T * (rank + r) + H * 2 * D * rank + T * n), **lk(n3, E, 2.0 * T * n3))
+            ws, as_ = _randn(H * 2 * D, rank, scale=0.02), _randn(T, rank)  # the same keys and values without their rotated part
+            tb.pair(f"T={T}: whole keys and values from the latent", lambda: project(lat, whole), f"Llama product {rank} -> {H * 2 * D}", lambda: linear(as_, ws),
+                    flops=2.0 * T * H * 2 * D * rank, nbytes=2.0 * (T * (rank + r) + H * 2 * D * rank + T * n), **lk(H * 2 * D, rank, 2.0 * T * H * 2 * D))
 
 
 def recurrence(tb: Table, W=4096):
