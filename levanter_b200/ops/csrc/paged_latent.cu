@@ -3,9 +3,9 @@
 // the product of the two rows, and the value is c itself (the caller applies W_uv(h) to the result).  So a key is read once for
 // all heads and used twice.
 //
-//  * paged_latent: one CTA per (packed query row, group of up to 32 query heads, partition of the visible keys).  A producer warp
-//    looks up the pages and brings the keys by TMA in tiles of 64 rows (128-byte swizzle; boxes of the rows of a page, at most
-//    64), two to four tiles deep.  Eight warps compute: scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the
+//  * paged_latent: one CTA per (packed query row, group of up to 32 query heads, partition of the visible keys).  The keys come
+//    by TMA in tiles of 64 rows (128-byte swizzle; boxes of the rows of a page, at most 64), two to four tiles deep.  Eight warps
+//    compute: scores are warp-level MMAs (m16n8k16, bf16, fp32 accumulation) with the
 //    query heads as the M rows, a warp taking 32 keys and a quarter of the row; then every warp owns the online softmax of a few
 //    heads, which adds up the quarters; then a set of 16-column pieces of the output, with the value operand read from the key
 //    tile by transposing ldmatrix.  Shared-memory reads bound a tile as much as its transfer does, hence the large share per
@@ -18,13 +18,17 @@ namespace lvb {
 namespace latent {
 
 constexpr int kWarps = 8;              // computing warps
-constexpr int kThreads = kWarps * 32;  // computing threads; the producer warp comes after them
+constexpr int kThreads = kWarps * 32;
+// A ninth warp is the producer, except where two M tiles and a long row want all registers that eight warps can have: there the first
+// computing warp issues the copies.
+__host__ __device__ constexpr bool has_producer(int m_tiles, int pieces) { return m_tiles == 1 || pieces <= 2; }
+__host__ __device__ constexpr int cta_threads(int m_tiles, int pieces) { return kThreads + (has_producer(m_tiles, pieces) ? 32 : 0); }
 constexpr int kSplit = 4;      // parts that the inner dimension of the scores is cut into
 constexpr int kMaxStages = 4;
 constexpr int kMaxSmem = 226 * 1024;
 constexpr int kTileKeys = 64;
 constexpr int kMinPart = 64;   // keys of a partition, at least
-constexpr int kMaxPieces = 4;  // 16-column output pieces per warp: rank <= 4 * 8 * 16
+constexpr int kMaxRank = 512;
 constexpr int kScoreLd = 68;   // floats per row of the score tile
 constexpr int kProbLd = 72;    // bf16 per row of the probability tile
 
@@ -92,10 +96,11 @@ __host__ __device__ constexpr int smem_bytes(int m_tiles, int width, int stages)
   return 1024 + stages * stage_bytes(width) + m_tiles * 16 * (row_bytes(width) + kSplit * kScoreLd * 4 + kProbLd * 2 + 3 * 4) + 2 * kMaxStages * 8 + 16;
 }
 
-// kM: M tiles (16 query heads each) per CTA
-template <int kM>
-__global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __grid_constant__ CUtensorMap tm, Params p) {
-  constexpr int kHeads = kM * 16;
+// kM: M tiles (16 query heads each) per CTA.  kPieces: 16-column output pieces per warp, at most: rank <= kPieces * 8 * 16.
+template <int kM, int kPieces>
+__global__ void __launch_bounds__(cta_threads(kM, kPieces), 1) paged_latent_kernel(const __grid_constant__ CUtensorMap tm, Params p) {
+  constexpr int kHeads = kM * 16, kCta = cta_threads(kM, kPieces);
+  constexpr bool kProducer = has_producer(kM, kPieces);
   constexpr int kRowLanes = 16 / kM;             // lanes per head in the softmax: a warp owns 2 kM heads
   constexpr int kLaneKeys = kTileKeys / kRowLanes;
   extern __shared__ uint8_t smem_raw[];
@@ -122,7 +127,7 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
   const int k0 = base + part * per;
   if (!live || k0 >= ctx) {
     if (!live && part == 0) {
-      for (int i = threadIdx.x; i < heads * p.rank; i += kThreads + 32)
+      for (int i = threadIdx.x; i < heads * p.rank; i += kCta)
         p.out[(static_cast<long long>(t) * p.H + h0) * p.rank + i] = __float2bfloat16(0.f);
     }
     return;
@@ -141,7 +146,7 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
     tma_prefetch_desc(&tm);
   }
   // queries; rows beyond the heads and columns beyond the width are zeros
-  for (int i = threadIdx.x; i < kHeads * chunks * 8; i += kThreads + 32) {
+  for (int i = threadIdx.x; i < kHeads * chunks * 8; i += kCta) {
     const int r = i / (chunks * 8), c = i - r * (chunks * 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (r < heads && c * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(t) * p.H + h0 + r) * p.width + c * 8);
@@ -149,34 +154,45 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
   }
   __syncthreads();
 
-  if (warp == kWarps) {
-    // ---- producer: a lane per box
-    const int per_group = p.whole ? 1 : chunks, boxes = kTileKeys / p.box * per_group, boxb = p.box * 128 * (p.whole ? chunks : 1);
+  // ---- copies: a lane per box
+  const int per_group = p.whole ? 1 : chunks, boxes = kTileKeys / p.box * per_group, boxb = p.box * 128 * (p.whole ? chunks : 1);
+  auto lookup = [&](int tile, int i) -> int {  // cache row of box i; past the last key any rows will do, they are masked
+    const int key = k0 + tile * kTileKeys + i / per_group * p.box;
+    if (i >= boxes || key >= ctx) return 0;
+    const int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
+    return page >= 0 && page < p.num_pages ? page * p.page_size + key % p.page_size : 0;
+  };
+  auto issue = [&](int tile, int stage, int row_first) {
+    if (tile >= tiles) return;
+    if (lane == 0) mbar_expect_tx(&full[stage], stageb);
+    __syncwarp();
+    for (int i = lane; i < boxes; i += 32) {
+      const int row = i == lane ? row_first : lookup(tile, i);
+      uint8_t* dst = s_k + stage * stageb + i * boxb;
+      if (p.whole) tma_load_3d(dst, &tm, &full[stage], 0, 0, row);
+      else tma_load_2d(dst, &tm, &full[stage], i % chunks * 64, row);
+    }
+  };
+  if (kProducer && warp == kWarps) {
     int st = 0;
     uint32_t phase = 0;
     for (int it = 0; it < tiles; ++it) {
+      const int row_first = lookup(it, lane);
       bool ok = mbar_wait(&empty[st], phase ^ 1, abort_flag, p.status, 1500, it);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
-      if (lane == 0) mbar_expect_tx(&full[st], stageb);
-      __syncwarp();
-      for (int i = lane; i < boxes; i += 32) {
-        const int group = i / per_group, chunk = i - group * per_group;
-        const int key = k0 + it * kTileKeys + group * p.box;
-        int row = 0;  // past the last key: any rows will do, they are masked
-        if (key < ctx) {
-          const int page = p.page_indices[seq * p.pages_per_seq + key / p.page_size];
-          if (page >= 0 && page < p.num_pages) row = page * p.page_size + key % p.page_size;
-        }
-        if (p.whole) tma_load_3d(s_k + st * stageb + i * boxb, &tm, &full[st], 0, 0, row);
-        else tma_load_2d(s_k + st * stageb + i * boxb, &tm, &full[st], chunk * 64, row);
-      }
+      issue(it, st, row_first);
       if (++st == p.stages) {
         st = 0;
         phase ^= 1;
       }
     }
     return;
+  }
+  int row_next = 0;
+  if (!kProducer && warp == 0) {
+    for (int i = 0; i < p.stages - 1; ++i) issue(i, i, lookup(i, lane));
+    row_next = lookup(p.stages - 1, lane);
   }
 
   const float sc_log2 = p.scale * 1.4426950408889634f;
@@ -196,9 +212,9 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
   // this lane's part of the softmax: keys lk .. lk + kLaneKeys of head row
   const int row = warp * 2 * kM + lane / kRowLanes, lk = (lane % kRowLanes) * kLaneKeys;
   float m_run = -INFINITY, l_run = 0.f;
-  float o[kMaxPieces][kM][2][4];
+  float o[kPieces][kM][2][4];
 #pragma unroll
-  for (int a = 0; a < kMaxPieces; ++a)
+  for (int a = 0; a < kPieces; ++a)
 #pragma unroll
     for (int b = 0; b < kM; ++b)
 #pragma unroll
@@ -207,6 +223,13 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
   int st = 0;
   uint32_t phase = 0;
   for (int it = 0; it < tiles; ++it) {
+    if (!kProducer && warp == 0) {  // once everyone is done with the tile before this one, its buffer takes the next copies
+      const int prev = st == 0 ? p.stages - 1 : st - 1;
+      bool ok = it == 0 || mbar_wait(&empty[prev], st == 0 ? phase ^ 1 : phase, abort_flag, p.status, 1500, it);
+      ok = __all_sync(0xffffffffu, ok);
+      if (ok) issue(it + p.stages - 1, prev, row_next);
+      row_next = lookup(it + p.stages, lane);
+    }
     // after a wait that ran out the loop goes on without data, so that everyone still meets at the barriers
     mbar_wait(&full[st], phase, abort_flag, p.status, 1501, it);
     __syncwarp();
@@ -252,24 +275,16 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
             mma16816(acc[m][2 * j + 1], f.a[m], f.b[j][2], f.b[j][3]);
           }
       };
-      if constexpr (kM == 1) {  // the next step's fragments are read ahead; with two M tiles that would spill, and eight MMAs hide the reads
-        load(ks_lo, f0);
-        int ks = ks_lo;
+      load(ks_lo, f0);
+      int ks = ks_lo;
 #pragma unroll 1
-        for (; ks + 1 < ks_hi; ks += 2) {
-          load(ks + 1, f1);
-          mul(f0);
-          if (ks + 2 < ks_hi) load(ks + 2, f0);
-          mul(f1);
-        }
-        if (ks < ks_hi) mul(f0);
-      } else {
-#pragma unroll 1
-        for (int ks = ks_lo; ks < ks_hi; ++ks) {
-          load(ks, f0);
-          mul(f0);
-        }
+      for (; ks + 1 < ks_hi; ks += 2) {  // the next step's fragments are read ahead
+        load(ks + 1, f1);
+        mul(f0);
+        if (ks + 2 < ks_hi) load(ks + 2, f0);
+        mul(f1);
       }
+      if (ks < ks_hi) mul(f0);
 #pragma unroll
       for (int m = 0; m < kM; ++m)
 #pragma unroll
@@ -279,21 +294,19 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
         }
     }
     named_bar_sync(1, kThreads);
-    // the value operand of 16 keys for the warp's output pieces: (keys 0-7, columns 0-7), (keys 8-15, same), (keys 0-7, columns 8-15),
-    // (keys 8-15, same)
-    uint32_t vb[kMaxPieces][4];
-    auto load_values = [&](int h) {
-      const int at = row_at(h * 16 + val_row);
+    // the value operand of the warp's first output piece: (keys 0-7, columns 0-7), (keys 8-15, same), (keys 0-7, columns 8-15),
+    // (keys 8-15, same) of each 16 keys
+    uint32_t vb[4][4];
+    auto load_values = [&](int piece) {
 #pragma unroll
-      for (int a = 0; a < kMaxPieces; ++a) {
-        const int piece = warp + a * kWarps;
-        if (piece < out_pieces) {
-          const int line = at + (piece >> 2) * chunkb, unit = (piece & 3) * 2 + (lane >> 4);
-          ldm_x4_trans(kb + line + ((unit ^ ((line >> 7) & 7)) << 4), vb[a][0], vb[a][1], vb[a][2], vb[a][3]);
-        }
+      for (int h = 0; h < 4; ++h) {
+        int r = h * 16 + val_row;
+        asm volatile("" : "+r"(r));  // computed per tile: hoisted out of the loop, the addresses would spill
+        const int line = row_at(r) + (piece >> 2) * chunkb, unit = (piece & 3) * 2 + (lane >> 4);
+        ldm_x4_trans(kb + line + ((unit ^ ((line >> 7) & 7)) << 4), vb[h][0], vb[h][1], vb[h][2], vb[h][3]);
       }
     };
-    load_values(0);
+    if (warp < out_pieces) load_values(warp);
     {
       float v[kLaneKeys];
 #pragma unroll
@@ -302,10 +315,12 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
       for (int k = 0; k < kSplit; ++k) {
         const float* src = s_s + (k * kHeads + row) * kScoreLd + lk;
 #pragma unroll
-        for (int i = 0; i < kLaneKeys; i += 2) {
-          const float2 x = *reinterpret_cast<const float2*>(src + i);
+        for (int i = 0; i < kLaneKeys; i += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(src + i);
           v[i] += x.x;
           v[i + 1] += x.y;
+          v[i + 2] += x.z;
+          v[i + 3] += x.w;
         }
       }
       const int left = nk - it * kTileKeys - lk, hidden = below - it * kTileKeys - lk;
@@ -334,17 +349,25 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
     }
     named_bar_sync(1, kThreads);
     {
+      uint32_t pa[kM][4][4];
       float al[kM][2];
       bool moved = false;
 #pragma unroll
       for (int m = 0; m < kM; ++m) {
+#pragma unroll
+        for (int h = 0; h < 4; ++h)
+          ldm_x4(smem_u32(s_p) + (m * 16 + (lane & 15)) * kProbLd * 2 + h * 32 + (lane >> 4) * 16, pa[m][h][0], pa[m][h][1], pa[m][h][2], pa[m][h][3]);
         al[m][0] = s_alpha[m * 16 + (lane >> 2)];
         al[m][1] = s_alpha[m * 16 + 8 + (lane >> 2)];
         moved = moved || al[m][0] != 1.f || al[m][1] != 1.f;
       }
-      if (__any_sync(0xffffffffu, moved)) {
+      moved = __any_sync(0xffffffffu, moved);
 #pragma unroll
-        for (int a = 0; a < kMaxPieces; ++a)
+      for (int a = 0; a < kPieces; ++a) {
+        const int piece = warp + a * kWarps;
+        if (piece >= out_pieces) break;
+        if (a > 0) load_values(piece);
+        if (moved) {
 #pragma unroll
           for (int m = 0; m < kM; ++m)
 #pragma unroll
@@ -352,24 +375,14 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
               o[a][m][j][0] *= al[m][0]; o[a][m][j][1] *= al[m][0];
               o[a][m][j][2] *= al[m][1]; o[a][m][j][3] *= al[m][1];
             }
-      }
-      const uint32_t probs = smem_u32(s_p) + (lane & 15) * kProbLd * 2 + (lane >> 4) * 16;
-#pragma unroll 1
-      for (int h = 0; h < 4; ++h) {
-        uint32_t pa[kM][4];
-#pragma unroll
-        for (int m = 0; m < kM; ++m) ldm_x4(probs + m * 16 * kProbLd * 2 + h * 32, pa[m][0], pa[m][1], pa[m][2], pa[m][3]);
-        if (h > 0) load_values(h);
-#pragma unroll
-        for (int a = 0; a < kMaxPieces; ++a) {
-          if (warp + a * kWarps < out_pieces) {
-#pragma unroll
-            for (int m = 0; m < kM; ++m) {
-              mma16816(o[a][m][0], pa[m], vb[a][0], vb[a][1]);
-              mma16816(o[a][m][1], pa[m], vb[a][2], vb[a][3]);
-            }
-          }
         }
+#pragma unroll
+        for (int h = 0; h < 4; ++h)
+#pragma unroll
+          for (int m = 0; m < kM; ++m) {
+            mma16816(o[a][m][0], pa[m][h], vb[h][0], vb[h][1]);
+            mma16816(o[a][m][1], pa[m][h], vb[h][2], vb[h][3]);
+          }
       }
     }
     __syncwarp();
@@ -390,7 +403,7 @@ __global__ void __launch_bounds__(kThreads + 32, 1) paged_latent_kernel(const __
     ml[1] = s_l[threadIdx.x];
   }
 #pragma unroll
-  for (int a = 0; a < kMaxPieces; ++a) {
+  for (int a = 0; a < kPieces; ++a) {
     const int piece = warp + a * kWarps;
     if (piece >= out_pieces) break;
 #pragma unroll
@@ -439,16 +452,16 @@ __global__ void __launch_bounds__(128) merge_kernel(Params p) {
   }
 }
 
-template <int kM>
+template <int kM, int kPieces>
 int launch(const CUtensorMap& tm, const Params& p, cudaStream_t s) {
   static bool attr_set = false;
-  auto kern = paged_latent_kernel<kM>;
+  auto kern = paged_latent_kernel<kM, kPieces>;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem) != cudaSuccess) return kErrCuda;
     attr_set = true;
   }
   const int groups = (p.H + kM * 16 - 1) / (kM * 16);
-  kern<<<dim3(p.T, groups, p.parts), kThreads + 32, smem_bytes(kM, p.width, p.stages), s>>>(tm, p);
+  kern<<<dim3(p.T, groups, p.parts), cta_threads(kM, kPieces), smem_bytes(kM, p.width, p.stages), s>>>(tm, p);
   if (cudaGetLastError() != cudaSuccess) return kErrCuda;
   if (p.parts > 1) merge_kernel<<<dim3(p.T, p.H), 128, 0, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
@@ -570,7 +583,7 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   using namespace lvb::latent;
   if (T <= 0) return kErrOk;
   if (H <= 0 || width <= 0 || rank <= 0 || rank > width || ((width | rank) & 7) || S <= 0 || window < 0 || parts < 1) return kErrBadArg;
-  if (rank > kMaxPieces * kWarps * 16 || width > 576) return kErrTooLarge;
+  if (rank > kMaxRank || width > 576) return kErrTooLarge;
   if (parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv_pages) | reinterpret_cast<uintptr_t>(out)) & 15) return kErrBadArg;
   Params p;
@@ -594,7 +607,9 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   const int rc = p.whole ? make_tmap_chunked_bf16(&tm, kv_pages, rows, width, p.box) : make_tmap_2d_bf16(&tm, kv_pages, rows, width, width, p.box, 64);
   if (rc != kErrOk) return rc;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return m_tiles == 1 ? launch<1>(tm, p, s) : launch<2>(tm, p, s);
+  const bool narrow = rank <= 256;
+  if (m_tiles == 1) return narrow ? launch<1, 2>(tm, p, s) : launch<1, 4>(tm, p, s);
+  return narrow ? launch<2, 2>(tm, p, s) : launch<2, 4>(tm, p, s);
 }
 
 // out(t, h) [N] = A(t, h) [K] times B(h): [N, K] with b_trans, else [K, N].  A(t, h) starts at a + t * lda + h * a_head, B(h) at b + h * b_head (row
