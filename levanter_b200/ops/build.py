@@ -27,8 +27,8 @@ SERVING_LIBNAME = "liblevanter_b200_serving.so"
 SERVING_SOURCES = ("attention_any", "elementwise", "flash_attn_fwd2", "gated_scan", "gemm_bf16", "gemm_pair", "gemm_skinny", "moe_experts",
                    "page_table", "paged_attention", "paged_latent", "qkv_prep", "residual_stream", "sampler")
 
-# Kernels whose results are 32-bit throughout (norms of an fp32 stream, router scores, rotary angles, gated recurrences, fp32 attention): no approximate
-# exponentials, divisions or square roots.
+# Kernels whose results are 32-bit throughout (norms of an fp32 stream, router scores, rotary angles, gated recurrences, fp32
+# attention): no fast-math exponentials, divisions or square roots.
 ACCURATE_SOURCES = ("attention_any", "gated_scan", "moe_experts", "qkv_prep", "residual_stream")
 
 NVCC_FLAGS = [

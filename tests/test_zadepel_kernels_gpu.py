@@ -235,8 +235,7 @@ def test_paged_attention_in_a_window(dtype, H, G, dk, dv, window):
     data = []
     for i, n in enumerate(lens):
         q, k, v = _randn(n, H, dk, seed=i, dtype=dtype), _randn(n, G, dk, seed=50 + i, dtype=dtype), _randn(n, G, dv, seed=90 + i, dtype=dtype)
-        if window is not None:
-            _needles(q, k, window)
+        _needles(q, k, min(window or 300, 300))  # without a window (or with a wide one): keys far away
         data.append((q, k, v))
         if n > last[i]:
             b, _ = seqs.step([(i, n - last[i])], pad=1)
@@ -271,8 +270,7 @@ def test_latent_attention(dtype, H, rank, r, window, page):
     data = []
     for i, n in enumerate(lens):
         q, k = _randn(n, H, w, seed=i, dtype=dtype), _randn(n, 1, w, seed=50 + i, dtype=dtype)
-        if window is not None:
-            _needles(q, k, window)
+        _needles(q, k, min(window or 300, 300))  # without a window (or with a wide one): keys far away
         data.append((q, k))
         if n > last[i]:
             b, _ = seqs.step([(i, n - last[i])], pad=0)
@@ -317,8 +315,7 @@ def test_packed_prefill_in_a_window(H, G, dk, dv, window):
     at, want = 0, []
     for i, m in enumerate(lens):
         q, k, v = _randn(m, H, dk, seed=i), _randn(m, G, dk, seed=30 + i), _randn(m, G, dv, seed=60 + i)
-        if window is not None:
-            _needles(q, k, window)
+        _needles(q, k, min(window or 300, 300))  # without a window (or with a wide one): keys far away
         wide[at:at + m] = torch.cat([q.flatten(1), k.flatten(1), v.flatten(1)], dim=1)
         pos[at:at + m] = torch.arange(m)
         want.append(O.softmax_attention(q.double(), k.double(), v.double(), 0.35, window))
