@@ -392,9 +392,22 @@ class AttentionConfig:
     output_gate: bool = False                 # the heads are multiplied by sigmoid(W_g x) before the output projection
     head_temperature: bool = False            # a learned number per query head multiplies its scores
     value_mixing: bool = False                # v <- (1 - m) v + m v_first with a learned m and the first such layer's values
+    head_gate: bool = False                   # head h is multiplied by sigmoid((W_g x)_h), one number per head (no bias)
+    differential: Optional[float] = None      # two score maps per head over the same values, combined as in MapDifference; the number is the
+    #                                           constant part of the second map's weight
+    norm_eps: float = 1e-6                    # of the norm after the difference
 
     def __post_init__(self):
         assert self.num_heads % self.num_kv_heads == 0, "num_heads must be divisible by num_kv_heads"
+        if self.differential is not None and (self.qk_norm is not None or self.head_temperature or self.output_gate):
+            raise ValueError("differential attention takes neither qk_norm, nor head temperatures, nor a gate per element")
+        if self.head_gate and self.output_gate:
+            raise ValueError("a gate per head and a gate per element exclude each other")
+
+    @property
+    def maps(self) -> int:
+        """Score maps per head."""
+        return 1 if self.differential is None else 2
 
     @property
     def head_size(self) -> int:
@@ -425,7 +438,7 @@ class Attention(nn.Module):
         super().__init__()
         c = config
         self.config = c
-        D, Dv = c.head_size, c.v_head_size
+        D, Dv = c.maps * c.head_size, c.v_head_size
         self.tp = tp
         tp_size = tp.size if tp is not None else 1
         assert c.num_kv_heads % tp_size == 0 or tp_size == 1, "kv heads must divide the tensor-parallel size"
@@ -443,28 +456,44 @@ class Attention(nn.Module):
         if c.output_gate:
             self.g_proj = Linear(c.hidden_dim, self.local_heads * Dv, bias=c.use_bias, init_std=init_std,
                                  lev_out=(self.local_kv, c.q_heads_per_group, Dv), lev_in=(c.hidden_dim,), parallel=("column", tp))
+        if c.head_gate:
+            self.g_proj = Linear(c.hidden_dim, self.local_heads, init_std=init_std, lev_out=(self.local_kv, c.q_heads_per_group), lev_in=(c.hidden_dim,),
+                                 parallel=("column", tp))
+        if c.differential is not None:
+            for n in self.difference_names:
+                p = nn.Parameter(torch.randn(c.head_size) * 0.1)
+                p.lev_shape = (c.head_size,)
+                setattr(self, n, p)
+            self._difference = None
         if c.qk_norm is not None:
             self.q_norm = c.qk_norm.build(D)
             self.k_norm = c.qk_norm.build(D)
         else:
             self.q_norm = None
             self.k_norm = None
-        self.rot: Optional[RotaryEmbeddings] = c.rope.build(D) if c.rope is not None else None
+        self.rot: Optional[RotaryEmbeddings] = c.rope.build(c.head_size) if c.rope is not None else None
         if c.head_temperature:
             self.temperature = nn.Parameter(torch.ones(self.local_heads))
             self.temperature.lev_shape = (self.local_heads,)
         if c.value_mixing:
             self.value_mix = nn.Parameter(torch.tensor(0.5))
             self.value_mix.lev_shape = ()
-        self._rows, self._bias_rows = FusedRows(), FusedRows()
+        rows = sum(m.weight.shape[0] for m in self._projections())
+        pad = -rows % 8  # whole groups of 8 columns keep the slices of the joint product aligned
+        self._rows, self._bias_rows = FusedRows(pad), FusedRows(pad + (self.local_heads if c.head_gate else 0))
+
+    difference_names = ("lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2")
+
+    def _projections(self):
+        return [self.q_proj, self.k_proj, self.v_proj] + ([self.g_proj] if self.config.output_gate or self.config.head_gate else [])
 
     # -- projections shared by training and paged decode (src/levanter/layers/attention.py:1606-1635)
     def _compute_qkv(self, x: torch.Tensor, pos_ids: Optional[torch.Tensor], rotate: bool = True):
         c = self.config
         D = c.head_size
         lead = x.shape[:-1]
-        q = self.q_proj(x).view(*lead, self.local_heads, D)
-        k = self.k_proj(x).view(*lead, self.local_kv, D)
+        q = self.q_proj(x).view(*lead, c.maps * self.local_heads, D)
+        k = self.k_proj(x).view(*lead, c.maps * self.local_kv, D)
         v = self.v_proj(x).view(*lead, self.local_kv, c.v_head_size)
         if self.q_norm is not None:
             q = self.q_norm(q)
@@ -474,6 +503,25 @@ class Attention(nn.Module):
 
             q, k = rope_op.apply_rope(q, k, self.rot, pos_ids)
         return q, k, v
+
+    def map_difference(self):
+        """How the two score maps of a head are combined when serving (``ops.map_difference``); the weight of the second map is derived from
+        the learned vectors and made again when one of them has moved or changed, and after every change of mode."""
+        from ..ops.map_difference import MapDifference, difference_weight
+
+        c = self.config
+        vecs = [getattr(self, n) for n in self.difference_names]
+        if torch.is_grad_enabled():
+            return MapDifference(difference_weight(*vecs, c.differential), 1.0 - c.differential, c.norm_eps)
+        key = tuple((p.data_ptr(), p._version, p.dtype) for p in vecs)
+        if self._difference is None or self._difference[0] != key:
+            self._difference = (key, MapDifference(difference_weight(*(p.detach() for p in vecs), c.differential), 1.0 - c.differential, c.norm_eps))
+        return self._difference[1]
+
+    def train(self, mode: bool = True):
+        if self.config.differential is not None:
+            self._difference = None
+        return super().train(mode)
 
     def _temper_and_mix(self, q, v, v_first):
         """Differentiable forms of the head temperatures and of value mixing."""
@@ -510,12 +558,17 @@ class Attention(nn.Module):
         squeeze = q.dim() == 3
         if squeeze:
             q, k, v = q.unsqueeze(0), k.unsqueeze(0), v.unsqueeze(0)
-        attn = dot_product_attention(
-            q, k, v, mask, attention_dtype=torch.float32 if c.upcast_attn else None, attn_backend=c.attn_backend,
+        maps = [dot_product_attention(
+            q[:, :, i::c.maps], k[:, :, i::c.maps], v, mask, attention_dtype=torch.float32 if c.upcast_attn else None, attn_backend=c.attn_backend,
             flash_block_size=c.flash_attention_block_size, logits_soft_cap=c.logits_soft_cap,
-            scaling_factor=c.scaling_factor, inference=True)
+            scaling_factor=c.scaling_factor, inference=True) for i in range(c.maps)]
+        attn = maps[0]
+        if c.differential is not None:
+            attn = self.map_difference()(*maps)
         if squeeze:
             attn = attn.squeeze(0)
+        if c.head_gate:
+            attn = attn.float() * torch.sigmoid(self.g_proj(x).float()).unsqueeze(-1)
         attn = attn.reshape(*x.shape[:-1], self.local_heads * c.v_head_size).to(x.dtype)
         if c.output_gate:
             attn = attn * torch.sigmoid(self.g_proj(x).float()).to(attn.dtype)
@@ -541,7 +594,7 @@ class Attention(nn.Module):
 
         c = self.config
         if c.output_gate or c.attention_chunk_size is not None or c.v_head_size != c.head_size or c.sliding_window is not None \
-                or c.head_temperature or c.value_mixing or (self.rot is not None and not self.rot.is_plain):
+                or c.head_temperature or c.value_mixing or c.head_gate or c.differential is not None or (self.rot is not None and not self.rot.is_plain):
             out, _ = self._paged_heads(x, kv_cache, batch_info, pos_ids)
             return (self.o_proj(out) if residual is None else self.o_proj(out) + residual), kv_cache
         q, k, v = self._compute_qkv(x, pos_ids)
@@ -570,13 +623,16 @@ class Attention(nn.Module):
     def _fused_projection(self):
         """``(weight, bias or None)`` of the joint projection ``[q; k; v; gate]`` for serving: the projections read the same rows, so a
         decode step streams one matrix instead of launching four products.  None when a projection is wrapped (LoRA, fp8) or only
-        some have a bias, and for a model in training."""
-        mods = [self.q_proj, self.k_proj, self.v_proj] + ([self.g_proj] if self.config.output_gate else [])
-        biased = [m.bias is not None for m in mods] if all(type(m) is Linear for m in mods) else [True, False]
-        if self.training or any(biased) != all(biased):
+        some of q, k, v have a bias, and for a model in training.  (The gate per head has none: its rows of the bias are zeros.)"""
+        mods = self._projections()
+        if self.training or not all(type(m) is Linear for m in mods):
+            return None
+        with_bias = mods[:3] if self.config.head_gate else mods
+        biased = [m.bias is not None for m in with_bias]
+        if any(biased) != all(biased):
             return None
         w = self._rows.get([m.weight for m in mods])
-        b = self._bias_rows.get([m.bias for m in mods]) if w is not None and biased[0] else None
+        b = self._bias_rows.get([m.bias for m in with_bias]) if w is not None and biased[0] else None
         return None if w is None or (biased[0] and b is None) else (w, b)
 
     def _paged_heads(self, x, kv_cache: "KvPageCache", batch_info, pos_ids, v_first: Optional[torch.Tensor] = None):
@@ -590,17 +646,17 @@ class Attention(nn.Module):
 
         c = self.config
         T, D, Dv = x.shape[0], c.head_size, c.v_head_size
-        nq, nk, nv = self.local_heads * D, self.local_kv * D, self.local_kv * Dv
+        nq, nk, nv = c.maps * self.local_heads * D, c.maps * self.local_kv * D, self.local_kv * Dv
         fused = self._fused_projection() if (x.is_cuda and not torch.is_grad_enabled() and self.q_norm is None) else None
         gate = None
         if fused is not None:
             y = project(x, fused[0], bias=fused[1])
             q, k, v = y[:, :nq].unflatten(1, (-1, D)), y[:, nq:nq + nk].unflatten(1, (-1, D)), y[:, nq + nk:nq + nk + nv].unflatten(1, (-1, Dv))
-            if c.output_gate:
-                gate = y[:, nq + nk + nv:]
+            if c.output_gate or c.head_gate:
+                gate = y[:, nq + nk + nv:nq + nk + nv + self.g_proj.weight.shape[0]]
         else:
             q, k, v = self._compute_qkv(x, pos_ids, rotate=False)
-            if c.output_gate:
+            if c.output_gate or c.head_gate:
                 gate = self.g_proj(x)
         if self.rot is not None or c.head_temperature or c.value_mixing:
             q, k, v = prepare_qkv(q, k, v, kv_cache.kv_pages, batch_info.new_token_dests, pos_ids, rot=self.rot,
@@ -612,13 +668,12 @@ class Attention(nn.Module):
             PA.kv_page_write_general(kv_cache.kv_pages, k, v, batch_info.new_token_dests)
         scale = c.scaling_factor if c.scaling_factor is not None else 1.0 / math.sqrt(D)
         seg = getattr(batch_info, "prefill_segment_ids", None)
-        if seg is not None and FA.packed_supported(q, k, v, scale):
+        kw = dict(chunk=c.attention_chunk_size, window=c.sliding_window, gate=gate, difference=None if c.differential is None else self.map_difference())
+        if seg is not None and FA.packed_supported(q, k, v, scale, c.maps):
             # pure prefill: every sequence starts at position 0, nothing is read back from the cache
-            out = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=scale, chunk=c.attention_chunk_size, window=c.sliding_window, gate=gate,
-                                            logits_soft_cap=c.logits_soft_cap)
+            out = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=scale, logits_soft_cap=c.logits_soft_cap, **kw)
         else:
-            out = PA.paged_attention_general(q, kv_cache.kv_pages, self.local_kv, Dv, batch_info, sm_scale=scale, chunk=c.attention_chunk_size,
-                                             window=c.sliding_window, gate=gate, soft_cap=c.logits_soft_cap)
+            out = PA.paged_attention_general(q, kv_cache.kv_pages, self.local_kv, Dv, batch_info, sm_scale=scale, soft_cap=c.logits_soft_cap, **kw)
         return out.reshape(T, self.local_heads * Dv).to(x.dtype), v_first
 
     def paged_decode_stream(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor):
@@ -641,8 +696,8 @@ class Attention(nn.Module):
         return self.o_proj(out).float(), v_first
 
     def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
-        return KvPageCache.init(max_pages, page_size, self.local_kv, self.config.head_size, v_head_size=self.config.v_head_size, dtype=dtype,
-                                device=device)
+        c = self.config
+        return KvPageCache.init(max_pages, page_size, self.local_kv, c.maps * c.head_size, v_head_size=c.v_head_size, dtype=dtype, device=device)
 
 
 class AttentionWithSink(Attention):
@@ -689,6 +744,7 @@ class MultiHeadLatentAttentionConfig:
     logits_soft_cap: Optional[float] = None
     norm_eps: float = 1e-6
     sliding_window: Optional[int] = None  # a query sees itself and that many positions less one before it
+    sink: bool = False  # a learned number per head joins the softmax denominator (unscaled, with no key and no value)
 
     @property
     def softmax_scale(self) -> float:
@@ -700,7 +756,8 @@ class MultiHeadLatentAttentionConfig:
 
 
 class MultiHeadLatentAttention(nn.Module):
-    """K/V are reconstructed from a low-rank latent (``kv_lora_rank``) plus a decoupled RoPE key shared by all heads;
+    """K/V are reconstructed from a low-rank latent (``kv_lora_rank``) plus a decoupled RoPE key shared by all heads (none with
+    ``qk_rope_head_dim`` 0: attention without positions);
     queries optionally pass through their own low-rank bottleneck (src/levanter/layers/attention.py:2063-2213).
 
     Serving (:meth:`paged_decode`) caches the normed latent and the rotated key part of a token, ``kv_lora_rank + qk_rope_head_dim``
@@ -726,8 +783,21 @@ class MultiHeadLatentAttention(nn.Module):
         self.kv_b_proj = Linear(c.kv_lora_rank, H * (c.qk_nope_head_dim + c.v_head_dim), bias=c.use_bias, init_std=init_std)
         self.o_proj = Linear(H * c.v_head_dim, c.hidden_dim, bias=c.use_bias, init_std=init_std)
         rope = c.rope if c.rope is not None else DefaultRotaryEmbeddingsConfig()
-        self.rot = rope.build(c.qk_rope_head_dim)
-        self._rows, self._whole_kv = FusedRows(), None
+        self.rot = rope.build(c.qk_rope_head_dim) if c.qk_rope_head_dim > 0 else None
+        if c.sink:
+            self.sinks = nn.Parameter(torch.zeros(H))
+            self.sinks.lev_shape = (H,)
+        self._rows, self._whole_kv, self._sinks = FusedRows(-(H * c.qk_head_dim + c.kv_lora_rank + c.qk_rope_head_dim) % 8), None, None
+
+    def sinks_fp32(self) -> Optional[torch.Tensor]:
+        """The sink numbers in fp32 at a fixed address (it goes into captured graphs), made again like :meth:`_whole_kv_weight`."""
+        if not self.config.sink:
+            return None
+        s = self.sinks
+        key = (s.data_ptr(), s._version, s.dtype, s.device)
+        if self._sinks is None or self._sinks[0] != key:
+            self._sinks = (key, s.detach().float().contiguous().clone())
+        return self._sinks[1]
 
     def up_projections(self, weight: torch.Tensor):
         """``(W_uk [H, qk_nope_head_dim, rank], W_uv [H, v_head_dim, rank])``: views of ``kv_b_proj``'s weight (or of its gradient and the
@@ -755,7 +825,7 @@ class MultiHeadLatentAttention(nn.Module):
         return self._whole_kv[1]
 
     def train(self, mode: bool = True):
-        self._whole_kv = None
+        self._whole_kv = self._sinks = None
         return super().train(mode)
 
     def empty_page_cache(self, max_pages: int, page_size: int, *, dtype=torch.bfloat16, device=None) -> "KvPageCache":
@@ -764,6 +834,24 @@ class MultiHeadLatentAttention(nn.Module):
 
     def paged_decode(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids: torch.Tensor) -> torch.Tensor:
         """Packed rows ``x [T, hidden]`` of a serving step -> ``[T, hidden]`` in fp32; their latents enter the cache."""
+        from ..ops.residual_stream import project
+
+        heads = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        if type(self.o_proj) is Linear:
+            return project(heads, self.o_proj.weight, out_dtype=torch.float32)
+        return self.o_proj(heads).float()
+
+    def paged_decode_stream(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor):
+        """:meth:`paged_decode` for an fp32 residual stream: ``stream + o_proj(heads)``, added in the projection's epilogue."""
+        from ..ops.residual_stream import add_linear
+
+        heads = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        if type(self.o_proj) is Linear and self.o_proj.bias is None:
+            return add_linear(stream, heads, self.o_proj.weight), kv_cache
+        return stream + self.o_proj(heads).float(), kv_cache
+
+    def _paged_heads(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids: torch.Tensor) -> torch.Tensor:
+        """The concatenated heads ``[T, heads * v_head_dim]`` of packed rows."""
         from ..ops import flash_attention as FA
         from ..ops import paged_attention as PA
         from ..ops.qkv_prep import prepare_latent
@@ -780,30 +868,27 @@ class MultiHeadLatentAttention(nn.Module):
             w = self._rows.get([self.q_proj.weight, self.kv_a_proj.weight])
         if w is not None:
             y = project(x, w)
-            q, down = y[:, :nq], y[:, nq:]
+            q, down = y[:, :nq], y[:, nq:nq + rank + dr]
         else:
             q = self.q_proj(x) if self.q_proj is not None else self.q_b_proj(self.q_a_norm(self.q_a_proj(x)))
             down = self.kv_a_proj(x)
         q = q.unflatten(1, (H, c.qk_head_dim))
         pages, dests = kv_cache.kv_pages, batch_info.new_token_dests
         norm = (self.kv_a_norm.weight, self.kv_a_norm.eps)
-        weight = self.kv_b_proj.weight
+        weight, sink = self.kv_b_proj.weight, self.sinks_fp32()
         if getattr(batch_info, "prefill_segment_ids", None) is not None and self._packed_prefill_fits(q):
             latent, _ = prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:])
             kv = project(latent, self._whole_kv_weight())
             k, v = kv[:, :nq].unflatten(1, (H, c.qk_head_dim)), kv[:, nq:].unflatten(1, (H, dv))
-            heads = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=c.softmax_scale, window=c.sliding_window)
+            heads = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=c.softmax_scale, window=c.sliding_window, sink=sink)
         else:
             uk, uv = self.up_projections(weight)
             qa = q.new_empty(T, H, rank + dr)
             prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:], qa[..., rank:])
             PA.head_product(q[..., :dn], uk.to(q.dtype), qa[..., :rank], b_trans=False)
-            o = PA.paged_attention_latent(qa, pages, rank, batch_info, sm_scale=c.softmax_scale, window=c.sliding_window)
+            o = PA.paged_attention_latent(qa, pages, rank, batch_info, sm_scale=c.softmax_scale, window=c.sliding_window, sink=sink)
             heads = PA.head_product(o.to(q.dtype), uv.to(q.dtype), q.new_empty(T, H, dv), b_trans=True)
-        heads = heads.reshape(T, H * dv).to(x.dtype)
-        if type(self.o_proj) is Linear:
-            return project(heads, self.o_proj.weight, out_dtype=torch.float32)
-        return self.o_proj(heads).float()
+        return heads.reshape(T, H * dv).to(x.dtype)
 
     def _packed_prefill_fits(self, q: torch.Tensor) -> bool:
         """Whether the packed flash kernel takes this layer's sizes (the joint product of keys and values has the strides of its columns)."""
@@ -830,11 +915,24 @@ class MultiHeadLatentAttention(nn.Module):
         latent, k_rope = kv_a.split([c.kv_lora_rank, c.qk_rope_head_dim], dim=-1)
         kv = self.kv_b_proj(self.kv_a_norm(latent)).view(B, S, H, c.qk_nope_head_dim + c.v_head_dim)
         k_nope, v = kv.split([c.qk_nope_head_dim, c.v_head_dim], dim=-1)
-        q_rope = self.rot(q_rope, pos_ids)
-        k_rope = self.rot(k_rope.unsqueeze(2), pos_ids).expand(B, S, H, c.qk_rope_head_dim)
-        qf = torch.cat([q_nope, q_rope], dim=-1)
-        kf = torch.cat([k_nope, k_rope], dim=-1)
+        qf, kf = q_nope, k_nope
+        if self.rot is not None:
+            q_rope = self.rot(q_rope, pos_ids)
+            k_rope = self.rot(k_rope.unsqueeze(2), pos_ids).expand(B, S, H, c.qk_rope_head_dim)
+            qf = torch.cat([q_nope, q_rope], dim=-1)
+            kf = torch.cat([k_nope, k_rope], dim=-1)
         scale = c.softmax_scale
+        if c.sink:
+            if c.logits_soft_cap is not None:
+                raise NotImplementedError("latent attention with a sink takes no soft cap")
+            # the sink is a key column of its own whose value row is zero
+            s = torch.einsum("bqhd,bkhd->bhqk", qf.float() * scale, kf.float())
+            m = materialize_mask(mask, S, S, device=x.device)
+            if m is not None:
+                s = torch.where(m, s, torch.full_like(s, -1e9))
+            p = torch.softmax(torch.cat([s, self.sinks.float().view(1, H, 1, 1).expand(B, H, S, 1)], dim=-1), dim=-1)[..., :-1]
+            out = torch.einsum("bhqk,bkhd->bqhd", p.to(v.dtype), v)
+            return self.o_proj(out.reshape(B, S, H * c.v_head_dim).to(x.dtype))
         # value head size differs from the qk head size, so pad V for the shared kernel interface
         out = simple_attention_with_dropout(qf, kf, F.pad(v, (0, c.qk_head_dim - c.v_head_dim)) if c.v_head_dim < c.qk_head_dim else v,
                                             mask, attention_dtype=torch.float32 if c.upcast_attn else None,

@@ -213,6 +213,40 @@ class YarnRotaryEmbeddingsConfig(RotaryEmbeddingsConfig):
                             "original_max_position_embeddings": self.original_max_position_embeddings, "mscale": self.mscale}
 
 
+@RotaryEmbeddingsConfig.register_subclass("yarn_partial")
+@dataclass(frozen=True)
+class PartialYarnRotaryEmbeddingsConfig(RotaryEmbeddingsConfig):
+    """YaRN over the first ``rotary_dim`` dimensions of a head: a frequency that turns ``beta_fast`` times or more within the original
+    context stays, one that turns ``beta_slow`` times or less is divided by ``factor``, with a ramp over the pairs in between; cos and
+    sin are multiplied by ``0.1 ln(factor) + 1``.  (:class:`YarnRotaryEmbeddingsConfig` keeps another published variant's ramp,
+    position scale and temperature.)"""
+
+    theta: float = 10000
+    factor: float = 1.0
+    beta_fast: float = 32.0
+    beta_slow: float = 1.0
+    original_max_position_embeddings: int = 2048
+    rotary_dim: Optional[int] = None  # the first dimensions of a head that turn; None: all
+
+    def build(self, head_dim: int) -> RotaryEmbeddings:
+        r = self.rotary_dim if self.rotary_dim is not None else head_dim
+        if r % 2 != 0 or not 0 < r <= head_dim:
+            raise ValueError(f"cannot rotate {r} of {head_dim} dimensions")
+
+        def pair_of(turns: float) -> float:  # (fractional) pair that turns that often within the original context
+            return r * math.log(self.original_max_position_embeddings / (2 * math.pi * turns)) / (2 * math.log(self.theta))
+
+        low = max(math.floor(pair_of(self.beta_fast)), 0)
+        high = min(math.ceil(pair_of(self.beta_slow)), r - 1)
+        i = torch.arange(r // 2, dtype=torch.float64)
+        ramp = ((i - low) / max(high - low, 0.001)).clamp(0.0, 1.0)
+        freq = float(self.theta) ** (-2.0 * i / r)
+        return RotaryEmbeddings(head_dim, freq / self.factor * ramp + freq * (1.0 - ramp), temperature=0.1 * math.log(self.factor) + 1.0)
+
+    def to_hf_config(self):
+        raise ValueError("a partial rotation has no Hugging Face rope config")
+
+
 def rope_config_from_hf(get, default_theta: float = 10000.0) -> RotaryEmbeddingsConfig:
     """RoPE config from an HF config accessor ``get(key, default)``: understands both the legacy ``rope_theta`` +
     ``rope_scaling`` keys and the merged ``rope_parameters`` dict of newer ``transformers`` releases."""

@@ -44,9 +44,10 @@ class GemmaRMSNorm(nn.Module):
     def forward(self, x):
         return fused_norm(x, self.weight, None, self.eps, w_offset=1.0)[0]
 
-    def from_stream(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """The norm of an fp32 residual stream, in the weight's dtype (``rows``: of these rows only)."""
-        return rms_norm_stream(x, self.weight, self.eps, w_offset=1.0, rows=rows)
+    def from_stream(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The norm of an fp32 residual stream, in the weight's dtype (``rows``: of these rows only; ``add``: after adding a vector to the
+        stream in place)."""
+        return rms_norm_stream(x, self.weight, self.eps, w_offset=1.0, rows=rows, add=add)
 
 
 @LayerNormConfigBase.register_subclass("gemma")

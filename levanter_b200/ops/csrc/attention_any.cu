@@ -1,10 +1,11 @@
 // Paged attention and cache writes without restrictions on the element type or the sizes: fp32 serving, and bf16 models whose
 // head sizes the tensor-core kernels do not take (not a multiple of 8, above 256, more than 16 query heads per KV head).
 //
-// Same semantics as lvb_paged_attention_general (paged_attention.cu): packed query rows, pages, an optional chunk size or window and
-// an optional output gate; and of lvb_paged_latent (paged_latent.cu), where a key's first columns are its value.  Everything is fp32 arithmetic whatever the storage type (this file is built without fast-math).
-// One CTA per (query row, query head) walks the visible keys in blocks: a key per thread for the scores, an online softmax over
-// the block, then an output column per thread for P V.
+// Same semantics as lvb_paged_attention_general (paged_attention.cu): packed query rows, pages, an optional chunk size or window, an
+// optional output gate and the difference of two score maps; and of lvb_paged_latent (paged_latent.cu), where a key's first columns are
+// its value and a sink per head may join the softmax denominator.  Everything is fp32 arithmetic whatever the storage type (this file is
+// built without fast-math).  One CTA per (query row, query head or map of it) walks the visible keys in blocks: a key per thread for the
+// scores, an online softmax over the block, then an output column per thread for P V.  Maps leave their results in fp32 for a second kernel.
 #include "common.cuh"
 
 namespace lvb {
@@ -56,12 +57,25 @@ struct Params {
   const int* cu_q_lens;
   const int* num_seqs;
   const void* gate;
+  const float* sink;     // optional [H]
   void* out;
+  float* scratch;        // [T, H, dv] fp32: the maps' results
   int T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages, chunk, window;
   int row, v_at;         // elements of a KV head's row, and where in it the value starts
   long long ldq, ldg;
   float scale, soft_cap;
+  int gate_per_head;     // the gate has one number per head instead of one per element
+  const float* weight;   // with two maps (H counts both of every head): o = a1 - weight a2, then diff_scale * o / sqrt(mean(o^2) + eps)
+  float diff_scale, eps;
 };
+
+// the sigmoid of the gate of element d of head h
+template <typename T>
+__device__ __forceinline__ float gate_factor(const Params& p, int t, int h, int d) {
+  if (p.gate == nullptr) return 1.f;
+  const long long at = p.gate_per_head ? h : static_cast<long long>(h) * p.dv + d;
+  return 1.f / (1.f + expf(-to_f<T>(reinterpret_cast<const T*>(p.gate)[t * p.ldg + at])));
+}
 
 __device__ __forceinline__ float block_reduce(float v, float* s_red, bool is_max) {
   v = is_max ? warp_max(v) : warp_sum(v);
@@ -83,7 +97,12 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
   float* s_red = reinterpret_cast<float*>(s_slot + kThreads);
   const int t = blockIdx.x, h = blockIdx.y;
   const int kvh = h / (p.H / p.KV);
-  T* out = reinterpret_cast<T*>(p.out) + (static_cast<long long>(t) * p.H + h) * p.dv;
+  const int k_at = p.weight != nullptr ? (h & 1) * p.dk : 0;  // where in a KV head's row this row's key starts
+  const long long out_at = (static_cast<long long>(t) * p.H + h) * p.dv;
+  auto store = [&](int d, float v) {
+    if (p.weight != nullptr) p.scratch[out_at + d] = v;
+    else reinterpret_cast<T*>(p.out)[out_at + d] = from_f<T>(v);
+  };
 
   // which sequence owns row t, and its position in it
   int n = p.num_seqs[0];
@@ -95,7 +114,7 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
     if (kl > 0 && kl <= p.pages_per_seq * p.page_size) ctx = kl - p.cu_q_lens[seq + 1] + t + 1;
   }
   if (ctx <= 0) {
-    for (int d = threadIdx.x; d < p.dv; d += kThreads) out[d] = from_f<T>(0.f);
+    for (int d = threadIdx.x; d < p.dv; d += kThreads) store(d, 0.f);
     return;
   }
   const T* q = reinterpret_cast<const T*>(p.q) + t * p.ldq + static_cast<long long>(h) * p.dk;
@@ -116,7 +135,7 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
     __syncthreads();  // s_q / s_o written; the previous block's s_p and s_slot have been read
     float s = -INFINITY;
     if (slot >= 0) {
-      const T* kr = pages + (static_cast<long long>(slot) * p.KV + kvh) * per;
+      const T* kr = pages + (static_cast<long long>(slot) * p.KV + kvh) * per + k_at;
       float acc = 0.f;
       for (int d = 0; d < p.dk; ++d) acc = fmaf(s_q[d], to_f<T>(kr[d]), acc);
       s = acc * p.scale;
@@ -139,13 +158,33 @@ __global__ void __launch_bounds__(kThreads) attention_any_kernel(Params p) {
       s_o[d] = acc;
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + t * p.ldg + static_cast<long long>(h) * p.dv : nullptr;
-  for (int d = threadIdx.x; d < p.dv; d += kThreads) {
-    float o = s_o[d] * inv;
-    if (gate != nullptr) o /= 1.f + expf(-to_f<T>(gate[d]));
-    out[d] = from_f<T>(o);
+  float shrink = 1.f;
+  if (p.sink != nullptr) {  // one more column of the softmax, whose value is zero
+    const float m_new = fmaxf(m, p.sink[h]);
+    shrink = expf(m - m_new);
+    l = l * shrink + expf(p.sink[h] - m_new);
   }
+  const float inv = l > 0.f ? shrink / l : 0.f;
+  for (int d = threadIdx.x; d < p.dv; d += kThreads) store(d, p.weight != nullptr ? s_o[d] * inv : s_o[d] * inv * gate_factor<T>(p, t, h, d));
+}
+
+// One CTA per (query row, head): the two maps' results to the head's output.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) difference_kernel(Params p) {
+  __shared__ float s_red[kThreads / 32];
+  const int t = blockIdx.x, h = blockIdx.y;
+  const float* a1 = p.scratch + (static_cast<long long>(t) * p.H + 2 * h) * p.dv;
+  const float* a2 = a1 + p.dv;
+  const float lam = *p.weight;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < p.dv; d += kThreads) {
+    const float o = a1[d] - lam * a2[d];
+    ss = fmaf(o, o, ss);
+  }
+  ss = block_reduce(ss, s_red, false);
+  const float r = p.diff_scale / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
+  T* out = reinterpret_cast<T*>(p.out) + (static_cast<long long>(t) * (p.H / 2) + h) * p.dv;
+  for (int d = threadIdx.x; d < p.dv; d += kThreads) out[d] = from_f<T>((a1[d] - lam * a2[d]) * r * gate_factor<T>(p, t, h, d));
 }
 
 }  // namespace any
@@ -175,22 +214,31 @@ extern "C" int lvb_kv_page_write_general(void* kv_pages, const void* k, const vo
 }
 
 // window > 0: a query sees itself and the window - 1 positions before it.  shared: a KV head's row holds dk elements only and its first dv are
-// the value (dv <= dk).
+// the value (dv <= dk).  sink: optional [H] fp32.  gate: [T, heads * dv], or [T, heads] with gate_per_head.  weight: one number on the device;
+// rows 2h and 2h + 1 of q are then the maps of head h, a KV head's row holds two keys and a value, out is [T, H / 2, dv] and scratch fp32
+// [T, H, dv].
 extern "C" int lvb_attention_any(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices, const int* cu_q_lens,
-                                 const int* num_seqs, const void* gate, void* out, int T, int H, int KV, int dk, int dv, long long ldq,
-                                 long long ldg, int S, int pages_per_seq, int page_size, int num_pages, int chunk, int window,
-                                 int shared, float scale, float soft_cap, int is_f32, void* stream) {
+                                 const int* num_seqs, const void* gate, const float* sink, void* out, float* scratch, int T, int H, int KV, int dk,
+                                 int dv, long long ldq, long long ldg, int gate_per_head, int S, int pages_per_seq, int page_size,
+                                 int num_pages, int chunk, int window, int shared, float scale, float soft_cap, const float* weight,
+                                 float diff_scale, float eps, int is_f32, void* stream) {
   using namespace lvb;
   using namespace lvb::any;
   if (T <= 0) return kErrOk;
   if (H <= 0 || KV <= 0 || H % KV != 0 || dk <= 0 || dv <= 0 || S <= 0 || chunk < 0 || window < 0) return kErrBadArg;
-  if (shared && dv > dk) return kErrBadArg;
+  if (shared && (dv > dk || weight != nullptr)) return kErrBadArg;
+  if (weight != nullptr && ((H / KV) % 2 != 0 || scratch == nullptr || sink != nullptr)) return kErrBadArg;
   const size_t smem = (static_cast<size_t>(dk) + dv + 2 * kThreads + kThreads / 32) * 4;
   if (smem > 48 * 1024) return kErrTooLarge;
-  Params p{q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, gate, out, T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages,
-           chunk, window, shared ? dk : dk + dv, shared ? 0 : dk, ldq, ldg, scale, soft_cap};
+  const int keys = weight != nullptr ? 2 * dk : dk;
+  Params p{q, kv_pages, kv_lens, page_indices, cu_q_lens, num_seqs, gate, sink, out, scratch, T, H, KV, dk, dv, S, pages_per_seq, page_size, num_pages,
+           chunk, window, shared ? dk : keys + dv, shared ? 0 : keys, ldq, ldg, scale, soft_cap, gate_per_head, weight, diff_scale, eps};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (is_f32) attention_any_kernel<float><<<dim3(T, H), kThreads, smem, s>>>(p);
   else attention_any_kernel<__nv_bfloat16><<<dim3(T, H), kThreads, smem, s>>>(p);
+  if (weight != nullptr && cudaGetLastError() == cudaSuccess) {
+    if (is_f32) difference_kernel<float><<<dim3(T, H / 2), kThreads, 0, s>>>(p);
+    else difference_kernel<__nv_bfloat16><<<dim3(T, H / 2), kThreads, 0, s>>>(p);
+  }
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }

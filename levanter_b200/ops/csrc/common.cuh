@@ -357,6 +357,10 @@ __device__ __forceinline__ float warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
 }
+// cap * tanh(x / cap) with an absolute error of a few 1e-7 of cap, also in files built with fast-math (whose tanhf keeps about 11 bits)
+__device__ __forceinline__ float soft_capped(float x, float cap) {
+  return cap - __fdividef(2.f * cap, 1.f + exp2f(x * __fdividef(2.885390081777927f, cap)));
+}
 // Named barrier among `count` threads (count multiple of 32), id in [1, 15].
 __device__ __forceinline__ void named_bar_sync(int id, int count) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(count) : "memory");

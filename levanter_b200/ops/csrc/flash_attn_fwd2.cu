@@ -18,6 +18,11 @@
 // 128: the tensor maps are three-dimensional (size, head, row), columns past the size arrive as zeros, and the MMAs stop at
 // the next multiple of 16.  Keys of up to 192 leave shared memory for one V stage only.  An optional gate is applied to the
 // output on its way out.
+//
+// kMaps (kPacked only): differential attention.  The two tiles of a CTA are the two score maps of a head over the same 128 rows: each
+// has queries and keys of its own (the K ring holds single tiles, alternating between the maps), both multiply the same V tile, and the
+// epilogue forms a1 - weight * a2, its norm over the values and the gate straight from the two accumulators.  The warps of a tile
+// take alternate groups of 32 columns of the result.
 #include "common.cuh"
 
 namespace lvb {
@@ -48,27 +53,33 @@ struct Params {
   const int* pos;            // [S]: position of each packed row in its sequence
   int chunk;                 // > 0: a row at position i sees positions >= i - i % chunk only (window, above: positions > i - window)
   int dk, dv;                // query/key and value sizes (multiples of 8, at most HD)
-  const __nv_bfloat16* gate; // optional [S, Hq * dv] (row stride ldg): the output is multiplied by its sigmoid
+  const __nv_bfloat16* gate; // optional [S, Hq * dv], or [S, Hq] with gate_per_head (row stride ldg): the output is multiplied by its sigmoid
   long long ldg;
+  int gate_per_head;
+  // ---- kMaps: o = a1 - weight a2, then diff_scale * o / sqrt(mean(o^2) + eps)
+  const float* weight;
+  float diff_scale, eps;
 };
 
 // HDK, HDV: room for the query/key and the value size
-template <int HDK, int HDV>
+template <int HDK, int HDV, bool kMaps = false>
 struct SmemT {
   static constexpr int kQKTile = 128 * HDK * 2;               // a [128 rows, HDK] tile: HDK / 64 chunks of 64 columns
   static constexpr int kVTile = 128 * HDV * 2;
-  static constexpr int kVStages = HDK > 128 ? 1 : kStages;
+  static constexpr int kKStages = kMaps ? 2 * kStages : kStages;
+  static constexpr int kVStages = HDK > (kMaps ? 64 : 128) ? 1 : kStages;
   static constexpr int kQ = 0;                                // 2 tiles
   static constexpr int kK = kQ + 2 * kQKTile;
-  static constexpr int kV = kK + kStages * kQKTile;
+  static constexpr int kV = kK + kKStages * kQKTile;
   static constexpr int kBars = kV + kVStages * kVTile;
-  static constexpr int kNumBars = 1 + 4 * kStages + 2 + 2 + 2;
+  static constexpr int kNumBars = 1 + 2 * kKStages + 2 * kStages + 2 + 2 + 2;
   static constexpr int kTotal = kBars + kNumBars * 8 + 16 + 1024;
 };
 
 template <bool kCap>
 __device__ __forceinline__ float to_log2(float s, float scale_log2, float scale, float cap) {
-  if constexpr (kCap) return cap * tanhf(s * scale / cap) * kLog2e;
+  // cap * tanh(s * scale / cap), from an exponential: this file's tanhf keeps about 11 bits
+  if constexpr (kCap) return cap * kLog2e - __fdividef(2.f * kLog2e * cap, 1.f + exp2f(s * __fdividef(2.f * kLog2e * scale, cap)));
   else return s * scale_log2;
 }
 
@@ -79,20 +90,40 @@ __device__ __forceinline__ int row_lower_bound(const Params& p, int qi) {
   return qi - (p.window > 0 ? min(back, p.window - 1) : back);
 }
 
-template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false>
+// dst[0 .. 7] = f * e (times the sigmoid of gate[0 .. 7] when given)
+__device__ __forceinline__ void store_row_piece(__nv_bfloat16* dst, const float* e, float f, const __nv_bfloat16* gate) {
+  float v[8];
+#pragma unroll
+  for (int t = 0; t < 8; ++t) v[t] = e[t] * f;
+  if (gate != nullptr) {
+    const uint4 gw = __ldg(reinterpret_cast<const uint4*>(gate));
+    const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&gw);
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      const float2 g = __bfloat1622float2(gh[t]);
+      v[2 * t] *= 1.f / (1.f + __expf(-g.x));
+      v[2 * t + 1] *= 1.f / (1.f + __expf(-g.y));
+    }
+  }
+  *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+}
+
+template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false, bool kMaps = false>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, Params p) {
-  using Smem = SmemT<HDK, HDV>;
-  constexpr int kQKTile = Smem::kQKTile, kVTile = Smem::kVTile, kVStages = Smem::kVStages;
+  static_assert(kPacked || !kMaps, "maps need packed rows");
+  using Smem = SmemT<HDK, HDV, kMaps>;
+  constexpr int kQKTile = Smem::kQKTile, kVTile = Smem::kVTile, kKStages = Smem::kKStages, kVStages = Smem::kVStages;
+  constexpr int kRows = kMaps ? BT : 2 * BT;  // query rows per CTA
   const bool causal = p.causal != 0;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Smem::kBars);
   uint64_t* q_full = bars;
   uint64_t* k_full = q_full + 1;
-  uint64_t* k_empty = k_full + kStages;
-  uint64_t* v_full = k_empty + kStages;
+  uint64_t* k_empty = k_full + kKStages;
+  uint64_t* v_full = k_empty + kKStages;
   uint64_t* v_empty = v_full + kStages;
   uint64_t* s_full = v_empty + kStages;  // [2 tiles]
   uint64_t* p_full = s_full + 2;         // [2 tiles]
@@ -102,14 +133,14 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int ncta = p.S / (2 * BT);
+  const int ncta = p.S / kRows;
   const int cb = ncta - 1 - static_cast<int>(blockIdx.x);  // heaviest first
   const int b = blockIdx.y / p.Hq;
   const int h = blockIdx.y % p.Hq;
   const int hkv = h / (p.Hq / p.Hkv);
-  const int q0 = cb * 2 * BT;
+  const int q0 = cb * kRows;
   // without the causal part there is no diagonal block (the mask test below never matches -1) and both tiles see every block
-  const int jdiagA = causal ? 2 * cb : -1, jdiagB = causal ? 2 * cb + 1 : -1;
+  const int jdiagA = kMaps ? cb : causal ? 2 * cb : -1, jdiagB = kMaps ? cb : causal ? 2 * cb + 1 : -1;
   int jlo = 0;
   if (!kPacked && p.window > 0) {
     const int first_key = q0 - p.window + 1;
@@ -122,14 +153,16 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   }
   if constexpr (kPacked) jlo = row_lower_bound(p, q0) / BT;  // bounds do not decrease along the packed rows
   const int nB = (causal ? jdiagB : p.Sk / BT - 1) - jlo + 1;  // blocks processed by tile B
-  const int nA = causal ? nB - 1 : nB;                        // causal: tile A stops one block earlier (its diagonal)
+  const int nA = causal && !kMaps ? nB - 1 : nB;              // causal: tile A stops one block earlier (its diagonal)
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
     mbar_init(q_full, 1);
-    for (int s = 0; s < kStages; ++s) {
+    for (int s = 0; s < kKStages; ++s) {
       mbar_init(&k_full[s], 1);
       mbar_init(&k_empty[s], 1);
+    }
+    for (int s = 0; s < kStages; ++s) {
       mbar_init(&v_full[s], 1);
       mbar_init(&v_empty[s], 1);
     }
@@ -163,24 +196,27 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int c = 0; c < HDK / 64; ++c)
           if constexpr (kPacked) {
-            if (c < ck) tma_load_3d(smem + Smem::kQ + t * kQKTile + c * kChunkBytes, &tmQ, q_full, 64 * c, h, row_q + t * BT);
+            if (c < ck) tma_load_3d(smem + Smem::kQ + t * kQKTile + c * kChunkBytes, &tmQ, q_full, 64 * c, kMaps ? 2 * h + t : h, kMaps ? row_q : row_q + t * BT);
           } else
           tma_load_2d(smem + Smem::kQ + t * kQKTile + c * kChunkBytes, &tmQ, q_full, h * HDK + 64 * c, row_q + t * BT);
       bool ok = true;
       for (int it = 0; it < nB && ok; ++it) {
-        const int st = it % kStages;
-        const uint32_t ph = (it / kStages) & 1;
         const int row_k = b * p.Sk + (jlo + it) * BT;
-        ok = mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 1200, it);
-        if (!ok) break;
-        uint8_t* ks = smem + Smem::kK + st * kQKTile;
-        mbar_expect_tx(&k_full[st], ck * kChunkBytes);
 #pragma unroll
-        for (int c = 0; c < HDK / 64; ++c)
-          if constexpr (kPacked) {
-            if (c < ck) tma_load_3d(ks + c * kChunkBytes, &tmK, &k_full[st], 64 * c, hkv, row_k);
-          } else
-          tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * HDK + 64 * c, row_k);
+        for (int t = 0; t < (kMaps ? 2 : 1); ++t) {
+          const int n = kMaps ? 2 * it + t : it, st = n % kKStages;
+          ok = mbar_wait(&k_empty[st], ((n / kKStages) & 1) ^ 1, abort_flag, p.status, 1200, it);
+          if (!ok) break;
+          uint8_t* ks = smem + Smem::kK + st * kQKTile;
+          mbar_expect_tx(&k_full[st], ck * kChunkBytes);
+#pragma unroll
+          for (int c = 0; c < HDK / 64; ++c)
+            if constexpr (kPacked) {
+              if (c < ck) tma_load_3d(ks + c * kChunkBytes, &tmK, &k_full[st], 64 * c, kMaps ? 2 * hkv + t : hkv, row_k);
+            } else
+            tma_load_2d(ks + c * kChunkBytes, &tmK, &k_full[st], hkv * HDK + 64 * c, row_k);
+        }
+        if (!ok) break;
         const int sv = it % kVStages;
         ok = mbar_wait(&v_empty[sv], ((it / kVStages) & 1) ^ 1, abort_flag, p.status, 1201, it);
         if (!ok) break;
@@ -204,8 +240,9 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       const uint32_t sq = smem_u32(smem + Smem::kQ);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1300, 0);
 
+      auto k_tile = [&](int tile, int it) { return kMaps ? 2 * it + tile : it; };  // number of the K tile that a query tile meets
       auto qk = [&](int tile, int it) {
-        const int st = it % kStages;
+        const int st = k_tile(tile, it) % kKStages;
         const uint32_t sk = smem_u32(smem + Smem::kK + st * kQKTile);
         const uint32_t sqt = sq + tile * kQKTile;
 #pragma unroll
@@ -216,6 +253,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                        idesc_qk, kk > 0 ? 1u : 0u);
         }
         umma_commit(&s_full[tile]);
+        if (kMaps || tile == 1) umma_commit(&k_empty[st]);
       };
       auto pv = [&](int tile, int it) {
         const uint32_t sv = smem_u32(smem + Smem::kV + (it % kVStages) * kVTile);
@@ -226,15 +264,18 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                        make_smem_desc(sv + kk * 2048, kChunkBytes, 1024), idesc_pv, (it > 0 || kk > 0) ? 1u : 0u);
         }
       };
-      auto wait_k = [&](int it) { return mbar_wait(&k_full[it % kStages], (it / kStages) & 1, abort_flag, p.status, 1301, it); };
+      auto wait_k = [&](int tile, int it) {
+        const int n = k_tile(tile, it);
+        return mbar_wait(&k_full[n % kKStages], (n / kKStages) & 1, abort_flag, p.status, 1301, it);
+      };
       auto wait_v = [&](int it) { return mbar_wait(&v_full[it % kVStages], (it / kVStages) & 1, abort_flag, p.status, 1302, it); };
 
-      if (ok) ok = wait_k(0);
+      if (ok) ok = wait_k(0, 0);
+      if (kMaps && ok) ok = wait_k(1, 0);
       if (ok) {
         tc_fence_after();
         qk(0, 0);
         qk(1, 0);
-        umma_commit(&k_empty[0]);
       }
       for (int it = 0; it < nB && ok; ++it) {
         ok = wait_v(it);
@@ -248,7 +289,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         }
         const bool more = it + 1 < nB;
         if (more) {
-          ok = wait_k(it + 1);
+          ok = wait_k(0, it + 1);
           if (!ok) break;
           tc_fence_after();
           if (it + 1 < nA) qk(0, it + 1);
@@ -260,8 +301,12 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         umma_commit(&v_empty[it % kVStages]);
         if (it == nB - 1) umma_commit(&o_done[1]);
         if (more) {
+          if (kMaps) {
+            ok = wait_k(1, it + 1);
+            if (!ok) break;
+            tc_fence_after();
+          }
           qk(1, it + 1);
-          umma_commit(&k_empty[(it + 1) % kStages]);
         }
       }
     }
@@ -270,7 +315,8 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int tile = (warp - 2) >> 2;
     const int quad = warp & 3;
     const int r = quad * 32 + lane;
-    const int qi = q0 + tile * BT + r;
+    const int tile_q0 = kMaps ? q0 : q0 + tile * BT;
+    const int qi = tile_q0 + r;
     const int jdiag = tile == 0 ? jdiagA : jdiagB;
     const int nT = tile == 0 ? nA : nB;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
@@ -284,7 +330,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     int row_lo = 0, tile_lo = 0;  // kPacked: this row's first visible key, and the last row's (the largest of the tile)
     if constexpr (kPacked) {
       row_lo = row_lower_bound(p, qi);
-      tile_lo = row_lower_bound(p, q0 + tile * BT + BT - 1);
+      tile_lo = row_lower_bound(p, tile_q0 + BT - 1);
     }
 
     for (int it = 0; it < nT && ok; ++it) {
@@ -396,6 +442,53 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       if (lane == 0) mbar_arrive(&p_full[tile]);
     }
 
+    if constexpr (kMaps) {
+      // the queries are not needed any more: their memory carries the rows' sums and partial norms between the two tiles' warps
+      for (int i = 0; i < 2 && ok; ++i) ok = mbar_wait(&o_done[i], 0, abort_flag, p.status, 1410 + i, nT);
+      ok = __all_sync(0xffffffffu, ok);
+      tc_fence_after();
+      float* s_inv = reinterpret_cast<float*>(smem + Smem::kQ);  // [2][BT]
+      float* s_ss = s_inv + 2 * BT;                              // [2][BT]
+      if (ok) s_inv[tile * BT + r] = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      named_bar_sync(1, 8 * 32);
+      const uint32_t tO1 = tmem_base + 2 * BT + lane_addr, tO2 = tO1 + HDV;
+      constexpr int kGroups = HDV / 64;  // groups of 32 columns per warp
+      float o[kGroups][32], ss = 0.f;
+      const float c1 = s_inv[r], c2 = -*p.weight * s_inv[BT + r];
+#pragma unroll
+      for (int n = 0; n < kGroups; ++n) {
+        const int c = (2 * n + tile) * 32;
+        if (c < p.dv) {
+          uint32_t v1[32], v2[32];
+          tmem_ld_32x32(tO1 + c, v1);
+          tmem_ld_32x32(tO2 + c, v2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int t = 0; t < 32; ++t) {
+            o[n][t] = c + t < p.dv ? fmaf(c1, __uint_as_float(v1[t]), c2 * __uint_as_float(v2[t])) : 0.f;
+            ss = fmaf(o[n][t], o[n][t], ss);
+          }
+        }
+      }
+      if (ok) s_ss[tile * BT + r] = ss;
+      named_bar_sync(1, 8 * 32);
+      if (ok) {
+        float f = p.diff_scale * rsqrtf((s_ss[r] + s_ss[BT + r]) / static_cast<float>(p.dv) + p.eps);
+        const __nv_bfloat16* grow = nullptr;
+        if (p.gate != nullptr) {
+          if (p.gate_per_head) f *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(qi) * p.ldg + h])));
+          else grow = p.gate + static_cast<size_t>(qi) * p.ldg + static_cast<size_t>(h) * p.dv;
+        }
+        __nv_bfloat16* orow = p.O + (static_cast<size_t>(qi) * p.Hq + h) * p.dv;
+#pragma unroll
+        for (int n = 0; n < kGroups; ++n) {
+          const int c = (2 * n + tile) * 32;
+#pragma unroll
+          for (int q4 = 0; q4 < 4; ++q4)
+            if (c + 8 * q4 < p.dv) store_row_piece(orow + c + 8 * q4, &o[n][8 * q4], f, grow != nullptr ? grow + c + 8 * q4 : nullptr);
+        }
+      }
+    } else {
     if (ok) {
       ok = mbar_wait(&o_done[tile], 0, abort_flag, p.status, 1410 + tile, nT);
       ok = __all_sync(0xffffffffu, ok);
@@ -416,36 +509,23 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       const float inv = l_sum > 0.f ? o_scale / l_sum : 0.f;
       if constexpr (kPacked) {
         __nv_bfloat16* orow = p.O + static_cast<size_t>(qi) * (static_cast<size_t>(p.Hq) * p.dv) + static_cast<size_t>(h) * p.dv;
-        const __nv_bfloat16* grow = p.gate != nullptr ? p.gate + static_cast<size_t>(qi) * p.ldg + static_cast<size_t>(h) * p.dv : nullptr;
+        const __nv_bfloat16* grow = nullptr;
+        float f = inv;
+        if (p.gate != nullptr) {
+          if (p.gate_per_head) f *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(qi) * p.ldg + h])));
+          else grow = p.gate + static_cast<size_t>(qi) * p.ldg + static_cast<size_t>(h) * p.dv;
+        }
 #pragma unroll 1
         for (int c = 0; c < p.dv; c += 32) {
           uint32_t v[32];
           tmem_ld_32x32(tO + c, v);
           tmem_ld_wait();
+          float e[32];
 #pragma unroll
-          for (int q4 = 0; q4 < 4; ++q4) {
-            if (c + 8 * q4 < p.dv) {
-              float e[8];
+          for (int t = 0; t < 32; ++t) e[t] = __uint_as_float(v[t]);
 #pragma unroll
-              for (int t = 0; t < 8; ++t) e[t] = __uint_as_float(v[q4 * 8 + t]) * inv;
-              if (grow != nullptr) {
-                const uint4 gw = __ldg(reinterpret_cast<const uint4*>(grow + c) + q4);
-                const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&gw);
-#pragma unroll
-                for (int t = 0; t < 4; ++t) {
-                  const float2 f = __bfloat1622float2(gh[t]);
-                  e[2 * t] *= 1.f / (1.f + __expf(-f.x));
-                  e[2 * t + 1] *= 1.f / (1.f + __expf(-f.y));
-                }
-              }
-              uint4 w;
-              w.x = pack_bf16x2(e[0], e[1]);
-              w.y = pack_bf16x2(e[2], e[3]);
-              w.z = pack_bf16x2(e[4], e[5]);
-              w.w = pack_bf16x2(e[6], e[7]);
-              reinterpret_cast<uint4*>(orow + c)[q4] = w;
-            }
-          }
+          for (int q4 = 0; q4 < 4; ++q4)
+            if (c + 8 * q4 < p.dv) store_row_piece(orow + c + 8 * q4, e + 8 * q4, f, grow != nullptr ? grow + c + 8 * q4 : nullptr);
         }
       } else {
       __nv_bfloat16* orow = p.O + (static_cast<size_t>(b) * p.S + qi) * (static_cast<size_t>(p.Hq) * HDV) + static_cast<size_t>(h) * HDV;
@@ -467,6 +547,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       p.lse2[(static_cast<size_t>(b) * p.Hq + h) * p.S + qi] = (l_sum > 0.f) ? m_used + log2f(l_sum) : -INFINITY;
       }
     }
+    }
   }
 
   tc_fence_before();
@@ -477,17 +558,17 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   }
 }
 
-template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false>
+template <int HDK, int HDV, bool kSeg, bool kCap, bool kPacked = false, bool kMaps = false>
 int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const Params& p, cudaStream_t st) {
-  using Smem = SmemT<HDK, HDV>;
+  using Smem = SmemT<HDK, HDV, kMaps>;
   static_assert(Smem::kTotal <= 227 * 1024, "shared memory of one CTA");
-  auto kern = flash_fwd2_kernel<HDK, HDV, kSeg, kCap, kPacked>;
+  auto kern = flash_fwd2_kernel<HDK, HDV, kSeg, kCap, kPacked, kMaps>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem::kTotal) != cudaSuccess) return kErrCuda;
     attr_set = true;
   }
-  dim3 grid(p.S / (2 * BT), p.B * p.Hq);
+  dim3 grid(p.S / (kMaps ? BT : 2 * BT), p.B * p.Hq);
   kern<<<grid, kThreads, Smem::kTotal, st>>>(tmQ, tmK, tmV, p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
@@ -540,7 +621,8 @@ extern "C" int lvb_flash_attn_fwd2_hd(const void* q, const void* k, const void* 
   p.scale = scale; p.soft_cap = soft_cap; p.window = window;
   p.causal = causal ? 1 : 0;
   p.status = status;
-  p.pos = nullptr; p.chunk = 0; p.dk = p.dv = head_dim; p.gate = nullptr; p.ldg = 0;
+  p.pos = nullptr; p.chunk = 0; p.dk = p.dv = head_dim; p.gate = nullptr; p.ldg = 0; p.gate_per_head = 0;
+  p.weight = nullptr; p.diff_scale = p.eps = 0.f;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (head_dim == 128) return launch_hd<128>(q, k, v, p, st);
   if (head_dim == 64) return launch_hd<64>(q, k, v, p, st);
@@ -556,33 +638,44 @@ extern "C" int lvb_flash_attn_fwd2(const void* q, const void* k, const void* v, 
 
 // Causal attention over T packed rows (T a multiple of 256) of sequences that each start at position 0:
 //   q: row t, head h at q + t * ldq + h * dk     k / v: row t, head g at k + t * ldk + g * dk, v + t * ldv + g * dv
-//   o[T, Hq, dv] = softmax(scale q k^T over the visible keys) v  (* sigmoid(gate[t, h, :]))
+//   o[T, Hq, dv] = softmax(scale q k^T over the visible keys) v  (* sigmoid(gate[t, h, :]) or sigmoid(gate[t, h]) with gate_per_head)
 // pos[t] is the row's position in its sequence (padding rows: 0).  chunk > 0: positions are cut into chunks of that many, counted
 // from the sequence's start, and a row sees its own chunk only; window > 0: a row sees itself and the window - 1 positions before
-// it.  dk, dv: multiples of 8, at most 192 and 128; ldq, ldk, ldv and ldg
+// it.  sink (optional, fp32 [Hq]): joins the softmax denominator as it is.  weight (optional, one fp32 number on the device): q and k hold two
+// score maps per head side by side (rows of 2 Hq and 2 Hkv heads), and o = diff_scale * d / sqrt(mean(d^2) + eps) with d = a1 - weight * a2
+// (no sink then).  dk, dv: multiples of 8, at most 192 (128 with two maps) and 128; ldq, ldk, ldv and, for a gate per element, ldg
 // multiples of 8 and the pointers 16-byte aligned.
-extern "C" int lvb_flash_attn_fwd_packed(const void* q, const void* k, const void* v, const void* gate, void* o, const int* pos, int T,
-                                         int Hq, int Hkv, int dk, int dv, int ldq, int ldk, int ldv, int ldg, int chunk, int window,
-                                         float scale, float soft_cap, int* status, void* stream) {
+extern "C" int lvb_flash_attn_fwd_packed(const void* q, const void* k, const void* v, const void* gate, const float* sink, void* o, const int* pos,
+                                         int T, int Hq, int Hkv, int dk, int dv, int ldq, int ldk, int ldv, int ldg, int gate_per_head,
+                                         int chunk, int window, float scale, float soft_cap, const float* weight, float diff_scale,
+                                         float eps, int* status, void* stream) {
   using namespace lvb;
   using namespace lvb::fa2;
   if (T <= 0 || (T % (2 * BT)) != 0 || Hq <= 0 || Hkv <= 0 || (Hq % Hkv) != 0 || pos == nullptr || chunk < 0 || window < 0) return kErrBadArg;
-  if (dk <= 0 || dv <= 0 || dk > 192 || dv > 128 || (dk & 7) || (dv & 7) || (ldg & 7) || !(scale > 0.f)) return kErrBadArg;
-  if ((reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(o) & 15)) return kErrBadArg;
+  if (dk <= 0 || dv <= 0 || dk > (weight != nullptr ? 128 : 192) || dv > 128 || (dk & 7) || (dv & 7) || !(scale > 0.f)) return kErrBadArg;
+  if (gate != nullptr && !gate_per_head && ((ldg & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return kErrBadArg;
+  if ((reinterpret_cast<uintptr_t>(o) & 15) || (weight != nullptr && sink != nullptr)) return kErrBadArg;
   Params p;
   p.O = reinterpret_cast<__nv_bfloat16*>(o);
-  p.lse2 = nullptr; p.q_seg = nullptr; p.k_seg = nullptr; p.kblock_lo = nullptr; p.sink = nullptr;
+  p.lse2 = nullptr; p.q_seg = nullptr; p.k_seg = nullptr; p.kblock_lo = nullptr; p.sink = sink;
   p.B = 1; p.S = T; p.Sk = T; p.Hq = Hq; p.Hkv = Hkv;
   p.scale = scale; p.soft_cap = soft_cap; p.window = window; p.causal = 1; p.status = status;
   p.pos = pos; p.chunk = chunk; p.dk = dk; p.dv = dv;
-  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg; p.gate_per_head = gate_per_head;
+  p.weight = weight; p.diff_scale = diff_scale; p.eps = eps;
+  const int maps = weight != nullptr ? 2 : 1;
   CUtensorMap tmQ, tmK, tmV;
-  int rc = make_tmap_heads_bf16(&tmQ, q, T, Hq, dk, ldq, BT);
-  if (rc == kErrOk) rc = make_tmap_heads_bf16(&tmK, k, T, Hkv, dk, ldk, BT);
+  int rc = make_tmap_heads_bf16(&tmQ, q, T, Hq * maps, dk, ldq, BT);
+  if (rc == kErrOk) rc = make_tmap_heads_bf16(&tmK, k, T, Hkv * maps, dk, ldk, BT);
   if (rc == kErrOk) rc = make_tmap_heads_bf16(&tmV, v, T, Hkv, dv, ldv, BT);
   if (rc != kErrOk) return rc;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool small = dk <= 64 && dv <= 64;
+  if (maps == 2) {
+    if (soft_cap > 0.f)
+      return dk <= 64 ? launch<64, 128, false, true, true, true>(tmQ, tmK, tmV, p, st) : launch<128, 128, false, true, true, true>(tmQ, tmK, tmV, p, st);
+    return dk <= 64 ? launch<64, 128, false, false, true, true>(tmQ, tmK, tmV, p, st) : launch<128, 128, false, false, true, true>(tmQ, tmK, tmV, p, st);
+  }
   if (soft_cap > 0.f) {
     if (dk > 128) return launch<192, 128, false, true, true>(tmQ, tmK, tmV, p, st);
     return small ? launch<64, 64, false, true, true>(tmQ, tmK, tmV, p, st) : launch<128, 128, false, true, true>(tmQ, tmK, tmV, p, st);

@@ -1,4 +1,4 @@
-// Serving kernels of a mixture of experts whose router scores each expert by a sigmoid and picks within groups of neighbours:
+// Serving kernels of a mixture of experts whose router scores the experts by a sigmoid or a softmax and picks within groups of neighbours:
 //   route     one warp per token: scores, group choice, top-k, weights; tokens per expert
 //   dispatch  positions in the expert-sorted, block-padded layout of the grouped GEMMs, and the copy of the token rows into it
 //   combine   weighted sum of a token's expert outputs, added to the fp32 residual stream
@@ -31,6 +31,9 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n) {
   return at < n ? at : 0;
 }
 
+// kSoftmax: scores are the softmax over all experts, a group counts by its best score, and the weights are the chosen scores divided by
+// their sum.  Otherwise scores are sigmoids, a group counts by its two best choice scores, and the weights are scale * score.
+template <bool kSoftmax>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict__ correction, int c_f32, const int* __restrict__ live,
              int live_limit, int T, int E, int k, int groups, int keep, float scale, int* __restrict__ idx, float* __restrict__ w,
@@ -46,8 +49,16 @@ route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict_
     for (int j = lane; j < k; j += 32) { idx[static_cast<size_t>(t) * k + j] = -1; w[static_cast<size_t>(t) * k + j] = 0.f; }
     return;
   }
+  float top = -INFINITY, inv = 1.f;
+  if constexpr (kSoftmax) {
+    for (int e = lane; e < E; e += 32) top = fmaxf(top, z[t * ldz + e]);
+    top = warp_max(top);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(z[t * ldz + e] - top);
+    inv = 1.f / warp_sum(sum);
+  }
   for (int e = lane; e < E; e += 32) {
-    const float s = 1.f / (1.f + expf(-z[t * ldz + e]));
+    const float s = kSoftmax ? expf(z[t * ldz + e] - top) * inv : 1.f / (1.f + expf(-z[t * ldz + e]));
     s_score[e] = s;
     s_choice[e] = s + (correction != nullptr ? ldv(correction, c_f32, e) : 0.f);
   }
@@ -60,7 +71,7 @@ route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict_
         const float c = s_choice[e];
         if (c > a) { b = a; a = c; } else if (c > b) b = c;
       }
-      s_group[g] = size > 1 ? a + b : a;
+      s_group[g] = size > 1 && !kSoftmax ? a + b : a;
     }
     __syncwarp();
     unsigned long long kept[kMaxExperts / 64] = {};
@@ -77,8 +88,10 @@ route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict_
     }
     __syncwarp();
   }
+  float chosen = 0.f;
   for (int j = 0; j < k; ++j) {
     const int e = warp_argmax(s_choice, E);
+    chosen += s_score[e];
     __syncwarp();
     if (lane == 0) {
       idx[static_cast<size_t>(t) * k + j] = e;
@@ -87,6 +100,9 @@ route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict_
       atomicAdd(&counts[e], 1);
     }
     __syncwarp();
+  }
+  if constexpr (kSoftmax) {
+    for (int j = lane; j < k; j += 32) w[static_cast<size_t>(t) * k + j] /= chosen + 1e-20f;
   }
 }
 
@@ -241,12 +257,13 @@ grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ B, T* __restri
 }  // namespace experts
 }  // namespace lvb
 
-// Routing of z [T, E] fp32 (row stride ldz).  Choice score: sigmoid(z) + correction (optional, fp32 or bf16 [E]).  groups > 1: only experts
-// of the `keep` neighbour groups (E / groups experts each) with the largest sum of their two best choice scores can be chosen.
-// idx, w [T, k]: the k best choice scores, best first, and scale * sigmoid(z) of each.  live (optional) [T]: tokens with a value outside
+// Routing of z [T, E] fp32 (row stride ldz).  kind 0: choice score sigmoid(z) + correction (optional, fp32 or bf16 [E]); groups > 1: only
+// experts of the `keep` neighbour groups (E / groups experts each) with the largest sum of their two best choice scores can be
+// chosen; idx, w [T, k]: the k best choice scores, best first, and scale * sigmoid(z) of each.  kind 1: softmax(z) + correction, groups by
+// their best choice score, weights softmax(z) / (sum over the chosen + 1e-20).  live (optional) [T]: tokens with a value outside
 // [0, live_limit) are padding and get idx = -1.  counts: int32 [2 * E], cleared here; the first E receive the tokens per expert, the
 // rest are lvb_moe_dispatch's cursors.
-extern "C" int lvb_moe_route_sigmoid(const float* z, long long ldz, const void* correction, int c_f32, const int* live, int live_limit, int T,
+extern "C" int lvb_moe_route_grouped(int kind, const float* z, long long ldz, const void* correction, int c_f32, const int* live, int live_limit, int T,
                                      int E, int k, int groups, int keep, float scale, int* idx, float* w, int* counts, void* stream) {
   using namespace lvb;
   using namespace lvb::experts;
@@ -257,8 +274,9 @@ extern "C" int lvb_moe_route_sigmoid(const float* z, long long ldz, const void* 
   if (smem > 48 * 1024) return kErrTooLarge;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (cudaMemsetAsync(counts, 0, 2 * static_cast<size_t>(E) * sizeof(int), s) != cudaSuccess) return kErrCuda;
-  route_kernel<<<(T + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, s>>>(z, ldz, correction, c_f32, live, live_limit, T, E, k, groups,
-                                                                                 keep, scale, idx, w, counts);
+  auto kern = kind == 1 ? route_kernel<true> : route_kernel<false>;
+  kern<<<(T + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, s>>>(z, ldz, correction, c_f32, live, live_limit, T, E, k, groups, keep, scale,
+                                                                          idx, w, counts);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 

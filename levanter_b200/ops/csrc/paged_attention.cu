@@ -81,7 +81,14 @@ struct Params {
   int chunk;                  // > 0: a query at position i sees positions >= i - i % chunk only
   int window;                 // > 0: a query at position i sees positions > i - window only
   long long ldq, ldg;         // row strides of q and gate
-  const __nv_bfloat16* gate;  // optional [T, H * dv]: the output is multiplied by its sigmoid
+  const __nv_bfloat16* gate;  // optional [T, heads * dv], or [T, heads] with gate_per_head: the output is multiplied by its sigmoid
+  int gate_per_head;
+  // maps = 2: rows 2h and 2h + 1 of q are two score maps of head h over the same values (H counts both).  A slot's key row holds both maps'
+  // keys side by side (dk counts both), each query row meets its own half, and out [T, H / 2, dv] = o * diff_scale / sqrt(mean(o^2) + eps)
+  // with o = a1 - weight a2.
+  int maps;
+  const float* weight;
+  float diff_scale, eps;
 };
 
 // First visible key of a query whose context (its position + 1) is ctx.
@@ -92,7 +99,8 @@ __device__ __forceinline__ int first_key(const Params& p, int ctx) {
 
 __device__ __forceinline__ float gate_factor(const Params& p, int t, int h, int d) {
   if (p.gate == nullptr) return 1.f;
-  return 1.f / (1.f + __expf(-__bfloat162float(p.gate[t * p.ldg + static_cast<long long>(h) * p.dv + d])));
+  const long long at = p.gate_per_head ? h : static_cast<long long>(h) * p.dv + d;
+  return 1.f / (1.f + __expf(-__bfloat162float(p.gate[t * p.ldg + at])));
 }
 
 // Which sequence owns packed token t, and how many keys it may attend to.  Returns false for padding tokens.
@@ -183,7 +191,7 @@ __global__ void __launch_bounds__(kThreads) paged_attention_kernel(Params p) {
     for (int g = 0; g < kMaxG; ++g) {
       if (g < G) {
         float v = (r >= 0) ? acc[g] : -INFINITY;
-        if (p.soft_cap > 0.f && r >= 0) v = p.soft_cap * tanhf(v / p.soft_cap);
+        if (p.soft_cap > 0.f && r >= 0) v = soft_capped(v, p.soft_cap);
         s_p[g * kPart + i] = v;
       }
     }
@@ -377,7 +385,7 @@ __global__ void __launch_bounds__(kThreads) paged_attention_staged_kernel(Params
           float v = acc[g];
           v += __shfl_xor_sync(0xffffffffu, v, 1);
           v += __shfl_xor_sync(0xffffffffu, v, 2);
-          if (p.soft_cap > 0.f) v = p.soft_cap * tanhf(v / p.soft_cap);
+          if (p.soft_cap > 0.f) v = soft_capped(v, p.soft_cap);
           if (quarter == 0) s_p[g * kStageKeys + key_l] = valid ? v : -INFINITY;
         }
       }
@@ -503,8 +511,9 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
   const int k0 = (live ? first_key(p, ctx) : 0) + part * kPart;
   if (!live || k0 >= ctx) {
     if (part == 0 && !live) {
-      for (int i = threadIdx.x; i < G * dv; i += kThreads)
-        p.out[(static_cast<long long>(t) * p.H + kvh * G) * dv + i] = __float2bfloat16(0.f);
+      const int per = G / p.maps;
+      for (int i = threadIdx.x; i < per * dv; i += kThreads)
+        p.out[(static_cast<long long>(t) * p.KV + kvh) * per * dv + i] = __float2bfloat16(0.f);
     }
     return;
   }
@@ -524,15 +533,19 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
   const int row_lo = lane >> 2, row_hi = row_lo + 8, kq = (lane & 3) * 2;
   uint32_t qa[DKC / 16][4];
   {
-    const __nv_bfloat16* qbase = p.q + t * p.ldq + static_cast<long long>(kvh) * G * dk;
+    const int dm = p.maps == 1 ? dk : dk / 2;  // a query row meets dm dimensions of the key row, the second map's the last ones
+    const __nv_bfloat16* qbase = p.q + t * p.ldq + static_cast<long long>(kvh) * G * dm;
+    auto load = [&](int row, int d) -> uint32_t {
+      const int at = d - (p.maps == 1 ? 0 : (row & 1) * dm);
+      return row < G && at >= 0 && at < dm ? *reinterpret_cast<const uint32_t*>(qbase + row * dm + at) : 0u;
+    };
 #pragma unroll
     for (int ks = 0; ks < DKC / 16; ++ks) {
       const int d0 = ks * 16 + kq;
-      const bool in0 = kExact || d0 < dk, in1 = kExact || d0 + 8 < dk;
-      qa[ks][0] = row_lo < G && in0 ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * dk + d0) : 0u;
-      qa[ks][1] = row_hi < G && in0 ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * dk + d0) : 0u;
-      qa[ks][2] = row_lo < G && in1 ? *reinterpret_cast<const uint32_t*>(qbase + row_lo * dk + d0 + 8) : 0u;
-      qa[ks][3] = row_hi < G && in1 ? *reinterpret_cast<const uint32_t*>(qbase + row_hi * dk + d0 + 8) : 0u;
+      qa[ks][0] = load(row_lo, d0);
+      qa[ks][1] = load(row_hi, d0);
+      qa[ks][2] = load(row_lo, d0 + 8);
+      qa[ks][3] = load(row_hi, d0 + 8);
     }
   }
 
@@ -612,7 +625,7 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
         const int kcol = st * kMmaStageKeys + 8 * j + kq + (e & 1);
         const bool valid = kcol < wnk && s_rows[wk0 + kcol] >= 0;
         float v = sacc[j][e];
-        if (p.soft_cap > 0.f) v = p.soft_cap * tanhf(v * p.scale / p.soft_cap) * 1.4426950408889634f;
+        if (p.soft_cap > 0.f) v = soft_capped(v * p.scale, p.soft_cap) * 1.4426950408889634f;
         else v *= sc_log2;
         v = valid ? v : -INFINITY;
         sacc[j][e] = v;
@@ -689,6 +702,45 @@ __global__ void __launch_bounds__(kThreads) paged_attention_mma_kernel(Params p)
     *reinterpret_cast<float2*>(s_o + (warp * 16 + row_hi) * dv16 + d0) = make_float2(o[n][2], o[n][3]);
   }
   __syncthreads();
+  if (p.maps == 2 && p.parts == 1) {  // a warp per head: both maps of a head, their difference and its norm
+    for (int j = warp; j < G / 2; j += 4) {
+      float f[2][4];  // what a warp's sum of a map is multiplied by
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        float m = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) m = fmaxf(m, s_ml[(w * 16 + 2 * j + i) * 2]);
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+          const float mw = s_ml[(w * 16 + 2 * j + i) * 2];
+          f[i][w] = (mw == -INFINITY) ? 0.f : exp2f(mw - m);
+          l = fmaf(s_ml[(w * 16 + 2 * j + i) * 2 + 1], f[i][w], l);
+        }
+        const float inv = l > 0.f ? (i == 0 ? 1.f : -*p.weight) / l : 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) f[i][w] *= inv;
+      }
+      float v[DVC / 32], ss = 0.f;
+#pragma unroll
+      for (int n = 0; n < DVC / 32; ++n) {
+        const int d = n * 32 + lane;
+        v[n] = 0.f;
+        if (d < dv) {
+#pragma unroll
+          for (int w = 0; w < 4; ++w) v[n] = fmaf(s_o[(w * 16 + 2 * j) * dv16 + d], f[0][w], fmaf(s_o[(w * 16 + 2 * j + 1) * dv16 + d], f[1][w], v[n]));
+        }
+        ss = fmaf(v[n], v[n], ss);
+      }
+      const float r = p.diff_scale * rsqrtf(warp_sum(ss) / static_cast<float>(dv) + p.eps);
+      const int h = kvh * (G / 2) + j;
+#pragma unroll
+      for (int n = 0; n < DVC / 32; ++n) {
+        const int d = n * 32 + lane;
+        if (d < dv) p.out[(static_cast<long long>(t) * (p.H / 2) + h) * dv + d] = __float2bfloat16(v[n] * r * gate_factor(p, t, h, d));
+      }
+    }
+    return;
+  }
   for (int idx = threadIdx.x; idx < G * dv; idx += kThreads) {
     const int g = idx / dv, d = idx - g * dv;
     float m = -INFINITY;
@@ -744,6 +796,52 @@ __global__ void __launch_bounds__(kThreadsM) paged_merge_kernel(Params p) {
   }
 }
 
+// The same with two score maps per head: one CTA per (token, head) merges both, and their difference is normed.
+template <int kThreadsM>
+__global__ void __launch_bounds__(kThreadsM) paged_merge_maps_kernel(Params p) {
+  constexpr int kPer = 256 / kThreadsM;  // output dimensions per thread, at most
+  __shared__ float s_red[kThreadsM / 32];
+  const int t = blockIdx.x, h = blockIdx.y;
+  int seq = 0, ctx = 0;
+  if (!locate(p, t, seq, ctx)) return;  // zeros were written by the attention kernel
+  const int np = (ctx - first_key(p, ctx) + kPart - 1) / kPart;
+  float o[kPer], ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < kPer; ++n) o[n] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const long long row = (static_cast<long long>(t) * p.H + 2 * h + i) * p.parts;
+    float m = -INFINITY, l = 0.f;
+    for (int k = 0; k < np; ++k) m = fmaxf(m, p.part_ml[(row + k) * 2]);
+    for (int k = 0; k < np; ++k) l += p.part_ml[(row + k) * 2] == -INFINITY ? 0.f : p.part_ml[(row + k) * 2 + 1] * __expf(p.part_ml[(row + k) * 2] - m);
+    const float inv = l > 0.f ? (i == 0 ? 1.f : -*p.weight) / l : 0.f;
+    for (int k = 0; k < np; ++k) {
+      const float mk = p.part_ml[(row + k) * 2];
+      if (mk == -INFINITY) continue;
+      const float f = __expf(mk - m) * inv;
+#pragma unroll
+      for (int n = 0; n < kPer; ++n) {
+        const int d = n * kThreadsM + threadIdx.x;
+        if (d < p.dv) o[n] = fmaf(p.part_o[(row + k) * p.dv + d], f, o[n]);
+      }
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < kPer; ++n) ss = fmaf(o[n], o[n], ss);
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int w = 0; w < kThreadsM / 32; ++w) ss += s_red[w];
+  const float r = p.diff_scale * rsqrtf(ss / static_cast<float>(p.dv) + p.eps);
+#pragma unroll
+  for (int n = 0; n < kPer; ++n) {
+    const int d = n * kThreadsM + threadIdx.x;
+    if (d < p.dv) p.out[(static_cast<long long>(t) * (p.H / 2) + h) * p.dv + d] = __float2bfloat16(o[n] * r * gate_factor(p, t, h, d));
+  }
+}
+
 // LVB_PAGED_ATTENTION=direct selects the kernel that reads the cache rows straight from global memory for every shape,
 // LVB_PAGED_ATTENTION=staged the scalar kernel on staged rows; the default for D = 128 is the tensor-core kernel.
 inline int paged_variant() {
@@ -770,7 +868,10 @@ int launch_mma(const Params& p, cudaStream_t s) {
 }
 
 int launch_merge(const Params& p, cudaStream_t s) {
-  if (p.parts > 1) {
+  if (p.parts > 1 && p.maps == 2) {
+    if (p.dv <= 128) paged_merge_maps_kernel<128><<<dim3(p.T, p.H / 2), 128, 0, s>>>(p);
+    else paged_merge_maps_kernel<256><<<dim3(p.T, p.H / 2), 256, 0, s>>>(p);
+  } else if (p.parts > 1) {
     if (p.dv <= 128) paged_merge_kernel<128><<<dim3(p.T, p.H), 128, 0, s>>>(p);
     else paged_merge_kernel<256><<<dim3(p.T, p.H), 256, 0, s>>>(p);
   }
@@ -830,6 +931,7 @@ extern "C" int lvb_paged_attention(const void* q, const void* kv_pages, const in
   p.parts = lvb_paged_attention_parts(pages_per_seq * page_size);
   p.scale = scale; p.soft_cap = soft_cap;
   p.dk = p.dv = D; p.chunk = 0; p.window = 0; p.ldq = static_cast<long long>(H) * D; p.gate = nullptr; p.ldg = 0;
+  p.gate_per_head = 0; p.maps = 1; p.weight = nullptr; p.diff_scale = p.eps = 0.f;
   if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (D) {
@@ -851,18 +953,23 @@ extern "C" int lvb_paged_attention_general_parts(int max_context, int chunk, int
 //   * kv_pages [num_pages, page_size, KV, dk + dv]: a key row followed by a value row per KV head,
 //   * chunk > 0: positions are cut into chunks of that many, counted from the sequence's start, and a query sees its own chunk,
 //   * window > 0: a query sees itself and the window - 1 positions before it,
-//   * gate (optional, [T, H * dv], row stride ldg): the output is multiplied by its sigmoid,
-//   * ldq: row stride of q.  At most 16 query heads per KV head.
+//   * gate (optional, [T, heads * dv], or [T, heads] with gate_per_head; row stride ldg): the output is multiplied by its sigmoid,
+//   * weight (optional, one fp32 number on the device): rows 2h and 2h + 1 of q are two score maps of head h, a slot holds two key rows and a
+//     value row per KV head, and out [T, H / 2, dv] = diff_scale * o / sqrt(mean(o^2) + eps) with o = a1 - weight * a2,
+//   * ldq: row stride of q.  At most 16 query rows per KV head, and with two maps dk up to 128.
 extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices,
                                            const int* cu_q_lens, const int* num_seqs, const void* gate, void* out, float* part_o,
-                                           float* part_ml, int T, int H, int KV, int dk, int dv, int ldq, int ldg, int S,
+                                           float* part_ml, int T, int H, int KV, int dk, int dv, int ldq, int ldg, int gate_per_head, int S,
                                            int pages_per_seq, int page_size, int num_pages, int chunk, int window, float scale,
-                                           float soft_cap, void* stream) {
+                                           float soft_cap, const float* weight, float diff_scale, float eps, void* stream) {
   using namespace lvb;
   using namespace lvb::paged;
   if (T <= 0) return kErrOk;
   if (H <= 0 || KV <= 0 || H % KV != 0 || H / KV > kMaxG || S <= 0 || chunk < 0 || window < 0) return kErrBadArg;
-  if (dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || (dk & 7) || (dv & 7) || (ldq & 1)) return kErrBadArg;
+  if (weight != nullptr && (H / KV) % 2 != 0) return kErrBadArg;
+  if (dk <= 0 || dv <= 0 || (dk & 7) || (dv & 7) || (ldq & 1)) return kErrBadArg;
+  if (weight != nullptr) dk *= 2;
+  if (dk > 256 || dv > 256) return kErrBadArg;
   Params p;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.kv_pages = reinterpret_cast<const __nv_bfloat16*>(kv_pages);
@@ -873,7 +980,8 @@ extern "C" int lvb_paged_attention_general(const void* q, const void* kv_pages, 
   p.parts = lvb_paged_attention_general_parts(pages_per_seq * page_size, chunk, window);
   p.scale = scale; p.soft_cap = soft_cap;
   p.dk = dk; p.dv = dv; p.chunk = chunk; p.window = window; p.ldq = ldq; p.ldg = ldg;
-  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.gate_per_head = gate_per_head;
+  p.maps = weight != nullptr ? 2 : 1; p.weight = weight; p.diff_scale = diff_scale; p.eps = eps;
   if (p.parts > 1 && (part_o == nullptr || part_ml == nullptr)) return kErrBadArg;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   int rc;

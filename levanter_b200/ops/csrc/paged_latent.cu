@@ -52,6 +52,7 @@ struct Params {
   const __nv_bfloat16* q;         // [T, H, width]
   const __nv_bfloat16* kv_pages;  // [num_pages, page_size, width]
   const int *kv_lens, *page_indices, *cu_q_lens, *num_seqs;
+  const float* sink;              // optional [H]: joins the softmax denominator of its head as it is
   __nv_bfloat16* out;             // [T, H, rank]
   float* part_o;                  // [T, H, parts, rank]
   float* part_ml;                 // [T, H, parts, 2]: maximum (base 2) and sum
@@ -86,6 +87,9 @@ __device__ __forceinline__ int part_keys(const Params& p, int visible) {
   const int n = even > kMinPart ? even : kMinPart;
   return (n + kTileKeys - 1) / kTileKeys * kTileKeys;
 }
+
+// What head h's sink adds to a softmax sum relative to the maximum m (base 2).  Far above the maximum it is infinite and the output zero.
+__device__ __forceinline__ float sink_term(const Params& p, int h, float m) { return exp2f(p.sink[h] * 1.4426950408889634f - m); }
 
 // Key tiles are cut into chunks of 64 columns (128 bytes); columns past the width are zeros.
 __host__ __device__ constexpr int chunks_of(int width) { return (width + 63) / 64; }
@@ -393,6 +397,7 @@ __global__ void __launch_bounds__(cta_threads(kM, kPieces), 1) paged_latent_kern
     }
   }
   if (lk == 0) {
+    if (p.parts == 1 && p.sink != nullptr && row < heads) l_run += sink_term(p, h0 + row, m_run);
     s_m[row] = m_run;
     s_l[row] = l_run;
   }
@@ -440,6 +445,7 @@ __global__ void __launch_bounds__(128) merge_kernel(Params p) {
   float m = -INFINITY, l = 0.f;
   for (int i = 0; i < np; ++i) m = fmaxf(m, ml[2 * i]);
   for (int i = 0; i < np; ++i) l += ml[2 * i + 1] * exp2f(ml[2 * i] - m);
+  if (p.sink != nullptr) l += sink_term(p, h, m);
   const float inv = l > 0.f ? 1.f / l : 0.f;
   for (int d = threadIdx.x * 4; d < p.rank; d += 128 * 4) {
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -574,11 +580,12 @@ extern "C" int lvb_paged_latent_parts(int T, int H, int width, int rank, int max
 }
 
 // Packed query rows q [T, H, width] over pages [num_pages, page_size, width] whose rows' first `rank` elements are the values -> out [T, H, rank];
-// causal, window > 0: a row sees itself and the window - 1 positions before it.  width and rank: multiples of 8, rank <= 512, width <= 576.
+// causal, window > 0: a row sees itself and the window - 1 positions before it; sink (optional, fp32 [H]): joins the softmax denominator of its
+// head, unscaled.  width and rank: multiples of 8, rank <= 512, width <= 576.
 extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* kv_lens, const int* page_indices, const int* cu_q_lens,
-                                const int* num_seqs, void* out, float* part_o, float* part_ml, int T, int H, int width, int rank, int S,
-                                int pages_per_seq, int page_size, int num_pages, int window, int parts, float scale, int* status,
-                                void* stream) {
+                                const int* num_seqs, const float* sink, void* out, float* part_o, float* part_ml, int T, int H, int width,
+                                int rank, int S, int pages_per_seq, int page_size, int num_pages, int window, int parts, float scale,
+                                int* status, void* stream) {
   using namespace lvb;
   using namespace lvb::latent;
   if (T <= 0) return kErrOk;
@@ -590,6 +597,7 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.kv_pages = reinterpret_cast<const __nv_bfloat16*>(kv_pages);
   p.kv_lens = kv_lens; p.page_indices = page_indices; p.cu_q_lens = cu_q_lens; p.num_seqs = num_seqs;
+  p.sink = sink;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml;
   p.T = T; p.H = H; p.width = width; p.rank = rank; p.S = S; p.pages_per_seq = pages_per_seq; p.page_size = page_size; p.num_pages = num_pages;

@@ -63,17 +63,18 @@ __device__ __forceinline__ void fill_angles(const Rotation& r, int pos, float* s
 }
 
 // Rotate (and scale) `heads` rows of `size` elements at src, writing to dst and, when given, to dst2; the head strides are in
-// elements.  Elements past r.dims pass (scaled).  head_scale: optional factor per head.  `vec`: sizes and strides are multiples
+// elements, and at dst2 `maps2` heads lie side by side within one stride.  Elements past r.dims pass (scaled).  head_scale: optional factor per head.  `vec`: sizes and strides are multiples
 // of 8, pointers aligned and pairs fall into whole groups of 8.
 template <typename T>
 __device__ __forceinline__ void rotate_heads(const T* src, long long src_stride, T* dst, long long dst_stride, T* dst2, long long dst2_stride,
-                                             int heads, int size, const Rotation& r, const float* s_cos, const float* s_sin,
+                                             int maps2, int heads, int size, const Rotation& r, const float* s_cos, const float* s_sin,
                                              const void* head_scale, int scale_f32, bool vec) {
   auto factor = [&](int h) -> float {
     if (head_scale == nullptr) return 1.f;
     return scale_f32 ? reinterpret_cast<const float*>(head_scale)[h] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(head_scale)[h]);
   };
   const int dims = r.inv_freq != nullptr ? r.dims : 0, half = dims / 2;
+  auto second = [&](int h) { return dst2 + (maps2 == 1 ? h * dst2_stride : h / maps2 * dst2_stride + h % maps2 * size); };
   if (vec) {
     // units of 8 elements: half / 8 pair units of two groups each (or dims / 8 units of interleaved pairs), then the rest
     const int turn = r.interleaved ? dims / 8 : half / 8, units = turn + (size - dims) / 8;
@@ -82,7 +83,7 @@ __device__ __forceinline__ void rotate_heads(const T* src, long long src_stride,
       const float f = factor(h);
       const T* s = src + h * src_stride;
       T* d = dst + h * dst_stride;
-      T* d2 = dst2 != nullptr ? dst2 + h * dst2_stride : nullptr;
+      T* d2 = dst2 != nullptr ? second(h) : nullptr;
       float a[8];
       if (u < turn && !r.interleaved) {
         float b[8], x[8], y[8];
@@ -131,14 +132,14 @@ __device__ __forceinline__ void rotate_heads(const T* src, long long src_stride,
       dst[h * dst_stride + lo] = x;
       dst[h * dst_stride + hi] = y;
       if (dst2 != nullptr) {
-        dst2[h * dst2_stride + lo] = x;
-        dst2[h * dst2_stride + hi] = y;
+        second(h)[lo] = x;
+        second(h)[hi] = y;
       }
     } else {
       const int c = dims + u - half;
       const T x = from_f<T>(to_f<T>(s[c]) * f);
       dst[h * dst_stride + c] = x;
-      if (dst2 != nullptr) dst2[h * dst2_stride + c] = x;
+      if (dst2 != nullptr) second(h)[c] = x;
     }
   }
 }
@@ -148,9 +149,9 @@ struct QkvParams {
   const void* v_first;      // optional rows of an earlier layer's values: v <- (1 - mix) v + mix v_first
   const void* mix;          // one number
   const void* q_head_scale; // optional [H]
-  void* kv_pages;           // [slots, KV, dk + dv]
+  void* kv_pages;           // [slots, KV, maps * dk + dv]
   const int *pos, *dests;
-  int H, KV, dk, dv;
+  int H, KV, maps, dk, dv;  // maps: keys per KV head; k has KV * maps heads
   long long ldq, ldk, ldv, ldf, slots;
   Rotation rot;
   int small_f32;            // type of mix and q_head_scale
@@ -170,15 +171,15 @@ __global__ void __launch_bounds__(kThreads) qkv_prep_kernel(QkvParams p) {
   }
   const long long dest = p.dests[t];
   const bool live = dest >= 0 && dest < p.slots;
-  const int per = p.dk + p.dv;
+  const int keys = p.maps * p.dk, per = keys + p.dv;
   T* cache = live ? reinterpret_cast<T*>(p.kv_pages) + dest * p.KV * per : nullptr;
   T* q = reinterpret_cast<T*>(p.q) + t * p.ldq;
   T* k = reinterpret_cast<T*>(p.k) + t * p.ldk;
   T* v = reinterpret_cast<T*>(p.v) + t * p.ldv;
   if (half > 0 || p.q_head_scale != nullptr) {
-    rotate_heads<T>(q, p.dk, q, p.dk, static_cast<T*>(nullptr), 0, p.H, p.dk, p.rot, s_cos, s_sin, p.q_head_scale, p.small_f32, p.vec != 0);
+    rotate_heads<T>(q, p.dk, q, p.dk, static_cast<T*>(nullptr), 0, 1, p.H, p.dk, p.rot, s_cos, s_sin, p.q_head_scale, p.small_f32, p.vec != 0);
   }
-  if (half > 0 || live) rotate_heads<T>(k, p.dk, k, p.dk, cache, per, p.KV, p.dk, p.rot, s_cos, s_sin, nullptr, 0, p.vec != 0);
+  if (half > 0 || live) rotate_heads<T>(k, p.dk, k, p.dk, cache, per, p.maps, p.KV * p.maps, p.dk, p.rot, s_cos, s_sin, nullptr, 0, p.vec != 0);
   const T* first = p.v_first != nullptr ? reinterpret_cast<const T*>(p.v_first) + t * p.ldf : nullptr;
   float lam = 0.f;
   if (first != nullptr) lam = p.small_f32 ? *reinterpret_cast<const float*>(p.mix) : __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.mix));
@@ -195,7 +196,7 @@ __global__ void __launch_bounds__(kThreads) qkv_prep_kernel(QkvParams p) {
         for (int j = 0; j < 8; ++j) a[j] = (1.f - lam) * a[j] + lam * b[j];
         Vec8<T>::store(v + e, a);
       }
-      if (cache != nullptr) Vec8<T>::store(cache + h * per + p.dk + c, a);
+      if (cache != nullptr) Vec8<T>::store(cache + h * per + keys + c, a);
     }
     return;
   }
@@ -206,7 +207,7 @@ __global__ void __launch_bounds__(kThreads) qkv_prep_kernel(QkvParams p) {
       a = (1.f - lam) * a + lam * to_f<T>(first[e]);
       v[e] = from_f<T>(a);
     }
-    if (cache != nullptr) cache[h * per + p.dk + c] = from_f<T>(a);
+    if (cache != nullptr) cache[h * per + keys + c] = from_f<T>(a);
   }
 }
 
@@ -232,7 +233,7 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(LatentParams p) {
   float* s_cos = s_angles;
   float* s_sin = s_angles + p.rot.dims / 2;
   const int t = blockIdx.x;
-  fill_angles(p.rot, p.pos[t], s_cos, s_sin);
+  if (p.rotd > 0) fill_angles(p.rot, p.pos[t], s_cos, s_sin);
   const long long dest = p.dests[t];
   const int width = p.rank + p.rotd;
   T* cache = dest >= 0 && dest < p.slots ? reinterpret_cast<T*>(p.kv_pages) + dest * width : nullptr;
@@ -278,10 +279,11 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(LatentParams p) {
       if (cache != nullptr) cache[c] = a;
     }
   }
-  rotate_heads<T>(down + p.rank, 0, latent + p.rank, 0, cache != nullptr ? cache + p.rank : nullptr, 0, 1, p.rotd, p.rot, s_cos, s_sin, nullptr, 0,
+  if (p.rotd == 0) return;
+  rotate_heads<T>(down + p.rank, 0, latent + p.rank, 0, cache != nullptr ? cache + p.rank : nullptr, 0, 1, 1, p.rotd, p.rot, s_cos, s_sin, nullptr, 0,
                   p.vec_c != 0 && p.vec_q != 0);
   rotate_heads<T>(reinterpret_cast<const T*>(p.q_rot) + t * p.ldq, p.q_head, reinterpret_cast<T*>(p.q_out) + t * p.ldo, p.o_head,
-                  static_cast<T*>(nullptr), 0, p.H, p.rotd, p.rot, s_cos, s_sin, nullptr, 0, p.vec_q != 0);
+                  static_cast<T*>(nullptr), 0, 1, p.H, p.rotd, p.rot, s_cos, s_sin, nullptr, 0, p.vec_q != 0);
 }
 
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
@@ -294,26 +296,26 @@ inline bool groups_of_8(const float* inv_freq, int dims, int interleaved) {
 }  // namespace prep
 }  // namespace lvb
 
-// Rows of q [T, H, dk], k [T, KV, dk], v [T, KV, dv] (row strides ldq, ldk, ldv), in place:
+// Rows of q [T, H, dk], k [T, KV * maps, dk], v [T, KV, dv] (row strides ldq, ldk, ldv), in place:
 //   q, k: the first rot_dims dimensions of each head rotated by pos[t] * pos_scale * inv_freq[i] (pairs as `interleaved` says; inv_freq
 //         null: no rotation), q multiplied by q_head_scale[h] when given;
 //   v:    (1 - mix) v + mix v_first[t] when v_first is given;
-// and k, v written to flat slots dests[t] of kv_pages [slots, KV, dk + dv] (out-of-range slots are skipped).  is_f32: type of the rows and the
+// and k, v written to flat slots dests[t] of kv_pages [slots, KV, maps * dk + dv] (out-of-range slots are skipped).  is_f32: type of the rows and the
 // cache; small_f32: type of mix and q_head_scale.
 extern "C" int lvb_qkv_prep(void* q, void* k, void* v, const void* v_first, const void* mix, const void* q_head_scale, void* kv_pages,
-                            const int* pos, const int* dests, int T, int H, int KV, int dk, int dv, long long ldq, long long ldk,
+                            const int* pos, const int* dests, int T, int H, int KV, int maps, int dk, int dv, long long ldq, long long ldk,
                             long long ldv, long long ldf, long long slots, const float* inv_freq, int rot_dims, int interleaved,
                             float pos_scale, float magnitude, int is_f32, int small_f32, void* stream) {
   using namespace lvb;
   using namespace lvb::prep;
   if (T <= 0) return kErrOk;
-  if (H <= 0 || KV <= 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims > dk || (rot_dims & 1)) return kErrBadArg;
+  if (H <= 0 || KV <= 0 || maps <= 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims > dk || (rot_dims & 1)) return kErrBadArg;
   if (inv_freq != nullptr && (rot_dims == 0 || pos == nullptr)) return kErrBadArg;
   if (v_first != nullptr && mix == nullptr) return kErrBadArg;
   if (rot_dims > 4096) return kErrTooLarge;
   QkvParams p;
   p.q = q; p.k = k; p.v = v; p.v_first = v_first; p.mix = mix; p.q_head_scale = q_head_scale; p.kv_pages = kv_pages; p.pos = pos; p.dests = dests;
-  p.H = H; p.KV = KV; p.dk = dk; p.dv = dv; p.ldq = ldq; p.ldk = ldk; p.ldv = ldv; p.ldf = ldf; p.slots = slots;
+  p.H = H; p.KV = KV; p.maps = maps; p.dk = dk; p.dv = dv; p.ldq = ldq; p.ldk = ldk; p.ldv = ldv; p.ldf = ldf; p.slots = slots;
   p.rot = Rotation{inv_freq, inv_freq != nullptr ? rot_dims : 0, interleaved, pos_scale, magnitude};
   p.small_f32 = small_f32;
   p.vec = ((dk | dv | ldq | ldk | ldv) & 7) == 0 && (v_first == nullptr || ((ldf & 7) == 0 && aligned16(v_first))) && aligned16(q) && aligned16(k) &&
@@ -327,7 +329,8 @@ extern "C" int lvb_qkv_prep(void* q, void* k, void* v, const void* v_first, cons
 
 // Latent attention.  Row t of down (stride ldd) holds `rank` compressed dimensions and a key part of rot_dims dimensions shared by the
 // heads.  latent[t] = [RMS norm of the former with weight norm_w, the latter rotated], also written to slot dests[t] of kv_pages [slots,
-// rank + rot_dims]; head h's rotated query part goes from q_rot + t * ldq + h * q_head to q_out + t * ldo + h * o_head.
+// rank + rot_dims]; head h's rotated query part goes from q_rot + t * ldq + h * q_head to q_out + t * ldo + h * o_head.  rot_dims 0: the norm and
+// the cache write only.
 extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* latent, void* kv_pages, const void* q_rot, void* q_out, const int* pos,
                                const int* dests, int T, int H, int rank, int rot_dims, long long ldd, long long ldq, long long q_head,
                                long long ldo, long long o_head, long long slots, float eps, const float* inv_freq, int interleaved,
@@ -335,7 +338,8 @@ extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* laten
   using namespace lvb;
   using namespace lvb::prep;
   if (T <= 0) return kErrOk;
-  if (H <= 0 || rank <= 0 || rot_dims <= 0 || (rot_dims & 1) || inv_freq == nullptr || pos == nullptr) return kErrBadArg;
+  if (H <= 0 || rank <= 0 || rot_dims < 0 || (rot_dims & 1)) return kErrBadArg;
+  if (rot_dims > 0 && (inv_freq == nullptr || pos == nullptr)) return kErrBadArg;
   if (rot_dims > 4096) return kErrTooLarge;
   LatentParams p;
   p.down = down; p.norm_w = norm_w; p.latent = latent; p.kv_pages = kv_pages; p.q_rot = q_rot; p.q_out = q_out; p.pos = pos; p.dests = dests;

@@ -38,9 +38,11 @@ __global__ void embed_kernel(const int* __restrict__ ids, const void* __restrict
 }
 
 // y[r, :] = x[r, :] / sqrt(mean(x[r, :]^2) + eps) * (w + w_offset); x fp32, y fp32 or bf16.  rows: optional int64 gather of the rows.
-// One CTA per row; the row's second read comes from L1.
+// One CTA per row; the row's second read comes from L1.  kAdd: the vector `add` (w's type) joins the row first, and the sum is written
+// back; every thread reads back the columns that it wrote.
+template <bool kAdd>
 __global__ void __launch_bounds__(256)
-rms_kernel(const float* __restrict__ x, const long long* __restrict__ rows, const void* __restrict__ w, int w_f32, void* __restrict__ y,
+rms_kernel(float* x, const long long* __restrict__ rows, const void* __restrict__ add, const void* __restrict__ w, int w_f32, void* __restrict__ y,
            int y_f32, int dim, float eps, float w_offset, int vec) {
   __shared__ float s_red[8];
   const size_t src = static_cast<size_t>(rows != nullptr ? rows[blockIdx.x] : blockIdx.x) * dim;
@@ -48,11 +50,23 @@ rms_kernel(const float* __restrict__ x, const long long* __restrict__ rows, cons
   float ss = 0.f;
   if (vec) {
     for (int c = threadIdx.x * 4; c < dim; c += blockDim.x * 4) {
-      const float4 v = *reinterpret_cast<const float4*>(x + src + c);
+      float4 v = *reinterpret_cast<const float4*>(x + src + c);
+      if constexpr (kAdd) {
+        const float4 a = ld4(add, w_f32, c);
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        *reinterpret_cast<float4*>(x + src + c) = v;
+      }
       ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
     }
   } else {
-    for (int c = threadIdx.x; c < dim; c += blockDim.x) ss = fmaf(x[src + c], x[src + c], ss);
+    for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+      float v = x[src + c];
+      if constexpr (kAdd) {
+        v += ld1(add, w_f32, c);
+        x[src + c] = v;
+      }
+      ss = fmaf(v, v, ss);
+    }
   }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = ss;
@@ -146,14 +160,37 @@ add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const long l
   }
 }
 
-// out[r, c] = gelu(gate[r, c]) * up[r, c] with the tanh form of gelu, any size and either type
-__global__ void gelu_glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, void* __restrict__ out, int f32, long long total,
-                                int cols, long long ldg, long long ldu) {
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+// act(g) * u: tanh-gelu (0) or silu (1).  kFast: for results that are rounded to bf16.
+template <bool kFast>
+__device__ __forceinline__ float glu(int act, float g, float u) {
+  if (act == 1) return kFast ? g * u * __fdividef(1.f, 1.f + __expf(-g)) : g / (1.f + expf(-g)) * u;
+  return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+}
+
+// out[r, c] = act(gate[r, c]) * up[r, c] (* sigmoid(row_gate[r * ldr])), any size; gate and up of one type, out of that type or bf16
+template <bool kOutF32>
+__global__ void __launch_bounds__(256)
+glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const float* __restrict__ row_gate, void* __restrict__ out, int act, int f32,
+           long long total, int cols, long long ldg, long long ldu, long long ldr, int vec) {
+  auto factor = [&](long long r) { return row_gate != nullptr ? 1.f / (1.f + expf(-row_gate[r * ldr])) : 1.f; };
+  const long long step = static_cast<long long>(gridDim.x) * blockDim.x;
+  if (vec) {  // groups of 4 columns; cols is a multiple of 4
+    const int per = cols / 4;
+    for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total / 4; i += step) {
+      const long long r = i / per, c = (i - r * per) * 4;
+      const float4 g = ld4(gate, f32, r * ldg + c), u = ld4(up, f32, r * ldu + c);
+      const float f = factor(r);
+      const float4 o = make_float4(glu<!kOutF32>(act, g.x, u.x) * f, glu<!kOutF32>(act, g.y, u.y) * f, glu<!kOutF32>(act, g.z, u.z) * f,
+                                   glu<!kOutF32>(act, g.w, u.w) * f);
+      if constexpr (kOutF32) reinterpret_cast<float4*>(out)[i] = o;
+      else reinterpret_cast<uint2*>(out)[i] = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    }
+    return;
+  }
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += step) {
     const long long r = i / cols, c = i - r * cols;
-    const float g = ld1(gate, f32, r * ldg + c), u = ld1(up, f32, r * ldu + c);
-    const float o = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-    if (f32) reinterpret_cast<float*>(out)[i] = o;
+    const float o = glu<!kOutF32>(act, ld1(gate, f32, r * ldg + c), ld1(up, f32, r * ldu + c)) * factor(r);
+    if constexpr (kOutF32) reinterpret_cast<float*>(out)[i] = o;
     else reinterpret_cast<__nv_bfloat16*>(out)[i] = __float2bfloat16(o);
   }
 }
@@ -176,14 +213,16 @@ extern "C" int lvb_embed_stream(const int* ids, const void* weight, int w_f32, f
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
-// n_rows output rows; rows: int64 [n_rows] source rows (each in range: the caller's responsibility), or null for row i = i.
-extern "C" int lvb_rms_stream(const float* x, const long long* rows, const void* w, int w_f32, void* y, int y_f32, int n_rows, int dim,
+// n_rows output rows; rows: int64 [n_rows] source rows (each in range: the caller's responsibility), or null for row i = i.  add: null, or a
+// vector [dim] of w's type that is added to every row of x first (in place; rows must be null then).
+extern "C" int lvb_rms_stream(float* x, const long long* rows, const void* add, const void* w, int w_f32, void* y, int y_f32, int n_rows, int dim,
                               float eps, float w_offset, void* stream) {
   using namespace lvb;
-  if (n_rows <= 0 || dim <= 0) return kErrBadArg;
-  const int vec = (dim & 3) == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
-  stream32::rms_kernel<<<n_rows, stream32::threads_for(dim), 0, reinterpret_cast<cudaStream_t>(stream)>>>(x, rows, w, w_f32, y, y_f32, dim, eps,
-                                                                                                       w_offset, vec);
+  if (n_rows <= 0 || dim <= 0 || (add != nullptr && rows != nullptr)) return kErrBadArg;
+  const int vec = (dim & 3) == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y) |
+                                      reinterpret_cast<uintptr_t>(add)) & 15) == 0;
+  auto kern = add != nullptr ? stream32::rms_kernel<true> : stream32::rms_kernel<false>;
+  kern<<<n_rows, stream32::threads_for(dim), 0, reinterpret_cast<cudaStream_t>(stream)>>>(x, rows, add, w, w_f32, y, y_f32, dim, eps, w_offset, vec);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
@@ -206,13 +245,19 @@ extern "C" int lvb_add_norm_stream(float* x, const float* y, const long long* ro
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
-// out [rows, cols] = gelu_tanh(gate) * up; gate and up with row strides ldg and ldu; f32: type of all three.
-extern "C" int lvb_gelu_glu_any(const void* gate, const void* up, void* out, int f32, int rows, int cols, long long ldg, long long ldu, void* stream) {
+// out [rows, cols] = act(gate) * up (* the sigmoid of row_gate[r * ldr], fp32, when given) with act = tanh-gelu (0) or silu (1); gate and up with row
+// strides ldg and ldu; in_f32, out_f32: types (fp32 results need fp32 operands).
+extern "C" int lvb_glu_any(const void* gate, const void* up, const float* row_gate, void* out, int act, int in_f32, int out_f32, int rows, int cols,
+                           long long ldg, long long ldu, long long ldr, void* stream) {
   using namespace lvb;
-  if (rows <= 0 || cols <= 0) return kErrBadArg;
+  if (rows <= 0 || cols <= 0 || act < 0 || act > 1 || (out_f32 && !in_f32)) return kErrBadArg;
+  const uintptr_t mis = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out);
+  const int vec = ((cols | ldg | ldu) & 3) == 0 && (mis & 15) == 0;
   const long long total = static_cast<long long>(rows) * cols, cap = static_cast<long long>(num_sms()) * 16;
-  long long blocks = (total + 255) / 256;
+  long long blocks = (total / (vec ? 4 : 1) + 255) / 256;
   if (blocks > cap) blocks = cap;
-  stream32::gelu_glu_kernel<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, out, f32, total, cols, ldg, ldu);
+  auto kern = out_f32 ? stream32::glu_kernel<true> : stream32::glu_kernel<false>;
+  kern<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, row_gate, out, act, in_f32, total, cols, ldg, ldu, ldr,
+                                                                                   vec);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }

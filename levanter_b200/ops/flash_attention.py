@@ -11,6 +11,7 @@ from typing import Optional
 import torch
 
 from . import lib
+from .map_difference import MapDifference
 
 
 def kernel_built() -> bool:
@@ -47,10 +48,11 @@ def supported(q, k, v, mask, bias, no_dropout: bool, attention_dtype) -> bool:
 _packed = {}
 
 
-def packed_supported(q, k, v, scale: float) -> bool:
-    """Shapes :func:`flash_attention_packed` takes: bf16 rows on a B200, sizes that are multiples of 8 (keys up to 192, values up to 128), a
-    positive scale (the running maximum is taken over unscaled scores) and 16-byte aligned rows."""
-    return packed_rows_ok(q, 192) and packed_rows_ok(k, 192) and packed_rows_ok(v, 128) and q.shape[0] % 256 == 0 and scale > 0.0
+def packed_supported(q, k, v, scale: float, maps: int = 1) -> bool:
+    """Shapes :func:`flash_attention_packed` takes: bf16 rows on a B200, sizes that are multiples of 8 (keys up to 192, with two score maps up
+    to 128; values up to 128), a positive scale (the running maximum is taken over unscaled scores) and 16-byte aligned rows."""
+    most = 192 if maps == 1 else 128
+    return packed_rows_ok(q, most) and packed_rows_ok(k, most) and packed_rows_ok(v, 128) and q.shape[0] % 256 == 0 and scale > 0.0
 
 
 def packed_rows_ok(t: torch.Tensor, most: int) -> bool:
@@ -60,26 +62,35 @@ def packed_rows_ok(t: torch.Tensor, most: int) -> bool:
 
 
 def flash_attention_packed(q, k, v, pos, *, scaling_factor: float, chunk: Optional[int] = None, window: Optional[int] = None, gate=None,
-                           logits_soft_cap: Optional[float] = None) -> torch.Tensor:
+                           logits_soft_cap: Optional[float] = None, sink: Optional[torch.Tensor] = None,
+                           difference: Optional[MapDifference] = None) -> torch.Tensor:
     """Causal attention over packed rows of sequences that start at position 0: ``q [T, Hq, dk]``, ``k [T, Hkv, dk]``, ``v [T, Hkv, dv]``
     (slices of one wider row are fine), ``pos [T]`` int32 positions with padding rows at 0, ``T`` a multiple of 256 ->
     ``[T, Hq, dv]``.  ``chunk``: a row sees its own chunk of that many positions only.  ``window``: a row sees itself and the
-    ``window - 1`` positions before it.  ``gate [T, Hq * dv]``: the result is multiplied by its sigmoid.  Forward only; shapes as in :func:`packed_supported`."""
+    ``window - 1`` positions before it.  ``gate [T, Hq * dv]`` or ``[T, Hq]``: the result is multiplied by its sigmoid.  ``sink [Hq]`` (fp32):
+    a number per head that joins the softmax denominator as it is.  ``difference``: ``q [T, 2 Hq, dk]`` and ``k [T, 2 Hkv, dk]`` hold the two
+    score maps of a head side by side, and their results are combined.  Forward only; shapes as in :func:`packed_supported`."""
     c = lib
     if "f" not in _packed:
-        _packed["f"] = lib.fn("lvb_flash_attn_fwd_packed", [c.c_void_p] * 6 + [c.c_int] * 11 + [c.c_float, c.c_float, c.c_void_p, c.c_void_p])
-    T, Hq, dk = q.shape
+        _packed["f"] = lib.fn("lvb_flash_attn_fwd_packed", [c.c_void_p] * 7 + [c.c_int] * 12 + [c.c_float, c.c_float, c.c_void_p, c.c_float, c.c_float,
+                                                                                               c.c_void_p, c.c_void_p])
+    T, rows, dk = q.shape
+    Hq = rows if difference is None else rows // 2
     Hkv, dv = v.shape[1], v.shape[2]
+    if difference is not None and sink is not None:
+        raise NotImplementedError("differential attention takes no sink")
     pos = pos.to(torch.int32).contiguous()
-    ldg = 0
+    ldg = per_head = 0
     if gate is not None:
-        if gate.dtype != torch.bfloat16 or gate.stride(1) != 1 or gate.stride(0) % 8 != 0 or gate.data_ptr() % 16 != 0:
+        per_head = int(gate.shape[1] == Hq)
+        if gate.dtype != torch.bfloat16 or gate.stride(1) != 1 or (not per_head and (gate.stride(0) % 8 != 0 or gate.data_ptr() % 16 != 0)):
             gate = gate.to(torch.bfloat16).contiguous()
         ldg = gate.stride(0)
+    diff = (0, 0.0, 0.0) if difference is None else (difference.weight.data_ptr(), float(difference.scale), float(difference.eps))
     out = torch.empty(T, Hq, dv, dtype=torch.bfloat16, device=q.device)
-    rc = _packed["f"](q.data_ptr(), k.data_ptr(), v.data_ptr(), lib.ptr(gate), out.data_ptr(), pos.data_ptr(), T, Hq, Hkv, dk, dv, q.stride(0),
-                      k.stride(0), v.stride(0), ldg, int(chunk or 0), int(window or 0), float(scaling_factor), float(logits_soft_cap or 0.0),
-                      lib.status_buffer().data_ptr(), lib.stream_ptr())
+    rc = _packed["f"](q.data_ptr(), k.data_ptr(), v.data_ptr(), lib.ptr(gate), lib.ptr(sink), out.data_ptr(), pos.data_ptr(), T, Hq, Hkv, dk, dv, q.stride(0),
+                      k.stride(0), v.stride(0), ldg, per_head, int(chunk or 0), int(window or 0), float(scaling_factor), float(logits_soft_cap or 0.0),
+                      *diff, lib.status_buffer().data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_flash_attn_fwd_packed")
     return out
 

@@ -240,41 +240,50 @@ def moe_route(router_logits: torch.Tensor, k: int):
     return moe_route_reference(router_logits, k)
 
 
-# ------------------------------------------------------------------------------------------------ sigmoid routing within groups
-# Serving form of a mixture whose router scores experts by a sigmoid, chooses by score + correction within the best groups of
-# neighbouring experts, and whose experts are plain (ungated) two-matrix layers.  ``csrc/moe_experts.cu``.
+# ------------------------------------------------------------------------------------------------ routing within groups, for serving
+# The router scores experts by a sigmoid or a softmax, chooses by score (+ correction) within the best groups of neighbouring experts;
+# experts are plain (squared ReLU) or gated (SiLU) layers.  ``csrc/moe_experts.cu``.
+def _within_groups(choice: torch.Tensor, groups: int, keep: int, best: int) -> torch.Tensor:
+    """``choice [T, E]`` with -inf outside the ``keep`` groups of neighbours whose ``best`` largest choice scores sum highest."""
+    if groups <= 1 or keep >= groups:
+        return choice
+    T, E = choice.shape
+    size = E // groups
+    gs = choice.view(T, groups, size).topk(min(best, size), dim=-1).values.sum(-1)
+    kept = torch.zeros(T, groups, dtype=torch.bool, device=choice.device)
+    kept.scatter_(1, gs.topk(keep, dim=-1).indices, True)
+    return choice.masked_fill(~kept.repeat_interleave(size, dim=1), float("-inf"))
+
+
 def route_sigmoid_reference(logits: torch.Tensor, correction, k: int, groups: int, keep: int, scale: float):
     """``(idx[T, k], w[T, k])``: see :func:`route_sigmoid`.  Differentiable in the weights."""
-    T, E = logits.shape
     s = torch.sigmoid(logits.float())
     c = s.detach() if correction is None else s.detach() + correction.float()
-    if groups > 1 and keep < groups:
-        size = E // groups
-        gs = c.view(T, groups, size).topk(min(2, size), dim=-1).values.sum(-1)
-        kept = torch.zeros(T, groups, dtype=torch.bool, device=c.device)
-        kept.scatter_(1, gs.topk(keep, dim=-1).indices, True)
-        c = c.masked_fill(~kept.repeat_interleave(size, dim=1), float("-inf"))
-    idx = c.topk(k, dim=-1).indices
+    idx = _within_groups(c, groups, keep, 2).topk(k, dim=-1).indices
     return idx, s.gather(1, idx) * scale
 
 
+def route_softmax_reference(logits: torch.Tensor, k: int, groups: int, keep: int):
+    """``(idx[T, k], w[T, k])``: see :func:`route_softmax`.  Differentiable in the weights."""
+    s = torch.softmax(logits.float(), dim=-1)
+    idx = _within_groups(s.detach(), groups, keep, 1).topk(k, dim=-1).indices
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20)
+
+
 class RoutedTokens:
-    """What :func:`route_sigmoid` leaves on the device for the expert products: choices, weights and tokens per expert."""
+    """What routing leaves on the device for the expert products: choices, weights and tokens per expert."""
 
     def __init__(self, idx, w, counts):
         self.idx, self.w, self.counts = idx, w, counts
 
 
-def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, keep: int = 1, scale: float = 1.0, live=None,
-                  live_limit: int = 0) -> RoutedTokens:
-    """Routing of fp32 ``logits [T, E]``: the ``k`` experts with the largest ``sigmoid(logits) + correction`` among those of the
-    ``keep`` (of ``groups``) neighbour groups whose two best choice scores sum highest; weights ``scale * sigmoid(logits)``.
-    ``live [T]`` int32: tokens whose value lies outside ``[0, live_limit)`` are padding and are sent to no expert (index -1)."""
+def _route(kind: int, logits, correction, k, groups, keep, scale, live, live_limit) -> RoutedTokens:
     from . import lib
 
     T, E = logits.shape
     if not (logits.is_cuda and lib.available()):
-        idx, w = route_sigmoid_reference(logits, correction, k, groups, keep, scale)
+        idx, w = route_softmax_reference(logits, k, groups, keep) if kind else route_sigmoid_reference(logits, correction, k, groups, keep, scale)
         idx = idx.to(torch.int32)
         if live is not None:
             dead = (live < 0) | (live >= live_limit)
@@ -282,7 +291,7 @@ def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, 
         return RoutedTokens(idx, w, None)
     c = lib
     if "rs" not in _g:
-        _g["rs"] = lib.fn("lvb_moe_route_sigmoid", [c.c_void_p, c.c_longlong, c.c_void_p, c.c_int, c.c_void_p] + [c.c_int] * 6 +
+        _g["rs"] = lib.fn("lvb_moe_route_grouped", [c.c_int, c.c_void_p, c.c_longlong, c.c_void_p, c.c_int, c.c_void_p] + [c.c_int] * 6 +
                           [c.c_float, c.c_void_p, c.c_void_p, c.c_void_p, c.c_void_p])
     dev = logits.device
     z = logits if logits.stride(1) == 1 else logits.contiguous()
@@ -291,10 +300,25 @@ def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, 
     idx = torch.empty(T, k, dtype=torch.int32, device=dev)
     w = torch.empty(T, k, dtype=torch.float32, device=dev)
     counts = torch.empty(2 * E, dtype=torch.int32, device=dev)
-    rc = _g["rs"](z.data_ptr(), z.stride(0), lib.ptr(correction), int(correction is not None and correction.dtype == torch.float32), lib.ptr(live),
+    rc = _g["rs"](kind, z.data_ptr(), z.stride(0), lib.ptr(correction), int(correction is not None and correction.dtype == torch.float32), lib.ptr(live),
                   int(live_limit), T, E, k, groups, keep, float(scale), idx.data_ptr(), w.data_ptr(), counts.data_ptr(), lib.stream_ptr())
-    lib.check_rc(rc, "lvb_moe_route_sigmoid")
+    lib.check_rc(rc, "lvb_moe_route_grouped")
     return RoutedTokens(idx, w, counts)
+
+
+def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, keep: int = 1, scale: float = 1.0, live=None,
+                  live_limit: int = 0) -> RoutedTokens:
+    """Routing of fp32 ``logits [T, E]``: the ``k`` experts with the largest ``sigmoid(logits) + correction`` among those of the
+    ``keep`` (of ``groups``) neighbour groups whose two best choice scores sum highest; weights ``scale * sigmoid(logits)``.
+    ``live [T]`` int32: tokens whose value lies outside ``[0, live_limit)`` are padding and are sent to no expert (index -1)."""
+    return _route(0, logits, correction, k, groups, keep, scale, live, live_limit)
+
+
+def route_softmax(logits: torch.Tensor, k: int, *, groups: int = 1, keep: int = 1, live=None, live_limit: int = 0) -> RoutedTokens:
+    """Routing of fp32 ``logits [T, E]`` (rows may be strided): the ``k`` experts with the largest softmax scores among those of the ``keep``
+    (of ``groups``) neighbour groups whose best score is largest; weights are the chosen scores divided by their sum.  ``live`` as in
+    :func:`route_sigmoid`."""
+    return _route(1, logits, None, k, groups, keep, 1.0, live, live_limit)
 
 
 def _block_rows(pairs: int, experts: int) -> int:
@@ -332,15 +356,18 @@ def grouped_product(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, 
     return y
 
 
-def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedTokens, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
+def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedTokens, up: torch.Tensor, down: torch.Tensor, *,
+                       gated: bool = False) -> torch.Tensor:
     """``stream[t] += sum_j w[t, j] * down[e] relu(up[e] h[t])^2`` with ``e = idx[t, j]``, in place on the fp32 stream; ``up [E, ff, width]``,
-    ``down [E, width, ff]``.  Forward only, CUDA only: dispatch into the block-padded expert-sorted layout, two grouped products (the
-    activation in the epilogue of the first), combine."""
+    ``down [E, width, ff]``.  ``gated``: ``up [E, 2 ff, width]`` holds a gate and an up projection, and the inner layer is ``silu(gate h) *
+    (up h)``.  Forward only, CUDA only: dispatch into the block-padded expert-sorted layout, two grouped products (the
+    activation in the epilogue of the first, or a gated activation between them), combine."""
     from . import lib
+    from .residual_stream import glu_of_rows
 
     c = lib
     T, k = routed.idx.shape
-    E, ff, width = up.shape
+    E, width, ff = down.shape
     dev = h.device
     tma = h.dtype == torch.bfloat16 and up.dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
     rows = _block_rows(T * k, E) if tma else 64  # 64: the tile of the fp32 product
@@ -356,19 +383,25 @@ def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedToke
                  dest.data_ptr(), tile_group.data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_moe_dispatch")
 
-    a = grouped_product(x_pad, up.to(h.dtype), tile_group, rows, True)
+    a = grouped_product(x_pad, up.to(h.dtype), tile_group, rows, not gated)
+    if gated:
+        a = glu_of_rows(a, ff, ActivationFunctionEnum.silu)
     y = grouped_product(a, down.to(h.dtype), tile_group, rows, False)
     rc = _g["c"](y.data_ptr(), int(y.dtype == torch.float32), dest.data_ptr(), routed.w.data_ptr(), T, k, width, stream.data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_moe_combine")
     return stream
 
 
-def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
+def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torch.Tensor, down: torch.Tensor, *, gated: bool = False) -> torch.Tensor:
     """The sum :func:`add_expert_outputs` adds, as differentiable framework ops (training, and the CPU path): ``[T, width]`` fp32."""
     T, k = idx.shape
     keep = idx >= 0
     dest, offsets, tile_group, capacity = padded_layout(idx.clamp_min(0).reshape(-1), up.shape[0])
     x_pad = h.new_zeros(capacity, h.shape[1]).index_copy(0, dest, h.repeat_interleave(k, dim=0))
-    a = torch.relu(grouped_linear(x_pad, up.to(h.dtype), tile_group, offsets)).square()
+    a = grouped_linear(x_pad, up.to(h.dtype), tile_group, offsets)
+    if gated:
+        a = gated_activation(a[:, :down.shape[2]], a[:, down.shape[2]:], ActivationFunctionEnum.silu)
+    else:
+        a = torch.relu(a).square()
     y = grouped_linear(a, down.to(h.dtype), tile_group, offsets).index_select(0, dest).view(T, k, -1)
     return (y.float() * (w.float() * keep).unsqueeze(-1)).sum(1)

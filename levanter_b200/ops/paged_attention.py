@@ -12,6 +12,7 @@ from typing import Optional
 import torch
 
 from . import lib
+from .map_difference import MapDifference
 
 INVALID = 2_000_000
 _f = {}
@@ -121,21 +122,44 @@ def kv_page_write_general(kv_pages: torch.Tensor, new_k: torch.Tensor, new_v: to
     flat[dests[sel].long()] = torch.cat([new_k[sel], new_v[sel]], dim=-1).to(kv.dtype)
 
 
+def _gate_args(gate: Optional[torch.Tensor], dtype: torch.dtype, heads: int, v_size: int):
+    """``(gate as the kernels take it, row stride, whether it has one number per head)`` of a gate ``[T, heads * v_size]`` or ``[T, heads]``."""
+    if gate is None:
+        return None, 0, 0
+    assert gate.shape[1] in (heads, heads * v_size)
+    gate = gate if gate.stride(1) == 1 and gate.dtype == dtype else gate.to(dtype).contiguous()
+    return gate, gate.stride(0), int(gate.shape[1] == heads)
+
+
+def _apply_gate(out: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``out [T, heads, v_size]`` times the sigmoid of either form of gate."""
+    return out * torch.sigmoid(gate.float()).view(out.shape[0], out.shape[1], -1)
+
+
+def _difference_args(d: Optional[MapDifference]):
+    return (0, 0.0, 0.0) if d is None else (d.weight.data_ptr(), float(d.scale), float(d.eps))
+
+
 def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: int, v_size: int, batch_info, *, sm_scale: float,
                             chunk: Optional[int] = None, window: Optional[int] = None, gate: Optional[torch.Tensor] = None,
-                            soft_cap: Optional[float] = None) -> torch.Tensor:
+                            soft_cap: Optional[float] = None, difference: Optional[MapDifference] = None) -> torch.Tensor:
     """:func:`ragged_paged_attention` of ``q [T, H, k_size]`` (rows may be strided) over pages of ``kv_heads * (k_size + v_size)``
     elements per slot -> ``[T, H, v_size]``.
 
     ``chunk``: positions are cut into chunks of that many, counted from the start of the sequence, and a query sees the keys of
-    its own chunk only.  ``window``: a query sees itself and the ``window - 1`` positions before it.  ``gate [T, H * v_size]``: the result is multiplied by its sigmoid.  bf16 with sizes that are multiples of 8
-    up to 256 and at most 16 query heads per KV head runs on tensor cores; everything else in fp32 arithmetic."""
-    T, H, dk = q.shape
+    its own chunk only.  ``window``: a query sees itself and the ``window - 1`` positions before it.  ``gate [T, H * v_size]`` or
+    ``[T, H]``: the result is multiplied by its sigmoid.  ``difference``: rows ``2h`` and ``2h + 1`` of ``q`` are the two score maps of head
+    ``h``, a slot holds ``2 * k_size + v_size`` elements per KV head, and the maps' results are combined -> ``[T, H / 2, v_size]``.  bf16
+    with sizes that are multiples of 8 up to 256 (with two maps: the sum of both keys) and at most 16 query rows per KV head runs
+    on tensor cores; everything else in fp32 arithmetic."""
+    T, rows, dk = q.shape
+    maps = 1 if difference is None else 2
+    H = rows // maps
     b = batch_info
     if not _use_kernel(q, kv_pages):
         return paged_attention_general_reference(q, kv_pages, kv_heads, v_size, b, sm_scale=sm_scale, chunk=chunk, window=window, gate=gate,
-                                                 soft_cap=soft_cap)
-    kv = _kv_view(kv_pages, kv_heads, dk, v_size)
+                                                 soft_cap=soft_cap, difference=difference)
+    kv = _kv_view(kv_pages, kv_heads, maps * dk, v_size)
     if kv.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"the cache must be bf16 or fp32, got {kv.dtype}")
     q = q.to(kv.dtype)  # attention runs in the cache's type
@@ -146,30 +170,30 @@ def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: i
     i32 = lambda t: t.to(device=dev, dtype=torch.int32).contiguous()  # noqa: E731
     lens, pages, cu = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens)
     ns = i32(b.num_seqs.reshape(1))
-    q = _strided_rows(q, H * dk)
-    ldg = 0
-    if gate is not None:
-        gate = gate if gate.stride(1) == 1 and gate.dtype == q.dtype else gate.to(q.dtype).contiguous()
-        ldg = gate.stride(0)
+    q = _strided_rows(q, rows * dk)
+    gate, ldg, per_head = _gate_args(gate, q.dtype, H, v_size)
+    diff = _difference_args(difference)
     out = torch.empty(T, H, v_size, dtype=q.dtype, device=dev)
-    tensor_cores = (q.dtype == torch.bfloat16 and dk % 8 == 0 and v_size % 8 == 0 and max(dk, v_size) <= 256 and H // kv_heads <= 16
+    tensor_cores = (q.dtype == torch.bfloat16 and dk % 8 == 0 and v_size % 8 == 0 and max(maps * dk, v_size) <= 256 and rows // kv_heads <= 16
                     and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0)
     if not tensor_cores:
-        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), T, H,
-                       kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), int(window or 0), 0, float(sm_scale),
-                       float(soft_cap or 0.0), int(q.dtype == torch.float32), lib.stream_ptr())
+        scratch = None if difference is None else torch.empty(T * rows * v_size, dtype=torch.float32, device=dev)
+        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), 0, out.data_ptr(),
+                       lib.ptr(scratch), T, rows, kv_heads, dk, v_size, q.stride(0), ldg, per_head, S, PP, ps, P, int(chunk or 0), int(window or 0), 0,
+                       float(sm_scale), float(soft_cap or 0.0), *diff, int(q.dtype == torch.float32), lib.stream_ptr())
         lib.check_rc(rc, "lvb_attention_any")
         return out
     if "g" not in _f:
-        _f["g"] = lib.fn("lvb_paged_attention_general", [c.c_void_p] * 10 + [c.c_int] * 13 + [c.c_float, c.c_float, c.c_void_p], launches=2)
+        _f["g"] = lib.fn("lvb_paged_attention_general", [c.c_void_p] * 10 + [c.c_int] * 14 + [c.c_float, c.c_float, c.c_void_p, c.c_float, c.c_float, c.c_void_p],
+                         launches=2)
         _f["gparts"] = lib.fn("lvb_paged_attention_general_parts", [c.c_int] * 3, launches=0)
     parts = _f["gparts"](PP * ps, int(chunk or 0), int(window or 0))
     po = pml = None
     if parts > 1:
-        po, pml = _part_scratch(dev, T * H * parts * v_size, T * H * parts * 2)
+        po, pml = _part_scratch(dev, T * rows * parts * v_size, T * rows * parts * 2)
     rc = _f["g"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(gate), out.data_ptr(), lib.ptr(po),
-                 lib.ptr(pml), T, H, kv_heads, dk, v_size, q.stride(0), ldg, S, PP, ps, P, int(chunk or 0), int(window or 0),
-                 float(sm_scale), float(soft_cap or 0.0), lib.stream_ptr())
+                 lib.ptr(pml), T, rows, kv_heads, dk, v_size, q.stride(0), ldg, per_head, S, PP, ps, P, int(chunk or 0), int(window or 0),
+                 float(sm_scale), float(soft_cap or 0.0), *diff, lib.stream_ptr())
     lib.check_rc(rc, "lvb_paged_attention_general")
     return out
 
@@ -177,8 +201,8 @@ def paged_attention_general(q: torch.Tensor, kv_pages: torch.Tensor, kv_heads: i
 def _any_fn():
     if "any" not in _f:
         c = lib
-        _f["any"] = lib.fn("lvb_attention_any", [c.c_void_p] * 8 + [c.c_int] * 5 + [c.c_longlong] * 2 + [c.c_int] * 7 +
-                           [c.c_float, c.c_float, c.c_int, c.c_void_p])
+        _f["any"] = lib.fn("lvb_attention_any", [c.c_void_p] * 10 + [c.c_int] * 5 + [c.c_longlong] * 2 + [c.c_int] * 8 +
+                           [c.c_float, c.c_float, c.c_void_p, c.c_float, c.c_float, c.c_int, c.c_void_p])
     return _f["any"]
 
 
@@ -200,15 +224,17 @@ def _part_scratch(dev, n_o: int, n_ml: int):
 
 def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, batch_info, *, sm_scale: float, chunk: Optional[int] = None,
                                       window: Optional[int] = None, gate: Optional[torch.Tensor] = None, soft_cap: Optional[float] = None,
-                                      shared: bool = False) -> torch.Tensor:
-    """PyTorch statement of :func:`paged_attention_general` (CPU path and test oracle).  ``shared``: a KV head's row is its key, whose
-    first ``v_size`` elements are the value."""
+                                      shared: bool = False, difference: Optional[MapDifference] = None,
+                                      sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """PyTorch statement of :func:`paged_attention_general` and, with ``shared``, of :func:`paged_attention_latent` (CPU path and test
+    oracle).  ``shared``: a KV head's row is its key, whose first ``v_size`` elements are the value."""
     T, H, dk = q.shape
+    maps = 1 if difference is None else 2
     b = batch_info
-    kv_all = _kv_view(kv_pages, kv_heads, dk, 0 if shared else v_size)
-    v_at = 0 if shared else dk
+    kv_all = _kv_view(kv_pages, kv_heads, maps * dk, 0 if shared else v_size)
+    v_at = 0 if shared else maps * dk
     ps = kv_all.shape[1]
-    G = H // kv_heads
+    G = H // kv_heads  # query rows per KV head: its query heads, with two maps (head, map)
     out = torch.zeros(T, H, v_size, dtype=torch.float32, device=q.device)
     cu, lens = b.cu_q_lens.tolist(), b.seq_lens.tolist()
     for i in range(int(b.num_seqs)):
@@ -217,7 +243,9 @@ def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, b
             continue
         n = (kl + ps - 1) // ps
         kv = kv_all[b.page_indices[i, :n].long()].reshape(n * ps, kv_heads, -1)[:kl].float()
-        s = torch.einsum("qkgd,skd->kgqs", q[q0:q1].float().view(q1 - q0, kv_heads, G, dk), kv[..., :dk]) * sm_scale
+        keys = kv[..., :maps * dk].unflatten(2, (maps, dk))
+        qi = q[q0:q1].float().view(q1 - q0, kv_heads, G // maps, maps, dk)
+        s = (torch.einsum("qkgmd,skmd->kgmqs", qi, keys) * sm_scale).flatten(1, 2)
         if soft_cap:
             s = torch.tanh(s / soft_cap) * soft_cap
         qpos = torch.arange(q1 - q0, device=q.device) + (kl - (q1 - q0))
@@ -227,23 +255,29 @@ def paged_attention_general_reference(q, kv_pages, kv_heads: int, v_size: int, b
             see = see & (kpos[None, :] // chunk == qpos[:, None] // chunk)
         if window:
             see = see & (qpos[:, None] - kpos[None, :] < window)
-        p = torch.softmax(s.masked_fill(~see, -float("inf")), dim=-1)
+        s = s.masked_fill(~see, -float("inf"))
+        if sink is not None:  # one more column, without a value
+            s = torch.cat([s, sink.float().view(kv_heads, G, 1, 1).expand(kv_heads, G, q1 - q0, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :kl]
         out[q0:q1] = torch.einsum("kgqs,skd->qkgd", p, kv[..., v_at:v_at + v_size]).reshape(q1 - q0, H, v_size)
+    if difference is not None:
+        out = difference(out[:, 0::2], out[:, 1::2])
     if gate is not None:
-        out = out * torch.sigmoid(gate.float()).view(T, H, v_size)
+        out = _apply_gate(out, gate)
     return out.to(q.dtype)
 
 
 # ------------------------------------------------------------------------------------------------ latent form
 def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, batch_info, *, sm_scale: float,
-                           window: Optional[int] = None) -> torch.Tensor:
+                           window: Optional[int] = None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of ``q [T, H, width]`` over pages of ``width`` elements per slot whose first ``rank`` are the value: all heads read
-    the same row per key -> ``[T, H, rank]``.  ``window`` as in :func:`paged_attention_general`.  bf16 with sizes that are multiples of
+    the same row per key -> ``[T, H, rank]``.  ``window`` as in :func:`paged_attention_general`.  ``sink [H]`` (fp32): one number per head
+    that joins the softmax denominator as it is, without a key or a value.  bf16 with sizes that are multiples of
     8 (rank up to 512, width up to 576) runs on tensor cores; everything else in fp32 arithmetic."""
     T, H, w = q.shape
     b = batch_info
     if not _use_kernel(q, kv_pages):
-        return paged_attention_general_reference(q, kv_pages, 1, rank, b, sm_scale=sm_scale, window=window, shared=True)
+        return paged_attention_general_reference(q, kv_pages, 1, rank, b, sm_scale=sm_scale, window=window, shared=True, sink=sink)
     kv = kv_pages.view(kv_pages.shape[0], kv_pages.shape[1], w)
     if kv.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"the cache must be bf16 or fp32, got {kv.dtype}")
@@ -256,18 +290,19 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
     lens, pages, cu, ns = i32(b.seq_lens), i32(b.page_indices), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
     out = torch.empty(T, H, rank, dtype=q.dtype, device=dev)
     if q.dtype != torch.bfloat16 or w % 8 != 0 or rank % 8 != 0 or rank > 512 or w > 576:
-        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), 0, out.data_ptr(), T, H, 1, w, rank,
-                       H * w, 0, S, PP, ps, P, 0, int(window or 0), 1, float(sm_scale), 0.0, int(q.dtype == torch.float32), lib.stream_ptr())
+        rc = _any_fn()(q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), 0, lib.ptr(sink), out.data_ptr(), 0, T, H,
+                       1, w, rank, H * w, 0, 0, S, PP, ps, P, 0, int(window or 0), 1, float(sm_scale), 0.0, 0, 0.0, 0.0, int(q.dtype == torch.float32),
+                       lib.stream_ptr())
         lib.check_rc(rc, "lvb_attention_any")
         return out
     if "l" not in _f:
-        _f["l"] = lib.fn("lvb_paged_latent", [c.c_void_p] * 9 + [c.c_int] * 10 + [c.c_float, c.c_void_p, c.c_void_p], launches=2)
+        _f["l"] = lib.fn("lvb_paged_latent", [c.c_void_p] * 10 + [c.c_int] * 10 + [c.c_float, c.c_void_p, c.c_void_p], launches=2)
         _f["lparts"] = lib.fn("lvb_paged_latent_parts", [c.c_int] * 6, launches=0)
     parts = _f["lparts"](T, H, w, rank, PP * ps, int(window or 0))
     po = pml = None
     if parts > 1:
         po, pml = _part_scratch(dev, T * H * parts * rank, T * H * parts * 2)
-    rc = _f["l"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), out.data_ptr(), lib.ptr(po), lib.ptr(pml), T,
+    rc = _f["l"](q.data_ptr(), kv.data_ptr(), lens.data_ptr(), pages.data_ptr(), cu.data_ptr(), ns.data_ptr(), lib.ptr(sink), out.data_ptr(), lib.ptr(po), lib.ptr(pml), T,
                  H, w, rank, S, PP, ps, P, int(window or 0), parts, float(sm_scale), lib.status_buffer().data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_paged_latent")
     return out

@@ -38,27 +38,28 @@ def mix_values(v: torch.Tensor, v_first: torch.Tensor, mix: torch.Tensor) -> tor
 def prepare_qkv(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kv_pages: torch.Tensor, dests: torch.Tensor, pos: torch.Tensor, *,
                 rot: Optional[RotaryEmbeddings] = None, head_scale: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None,
                 mix: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
-    """``q [T, H, dk]``, ``k [T, KV, dk]``, ``v [T, KV, dv]`` (strided rows; they may be updated in place) -> what attention reads:
+    """``q [T, H, dk]``, ``k [T, KV * n, dk]``, ``v [T, KV, dv]`` (strided rows; they may be updated in place) -> what attention reads:
     ``q`` and ``k`` rotated by ``rot`` at ``pos``, ``q`` times ``head_scale[h]``, ``v`` mixed with ``v_first [T, KV, dv]``.  ``k`` and ``v``
-    are also written to slots ``dests`` of the cache."""
+    are also written to slots ``dests`` of the cache: per KV head its ``n`` keys (one per score map), then its value."""
     T, H, dk = q.shape
     KV, dv = v.shape[1], v.shape[2]
+    maps = k.shape[1] // KV
     dt = q.dtype
     small = [t for t in (head_scale, mix) if t is not None]
     if _kernel(q, k, v, kv_pages) and k.dtype == v.dtype == kv_pages.dtype == dt and all(t.dtype in (torch.bfloat16, torch.float32) for t in small) \
             and len({t.dtype for t in small}) <= 1 and (v_first is None or v_first.dtype == dt):
-        q, k, v = _strided_rows(q, H * dk), _strided_rows(k, KV * dk), _strided_rows(v, KV * dv)
+        q, k, v = _strided_rows(q, H * dk), _strided_rows(k, KV * maps * dk), _strided_rows(v, KV * dv)
         if v_first is not None:
             v_first = _strided_rows(v_first, KV * dv)
         c = lib
         if "q" not in _f:
-            _f["q"] = lib.fn("lvb_qkv_prep", [c.c_void_p] * 9 + [c.c_int] * 5 + [c.c_longlong] * 5 + [c.c_void_p, c.c_int, c.c_int, c.c_float, c.c_float,
+            _f["q"] = lib.fn("lvb_qkv_prep", [c.c_void_p] * 9 + [c.c_int] * 6 + [c.c_longlong] * 5 + [c.c_void_p, c.c_int, c.c_int, c.c_float, c.c_float,
                                                                                                     c.c_int, c.c_int, c.c_void_p])
         d, p = _i32(dests), _i32(pos)
         hs = None if head_scale is None else head_scale.contiguous()
         slots = kv_pages.shape[0] * kv_pages.shape[1]
         rc = _f["q"](q.data_ptr(), k.data_ptr(), v.data_ptr(), lib.ptr(v_first), lib.ptr(mix if v_first is not None else None), lib.ptr(hs),
-                     kv_pages.data_ptr(), p.data_ptr(), d.data_ptr(), T, H, KV, dk, dv, q.stride(0), k.stride(0), v.stride(0),
+                     kv_pages.data_ptr(), p.data_ptr(), d.data_ptr(), T, H, KV, maps, dk, dv, q.stride(0), k.stride(0), v.stride(0),
                      0 if v_first is None else v_first.stride(0), slots, *_rotation_args(rot, q.device), int(dt == torch.float32),
                      int(bool(small) and small[0].dtype == torch.float32), lib.stream_ptr())
         lib.check_rc(rc, "lvb_qkv_prep")
@@ -70,19 +71,20 @@ def prepare_qkv(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kv_pages: tor
         k = rot(k, pos)
     if v_first is not None:
         v = mix_values(v, v_first, mix)
-    kv_page_write_general(kv_pages, k, v, dests)
+    kv_page_write_general(kv_pages, k.reshape(T, KV, maps * dk), v, dests)
     return qf.to(dt), k, v
 
 
 def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_pages: torch.Tensor, dests: torch.Tensor, pos: torch.Tensor,
-                   rot: RotaryEmbeddings, q_rot: torch.Tensor, q_out: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
-    """``down [T, rank + r]``: a compressed row and a key part of ``r`` dimensions shared by the heads.  Returns ``(latent, q_out)``:
+                   rot: Optional[RotaryEmbeddings], q_rot: torch.Tensor, q_out: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``down [T, rank + r]``: a compressed row and a key part of ``r`` dimensions shared by the heads (0, and no ``rot``: there is none).  Returns ``(latent, q_out)``:
     ``latent [T, rank + r]`` is the RMS norm of the former (weight ``norm_weight [rank]``) and the latter rotated at ``pos``, also written
     to slots ``dests`` of the cache; the heads' query parts ``q_rot [T, H, r]`` are rotated into ``q_out`` (None: in place)."""
     T, width = down.shape
     rank, r = norm_weight.shape[0], width - norm_weight.shape[0]
     dt = down.dtype
     dst = q_rot if q_out is None else q_out
+    assert (rot.rotary_dim if rot is not None else 0) == r, "the shared key part is rotated as a whole"
     if _kernel(down, norm_weight, kv_pages, q_rot, dst) and q_rot.dtype == dst.dtype == kv_pages.dtype == dt and down.stride(1) == 1 \
             and norm_weight.dtype in (torch.bfloat16, torch.float32) and q_rot.stride(2) == dst.stride(2) == 1:
         c = lib
@@ -92,7 +94,6 @@ def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv
         latent = torch.empty(T, width, dtype=dt, device=down.device)
         d, p, w = _i32(dests), _i32(pos), norm_weight.contiguous()
         freq, dims, inter, pscale, mag = _rotation_args(rot, down.device)
-        assert dims == r, "the shared key part is rotated as a whole"
         rc = _f["l"](down.data_ptr(), w.data_ptr(), latent.data_ptr(), kv_pages.data_ptr(), q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), d.data_ptr(), T,
                      q_rot.shape[1], rank, r, down.stride(0), q_rot.stride(0), q_rot.stride(1), dst.stride(0), dst.stride(1),
                      kv_pages.shape[0] * kv_pages.shape[1], float(eps), freq, inter, pscale, mag, int(dt == torch.float32), int(w.dtype == torch.float32),
@@ -101,9 +102,10 @@ def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv
         return latent, dst
     x = down[:, :rank].float()
     c = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * norm_weight.float()).to(dt)
-    latent = torch.cat([c, rot(down[:, None, rank:], pos)[:, 0]], dim=1)
+    latent = c if rot is None else torch.cat([c, rot(down[:, None, rank:], pos)[:, 0]], dim=1)
     flat = kv_pages.view(-1, width)
     sel = ((dests >= 0) & (dests < flat.shape[0])).nonzero().squeeze(-1)
     flat[dests[sel].long()] = latent[sel].to(flat.dtype)
-    dst.copy_(rot(q_rot, pos))
+    if rot is not None:
+        dst.copy_(rot(q_rot, pos))
     return latent, dst

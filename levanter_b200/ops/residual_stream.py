@@ -42,15 +42,17 @@ def embed_stream(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch
 
 
 def rms_norm_stream(x: torch.Tensor, weight: torch.Tensor, eps: float, *, w_offset: float = 0.0, out_dtype: Optional[torch.dtype] = None,
-                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """RMS norm of the fp32 stream in ``out_dtype`` (default: the weight's dtype).  ``rows``: normalise these rows only."""
+                    rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm of the fp32 stream in ``out_dtype`` (default: the weight's dtype).  ``rows``: normalise these rows only.  ``add [D]``: a
+    vector that joins every row of the stream first, in place (serving only)."""
     dt = out_dtype or weight.dtype
-    if _kernels(x, weight) and x.dtype == torch.float32 and dt in (torch.float32, torch.bfloat16) and weight.dtype in (torch.float32, torch.bfloat16) \
+    if add is not None:
+        assert rows is None and x.is_contiguous() and not torch.is_grad_enabled()
+    if _kernels(x, weight) and (add is None or (add.is_contiguous() and add.dtype == weight.dtype)) and x.dtype == torch.float32 and dt in (torch.float32, torch.bfloat16) and weight.dtype in (torch.float32, torch.bfloat16) \
             and weight.is_contiguous():
         c = lib
         if "n" not in _f:
-            _f["n"] = lib.fn("lvb_rms_stream", [c.c_void_p, c.c_void_p, c.c_void_p, c.c_int, c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_float,
-                                                c.c_float, c.c_void_p])
+            _f["n"] = lib.fn("lvb_rms_stream", [c.c_void_p] * 4 + [c.c_int, c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_float, c.c_float, c.c_void_p])
         D = x.shape[-1]
         x2 = x.reshape(-1, D)
         x2 = x2 if x2.is_contiguous() else x2.contiguous()
@@ -58,10 +60,12 @@ def rms_norm_stream(x: torch.Tensor, weight: torch.Tensor, eps: float, *, w_offs
             rows = rows.to(torch.int64).contiguous()
         n = x2.shape[0] if rows is None else rows.numel()
         y = torch.empty(n, D, dtype=dt, device=x.device)
-        rc = _f["n"](x2.data_ptr(), lib.ptr(rows), weight.data_ptr(), int(weight.dtype == torch.float32), y.data_ptr(), int(dt == torch.float32), n, D,
+        rc = _f["n"](x2.data_ptr(), lib.ptr(rows), lib.ptr(add), weight.data_ptr(), int(weight.dtype == torch.float32), y.data_ptr(), int(dt == torch.float32), n, D,
                      float(eps), float(w_offset), lib.stream_ptr())
         lib.check_rc(rc, "lvb_rms_stream")
         return y.view(*x.shape[:-1], D) if rows is None else y
+    if add is not None:
+        x.add_(add.float())
     if rows is not None:
         x = x.index_select(0, rows.long())
     xf = x.float()
@@ -94,20 +98,31 @@ def add_norm_stream(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_ne
     return rms_norm_stream(x, w_next, eps)
 
 
-def glu_of_rows(y: torch.Tensor, cols: int, act: ActivationFunctionEnum) -> torch.Tensor:
-    """``act(y[:, :cols]) * y[:, cols:]`` of the joint product of a gate and an up projection."""
-    gate, up = y[:, :cols], y[:, cols:]
-    if act == ActivationFunctionEnum.gelu_new and _kernels(y) and not (y.dtype == torch.bfloat16 and cols % 8 == 0) \
-            and y.dtype in (torch.float32, torch.bfloat16):
+_GLU_ANY = {ActivationFunctionEnum.gelu_new: 0, ActivationFunctionEnum.silu: 1, ActivationFunctionEnum.swish: 1}
+
+
+def glu_of_rows(y: torch.Tensor, cols: int, act: ActivationFunctionEnum, *, gate_logit: Optional[torch.Tensor] = None,
+                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``act(y[:, :cols]) * y[:, cols:2 * cols]`` of the joint product of a gate and an up projection, in ``out_dtype`` (default: ``y``'s).
+    ``gate_logit [rows]``: every row is also multiplied by the sigmoid of its number."""
+    gate, up = y[:, :cols], y[:, cols:2 * cols]
+    dt = out_dtype or y.dtype
+    plain = gate_logit is None and dt == y.dtype
+    if act in _GLU_ANY and _kernels(y) and not (plain and y.dtype == torch.bfloat16 and cols % 8 == 0) \
+            and y.dtype in (torch.float32, torch.bfloat16) and dt in (y.dtype, torch.bfloat16) and y.stride(1) == 1 \
+            and (gate_logit is None or gate_logit.dtype == torch.float32):
         c = lib
         if "g" not in _f:
-            _f["g"] = lib.fn("lvb_gelu_glu_any", [c.c_void_p] * 3 + [c.c_int] * 3 + [c.c_longlong] * 2 + [c.c_void_p])
-        out = torch.empty(y.shape[0], cols, dtype=y.dtype, device=y.device)
-        rc = _f["g"](gate.data_ptr(), up.data_ptr(), out.data_ptr(), int(y.dtype == torch.float32), y.shape[0], cols, y.stride(0), y.stride(0),
-                     lib.stream_ptr())
-        lib.check_rc(rc, "lvb_gelu_glu_any")
+            _f["g"] = lib.fn("lvb_glu_any", [c.c_void_p] * 4 + [c.c_int] * 5 + [c.c_longlong] * 3 + [c.c_void_p])
+        out = torch.empty(y.shape[0], cols, dtype=dt, device=y.device)
+        rc = _f["g"](gate.data_ptr(), up.data_ptr(), lib.ptr(gate_logit), out.data_ptr(), _GLU_ANY[act], int(y.dtype == torch.float32),
+                     int(dt == torch.float32), y.shape[0], cols, y.stride(0), y.stride(0), 0 if gate_logit is None else gate_logit.stride(0), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_glu_any")
         return out
-    return gated_activation(gate, up, act)
+    out = gated_activation(gate, up, act)
+    if gate_logit is not None:
+        out = out * torch.sigmoid(gate_logit.float())[:, None]
+    return out.to(dt)
 
 
 def _gemm_ok(h: torch.Tensor, w: torch.Tensor) -> bool:
