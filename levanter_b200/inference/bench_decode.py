@@ -35,6 +35,13 @@ MODELS = {
     "tiny_zadepel": dict(family="zadepel", hidden_dim=256, num_layers=4, intermediate_dim=512, vocab=1024,
                          attention=dict(num_heads=4, num_kv_heads=2, head_dim=64, v_head_dim=64, attention_scale=0.125, rotary_dim=32), mingru=dict(width=320),
                          latent=dict(num_heads=4, head_dim=32, rotary_dim=16, v_head_dim=48, kv_lora_rank=64, attention_scale=0.15, sliding_window=96)),
+    # Zosipel beside fedolorn_moe: the same width, vocabulary, layer runs and expert weights (three matrices of 1024 instead of two of 1536), a
+    # shared expert, four of twelve layers run twice; of four layers one is differential attention in a window, three are latent attention
+    "zosipel_moe": dict(family="zosipel", hidden_dim=4096, num_layers=12, intermediate_dim=1024, vocab=128256, shared=2048, loop=(4, 8, 2)),
+    "tiny_zosipel": dict(family="zosipel", hidden_dim=256, num_layers=4, intermediate_dim=64, vocab=1024, shared=96, loop=(1, 3, 2),
+                         attention=dict(num_heads=4, num_kv_heads=2, head_dim=32, v_head_dim=64, attention_scale=0.18, sliding_window=96, soft_cap=20.0),
+                         latent=dict(num_heads=4, head_dim=48, v_head_dim=32, kv_lora_rank=64, attention_scale=0.15),
+                         moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=4, expert_groups_kept=2)),
     "tiny": dict(hidden_dim=256, intermediate_dim=512, num_layers=2, num_heads=4, num_kv_heads=2, vocab=1024),
 }
 
@@ -57,6 +64,20 @@ def model_config(m: dict, seq_len: int):
                  ZadepelLayerConfig(mixer="mingru", intermediate_dim=ff, **m.get("mingru", dict(width=4096))), latent]
         return ZadepelConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], gradient_checkpointing=False,
                              layers=tuple(group[i % 4] for i in range(m["num_layers"])))
+    if family == "zosipel":
+        from ..layers.rotary import PartialYarnRotaryEmbeddingsConfig
+        from ..models.zosipel import ZosipelConfig, ZosipelLayerConfig
+
+        moe = dict(intermediate_dim=m["intermediate_dim"], shared_intermediate_dim=m["shared"],
+                   **m.get("moe", dict(num_experts=64, num_experts_per_tok=8, expert_groups=8, expert_groups_kept=4)))
+        rope = PartialYarnRotaryEmbeddingsConfig(theta=500000.0, factor=4.0, original_max_position_embeddings=2048)
+        attn = dict(num_heads=32, num_kv_heads=8, head_dim=64, v_head_dim=128, attention_scale=0.125, sliding_window=1024, soft_cap=30.0)
+        latent = dict(num_heads=32, head_dim=128, v_head_dim=128, kv_lora_rank=512, attention_scale=128 ** -0.5)
+        layers = {False: ZosipelLayerConfig(mixer="latent_attention", rope=None, **m.get("latent", latent), **moe),
+                  True: ZosipelLayerConfig(mixer="attention", rope=rope, difference=0.5, **m.get("attention", attn), **moe)}
+        start, stop, times = m["loop"] if m["num_layers"] >= m["loop"][1] else (0, 0, 0)
+        return ZosipelConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], gradient_checkpointing=False, loop_start=start, loop_stop=stop, loop_times=times,
+                             layers=tuple(layers[i % 4 == 2] for i in range(m["num_layers"])))
     from ..models.fedolorn import FedolornConfig, FedolornLayerConfig
 
     layer = FedolornLayerConfig(intermediate_dim=m["intermediate_dim"], **m.get("heads", {}), **m.get("moe", {}))

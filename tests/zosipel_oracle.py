@@ -11,7 +11,7 @@ def rms(x, eps):
 
 
 def offset_rms_norm(x, w, eps):
-    """The weight is stored around zero."""
+    """``w`` is the offset of the weight from one."""
     return rms(x, eps) * (1.0 + w)
 
 
