@@ -884,7 +884,7 @@ class MultiHeadLatentAttention(nn.Module):
         else:
             uk, uv = self.up_projections(weight)
             qa = q.new_empty(T, H, rank + dr)
-            prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:], qa[..., rank:])
+            prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:], qa[..., rank:], to_cache_only=True)
             PA.head_product(q[..., :dn], uk.to(q.dtype), qa[..., :rank], b_trans=False)
             o = PA.paged_attention_latent(qa, pages, rank, batch_info, sm_scale=c.softmax_scale, window=c.sliding_window, sink=sink)
             heads = PA.head_product(o.to(q.dtype), uv.to(q.dtype), q.new_empty(T, H, dv), b_trans=True)

@@ -454,8 +454,8 @@ inline int make_tmap_heads_bf16(CUtensorMap* out, const void* ptr, uint64_t rows
 }
 
 // Dense row-major bf16 [rows, cols], cols a multiple of 64, as [rows, cols / 64, 64]; box = box_rows whole rows, each cols / 64 lines of 128
-// bytes in shared memory, 128-byte swizzle.
-inline int make_tmap_chunked_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows) {
+// bytes in shared memory, 128-byte swizzle.  chunk_major: as [cols / 64, rows, 64], so that a box holds the lines of a chunk side by side.
+inline int make_tmap_chunked_bf16(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, bool chunk_major = false) {
   ensure_context_for(ptr);
   EncodeTiledFn enc = get_encode_tiled();
   if (enc == nullptr) return kErrTensorMap;
@@ -463,6 +463,11 @@ inline int make_tmap_chunked_bf16(CUtensorMap* out, const void* ptr, uint64_t ro
   cuuint64_t gdim[3] = {64, cols / 64, rows};
   cuuint64_t gstr[2] = {128, cols * 2};
   cuuint32_t box[3] = {64, static_cast<cuuint32_t>(cols / 64), box_rows};
+  if (chunk_major) {
+    gdim[1] = rows; gdim[2] = cols / 64;
+    gstr[0] = cols * 2; gstr[1] = 128;
+    box[1] = box_rows; box[2] = static_cast<cuuint32_t>(cols / 64);
+  }
   cuuint32_t estr[3] = {1, 1, 1};
   CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), gdim, gstr, box, estr,
                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

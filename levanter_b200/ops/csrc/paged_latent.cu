@@ -61,7 +61,8 @@ struct Params {
   int* status;
   int box;   // rows of a TMA box: a power of two that divides the page size and 64
   int box_log;
-  int whole; // a box holds whole rows [box][chunks][128 bytes]; else one chunk of them [box][128 bytes]
+  int whole; // a box holds whole rows [box][chunks][128 bytes]; else all their chunks [chunks][box][128 bytes] (grouped) or one [box][128 bytes]
+  int grouped;
 };
 
 __device__ __forceinline__ bool locate(const Params& p, int t, int& seq, int& ctx) {
@@ -159,7 +160,7 @@ __global__ void __launch_bounds__(cta_threads(kM, kPieces), 1) paged_latent_kern
   __syncthreads();
 
   // ---- copies: a lane per box
-  const int per_group = p.whole ? 1 : chunks, boxes = kTileKeys / p.box * per_group, boxb = p.box * 128 * (p.whole ? chunks : 1);
+  const int per_group = p.whole || p.grouped ? 1 : chunks, boxes = kTileKeys / p.box * per_group, boxb = p.box * 128 * (chunks / per_group);
   auto lookup = [&](int tile, int i) -> int {  // cache row of box i; past the last key any rows will do, they are masked
     const int key = k0 + tile * kTileKeys + i / per_group * p.box;
     if (i >= boxes || key >= ctx) return 0;
@@ -174,6 +175,7 @@ __global__ void __launch_bounds__(cta_threads(kM, kPieces), 1) paged_latent_kern
       const int row = i == lane ? row_first : lookup(tile, i);
       uint8_t* dst = s_k + stage * stageb + i * boxb;
       if (p.whole) tma_load_3d(dst, &tm, &full[stage], 0, 0, row);
+      else if (p.grouped) tma_load_3d(dst, &tm, &full[stage], 0, row, 0);
       else tma_load_2d(dst, &tm, &full[stage], i % chunks * 64, row);
     }
   };
@@ -611,8 +613,10 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
   CUtensorMap tm;
   // rows of an odd number of chunks are free of bank conflicts as they are; else the chunks are kept apart
   p.whole = (width & 63) == 0 && (chunks_of(width) & 1) != 0;
+  p.grouped = (width & 63) == 0 && !p.whole;
   const uint64_t rows = static_cast<uint64_t>(num_pages) * page_size;
-  const int rc = p.whole ? make_tmap_chunked_bf16(&tm, kv_pages, rows, width, p.box) : make_tmap_2d_bf16(&tm, kv_pages, rows, width, width, p.box, 64);
+  const int rc = p.whole || p.grouped ? make_tmap_chunked_bf16(&tm, kv_pages, rows, width, p.box, p.grouped != 0)
+                                      : make_tmap_2d_bf16(&tm, kv_pages, rows, width, width, p.box, 64);
   if (rc != kErrOk) return rc;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool narrow = rank <= 256;

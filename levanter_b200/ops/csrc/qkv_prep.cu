@@ -233,7 +233,7 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(LatentParams p) {
   float* s_cos = s_angles;
   float* s_sin = s_angles + p.rot.dims / 2;
   const int t = blockIdx.x;
-  if (p.rotd > 0) fill_angles(p.rot, p.pos[t], s_cos, s_sin);
+  fill_angles(p.rot, p.pos[t], s_cos, s_sin);
   const long long dest = p.dests[t];
   const int width = p.rank + p.rotd;
   T* cache = dest >= 0 && dest < p.slots ? reinterpret_cast<T*>(p.kv_pages) + dest * width : nullptr;
@@ -279,11 +279,63 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(LatentParams p) {
       if (cache != nullptr) cache[c] = a;
     }
   }
-  if (p.rotd == 0) return;
   rotate_heads<T>(down + p.rank, 0, latent + p.rank, 0, cache != nullptr ? cache + p.rank : nullptr, 0, 1, 1, p.rotd, p.rot, s_cos, s_sin, nullptr, 0,
                   p.vec_c != 0 && p.vec_q != 0);
   rotate_heads<T>(reinterpret_cast<const T*>(p.q_rot) + t * p.ldq, p.q_head, reinterpret_cast<T*>(p.q_out) + t * p.ldo, p.o_head,
                   static_cast<T*>(nullptr), 0, 1, p.H, p.rotd, p.rot, s_cos, s_sin, nullptr, 0, p.vec_q != 0);
+}
+
+// latent_prep without a rotated part: the norm and the cache write, a warp per row, the row in registers.  latent may be null.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) latent_norm_kernel(LatentParams p, int rows) {
+  constexpr int kKeep = 4;  // groups of 8 columns per lane in registers
+  const int t = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= rows) return;
+  const long long dest = p.dests[t];
+  T* cache = dest >= 0 && dest < p.slots ? reinterpret_cast<T*>(p.kv_pages) + dest * p.rank : nullptr;
+  const T* down = reinterpret_cast<const T*>(p.down) + t * p.ldd;
+  T* latent = p.latent != nullptr ? reinterpret_cast<T*>(p.latent) + static_cast<long long>(t) * p.rank : nullptr;
+  auto weight = [&](int c) -> float {
+    return p.w_f32 ? reinterpret_cast<const float*>(p.norm_w)[c] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.norm_w)[c]);
+  };
+  auto scale = [&](float ss) { return 1.f / sqrtf(warp_sum(ss) / static_cast<float>(p.rank) + p.eps); };
+  float ss = 0.f;
+  if (p.vec_c && p.rank <= kKeep * 256) {
+    float a[kKeep][8];
+#pragma unroll
+    for (int n = 0; n < kKeep; ++n) {
+      const int c = n * 256 + lane * 8;
+      if (c < p.rank) Vec8<T>::load(down + c, a[n]);
+      else
+#pragma unroll
+        for (int j = 0; j < 8; ++j) a[n][j] = 0.f;
+    }
+#pragma unroll
+    for (int n = 0; n < kKeep; ++n)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(a[n][j], a[n][j], ss);
+    const float r = scale(ss);
+#pragma unroll
+    for (int n = 0; n < kKeep; ++n) {
+      const int c = n * 256 + lane * 8;
+      if (c >= p.rank) continue;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[n][j] *= r * weight(c + j);
+      if (latent != nullptr) Vec8<T>::store(latent + c, a[n]);
+      if (cache != nullptr) Vec8<T>::store(cache + c, a[n]);
+    }
+    return;
+  }
+  for (int c = lane; c < p.rank; c += 32) {
+    const float a = to_f<T>(down[c]);
+    ss = fmaf(a, a, ss);
+  }
+  const float r = scale(ss);
+  for (int c = lane; c < p.rank; c += 32) {
+    const T a = from_f<T>(to_f<T>(down[c]) * (r * weight(c)));
+    if (latent != nullptr) latent[c] = a;
+    if (cache != nullptr) cache[c] = a;
+  }
 }
 
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
@@ -330,7 +382,7 @@ extern "C" int lvb_qkv_prep(void* q, void* k, void* v, const void* v_first, cons
 // Latent attention.  Row t of down (stride ldd) holds `rank` compressed dimensions and a key part of rot_dims dimensions shared by the
 // heads.  latent[t] = [RMS norm of the former with weight norm_w, the latter rotated], also written to slot dests[t] of kv_pages [slots,
 // rank + rot_dims]; head h's rotated query part goes from q_rot + t * ldq + h * q_head to q_out + t * ldo + h * o_head.  rot_dims 0: the norm and
-// the cache write only.
+// the cache write only; latent may be null then.
 extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* latent, void* kv_pages, const void* q_rot, void* q_out, const int* pos,
                                const int* dests, int T, int H, int rank, int rot_dims, long long ldd, long long ldq, long long q_head,
                                long long ldo, long long o_head, long long slots, float eps, const float* inv_freq, int interleaved,
@@ -339,7 +391,7 @@ extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* laten
   using namespace lvb::prep;
   if (T <= 0) return kErrOk;
   if (H <= 0 || rank <= 0 || rot_dims < 0 || (rot_dims & 1)) return kErrBadArg;
-  if (rot_dims > 0 && (inv_freq == nullptr || pos == nullptr)) return kErrBadArg;
+  if (rot_dims > 0 && (inv_freq == nullptr || pos == nullptr || latent == nullptr)) return kErrBadArg;
   if (rot_dims > 4096) return kErrTooLarge;
   LatentParams p;
   p.down = down; p.norm_w = norm_w; p.latent = latent; p.kv_pages = kv_pages; p.q_rot = q_rot; p.q_out = q_out; p.pos = pos; p.dests = dests;
@@ -351,7 +403,11 @@ extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* laten
   p.vec_q = ((rot_dims | ldq | q_head | ldo | o_head) & 7) == 0 && aligned16(q_rot) && aligned16(q_out) && groups_of_8(inv_freq, rot_dims, interleaved);
   const size_t smem = static_cast<size_t>(rot_dims) * 4;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (is_f32) latent_prep_kernel<float><<<T, kThreads, smem, s>>>(p);
+  if (rot_dims == 0) {
+    const int per = kThreads / 32;
+    if (is_f32) latent_norm_kernel<float><<<(T + per - 1) / per, kThreads, 0, s>>>(p, T);
+    else latent_norm_kernel<__nv_bfloat16><<<(T + per - 1) / per, kThreads, 0, s>>>(p, T);
+  } else if (is_f32) latent_prep_kernel<float><<<T, kThreads, smem, s>>>(p);
   else latent_prep_kernel<__nv_bfloat16><<<T, kThreads, smem, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }

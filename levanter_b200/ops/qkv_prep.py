@@ -76,10 +76,12 @@ def prepare_qkv(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kv_pages: tor
 
 
 def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_pages: torch.Tensor, dests: torch.Tensor, pos: torch.Tensor,
-                   rot: Optional[RotaryEmbeddings], q_rot: torch.Tensor, q_out: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+                   rot: Optional[RotaryEmbeddings], q_rot: torch.Tensor, q_out: Optional[torch.Tensor] = None,
+                   to_cache_only: bool = False) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
     """``down [T, rank + r]``: a compressed row and a key part of ``r`` dimensions shared by the heads (0, and no ``rot``: there is none).  Returns ``(latent, q_out)``:
     ``latent [T, rank + r]`` is the RMS norm of the former (weight ``norm_weight [rank]``) and the latter rotated at ``pos``, also written
-    to slots ``dests`` of the cache; the heads' query parts ``q_rot [T, H, r]`` are rotated into ``q_out`` (None: in place)."""
+    to slots ``dests`` of the cache; the heads' query parts ``q_rot [T, H, r]`` are rotated into ``q_out`` (None: in place).
+    ``to_cache_only``: the caller does not read ``latent``, which may come back as None."""
     T, width = down.shape
     rank, r = norm_weight.shape[0], width - norm_weight.shape[0]
     dt = down.dtype
@@ -91,10 +93,10 @@ def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv
         if "l" not in _f:
             _f["l"] = lib.fn("lvb_latent_prep", [c.c_void_p] * 8 + [c.c_int] * 4 + [c.c_longlong] * 6 + [c.c_float, c.c_void_p, c.c_int, c.c_float, c.c_float,
                                                                                                        c.c_int, c.c_int, c.c_void_p])
-        latent = torch.empty(T, width, dtype=dt, device=down.device)
+        latent = None if to_cache_only and rot is None else torch.empty(T, width, dtype=dt, device=down.device)
         d, p, w = _i32(dests), _i32(pos), norm_weight.contiguous()
         freq, dims, inter, pscale, mag = _rotation_args(rot, down.device)
-        rc = _f["l"](down.data_ptr(), w.data_ptr(), latent.data_ptr(), kv_pages.data_ptr(), q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), d.data_ptr(), T,
+        rc = _f["l"](down.data_ptr(), w.data_ptr(), lib.ptr(latent), kv_pages.data_ptr(), q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), d.data_ptr(), T,
                      q_rot.shape[1], rank, r, down.stride(0), q_rot.stride(0), q_rot.stride(1), dst.stride(0), dst.stride(1),
                      kv_pages.shape[0] * kv_pages.shape[1], float(eps), freq, inter, pscale, mag, int(dt == torch.float32), int(w.dtype == torch.float32),
                      lib.stream_ptr())

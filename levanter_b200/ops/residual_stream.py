@@ -107,8 +107,8 @@ def glu_of_rows(y: torch.Tensor, cols: int, act: ActivationFunctionEnum, *, gate
     ``gate_logit [rows]``: every row is also multiplied by the sigmoid of its number."""
     gate, up = y[:, :cols], y[:, cols:2 * cols]
     dt = out_dtype or y.dtype
-    plain = gate_logit is None and dt == y.dtype
-    if act in _GLU_ANY and _kernels(y) and not (plain and y.dtype == torch.bfloat16 and cols % 8 == 0) \
+    plain = gate_logit is None and dt == y.dtype == torch.bfloat16 and cols % 8 == 0 and y.stride(0) % 8 == 0 and y.data_ptr() % 16 == 0
+    if act in _GLU_ANY and _kernels(y) and not plain \
             and y.dtype in (torch.float32, torch.bfloat16) and dt in (y.dtype, torch.bfloat16) and y.stride(1) == 1 \
             and (gate_logit is None or gate_logit.dtype == torch.float32):
         c = lib

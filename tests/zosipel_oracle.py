@@ -196,3 +196,46 @@ def logits(cfg, weights, tokens, dtype=torch.float64, streams=None):
         if streams is not None:
             streams.append(x)
     return offset_rms_norm(x, W["final.norm"], cfg["norm"]["eps"]) @ W["head"].T
+
+
+def random_weights(cfg, seed=0, dtype=torch.bfloat16):
+    """Small random weights under the checkpoint's names, for tests."""
+    gen = torch.Generator().manual_seed(seed)
+    E = cfg["width"]
+
+    def mat(o, i, s=1.0):
+        return (torch.randn(o, i, generator=gen) * (s / i ** 0.5)).to(dtype)
+
+    def vec(n, s, mean=0.0):
+        return (torch.randn(n, generator=gen) * s + mean).to(dtype)
+
+    def gated(pre, ff):
+        W[pre + "gate"], W[pre + "up"], W[pre + "down"] = mat(ff, E), mat(ff, E), mat(E, ff, 0.6)
+
+    W = {"embed": mat(cfg["vocab"], E, E ** 0.5), "head": mat(cfg["vocab"], E), "final.norm": vec(E, 0.2)}
+    if cfg.get("loop"):
+        W["loop.step"] = mat(cfg["loop"]["times"], E, E ** 0.5)
+    for i, L in enumerate(cfg["layers"]):
+        p, m, f = "l%d." % i, L["mixer"], L["mlp"]
+        for n in ("norm1",) + (() if f is None else ("norm2",)):
+            W[p + n] = vec(E, 0.2)
+        x = p + "mix."
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            for n, rows in (("q", 2 * H * d), ("k", 2 * m["kv_heads"] * d), ("v", m["kv_heads"] * dv)):
+                W[x + n], W[x + n + ".b"] = mat(rows, E, 1.5), vec(rows, 0.3)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                W[x + n] = vec(d, 0.4)
+            W[x + "g"], W[x + "o"] = mat(H, E, 2.0), mat(E, H * dv, 2.0)
+        else:
+            r = m["kv_rank"]
+            W[x + "q"], W[x + "dkv"], W[x + "dkv.norm"] = mat(H * d, E, 1.5), mat(r, E, 1.5), vec(r, 0.2, 1.0)
+            W[x + "uk"], W[x + "uv"], W[x + "sink"], W[x + "o"] = mat(H * d, r, 1.5), mat(H * dv, r, 1.5), vec(H, 1.0, 1.0), mat(E, H * dv, 1.5)
+        if f is not None:
+            W[p + "mlp.router"] = mat(f["router"]["experts"], E, 5.0)  # sharp scores: what a close call swaps weighs little
+            for j in range(f["router"]["experts"]):
+                gated(p + "mlp.e%d." % j, f["expert"]["ff"])
+            if f.get("shared"):
+                gated(p + "mlp.shared.", f["shared"]["ff"])
+                W[p + "mlp.shared.sg"] = mat(1, E, 2.0)
+    return W
