@@ -25,8 +25,6 @@ def attention(tb: Table, T=8192, n_seq=4, H=32, KV=8, S=64, ctx=4096):
     diff = _difference()
     L = T // n_seq
     pos = (torch.arange(T, device="cuda") % L).int()
-    ql, kl, vl = (_randn(T, h, 128) for h in (H, KV, KV))
-    klh, vlh = _randn(T, H, 128), _randn(T, H, 128)
 
     def seen(window):
         w = min(window or L, L)
@@ -36,12 +34,14 @@ def attention(tb: Table, T=8192, n_seq=4, H=32, KV=8, S=64, ctx=4096):
         y = _randn(T, 2 * H * dk + KV * (2 * dk + dv) + H)
         q, k = y[:, :2 * H * dk].unflatten(1, (2 * H, dk)), y[:, 2 * H * dk:2 * (H + KV) * dk].unflatten(1, (2 * KV, dk))
         v, gate = y[:, 2 * (H + KV) * dk:-H].unflatten(1, (KV, dv)), y[:, -H:]
-        like = lambda: FA.flash_attention_packed(ql, kl, vl, pos, scaling_factor=128 ** -0.5, window=window, logits_soft_cap=cap)  # noqa: E731
+        d = 64 if max(2 * dk, dv) <= 64 else 128
+        ql, kl, vl = (_randn(T, h, d) for h in (H, KV, KV))
         tb.pair(f"prefill differential 2x{dk}/{dv}, window {window or 'none'}, cap {cap or 'none'}, gated",
                 lambda: FA.flash_attention_packed(q, k, v, pos, scaling_factor=dk ** -0.5, window=window, gate=gate, logits_soft_cap=cap, difference=diff),
-                f"Fedolorn prefill attention 128/128, window {window or 'none'}, cap {cap or 'none'}", like,
+                f"Fedolorn prefill attention {d}/{d}, window {window or 'none'}, cap {cap or 'none'}",
+                lambda: FA.flash_attention_packed(ql, kl, vl, pos, scaling_factor=d ** -0.5, window=window, logits_soft_cap=cap),
                 flops=4.0 * H * (dk + dv) * seen(window), nbytes=2.0 * (y.numel() + T * H * dv),
-                like_flops=4.0 * H * 128 * seen(window), like_bytes=4.0 * T * (H + KV) * 128)
+                like_flops=4.0 * H * d * seen(window), like_bytes=4.0 * T * (H + KV) * d)
     sink = _randn(H, dtype=F32)
     for dk, dv in ((128, 128), (64, 64)):
         y = _randn(T, H * (2 * dk + dv))
@@ -75,6 +75,7 @@ def attention(tb: Table, T=8192, n_seq=4, H=32, KV=8, S=64, ctx=4096):
 
 def around_attention(tb: Table, H=32, KV=8, D=64, Dv=128, rank=512, E=4096):
     from ..layers.rotary import DefaultRotaryEmbeddingsConfig, PartialYarnRotaryEmbeddingsConfig
+    from ..ops.norm import rms_norm
     from ..ops.qkv_prep import prepare_latent, prepare_qkv
     from ..ops.residual_stream import project, rms_norm_stream
 
@@ -100,8 +101,12 @@ def around_attention(tb: Table, H=32, KV=8, D=64, Dv=128, rank=512, E=4096):
         yl = _randn(T, H * 192 + rank + 64)
         down, downz, qr = yl[:, H * 192:H * 192 + rank], yl[:, H * 192:], yl[:, :H * 192].unflatten(1, (H, 192))[..., 128:]
         pl, plz = _randn(T // 16 + 1, 16, 1, rank), _randn(T // 16 + 1, 16, 1, rank + 64)
-        tb.pair(f"T={T}: latent norm, cache write", lambda: prepare_latent(down, wn, 1e-6, pl, dest, pos, None, qr), "Zadepel latent norm, rotations, cache write",
+        xr = down.contiguous()
+        new = lambda: prepare_latent(down, wn, 1e-6, pl, dest, pos, None, qr)  # noqa: E731
+        tb.pair(f"T={T}: latent norm, cache write", new, "Zadepel latent norm, rotations, cache write",
                 lambda: prepare_latent(downz, wn, 1e-6, plz, dest, pos, roti, qr), nbytes=6.0 * T * rank, like_bytes=2.0 * T * (3 * (rank + 64) + 2 * H * 64))
+        tb.pair(f"T={T}: latent norm, cache write (again)", new, f"Llama RMS norm of {rank}", lambda: rms_norm(xr, wn), nbytes=6.0 * T * rank,
+                like_bytes=4.0 * T * rank)
         x, h = _randn(T, E, dtype=F32), _randn(T, E)
         tb.pair(f"T={T}: add a vector to the stream, RMS norm", lambda: rms_norm_stream(x, wx, 1e-6, w_offset=1.0, add=add), "Fedolorn RMS norm",
                 lambda: rms_norm_stream(x, wx, 1e-6, w_offset=1.0), nbytes=10.0 * T * E, like_bytes=6.0 * T * E)

@@ -335,6 +335,15 @@ __device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r
       "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
       : "memory");
 }
+__device__ __forceinline__ void tmem_ld_32x16(uint32_t taddr, uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+        "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr)
+      : "memory");
+}
 __device__ __forceinline__ void tmem_ld_wait() {
   asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
@@ -360,6 +369,39 @@ __device__ __forceinline__ float warp_max(float v) {
 // cap * tanh(x / cap) with an absolute error of a few 1e-7 of cap, also in files built with fast-math (whose tanhf keeps about 11 bits)
 __device__ __forceinline__ float soft_capped(float x, float cap) {
   return cap - __fdividef(2.f * cap, 1.f + exp2f(x * __fdividef(2.885390081777927f, cap)));
+}
+// Two fp32 numbers in a register pair, for the two-wide arithmetic instructions
+struct F32x2 {
+  unsigned long long v;
+};
+__device__ __forceinline__ F32x2 f2(float a, float b) {
+  F32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void f2_split(F32x2 x, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(x.v)); }
+__device__ __forceinline__ F32x2 f2_fma(F32x2 a, F32x2 b, F32x2 c) {
+  F32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return r;
+}
+__device__ __forceinline__ F32x2 f2_mul(F32x2 a, F32x2 b) {
+  F32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+__device__ __forceinline__ F32x2 f2_add(F32x2 a, F32x2 b) {
+  F32x2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+// tanh(x) / x as a polynomial of u = x^2 for |x| <= 0.75, interpolated at the Chebyshev nodes of [0, 0.5625]; relative error 3e-8
+__device__ __forceinline__ F32x2 tanh_ratio(F32x2 u) {
+  F32x2 p = f2_fma(f2(-0.0047115222f, -0.0047115222f), u, f2(0.0195762164f, 0.0195762164f));
+  p = f2_fma(p, u, f2(-0.0533411153f, -0.0533411153f));
+  p = f2_fma(p, u, f2(0.1332533885f, 0.1332533885f));
+  p = f2_fma(p, u, f2(-0.3333295410f, -0.3333295410f));
+  return f2_fma(p, u, f2(0.9999999705f, 0.9999999705f));
 }
 // Named barrier among `count` threads (count multiple of 32), id in [1, 15].
 __device__ __forceinline__ void named_bar_sync(int id, int count) {

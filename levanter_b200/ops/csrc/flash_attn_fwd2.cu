@@ -76,6 +76,11 @@ struct SmemT {
   static constexpr int kTotal = kBars + kNumBars * 8 + 16 + 1024;
 };
 
+template <bool kValue>
+struct Yes {  // a compile-time answer as an argument
+  static constexpr bool value = kValue;
+};
+
 template <bool kCap>
 __device__ __forceinline__ float to_log2(float s, float scale_log2, float scale, float cap) {
   // cap * tanh(s * scale / cap), from an exponential: this file's tanhf keeps about 11 bits
@@ -323,6 +328,7 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const uint32_t tS = tmem_base + tile * BT + lane_addr;
     const uint32_t tO = tmem_base + 2 * BT + tile * HDV + lane_addr;
     const float scale_log2 = p.scale * kLog2e;
+    const float cap_inv = kCap ? __fdividef(p.scale, p.soft_cap) : 0.f;
     const int my_seg = kSeg ? p.q_seg[b * p.S + qi] : 0;
     const int* kseg_row = kSeg ? p.k_seg + b * p.Sk : nullptr;
     float m_used = -INFINITY, l_sum = 0.f;
@@ -342,32 +348,64 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       tc_fence_after();
       const bool need_mask = (j == jdiag) || kSeg || (kPacked && k0 < tile_lo) || (!kPacked && p.window > 0 && k0 <= q0 + tile * BT + BT - 1 - p.window);
 
-      // ---- pass 1: row maximum (raw logits; the scale is positive and the soft-cap monotonic)
-      float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
-#pragma unroll 1
-      for (int c = 0; c < BT; c += 32) {
-        uint32_t v[32];
-        tmem_ld_32x32(tS + c, v);
-        tmem_ld_wait();
-        if (need_mask) {
+      // what the row sees of the block: columns col_lo .. col_lo + col_span (with segment ids: those of its segment)
+      const int col_lo = (kPacked ? row_lo : p.window > 0 ? qi - p.window + 1 : 0) - k0;
+      const unsigned col_span = causal ? static_cast<unsigned>(qi - k0 - col_lo) : 0x7fffffffu;
+      uint32_t same[4] = {0u, 0u, 0u, 0u};  // kSeg: a bit per column, set in pass 1
+      auto mask = [&](uint32_t (&v)[2][32], int c) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const uint32_t bits = c == 0 ? same[i] : same[2 + i];
 #pragma unroll
           for (int t = 0; t < 32; ++t) {
-            const int kj = k0 + c + t;
-            bool valid = !causal || kj <= qi;
-            if (!kPacked && p.window > 0) valid = valid && (qi - kj < p.window);
-            if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
-            if (kPacked) valid = valid && kj >= row_lo;
-            if (!valid) v[t] = __float_as_uint(-INFINITY);
+            bool valid = static_cast<unsigned>(c + 32 * i + t - col_lo) <= col_span;
+            if (kSeg) valid = valid && ((bits >> t) & 1u);
+            if (!valid) v[i][t] = __float_as_uint(-INFINITY);
           }
         }
+      };
+      if constexpr (kSeg) {
 #pragma unroll
-        for (int t = 0; t < 32; t += 4) {
-          mx0 = fmaxf(mx0, __uint_as_float(v[t]));
-          mx1 = fmaxf(mx1, __uint_as_float(v[t + 1]));
-          mx2 = fmaxf(mx2, __uint_as_float(v[t + 2]));
-          mx3 = fmaxf(mx3, __uint_as_float(v[t + 3]));
-        }
+        for (int i = 0; i < 4; ++i)
+#pragma unroll 2
+          for (int t = 0; t < 32; t += 4) {
+            const int4 seg = __ldg(reinterpret_cast<const int4*>(kseg_row + k0 + 32 * i + t));
+            same[i] |= (seg.x == my_seg ? 1u << t : 0u) | (seg.y == my_seg ? 2u << t : 0u) | (seg.z == my_seg ? 4u << t : 0u) |
+                       (seg.w == my_seg ? 8u << t : 0u);
+          }
       }
+
+      // ---- pass 1: row maximum (raw logits; the scale is positive and the soft-cap monotonic).  Rolled loops over 64 columns: unrolled
+      // further, the code no longer fits the instruction cache
+      float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY, far0 = 0.f, far1 = 0.f;
+#pragma unroll 1
+      for (int c = 0; c < BT; c += 64) {
+        uint32_t v[2][32];
+        tmem_ld_32x32(tS + c, v[0]);
+        tmem_ld_32x32(tS + c + 32, v[1]);
+        tmem_ld_wait();
+        if constexpr (kCap) {
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int t = 0; t < 32; t += 2) {
+              far0 = fmaxf(far0, fabsf(__uint_as_float(v[i][t])));
+              far1 = fmaxf(far1, fabsf(__uint_as_float(v[i][t + 1])));
+            }
+        }
+        if (need_mask) mask(v, c);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int t = 0; t < 32; t += 4) {
+            mx0 = fmaxf(mx0, __uint_as_float(v[i][t]));
+            mx1 = fmaxf(mx1, __uint_as_float(v[i][t + 1]));
+            mx2 = fmaxf(mx2, __uint_as_float(v[i][t + 2]));
+            mx3 = fmaxf(mx3, __uint_as_float(v[i][t + 3]));
+          }
+      }
+      // kCap: whether all logits of the warp lie where the cap is a polynomial
+      const bool near = kCap && __all_sync(0xffffffffu, fmaxf(far0, far1) * p.scale <= 0.75f * p.soft_cap);
       const float m_raw = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
       const float m_blk = (m_raw == -INFINITY) ? -INFINITY : to_log2<kCap>(m_raw, scale_log2, p.scale, p.soft_cap);
 
@@ -382,13 +420,13 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           const float alpha = scale_row ? exp2f(m_used - m_new) : 1.f;
           l_sum *= alpha;
 #pragma unroll 1
-          for (int c = 0; c < HDV; c += 32) {
-            uint32_t v[32];
-            tmem_ld_32x32(tO + c, v);
+          for (int c = 0; c < HDV; c += 16) {  // few columns at a time: the logits hold most registers
+            uint32_t w[16];
+            tmem_ld_32x16(tO + c, w);
             tmem_ld_wait();
 #pragma unroll
-            for (int t = 0; t < 32; ++t) v[t] = __float_as_uint(__uint_as_float(v[t]) * alpha);
-            tmem_st_32x32(tO + c, v);
+            for (int t = 0; t < 16; ++t) w[t] = __float_as_uint(__uint_as_float(w[t]) * alpha);
+            tmem_st_32x16(tO + c, w);
           }
         }
         m_used = m_new;
@@ -396,46 +434,53 @@ flash_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       const float neg_m = (m_used == -INFINITY) ? 0.f : -m_used;
 
       // ---- pass 2: P = exp2(s - m) -> bf16 pairs written over the first 64 columns of S
-      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+      const F32x2 scale2 = f2(scale_log2, scale_log2), cap2 = f2(cap_inv, cap_inv), neg2 = f2(neg_m, neg_m);
+      F32x2 sum[4] = {f2(0.f, 0.f), f2(0.f, 0.f), f2(0.f, 0.f), f2(0.f, 0.f)};
+      auto exponentials = [&](auto masked, auto polynomial) {
+        constexpr bool kMasked = decltype(masked)::value, kPoly = decltype(polynomial)::value;
 #pragma unroll 1
-      for (int c = 0; c < BT; c += 32) {
-        uint32_t v[32];
-        tmem_ld_32x32(tS + c, v);
-        tmem_ld_wait();
-        float e[32];
-        if (need_mask) {
+        for (int c = 0; c < BT; c += 64) {
+          uint32_t v[2][32];
+          tmem_ld_32x32(tS + c, v[0]);
+          tmem_ld_32x32(tS + c + 32, v[1]);
+          tmem_ld_wait();
+          if constexpr (kMasked) mask(v, c);
 #pragma unroll
-          for (int t = 0; t < 32; ++t) {
-            const int kj = k0 + c + t;
-            bool valid = !causal || kj <= qi;
-            if (!kPacked && p.window > 0) valid = valid && (qi - kj < p.window);
-            if (kSeg) valid = valid && (kseg_row[kj] == my_seg);
-            if (kPacked) valid = valid && kj >= row_lo;
-            const float x = kCap ? to_log2<kCap>(__uint_as_float(v[t]), scale_log2, p.scale, p.soft_cap) + neg_m
-                                 : fmaf(__uint_as_float(v[t]), scale_log2, neg_m);
-            e[t] = valid ? exp2f(x) : 0.f;
-          }
-        } else {
+          for (int i = 0; i < 2; ++i) {
+            uint32_t pk[16];
 #pragma unroll
-          for (int t = 0; t < 32; ++t) {
-            const float x = kCap ? to_log2<kCap>(__uint_as_float(v[t]), scale_log2, p.scale, p.soft_cap) + neg_m
-                                 : fmaf(__uint_as_float(v[t]), scale_log2, neg_m);
-            e[t] = exp2f(x);
+            for (int t = 0; t < 16; ++t) {
+              const float x0 = __uint_as_float(v[i][2 * t]), x1 = __uint_as_float(v[i][2 * t + 1]);
+              const F32x2 x = f2(x0, x1);
+              float a, b;
+              if constexpr (!kCap) {
+                f2_split(f2_fma(x, scale2, neg2), a, b);
+              } else if constexpr (kPoly) {
+                const F32x2 y = f2_mul(x, cap2);
+                f2_split(f2_fma(f2_mul(x, scale2), tanh_ratio(f2_mul(y, y)), neg2), a, b);
+              } else {
+                a = to_log2<kCap>(x0, scale_log2, p.scale, p.soft_cap) + neg_m;
+                b = to_log2<kCap>(x1, scale_log2, p.scale, p.soft_cap) + neg_m;
+              }
+              if constexpr (kCap && kMasked) {  // a masked logit does not stay masked under the cap
+                a = x0 == -INFINITY ? -INFINITY : a;
+                b = x1 == -INFINITY ? -INFINITY : b;
+              }
+              a = exp2f(a);
+              b = exp2f(b);
+              sum[t & 3] = f2_add(sum[t & 3], f2(a, b));
+              pk[t] = pack_bf16x2(a, b);
+            }
+            tmem_st_32x16(tS + (c >> 1) + 16 * i, pk);
           }
         }
-        uint32_t pk[16];
-#pragma unroll
-        for (int t = 0; t < 16; ++t) pk[t] = pack_bf16x2(e[2 * t], e[2 * t + 1]);
-#pragma unroll
-        for (int t = 0; t < 32; t += 4) {
-          s0 += e[t];
-          s1 += e[t + 1];
-          s2 += e[t + 2];
-          s3 += e[t + 3];
-        }
-        tmem_st_32x16(tS + (c >> 1), pk);
-      }
-      l_sum += (s0 + s1) + (s2 + s3);
+      };
+      if (kCap && !near) exponentials(Yes<true>{}, Yes<false>{});
+      else if (need_mask) exponentials(Yes<true>{}, Yes<true>{});
+      else exponentials(Yes<false>{}, Yes<true>{});
+      float s0, s1;
+      f2_split(f2_add(f2_add(sum[0], sum[1]), f2_add(sum[2], sum[3])), s0, s1);
+      l_sum += s0 + s1;
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -610,6 +655,7 @@ extern "C" int lvb_flash_attn_fwd2_hd(const void* q, const void* k, const void* 
   if (B <= 0 || S <= 0 || (S % (2 * BT)) != 0 || Hq <= 0 || Hkv <= 0 || (Hq % Hkv) != 0) return kErrBadArg;
   if (!causal && (window != 0 || kblock_lo != nullptr)) return kErrBadArg;
   if (Sk <= 0 || (Sk % BT) != 0 || (causal && Sk != S)) return kErrBadArg;
+  if (reinterpret_cast<uintptr_t>(k_seg) & 15) return kErrBadArg;
   Params p;
   p.O = reinterpret_cast<__nv_bfloat16*>(o);
   p.lse2 = lse2;
