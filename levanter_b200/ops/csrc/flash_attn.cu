@@ -269,7 +269,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
         for (int t = 0; t < 32; ++t) {
           float s = __uint_as_float(v[t]);
-          if (p.soft_cap > 0.f) s = p.soft_cap * tanhf(s * p.scale / p.soft_cap) * 1.4426950408889634f;
+          if (p.soft_cap > 0.f) s = soft_capped(s * p.scale, p.soft_cap) * 1.4426950408889634f;
           else s *= scale_log2;
           if (need_mask) {
             const int kj = k0 + c + t;
@@ -322,7 +322,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
         for (int t = 0; t < 32; ++t) {
           float s = __uint_as_float(v[t]);
-          if (p.soft_cap > 0.f) s = p.soft_cap * tanhf(s * p.scale / p.soft_cap) * 1.4426950408889634f;
+          if (p.soft_cap > 0.f) s = soft_capped(s * p.scale, p.soft_cap) * 1.4426950408889634f;
           else s *= scale_log2;
           if (need_mask) {
             const int kj = k0 + c + t;

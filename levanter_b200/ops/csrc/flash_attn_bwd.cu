@@ -250,7 +250,7 @@ flash_bwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         for (int u = 0; u < 32; ++u) {
           float x, dcap = p.scale;
           if constexpr (kCap) {
-            const float th = tanhf(__uint_as_float(sv[u]) * p.scale / p.soft_cap);
+            const float th = soft_capped(__uint_as_float(sv[u]) * (p.scale / p.soft_cap), 1.f);
             x = p.soft_cap * th * 1.4426950408889634f + neg_lse;
             dcap = p.scale * (1.f - th * th);
           } else {

@@ -322,7 +322,7 @@ flash_bwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             float x, dcap = p.scale;
             const float neg_lse = s_lse[c + u];
             if constexpr (kCap) {
-              const float th = tanhf(__uint_as_float(sv[u]) * p.scale / p.soft_cap);
+              const float th = soft_capped(__uint_as_float(sv[u]) * (p.scale / p.soft_cap), 1.f);
               x = p.soft_cap * th * 1.4426950408889634f + neg_lse;
               dcap = p.scale * (1.f - th * th);
             } else {
