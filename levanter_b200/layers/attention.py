@@ -745,6 +745,8 @@ class MultiHeadLatentAttentionConfig:
     norm_eps: float = 1e-6
     sliding_window: Optional[int] = None  # a query sees itself and that many positions less one before it
     sink: bool = False  # a learned number per head joins the softmax denominator (unscaled, with no key and no value)
+    output_gate: bool = False  # the heads are multiplied by sigmoid(W_g x) before the output projection
+    shares_latent: bool = False  # no down projection of its own: keys and values come from the latents that an earlier layer keeps
 
     @property
     def softmax_scale(self) -> float:
@@ -763,7 +765,10 @@ class MultiHeadLatentAttention(nn.Module):
     Serving (:meth:`paged_decode`) caches the normed latent and the rotated key part of a token, ``kv_lora_rank + qk_rope_head_dim``
     numbers for all heads.  Prompts that start in a step are attended to with per-head keys and values: one product of the cache
     rows with ``[[W_uk, 0], [0, 1]]`` yields whole keys, the identity block putting the shared part into every head.  Otherwise
-    (decoding, portions) ``W_uk`` is applied to the queries and ``W_uv`` to the result, and the heads read the cache rows as they are."""
+    (decoding, portions) ``W_uk`` is applied to the queries and ``W_uv`` to the result, and the heads read the cache rows as they are.
+
+    With ``shares_latent`` a layer is handed what an earlier layer of the same latent size and rotation keeps: its pages and, for prompts that
+    start in a step, its rows of the step."""
 
     def __init__(self, config: MultiHeadLatentAttentionConfig, init_std: float = 0.02):
         super().__init__()
@@ -778,8 +783,11 @@ class MultiHeadLatentAttention(nn.Module):
             self.q_a_proj = Linear(c.hidden_dim, c.q_lora_rank, bias=c.use_bias, init_std=init_std)
             self.q_a_norm = RmsNorm(c.q_lora_rank, eps=c.norm_eps)
             self.q_b_proj = Linear(c.q_lora_rank, H * c.qk_head_dim, bias=c.use_bias, init_std=init_std)
-        self.kv_a_proj = Linear(c.hidden_dim, c.kv_lora_rank + c.qk_rope_head_dim, bias=c.use_bias, init_std=init_std)
-        self.kv_a_norm = RmsNorm(c.kv_lora_rank, eps=c.norm_eps)
+        self.kv_a_proj = self.kv_a_norm = None
+        if not c.shares_latent:
+            self.kv_a_proj = Linear(c.hidden_dim, c.kv_lora_rank + c.qk_rope_head_dim, bias=c.use_bias, init_std=init_std)
+            self.kv_a_norm = RmsNorm(c.kv_lora_rank, eps=c.norm_eps)
+        self.g_proj = Linear(c.hidden_dim, H * c.v_head_dim, init_std=init_std) if c.output_gate else None
         self.kv_b_proj = Linear(c.kv_lora_rank, H * (c.qk_nope_head_dim + c.v_head_dim), bias=c.use_bias, init_std=init_std)
         self.o_proj = Linear(H * c.v_head_dim, c.hidden_dim, bias=c.use_bias, init_std=init_std)
         rope = c.rope if c.rope is not None else DefaultRotaryEmbeddingsConfig()
@@ -787,7 +795,11 @@ class MultiHeadLatentAttention(nn.Module):
         if c.sink:
             self.sinks = nn.Parameter(torch.zeros(H))
             self.sinks.lev_shape = (H,)
-        self._rows, self._whole_kv, self._sinks = FusedRows(-(H * c.qk_head_dim + c.kv_lora_rank + c.qk_rope_head_dim) % 8), None, None
+        self._rows, self._whole_kv, self._sinks = FusedRows(-sum(m.weight.shape[0] for m in self._from_input()) % 8), None, None
+
+    def _from_input(self):
+        """The projections that read the layer's input."""
+        return [m for m in (self.q_proj, self.q_a_proj, self.kv_a_proj, self.g_proj) if m is not None]
 
     def sinks_fp32(self) -> Optional[torch.Tensor]:
         """The sink numbers in fp32 at a fixed address (it goes into captured graphs), made again like :meth:`_whole_kv_weight`."""
@@ -836,25 +848,33 @@ class MultiHeadLatentAttention(nn.Module):
         """Packed rows ``x [T, hidden]`` of a serving step -> ``[T, hidden]`` in fp32; their latents enter the cache."""
         from ..ops.residual_stream import project
 
-        heads = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        heads, _ = self._paged_heads(x, kv_cache, batch_info, pos_ids)
         if type(self.o_proj) is Linear:
             return project(heads, self.o_proj.weight, out_dtype=torch.float32)
         return self.o_proj(heads).float()
 
     def paged_decode_stream(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor):
         """:meth:`paged_decode` for an fp32 residual stream: ``stream + o_proj(heads)``, added in the projection's epilogue."""
+        return self.paged_decode_stream_sharing(x, kv_cache, batch_info, pos_ids, stream)[0], kv_cache
+
+    def paged_decode_stream_sharing(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids, stream: torch.Tensor,
+                                    latent: Optional[torch.Tensor] = None):
+        """``(stream + o_proj(heads), latent)`` for layers of which some read what others keep.  ``latent [T, rank + rope]``: the rows of the
+        step that entered the cache, where a layer had use for them (None otherwise, and then they are read from the cache); a layer that
+        shares them is given them, with the pages of the layer that keeps them."""
         from ..ops.residual_stream import add_linear
 
-        heads = self._paged_heads(x, kv_cache, batch_info, pos_ids)
+        heads, latent = self._paged_heads(x, kv_cache, batch_info, pos_ids, latent)
         if type(self.o_proj) is Linear and self.o_proj.bias is None:
-            return add_linear(stream, heads, self.o_proj.weight), kv_cache
-        return stream + self.o_proj(heads).float(), kv_cache
+            return add_linear(stream, heads, self.o_proj.weight), latent
+        return stream + self.o_proj(heads).float(), latent
 
-    def _paged_heads(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids: torch.Tensor) -> torch.Tensor:
-        """The concatenated heads ``[T, heads * v_head_dim]`` of packed rows."""
+    def _paged_heads(self, x: torch.Tensor, kv_cache: "KvPageCache", batch_info, pos_ids: torch.Tensor, latent: Optional[torch.Tensor] = None):
+        """``(heads, latent)``: the concatenated (gated) heads ``[T, heads * v_head_dim]`` of packed rows; ``latent`` as in
+        :meth:`paged_decode_stream_sharing`."""
         from ..ops import flash_attention as FA
         from ..ops import paged_attention as PA
-        from ..ops.qkv_prep import prepare_latent
+        from ..ops.qkv_prep import norm_rows, prepare_latent, rotate_queries
         from ..ops.residual_stream import project
 
         c = self.config
@@ -862,33 +882,46 @@ class MultiHeadLatentAttention(nn.Module):
             raise NotImplementedError("serving latent attention takes neither a soft cap nor biases")
         T, H, dn, dr, dv, rank = x.shape[0], c.num_heads, c.qk_nope_head_dim, c.qk_rope_head_dim, c.v_head_dim, c.kv_lora_rank
         nq = H * c.qk_head_dim
+        mods = self._from_input()
         w = None
-        if self.q_proj is not None and type(self.q_proj) is Linear and type(self.kv_a_proj) is Linear and x.is_cuda and not self.training \
-                and not torch.is_grad_enabled():
-            w = self._rows.get([self.q_proj.weight, self.kv_a_proj.weight])
+        if all(type(m) is Linear for m in mods) and x.is_cuda and not self.training and not torch.is_grad_enabled():
+            w = self._rows.get([m.weight for m in mods])
         if w is not None:
-            y = project(x, w)
-            q, down = y[:, :nq], y[:, nq:nq + rank + dr]
+            parts = project(x, w).split([m.weight.shape[0] for m in mods] + [self._rows.pad], dim=1)
         else:
-            q = self.q_proj(x) if self.q_proj is not None else self.q_b_proj(self.q_a_norm(self.q_a_proj(x)))
-            down = self.kv_a_proj(x)
+            parts = [m(x) for m in mods]
+        q, rest = parts[0], list(parts[1:])
+        down = rest.pop(0) if self.kv_a_proj is not None else None
+        gate = rest.pop(0) if self.g_proj is not None else None
+        if self.q_a_proj is not None:
+            q = norm_rows(q, self.q_a_norm.weight, self.q_a_norm.eps)
+            q = project(q, self.q_b_proj.weight) if type(self.q_b_proj) is Linear else self.q_b_proj(q)
         q = q.unflatten(1, (H, c.qk_head_dim))
         pages, dests = kv_cache.kv_pages, batch_info.new_token_dests
-        norm = (self.kv_a_norm.weight, self.kv_a_norm.eps)
         weight, sink = self.kv_b_proj.weight, self.sinks_fp32()
-        if getattr(batch_info, "prefill_segment_ids", None) is not None and self._packed_prefill_fits(q):
-            latent, _ = prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:])
+
+        def prepare(q_out, to_cache_only):
+            """Rotated queries (into ``q_out``, or in place) and, unless another layer has seen to it, the latents in the cache."""
+            if c.shares_latent:
+                if self.rot is not None:
+                    rotate_queries(q[..., dn:], pos_ids, self.rot, q_out)
+                return latent
+            return prepare_latent(down, self.kv_a_norm.weight, self.kv_a_norm.eps, pages, dests, pos_ids, self.rot, q[..., dn:], q_out,
+                                  to_cache_only=to_cache_only)[0]
+
+        if getattr(batch_info, "prefill_segment_ids", None) is not None and self._packed_prefill_fits(q) and (latent is not None or not c.shares_latent):
+            latent = prepare(None, False)
             kv = project(latent, self._whole_kv_weight())
             k, v = kv[:, :nq].unflatten(1, (H, c.qk_head_dim)), kv[:, nq:].unflatten(1, (H, dv))
-            heads = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=c.softmax_scale, window=c.sliding_window, sink=sink)
+            heads = FA.flash_attention_packed(q, k, v, pos_ids, scaling_factor=c.softmax_scale, window=c.sliding_window, sink=sink, gate=gate)
         else:
             uk, uv = self.up_projections(weight)
             qa = q.new_empty(T, H, rank + dr)
-            prepare_latent(down, *norm, pages, dests, pos_ids, self.rot, q[..., dn:], qa[..., rank:], to_cache_only=True)
+            latent = prepare(qa[..., rank:], True)
             PA.head_product(q[..., :dn], uk.to(q.dtype), qa[..., :rank], b_trans=False)
             o = PA.paged_attention_latent(qa, pages, rank, batch_info, sm_scale=c.softmax_scale, window=c.sliding_window, sink=sink)
-            heads = PA.head_product(o.to(q.dtype), uv.to(q.dtype), q.new_empty(T, H, dv), b_trans=True)
-        return heads.reshape(T, H * dv).to(x.dtype)
+            heads = PA.head_product(o.to(q.dtype), uv.to(q.dtype), q.new_empty(T, H, dv), b_trans=True, gate=gate)
+        return heads.reshape(T, H * dv).to(x.dtype), latent
 
     def _packed_prefill_fits(self, q: torch.Tensor) -> bool:
         """Whether the packed flash kernel takes this layer's sizes (the joint product of keys and values has the strides of its columns)."""
@@ -900,6 +933,11 @@ class MultiHeadLatentAttention(nn.Module):
                 and not torch.is_grad_enabled())
 
     def forward(self, x, mask=None, pos_ids=None):
+        return self.forward_sharing(x, mask, pos_ids)[0]
+
+    def forward_sharing(self, x, mask=None, pos_ids=None, kept=None):
+        """``(attention(x), kept)`` for layers of which some read what others keep: ``kept`` is ``(latent [B, S, rank], rotated key part)``, made
+        here unless the layer shares an earlier one's."""
         c = self.config
         if c.sliding_window is not None:
             mask = (mask if isinstance(mask, AttentionMask) else AttentionMask.explicit(mask) if mask is not None
@@ -911,17 +949,24 @@ class MultiHeadLatentAttention(nn.Module):
         q = self.q_proj(x) if self.q_proj is not None else self.q_b_proj(self.q_a_norm(self.q_a_proj(x)))
         q = q.view(B, S, H, c.qk_head_dim)
         q_nope, q_rope = q.split([c.qk_nope_head_dim, c.qk_rope_head_dim], dim=-1)
-        kv_a = self.kv_a_proj(x)
-        latent, k_rope = kv_a.split([c.kv_lora_rank, c.qk_rope_head_dim], dim=-1)
-        kv = self.kv_b_proj(self.kv_a_norm(latent)).view(B, S, H, c.qk_nope_head_dim + c.v_head_dim)
+        if not c.shares_latent:
+            latent, k_rope = self.kv_a_proj(x).split([c.kv_lora_rank, c.qk_rope_head_dim], dim=-1)
+            kept = (self.kv_a_norm(latent), k_rope if self.rot is None else self.rot(k_rope.unsqueeze(2), pos_ids).squeeze(2))
+        latent, k_rope = kept
+        kv = self.kv_b_proj(latent).view(B, S, H, c.qk_nope_head_dim + c.v_head_dim)
         k_nope, v = kv.split([c.qk_nope_head_dim, c.v_head_dim], dim=-1)
         qf, kf = q_nope, k_nope
         if self.rot is not None:
-            q_rope = self.rot(q_rope, pos_ids)
-            k_rope = self.rot(k_rope.unsqueeze(2), pos_ids).expand(B, S, H, c.qk_rope_head_dim)
-            qf = torch.cat([q_nope, q_rope], dim=-1)
-            kf = torch.cat([k_nope, k_rope], dim=-1)
+            qf = torch.cat([q_nope, self.rot(q_rope, pos_ids)], dim=-1)
+            kf = torch.cat([k_nope, k_rope.unsqueeze(2).expand(B, S, H, c.qk_rope_head_dim)], dim=-1)
         scale = c.softmax_scale
+
+        def project_out(heads):
+            heads = heads.reshape(B, S, H * c.v_head_dim)
+            if self.g_proj is not None:
+                heads = heads.float() * torch.sigmoid(self.g_proj(x).float())
+            return self.o_proj(heads.to(x.dtype))
+
         if c.sink:
             if c.logits_soft_cap is not None:
                 raise NotImplementedError("latent attention with a sink takes no soft cap")
@@ -931,14 +976,12 @@ class MultiHeadLatentAttention(nn.Module):
             if m is not None:
                 s = torch.where(m, s, torch.full_like(s, -1e9))
             p = torch.softmax(torch.cat([s, self.sinks.float().view(1, H, 1, 1).expand(B, H, S, 1)], dim=-1), dim=-1)[..., :-1]
-            out = torch.einsum("bhqk,bkhd->bqhd", p.to(v.dtype), v)
-            return self.o_proj(out.reshape(B, S, H * c.v_head_dim).to(x.dtype))
+            return project_out(torch.einsum("bhqk,bkhd->bqhd", p.to(v.dtype), v)), kept
         # value head size differs from the qk head size, so pad V for the shared kernel interface
         out = simple_attention_with_dropout(qf, kf, F.pad(v, (0, c.qk_head_dim - c.v_head_dim)) if c.v_head_dim < c.qk_head_dim else v,
                                             mask, attention_dtype=torch.float32 if c.upcast_attn else None,
                                             logits_soft_cap=c.logits_soft_cap, scaling_factor=scale)
-        out = out[..., : c.v_head_dim]
-        return self.o_proj(out.reshape(B, S, H * c.v_head_dim).to(x.dtype))
+        return project_out(out[..., : c.v_head_dim]), kept
 
 
 # --------------------------------------------------------------------------------------------- paged KV cache

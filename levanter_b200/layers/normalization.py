@@ -1,4 +1,4 @@
-"""Normalisation configs selectable by ``type:`` (``rms`` | ``layer``; Gemma registers ``gemma``)
+"""Normalisation configs selectable by ``type:`` (``rms`` | ``rms_grouped`` | ``layer``; Gemma registers ``gemma``)
 (src/levanter/layers/normalization.py:15-48)."""
 from __future__ import annotations
 
@@ -29,6 +29,21 @@ class RmsNormConfig(LayerNormConfigBase):
         from ..nn import RmsNorm
 
         return RmsNorm(dim, eps=self.eps, use_weight=self.use_weight, use_bias=self.use_bias)
+
+
+@LayerNormConfigBase.register_subclass("rms_grouped")
+@dataclass(frozen=True)
+class GroupedRmsNormConfig(LayerNormConfigBase):
+    """``groups`` equal consecutive parts of a row, each divided by its own root mean square."""
+
+    groups: int = 1
+
+    def build(self, dim: int):
+        from ..nn import GroupedRmsNorm
+
+        if not self.use_weight or self.use_bias:
+            raise ValueError("a grouped RMS norm has a weight and no bias")
+        return GroupedRmsNorm(dim, self.groups, eps=self.eps)
 
 
 @LayerNormConfigBase.register_subclass("layer")

@@ -2,14 +2,15 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import Dict, Optional, Tuple
 
 import torch
 import torch.nn as nn
 
-from ..nn import FusedRows, Linear
+from ..nn import FusedRows, Linear, RmsNorm
 from ..ops.gated_scan import min_gru, min_gru_packed
-from ..ops.residual_stream import project
+from ..ops.linear_attention import fixed_decay_attention, gated_norm, linear_attention_packed
+from ..ops.residual_stream import add_linear, project
 from .attention import AttentionMask
 
 
@@ -32,6 +33,21 @@ class SlotStateCache:
         return self  # nothing is kept by pages
 
 
+def sequence_starts(mask) -> Optional[torch.Tensor]:
+    """``[B, L]`` bool: where packed sequences (segment ids of the mask) begin; None when rows are whole sequences."""
+    if not isinstance(mask, AttentionMask) or mask.segment_ids is None:
+        return None
+    seg = _segments(mask)
+    starts = torch.ones_like(seg, dtype=torch.bool)
+    starts[:, 1:] = seg[:, 1:] != seg[:, :-1]
+    return starts
+
+
+def _segments(mask: AttentionMask) -> torch.Tensor:
+    seg = mask.segment_ids[0]
+    return seg if seg.dim() == 2 else seg[None]
+
+
 class MinGru(nn.Module):
     """minGRU: ``o_proj(S_t * silu(g_proj x))`` over ``S_t = (1 - z) S_{t-1} + z c`` whose gates read the current token only: ``z =
     sigmoid(z_proj x)``, ``c = u + 1/2`` for ``u = x_proj x >= 0`` and ``sigmoid(u)`` below."""
@@ -50,12 +66,7 @@ class MinGru(nn.Module):
 
     def forward(self, x: torch.Tensor, mask=None, pos_ids=None) -> torch.Tensor:
         """``x [B, L, hidden]`` (or ``[L, hidden]``); packed sequences (segment ids of the mask) start from zero each."""
-        starts = None
-        if isinstance(mask, AttentionMask) and mask.segment_ids is not None:
-            seg = mask.segment_ids[0]
-            seg = seg if seg.dim() == 2 else seg[None]
-            starts = torch.ones_like(seg, dtype=torch.bool)
-            starts[:, 1:] = seg[:, 1:] != seg[:, :-1]
+        starts = sequence_starts(mask)
         z, u, g = self.z_proj(x), self.x_proj(x), self.g_proj(x)
         z3, u3 = (z, u) if z.dim() == 3 else (z[None], u[None])
         s = min_gru(z3, u3, starts)
@@ -78,3 +89,90 @@ class MinGru(nn.Module):
 
     def empty_state(self, max_seqs: int, device=None) -> SlotStateCache:
         return SlotStateCache.init(max_seqs, self.width, device=device)
+
+
+@dataclass(frozen=True)
+class LinearAttentionConfig:
+    """Linear attention with a fixed decay per head (:class:`LinearAttention`)."""
+
+    hidden_dim: int
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    decay: Tuple[float, ...]
+    key_scale: float = 1.0
+    silu: bool = False          # q, k and v pass through silu
+    norm_per_head: bool = True  # the heads' outputs are normed one by one without a weight; else all together with one
+    sigmoid_gate: bool = False  # the gate is a sigmoid; else a silu
+    norm_eps: float = 1e-6
+
+    def __post_init__(self):
+        if len(self.decay) != self.num_heads:
+            raise ValueError(f"{len(self.decay)} decays for {self.num_heads} heads")
+
+
+class LinearAttention(nn.Module):
+    """``o_proj(norm(o) * act(g_proj x))`` with, per head, ``S_t = decay S_{t-1} + key_scale k_t v_t^T`` and ``o_t = S_t^T q_t`` of q, k, v projected from
+    ``x``: retention (Sun et al., "Retentive Network", 2023; ``key_scale = head_dim^-1/2``, norm per head, silu gate) or lightning attention (silu
+    on q, k and v, one norm with a weight, sigmoid gate)."""
+
+    def __init__(self, config: LinearAttentionConfig, *, init_std: float = 0.02):
+        super().__init__()
+        c = self.config = config
+        qk, v = c.num_heads * c.head_dim, c.num_heads * c.v_head_dim
+        self.q_proj = Linear(c.hidden_dim, qk, init_std=init_std)
+        self.k_proj = Linear(c.hidden_dim, qk, init_std=init_std)
+        self.v_proj = Linear(c.hidden_dim, v, init_std=init_std)
+        self.g_proj = Linear(c.hidden_dim, v, init_std=init_std)
+        self.o_proj = Linear(v, c.hidden_dim, init_std=init_std)
+        self.o_norm = None if c.norm_per_head else RmsNorm(v, eps=c.norm_eps)
+        self._rows = FusedRows(-(2 * qk + 2 * v) % 8)
+        self._decay: Dict[torch.device, torch.Tensor] = {}
+
+    def decay_on(self, device) -> torch.Tensor:
+        """The decays in fp32 (whatever the parameters' type), made once per device."""
+        device = torch.device(device)
+        if device not in self._decay:
+            self._decay[device] = torch.tensor(self.config.decay, dtype=torch.float32, device=device)
+        return self._decay[device]
+
+    def _gated(self, o: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
+        """``o, g [T, heads * v_head_dim]``."""
+        c = self.config
+        return gated_norm(o, g, c.norm_eps, groups=c.num_heads if c.norm_per_head else 1, weight=None if self.o_norm is None else self.o_norm.weight,
+                          sigmoid=c.sigmoid_gate)
+
+    def forward(self, x: torch.Tensor, mask=None, pos_ids=None) -> torch.Tensor:
+        """``x [B, L, hidden]``; packed sequences (segment ids of the mask) start from zero each."""
+        c = self.config
+        B, L, _ = x.shape
+        q, k, v = (m(x).view(B, L, c.num_heads, -1) for m in (self.q_proj, self.k_proj, self.v_proj))
+        if c.silu:
+            q, k, v = (torch.nn.functional.silu(t.float()) for t in (q, k, v))
+        seg = None
+        if isinstance(mask, AttentionMask) and mask.segment_ids is not None:
+            seg = _segments(mask).expand(B, L)
+        o = fixed_decay_attention(q, k.float() * c.key_scale, v, self.decay_on(x.device), seg).reshape(B * L, -1)
+        return self.o_proj(self._gated(o, self.g_proj(x).reshape(B * L, -1).float()).to(x.dtype).view(B, L, -1))
+
+    def paged_decode_stream(self, x: torch.Tensor, cache: SlotStateCache, batch_info, pos_ids, stream: torch.Tensor):
+        """Packed rows ``x [T, hidden]`` of a serving step: ``stream + o_proj(...)`` on the fp32 stream, added in the projection's epilogue; the
+        sequences' states go on from their slots."""
+        c = self.config
+        mods = (self.q_proj, self.k_proj, self.v_proj, self.g_proj)
+        w = None
+        if all(type(m) is Linear for m in mods) and x.is_cuda and not self.training and not torch.is_grad_enabled():
+            w = self._rows.get([m.weight for m in mods])
+        y = project(x, w) if w is not None else torch.cat([m(x) for m in mods], dim=1)
+        qk, nv = c.num_heads * c.head_dim, c.num_heads * c.v_head_dim
+        q, k, v, g = y[:, :2 * qk + 2 * nv].split([qk, qk, nv, nv], dim=1)
+        heads = lambda t: t.unflatten(1, (c.num_heads, -1))  # noqa: E731
+        o = linear_attention_packed(heads(q), heads(k), heads(v), self.decay_on(x.device), cache.state, batch_info, key_scale=c.key_scale, silu=c.silu)
+        h = self._gated(o.flatten(1), g)
+        if type(self.o_proj) is Linear:
+            return add_linear(stream, h, self.o_proj.weight), cache
+        return stream + self.o_proj(h).float(), cache
+
+    def empty_state(self, max_seqs: int, device=None) -> SlotStateCache:
+        c = self.config
+        return SlotStateCache.init(max_seqs, c.num_heads, c.head_dim, c.v_head_dim, device=device)

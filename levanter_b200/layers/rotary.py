@@ -274,3 +274,24 @@ def rope_to_hf_dict(rope: RotaryEmbeddingsConfig) -> dict:
         params["rope_type"] = scaling.get("rope_type", scaling.get("type", "default"))
         params.pop("type", None)
     return {"rope_theta": theta, "rope_scaling": scaling, "rope_parameters": params}
+
+
+def rope_from_entry(rot: Optional[dict]) -> Optional[RotaryEmbeddingsConfig]:
+    """The rotation that a layer's ``{base, dims, scaling: {factor, original, fast, slow}}`` entry describes (None: no rotation)."""
+    if rot is None:
+        return None
+    s = rot.get("scaling")
+    if s is None:
+        return DefaultRotaryEmbeddingsConfig(theta=float(rot["base"]), rotary_dim=rot["dims"])
+    return PartialYarnRotaryEmbeddingsConfig(theta=float(rot["base"]), rotary_dim=rot["dims"], factor=float(s["factor"]), beta_fast=float(s["fast"]),
+                                             beta_slow=float(s["slow"]), original_max_position_embeddings=s["original"])
+
+
+def rope_to_entry(rope: RotaryEmbeddingsConfig, head_dim: int) -> dict:
+    """The inverse of :func:`rope_from_entry` for heads of ``head_dim``."""
+    rot = dict(base=rope.theta, dims=head_dim if rope.rotary_dim is None else rope.rotary_dim)
+    if isinstance(rope, PartialYarnRotaryEmbeddingsConfig):
+        rot["scaling"] = dict(factor=rope.factor, original=rope.original_max_position_embeddings, fast=rope.beta_fast, slow=rope.beta_slow)
+    elif not isinstance(rope, DefaultRotaryEmbeddingsConfig) or rope.interleaved or rope.factor != 1.0:
+        raise ValueError(f"a layer entry cannot describe {rope}")
+    return rot

@@ -23,8 +23,8 @@ from ..layers.normalization import LayerNormConfigBase, RmsNormConfig
 from ..layers.rotary import rope_config_from_hf, rope_to_hf_dict, DefaultRotaryEmbeddingsConfig, RotaryEmbeddingsConfig
 from ..nn import Embedding, FusedRows, Linear
 from ..ops.gemm import linear_residual
-from ..ops.glu import gated_activation
-from ..ops.residual_stream import glu_of_rows, project
+from ..ops.glu import ClampedGlu, GatedActivation, gated_activation
+from ..ops.residual_stream import add_linear, glu_of_rows, project
 from ..utils.activation import ActivationFunctionEnum
 from ..utils.flop_utils import lm_flops_per_token
 from ..utils.remat import ScanCheckpointPolicy, checkpoint_layer, keeps_attention, should_recompute
@@ -151,7 +151,7 @@ def _getter(hf_config):
 class LlamaMlp(nn.Module):
     """SwiGLU MLP: ``down(act(gate(x)) * up(x))`` (src/levanter/models/llama.py:243-280)."""
 
-    def __init__(self, hidden: int, intermediate: int, activation: ActivationFunctionEnum, *, use_bias: bool = False,
+    def __init__(self, hidden: int, intermediate: int, activation: GatedActivation, *, use_bias: bool = False,
                  init_std: float = 0.02, tp=None):
         super().__init__()
         tp_size = tp.size if tp is not None else 1
@@ -161,23 +161,33 @@ class LlamaMlp(nn.Module):
         self.gate_proj = Linear(hidden, local, bias=use_bias, init_std=init_std, parallel=("column", tp))
         self.up_proj = Linear(hidden, local, bias=use_bias, init_std=init_std, parallel=("column", tp))
         self.down_proj = Linear(local, hidden, bias=use_bias, init_std=init_std, parallel=("row", tp))
-        self.act = activation if isinstance(activation, ActivationFunctionEnum) else ActivationFunctionEnum(activation)
+        self.act = activation if isinstance(activation, (ActivationFunctionEnum, ClampedGlu)) else ActivationFunctionEnum(activation)
         self._rows = FusedRows()
 
-    def forward_fp32(self, x: torch.Tensor) -> torch.Tensor:
-        """The MLP of packed rows ``x [T, hidden]`` in fp32 straight from the last product, for blocks whose output is normed before it
-        joins an fp32 stream; gate and up are one product when serving (no biases, tanh-gelu or any activation of ``ops.glu``)."""
+    def _inner(self, x: torch.Tensor) -> torch.Tensor:
+        """The gated activation of packed rows; gate and up are one product when serving (no biases)."""
         mods = (self.gate_proj, self.up_proj)
         w = None
         if all(type(m) is Linear and m.bias is None for m in mods) and x.is_cuda and not self.training and not torch.is_grad_enabled():
             w = self._rows.get([m.weight for m in mods])
         if w is not None:
-            h = glu_of_rows(project(x, w), self.gate_proj.weight.shape[0], self.act)
-        else:
-            h = gated_activation(self.gate_proj(x), self.up_proj(x), self.act)
+            return glu_of_rows(project(x, w), self.gate_proj.weight.shape[0], self.act)
+        return gated_activation(self.gate_proj(x), self.up_proj(x), self.act)
+
+    def forward_fp32(self, x: torch.Tensor) -> torch.Tensor:
+        """The MLP of packed rows ``x [T, hidden]`` in fp32 straight from the last product, for blocks whose output is normed before it
+        joins an fp32 stream."""
+        h = self._inner(x)
         if type(self.down_proj) is Linear:
             return project(h, self.down_proj.weight, bias=self.down_proj.bias, out_dtype=torch.float32)
         return self.down_proj(h).float()
+
+    def add_to_stream(self, stream: torch.Tensor, x: torch.Tensor, batch_info=None) -> torch.Tensor:
+        """``stream + mlp(x)`` on an fp32 stream, added in the epilogue of the last product."""
+        h = self._inner(x)
+        if type(self.down_proj) is Linear and self.down_proj.bias is None:
+            return add_linear(stream, h, self.down_proj.weight)
+        return stream + self.down_proj(h).float()
 
     def forward(self, x: torch.Tensor, residual: Optional[torch.Tensor] = None) -> torch.Tensor:
         if self.tp is not None and self.tp.size > 1:
@@ -367,3 +377,17 @@ class LlamaLMHeadModel(LmHeadModel):
     @staticmethod
     def hf_key_map() -> Dict[str, Optional[str]]:
         return {"transformer": "model", "embeddings": None, "token_embeddings": "model.embed_tokens"}
+
+
+class RecurrentLMHeadModel(LlamaLMHeadModel):
+    """The Llama head model with caches that hold state by sequence slot beside pages."""
+
+    def initial_cache(self, max_pages, page_size: Optional[int] = None, max_seqs: Optional[int] = None, *, dtype=torch.bfloat16, device=None):
+        """One cache per layer: pages, or recurrent state by sequence slot.  ``max_pages`` may be a page table (then its sizes are used)."""
+        if page_size is None and hasattr(max_pages, "num_pages"):
+            max_pages, page_size, max_seqs = max_pages.num_pages, max_pages.page_size, max_pages.max_seqs
+        if max_seqs is None:
+            raise ValueError("recurrent state is kept by sequence slot: give max_seqs, or a page table")
+        if device is None:
+            device = next(self.parameters()).device
+        return self.transformer.initial_cache(max_pages, page_size, max_seqs, dtype=dtype, device=device)

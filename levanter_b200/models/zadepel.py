@@ -34,7 +34,7 @@ from ..nn import Embedding
 from ..ops.residual_stream import add_norm_stream, embed_stream, project, rms_norm_stream
 from ..utils.activation import ActivationFunctionEnum
 from ..utils.remat import ScanCheckpointPolicy, should_recompute
-from .llama import LlamaLMHeadModel, LlamaMlp
+from .llama import LlamaMlp, RecurrentLMHeadModel
 from .lm_model import LmConfig
 
 MIXERS = ("attention", "latent_attention", "mingru")
@@ -300,7 +300,7 @@ class ZadepelEmbedding(nn.Module):
     forward = embed
 
 
-class ZadepelLMHeadModel(LlamaLMHeadModel):
+class ZadepelLMHeadModel(RecurrentLMHeadModel):
     """Shares the vocabulary handling of the Llama head model; the head is the embedding itself."""
 
     def __init__(self, vocab_size: int, config: ZadepelConfig, *, tp=None):
@@ -315,16 +315,6 @@ class ZadepelLMHeadModel(LlamaLMHeadModel):
 
     def activations(self, input_ids, attn_mask=None, *, pos_ids=None):
         return self.transformer(self.embeddings.embed(input_ids), attn_mask if attn_mask is not None else AttentionMask.causal(), pos_ids)
-
-    def initial_cache(self, max_pages, page_size: Optional[int] = None, max_seqs: Optional[int] = None, *, dtype=torch.bfloat16, device=None):
-        """One cache per layer: pages, or recurrent state by sequence slot.  ``max_pages`` may be a page table (then its sizes are used)."""
-        if page_size is None and hasattr(max_pages, "num_pages"):
-            max_pages, page_size, max_seqs = max_pages.num_pages, max_pages.page_size, max_pages.max_seqs
-        if max_seqs is None:
-            raise ValueError("recurrent state is kept by sequence slot: give max_seqs, or a page table")
-        if device is None:
-            device = next(self.parameters()).device
-        return self.transformer.initial_cache(max_pages, page_size, max_seqs, dtype=dtype, device=device)
 
     def decode(self, input_ids, kv_cache, batch_info, pos_ids, logit_rows: Optional[torch.Tensor] = None):
         x = self.embeddings.embed(input_ids)

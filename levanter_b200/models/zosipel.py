@@ -27,7 +27,7 @@ from ..layers.attention import (Attention, AttentionBackend, AttentionConfig, At
                                 MultiHeadLatentAttentionConfig)
 from ..layers.experts import GroupedSoftmaxMoe
 from ..layers.normalization import LayerNormConfigBase
-from ..layers.rotary import DefaultRotaryEmbeddingsConfig, PartialYarnRotaryEmbeddingsConfig, RotaryEmbeddingsConfig
+from ..layers.rotary import DefaultRotaryEmbeddingsConfig, RotaryEmbeddingsConfig, rope_from_entry, rope_to_entry
 from ..nn import Embedding, Linear
 from ..ops.residual_stream import embed_stream, project
 from ..utils.remat import ScanCheckpointPolicy, should_recompute
@@ -86,31 +86,12 @@ class ZosipelLayerConfig:
                 raise ValueError(f"{self.num_experts_per_tok} experts per token do not fit the kept groups")
 
 
-def _rope_from_checkpoint(rot: Optional[dict]) -> Optional[RotaryEmbeddingsConfig]:
-    if rot is None:
-        return None
-    s = rot.get("scaling")
-    if s is None:
-        return DefaultRotaryEmbeddingsConfig(theta=float(rot["base"]), rotary_dim=rot["dims"])
-    return PartialYarnRotaryEmbeddingsConfig(theta=float(rot["base"]), rotary_dim=rot["dims"], factor=float(s["factor"]), beta_fast=float(s["fast"]),
-                                             beta_slow=float(s["slow"]), original_max_position_embeddings=s["original"])
-
-
-def _rope_to_checkpoint(rope: RotaryEmbeddingsConfig, head_dim: int) -> dict:
-    rot = dict(base=rope.theta, dims=head_dim if rope.rotary_dim is None else rope.rotary_dim)
-    if isinstance(rope, PartialYarnRotaryEmbeddingsConfig):
-        rot["scaling"] = dict(factor=rope.factor, original=rope.original_max_position_embeddings, fast=rope.beta_fast, slow=rope.beta_slow)
-    elif not isinstance(rope, DefaultRotaryEmbeddingsConfig) or rope.interleaved or rope.factor != 1.0:
-        raise ValueError(f"a zosipel checkpoint cannot describe {rope}")
-    return rot
-
-
 def _layer_from_checkpoint(entry: dict) -> ZosipelLayerConfig:
     kind, m, f = entry["type"], entry["mixer"], entry.get("mlp")
     kw = dict(mixer=kind, num_heads=m["heads"], head_dim=m["dim"], v_head_dim=m["vdim"], attention_scale=float(m["scale"]), intermediate_dim=None)
     if kind == "attention":
         mask, cap = m.get("mask"), m.get("softcap")
-        kw.update(num_kv_heads=m["kv_heads"], rope=_rope_from_checkpoint(m.get("rot")), difference=float(m["diff"]),
+        kw.update(num_kv_heads=m["kv_heads"], rope=rope_from_entry(m.get("rot")), difference=float(m["diff"]),
                   soft_cap=None if cap is None else float(cap), sliding_window=None if mask is None else mask["size"])
     elif kind == "latent_attention":
         kw.update(kv_lora_rank=m["kv_rank"], rope=None)
@@ -129,7 +110,7 @@ def _layer_to_checkpoint(c: ZosipelLayerConfig) -> dict:
     if c.mixer == "attention":
         m.update(kv_heads=c.num_kv_heads, diff=c.difference)
         if c.rope is not None:
-            m["rot"] = _rope_to_checkpoint(c.rope, c.head_dim)
+            m["rot"] = rope_to_entry(c.rope, c.head_dim)
         if c.soft_cap is not None:
             m["softcap"] = c.soft_cap
         if c.sliding_window is not None:

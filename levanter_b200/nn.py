@@ -176,6 +176,33 @@ class RmsNorm(nn.Module):
         return rms_norm_stream(x, self.weight, self.eps, rows=rows)
 
 
+class GroupedRmsNorm(RmsNorm):
+    """:class:`RmsNorm` whose rows are split into ``groups`` equal consecutive parts with a root mean square each."""
+
+    def __init__(self, dim: int, groups: int, eps: float = 1e-6, device=None, dtype=None):
+        super().__init__(dim, eps=eps, device=device, dtype=dtype)
+        if groups <= 0 or dim % groups != 0:
+            raise ValueError(f"a row of {dim} elements has no {groups} equal groups")
+        self.groups = groups
+
+    def in_fp32(self, x: torch.Tensor) -> torch.Tensor:
+        from .ops.depth_stream import grouped_rms_norm
+
+        return grouped_rms_norm(x, self.weight, self.eps, self.groups)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.in_fp32(x).to(x.dtype)
+
+    def from_stream(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        from .ops.depth_stream import norm_of_depths
+
+        if torch.is_grad_enabled():
+            x = x if rows is None else x.index_select(0, rows.long())
+            return self.in_fp32(x).to(self.weight.dtype)
+        y = norm_of_depths(x.reshape(1, -1, self.dim), self.weight, self.eps, groups=self.groups, rows=rows)
+        return y.view_as(x) if rows is None else y
+
+
 class LayerNorm(nn.Module):
     def __init__(self, dim: int, eps: float = 1e-5, use_weight: bool = True, use_bias: bool = True, device=None, dtype=None):
         super().__init__()

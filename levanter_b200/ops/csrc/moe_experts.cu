@@ -31,8 +31,8 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n) {
   return at < n ? at : 0;
 }
 
-// kSoftmax: scores are the softmax over all experts, a group counts by its best score, and the weights are the chosen scores divided by
-// their sum.  Otherwise scores are sigmoids, a group counts by its two best choice scores, and the weights are scale * score.
+// kSoftmax: scores are the softmax over all experts of z + correction, a group counts by its best score, and the weights are the chosen
+// scores divided by their sum.  Otherwise scores are sigmoids, a group counts by its two best choice scores, and the weights are scale * score.
 template <bool kSoftmax>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict__ correction, int c_f32, const int* __restrict__ live,
@@ -49,18 +49,22 @@ route_kernel(const float* __restrict__ z, long long ldz, const void* __restrict_
     for (int j = lane; j < k; j += 32) { idx[static_cast<size_t>(t) * k + j] = -1; w[static_cast<size_t>(t) * k + j] = 0.f; }
     return;
   }
+  auto corrected = [&](float s, int e) { return correction != nullptr ? s + ldv(correction, c_f32, e) : s; };
   float top = -INFINITY, inv = 1.f;
   if constexpr (kSoftmax) {
-    for (int e = lane; e < E; e += 32) top = fmaxf(top, z[t * ldz + e]);
+    for (int e = lane; e < E; e += 32) {
+      s_score[e] = corrected(z[t * ldz + e], e);  // read back by this lane only
+      top = fmaxf(top, s_score[e]);
+    }
     top = warp_max(top);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(z[t * ldz + e] - top);
+    for (int e = lane; e < E; e += 32) sum += expf(s_score[e] - top);
     inv = 1.f / warp_sum(sum);
   }
   for (int e = lane; e < E; e += 32) {
-    const float s = kSoftmax ? expf(z[t * ldz + e] - top) * inv : 1.f / (1.f + expf(-z[t * ldz + e]));
+    const float s = kSoftmax ? expf(s_score[e] - top) * inv : 1.f / (1.f + expf(-z[t * ldz + e]));
     s_score[e] = s;
-    s_choice[e] = s + (correction != nullptr ? ldv(correction, c_f32, e) : 0.f);
+    s_choice[e] = kSoftmax ? s : corrected(s, e);
   }
   __syncwarp();
   if (groups > 1 && keep < groups) {
@@ -259,7 +263,7 @@ grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ B, T* __restri
 
 // Routing of z [T, E] fp32 (row stride ldz).  kind 0: choice score sigmoid(z) + correction (optional, fp32 or bf16 [E]); groups > 1: only
 // experts of the `keep` neighbour groups (E / groups experts each) with the largest sum of their two best choice scores can be
-// chosen; idx, w [T, k]: the k best choice scores, best first, and scale * sigmoid(z) of each.  kind 1: softmax(z) + correction, groups by
+// chosen; idx, w [T, k]: the k best choice scores, best first, and scale * sigmoid(z) of each.  kind 1: the softmax of z + correction, groups by
 // their best choice score, weights softmax(z) / (sum over the chosen + 1e-20).  live (optional) [T]: tokens with a value outside
 // [0, live_limit) are padding and get idx = -1.  counts: int32 [2 * E], cleared here; the first E receive the tokens per expert, the
 // rest are lvb_moe_dispatch's cursors.

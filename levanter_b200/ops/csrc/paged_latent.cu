@@ -484,6 +484,8 @@ struct ProductParams {
   __nv_bfloat16* out;
   long long lda, a_head, ldb, b_head, ldo, o_head;
   int T, N, K;
+  const __nv_bfloat16* gate;  // optional: the results of row t, head h are multiplied by the sigmoids of N numbers at gate + t * ldg + h * N
+  long long ldg;
 };
 
 // kTrans: B(h) is [N, K] (out = A B^T), else [K, N]
@@ -549,7 +551,14 @@ __global__ void __launch_bounds__(128) head_product_kernel(ProductParams p) {
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int t = t0 + warp * 16 + half * 8 + (lane >> 2);
-      if (t < p.T) *reinterpret_cast<uint32_t*>(p.out + t * p.ldo + h * p.o_head + n) = pack_bf16x2(acc[j][half * 2], acc[j][half * 2 + 1]);
+      if (t >= p.T) continue;
+      float a = acc[j][half * 2], b = acc[j][half * 2 + 1];
+      if (p.gate != nullptr) {
+        const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.gate + t * p.ldg + h * p.N + n));
+        a *= 1.f / (1.f + __expf(-g.x));
+        b *= 1.f / (1.f + __expf(-g.y));
+      }
+      *reinterpret_cast<uint32_t*>(p.out + t * p.ldo + h * p.o_head + n) = pack_bf16x2(a, b);
     }
   }
 }
@@ -625,18 +634,20 @@ extern "C" int lvb_paged_latent(const void* q, const void* kv_pages, const int* 
 }
 
 // out(t, h) [N] = A(t, h) [K] times B(h): [N, K] with b_trans, else [K, N].  A(t, h) starts at a + t * lda + h * a_head, B(h) at b + h * b_head (row
-// stride ldb), out(t, h) at out + t * ldo + h * o_head.  bf16; N, K, lda, a_head, ldb, b_head multiples of 8, ldo and o_head of 2, a and b
-// 16-byte aligned.
-extern "C" int lvb_head_product(const void* a, const void* b, void* out, int T, int H, int N, int K, long long lda, long long a_head, long long ldb,
-                                long long b_head, long long ldo, long long o_head, int b_trans, void* stream) {
+// stride ldb), out(t, h) at out + t * ldo + h * o_head.  bf16; N, K, lda, a_head, ldb, b_head multiples of 8, ldo, o_head and ldg of 2, a and b
+// 16-byte aligned.  gate: null, or rows of H * N numbers (stride ldg, 4-byte aligned) whose sigmoids multiply the results.
+extern "C" int lvb_head_product(const void* a, const void* b, void* out, const void* gate, int T, int H, int N, int K, long long lda,
+                                long long a_head, long long ldb, long long b_head, long long ldo, long long o_head, long long ldg, int b_trans,
+                                void* stream) {
   using namespace lvb;
   using namespace lvb::latent;
   if (T <= 0) return kErrOk;
   if (H <= 0 || N <= 0 || K <= 0 || ((N | K | lda | a_head | ldb | b_head) & 7) || ((ldo | o_head) & 1)) return kErrBadArg;
-  if (((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b)) & 15) || (reinterpret_cast<uintptr_t>(out) & 3)) return kErrBadArg;
+  if (((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b)) & 15) || ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate)) & 3) || (ldg & 1))
+    return kErrBadArg;
   if (H > 65535 || (T + kPT - 1) / kPT > 65535) return kErrTooLarge;
   ProductParams p{reinterpret_cast<const __nv_bfloat16*>(a), reinterpret_cast<const __nv_bfloat16*>(b), reinterpret_cast<__nv_bfloat16*>(out),
-                  lda, a_head, ldb, b_head, ldo, o_head, T, N, K};
+                  lda, a_head, ldb, b_head, ldo, o_head, T, N, K, reinterpret_cast<const __nv_bfloat16*>(gate), ldg};
   const dim3 grid((N + kPN - 1) / kPN, (T + kPT - 1) / kPT, H);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (b_trans) head_product_kernel<true><<<grid, 128, 0, s>>>(p);

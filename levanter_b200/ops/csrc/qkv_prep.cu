@@ -234,6 +234,12 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(LatentParams p) {
   float* s_sin = s_angles + p.rot.dims / 2;
   const int t = blockIdx.x;
   fill_angles(p.rot, p.pos[t], s_cos, s_sin);
+  if (p.down == nullptr) {  // the queries only
+    __syncthreads();
+    rotate_heads<T>(reinterpret_cast<const T*>(p.q_rot) + t * p.ldq, p.q_head, reinterpret_cast<T*>(p.q_out) + t * p.ldo, p.o_head,
+                    static_cast<T*>(nullptr), 0, 1, p.H, p.rotd, p.rot, s_cos, s_sin, nullptr, 0, p.vec_q != 0);
+    return;
+  }
   const long long dest = p.dests[t];
   const int width = p.rank + p.rotd;
   T* cache = dest >= 0 && dest < p.slots ? reinterpret_cast<T*>(p.kv_pages) + dest * width : nullptr;
@@ -291,7 +297,7 @@ __global__ void __launch_bounds__(kThreads) latent_norm_kernel(LatentParams p, i
   constexpr int kKeep = 4;  // groups of 8 columns per lane in registers
   const int t = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= rows) return;
-  const long long dest = p.dests[t];
+  const long long dest = p.dests != nullptr ? p.dests[t] : -1;
   T* cache = dest >= 0 && dest < p.slots ? reinterpret_cast<T*>(p.kv_pages) + dest * p.rank : nullptr;
   const T* down = reinterpret_cast<const T*>(p.down) + t * p.ldd;
   T* latent = p.latent != nullptr ? reinterpret_cast<T*>(p.latent) + static_cast<long long>(t) * p.rank : nullptr;
@@ -382,7 +388,7 @@ extern "C" int lvb_qkv_prep(void* q, void* k, void* v, const void* v_first, cons
 // Latent attention.  Row t of down (stride ldd) holds `rank` compressed dimensions and a key part of rot_dims dimensions shared by the
 // heads.  latent[t] = [RMS norm of the former with weight norm_w, the latter rotated], also written to slot dests[t] of kv_pages [slots,
 // rank + rot_dims]; head h's rotated query part goes from q_rot + t * ldq + h * q_head to q_out + t * ldo + h * o_head.  rot_dims 0: the norm and
-// the cache write only; latent may be null then.
+// the cache write only; latent may be null then, or dests (no cache write).  down null: the rotation of the queries only.
 extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* latent, void* kv_pages, const void* q_rot, void* q_out, const int* pos,
                                const int* dests, int T, int H, int rank, int rot_dims, long long ldd, long long ldq, long long q_head,
                                long long ldo, long long o_head, long long slots, float eps, const float* inv_freq, int interleaved,
@@ -390,8 +396,10 @@ extern "C" int lvb_latent_prep(const void* down, const void* norm_w, void* laten
   using namespace lvb;
   using namespace lvb::prep;
   if (T <= 0) return kErrOk;
-  if (H <= 0 || rank <= 0 || rot_dims < 0 || (rot_dims & 1)) return kErrBadArg;
-  if (rot_dims > 0 && (inv_freq == nullptr || pos == nullptr || latent == nullptr)) return kErrBadArg;
+  if (H <= 0 || rot_dims < 0 || (rot_dims & 1)) return kErrBadArg;
+  if (down == nullptr ? rot_dims == 0 : rank <= 0 || (rot_dims > 0 && (latent == nullptr || dests == nullptr)) || (latent == nullptr && dests == nullptr))
+    return kErrBadArg;
+  if (rot_dims > 0 && (inv_freq == nullptr || pos == nullptr)) return kErrBadArg;
   if (rot_dims > 4096) return kErrTooLarge;
   LatentParams p;
   p.down = down; p.norm_w = norm_w; p.latent = latent; p.kv_pages = kv_pages; p.q_rot = q_rot; p.q_out = q_out; p.pos = pos; p.dests = dests;

@@ -160,9 +160,15 @@ add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const long l
   }
 }
 
-// act(g) * u: tanh-gelu (0) or silu (1).  kFast: for results that are rounded to bf16.
+// act(g) * u: tanh-gelu (0) or silu (1); or (2) g sigmoid(1.702 g) (u + 1) with g at most `limit` and u within +-limit.  kFast: for results that
+// are rounded to bf16.
 template <bool kFast>
-__device__ __forceinline__ float glu(int act, float g, float u) {
+__device__ __forceinline__ float glu(int act, float limit, float g, float u) {
+  if (act == 2) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.f;
+    return kFast ? g * u * __fdividef(1.f, 1.f + __expf(-1.702f * g)) : g / (1.f + expf(-1.702f * g)) * u;
+  }
   if (act == 1) return kFast ? g * u * __fdividef(1.f, 1.f + __expf(-g)) : g / (1.f + expf(-g)) * u;
   return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
@@ -170,8 +176,8 @@ __device__ __forceinline__ float glu(int act, float g, float u) {
 // out[r, c] = act(gate[r, c]) * up[r, c] (* sigmoid(row_gate[r * ldr])), any size; gate and up of one type, out of that type or bf16
 template <bool kOutF32>
 __global__ void __launch_bounds__(256)
-glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const float* __restrict__ row_gate, void* __restrict__ out, int act, int f32,
-           long long total, int cols, long long ldg, long long ldu, long long ldr, int vec) {
+glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const float* __restrict__ row_gate, void* __restrict__ out, int act, float limit,
+           int f32, long long total, int cols, long long ldg, long long ldu, long long ldr, int vec) {
   auto factor = [&](long long r) { return row_gate != nullptr ? 1.f / (1.f + expf(-row_gate[r * ldr])) : 1.f; };
   const long long step = static_cast<long long>(gridDim.x) * blockDim.x;
   if (vec) {  // groups of 4 columns; cols is a multiple of 4
@@ -180,8 +186,8 @@ glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const flo
       const long long r = i / per, c = (i - r * per) * 4;
       const float4 g = ld4(gate, f32, r * ldg + c), u = ld4(up, f32, r * ldu + c);
       const float f = factor(r);
-      const float4 o = make_float4(glu<!kOutF32>(act, g.x, u.x) * f, glu<!kOutF32>(act, g.y, u.y) * f, glu<!kOutF32>(act, g.z, u.z) * f,
-                                   glu<!kOutF32>(act, g.w, u.w) * f);
+      const float4 o = make_float4(glu<!kOutF32>(act, limit, g.x, u.x) * f, glu<!kOutF32>(act, limit, g.y, u.y) * f, glu<!kOutF32>(act, limit, g.z, u.z) * f,
+                                   glu<!kOutF32>(act, limit, g.w, u.w) * f);
       if constexpr (kOutF32) reinterpret_cast<float4*>(out)[i] = o;
       else reinterpret_cast<uint2*>(out)[i] = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
     }
@@ -189,7 +195,7 @@ glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const flo
   }
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += step) {
     const long long r = i / cols, c = i - r * cols;
-    const float o = glu<!kOutF32>(act, ld1(gate, f32, r * ldg + c), ld1(up, f32, r * ldu + c)) * factor(r);
+    const float o = glu<!kOutF32>(act, limit, ld1(gate, f32, r * ldg + c), ld1(up, f32, r * ldu + c)) * factor(r);
     if constexpr (kOutF32) reinterpret_cast<float*>(out)[i] = o;
     else reinterpret_cast<__nv_bfloat16*>(out)[i] = __float2bfloat16(o);
   }
@@ -245,19 +251,20 @@ extern "C" int lvb_add_norm_stream(float* x, const float* y, const long long* ro
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
-// out [rows, cols] = act(gate) * up (* the sigmoid of row_gate[r * ldr], fp32, when given) with act = tanh-gelu (0) or silu (1); gate and up with row
-// strides ldg and ldu; in_f32, out_f32: types (fp32 results need fp32 operands).
-extern "C" int lvb_glu_any(const void* gate, const void* up, const float* row_gate, void* out, int act, int in_f32, int out_f32, int rows, int cols,
-                           long long ldg, long long ldu, long long ldr, void* stream) {
+// out [rows, cols] = act(gate) * up (* the sigmoid of row_gate[r * ldr], fp32, when given) with act = tanh-gelu (0), silu (1) or the clamped form
+// (2: min(gate, limit) sigmoid(1.702 min(gate, limit)) (clamp(up, -limit, limit) + 1)); gate and up with row strides ldg and ldu; in_f32, out_f32:
+// types (fp32 results need fp32 operands).
+extern "C" int lvb_glu_any(const void* gate, const void* up, const float* row_gate, void* out, int act, float limit, int in_f32, int out_f32, int rows,
+                           int cols, long long ldg, long long ldu, long long ldr, void* stream) {
   using namespace lvb;
-  if (rows <= 0 || cols <= 0 || act < 0 || act > 1 || (out_f32 && !in_f32)) return kErrBadArg;
+  if (rows <= 0 || cols <= 0 || act < 0 || act > 2 || (out_f32 && !in_f32)) return kErrBadArg;
   const uintptr_t mis = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out);
   const int vec = ((cols | ldg | ldu) & 3) == 0 && (mis & 15) == 0;
   const long long total = static_cast<long long>(rows) * cols, cap = static_cast<long long>(num_sms()) * 16;
   long long blocks = (total / (vec ? 4 : 1) + 255) / 256;
   if (blocks > cap) blocks = cap;
   auto kern = out_f32 ? stream32::glu_kernel<true> : stream32::glu_kernel<false>;
-  kern<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, row_gate, out, act, in_f32, total, cols, ldg, ldu, ldr,
+  kern<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, row_gate, out, act, limit, in_f32, total, cols, ldg, ldu, ldr,
                                                                                    vec);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }

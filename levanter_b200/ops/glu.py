@@ -2,6 +2,9 @@
 (src/levanter/models/llama.py:273-280)."""
 from __future__ import annotations
 
+from dataclasses import dataclass
+from typing import Union
+
 import torch
 
 from . import lib
@@ -12,6 +15,21 @@ _ACT = {
     ActivationFunctionEnum.gelu: 2, ActivationFunctionEnum.relu: 3, ActivationFunctionEnum.quick_gelu: 4,
 }
 _f = {}
+
+
+@dataclass(frozen=True)
+class ClampedGlu:
+    """A gated activation with bounded inputs, for where an activation of the gate alone is expected: ``g sigmoid(1.702 g) (u + 1)`` with ``g =
+    min(gate, limit)`` and ``u = clamp(up, -limit, limit)``."""
+
+    limit: float
+
+    def __call__(self, gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+        g, u = gate.float().clamp(max=self.limit), up.float().clamp(-self.limit, self.limit)
+        return (g * torch.sigmoid(1.702 * g) * (u + 1.0)).to(gate.dtype)
+
+
+GatedActivation = Union[ActivationFunctionEnum, ClampedGlu]
 
 
 def _fwd():
@@ -62,7 +80,9 @@ class _GluFn(torch.autograd.Function):
         return dg.view(ctx.shape), du.view(ctx.shape), None
 
 
-def gated_activation(gate: torch.Tensor, up: torch.Tensor, act: ActivationFunctionEnum) -> torch.Tensor:
+def gated_activation(gate: torch.Tensor, up: torch.Tensor, act: GatedActivation) -> torch.Tensor:
+    if isinstance(act, ClampedGlu):
+        return act(gate, up)
     act = ActivationFunctionEnum(act) if not isinstance(act, ActivationFunctionEnum) else act
     if (gate.is_cuda and lib.available() and gate.dtype == torch.bfloat16 and up.dtype == torch.bfloat16
             and gate.shape[-1] % 8 == 0 and act in _ACT):

@@ -10,7 +10,7 @@ import torch
 
 from ..utils.activation import ActivationFunctionEnum
 from .gemm import linear
-from .glu import gated_activation
+from .glu import GatedActivation, gated_activation
 
 
 def grouped_mlp(x_sorted: torch.Tensor, group_sizes: torch.Tensor, w1: torch.Tensor, w3: torch.Tensor, w2: torch.Tensor,
@@ -263,9 +263,9 @@ def route_sigmoid_reference(logits: torch.Tensor, correction, k: int, groups: in
     return idx, s.gather(1, idx) * scale
 
 
-def route_softmax_reference(logits: torch.Tensor, k: int, groups: int, keep: int):
+def route_softmax_reference(logits: torch.Tensor, k: int, groups: int, keep: int, bias=None):
     """``(idx[T, k], w[T, k])``: see :func:`route_softmax`.  Differentiable in the weights."""
-    s = torch.softmax(logits.float(), dim=-1)
+    s = torch.softmax(logits.float() if bias is None else logits.float() + bias.float(), dim=-1)
     idx = _within_groups(s.detach(), groups, keep, 1).topk(k, dim=-1).indices
     w = s.gather(1, idx)
     return idx, w / (w.sum(-1, keepdim=True) + 1e-20)
@@ -283,7 +283,7 @@ def _route(kind: int, logits, correction, k, groups, keep, scale, live, live_lim
 
     T, E = logits.shape
     if not (logits.is_cuda and lib.available()):
-        idx, w = route_softmax_reference(logits, k, groups, keep) if kind else route_sigmoid_reference(logits, correction, k, groups, keep, scale)
+        idx, w = route_softmax_reference(logits, k, groups, keep, correction) if kind else route_sigmoid_reference(logits, correction, k, groups, keep, scale)
         idx = idx.to(torch.int32)
         if live is not None:
             dead = (live < 0) | (live >= live_limit)
@@ -314,11 +314,11 @@ def route_sigmoid(logits: torch.Tensor, correction, k: int, *, groups: int = 1, 
     return _route(0, logits, correction, k, groups, keep, scale, live, live_limit)
 
 
-def route_softmax(logits: torch.Tensor, k: int, *, groups: int = 1, keep: int = 1, live=None, live_limit: int = 0) -> RoutedTokens:
-    """Routing of fp32 ``logits [T, E]`` (rows may be strided): the ``k`` experts with the largest softmax scores among those of the ``keep``
-    (of ``groups``) neighbour groups whose best score is largest; weights are the chosen scores divided by their sum.  ``live`` as in
-    :func:`route_sigmoid`."""
-    return _route(1, logits, None, k, groups, keep, 1.0, live, live_limit)
+def route_softmax(logits: torch.Tensor, k: int, *, groups: int = 1, keep: int = 1, bias=None, live=None, live_limit: int = 0) -> RoutedTokens:
+    """Routing of fp32 ``logits [T, E]`` (rows may be strided; plus ``bias [E]``): the ``k`` experts with the largest softmax scores among those
+    of the ``keep`` (of ``groups``) neighbour groups whose best score is largest; weights are the chosen scores divided by their sum, which is
+    the softmax over the chosen logits.  ``live`` as in :func:`route_sigmoid`."""
+    return _route(1, logits, bias, k, groups, keep, 1.0, live, live_limit)
 
 
 def _block_rows(pairs: int, experts: int) -> int:
@@ -357,9 +357,9 @@ def grouped_product(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, 
 
 
 def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedTokens, up: torch.Tensor, down: torch.Tensor, *,
-                       gated: bool = False) -> torch.Tensor:
+                       gated: bool = False, act: GatedActivation = ActivationFunctionEnum.silu) -> torch.Tensor:
     """``stream[t] += sum_j w[t, j] * down[e] relu(up[e] h[t])^2`` with ``e = idx[t, j]``, in place on the fp32 stream; ``up [E, ff, width]``,
-    ``down [E, width, ff]``.  ``gated``: ``up [E, 2 ff, width]`` holds a gate and an up projection, and the inner layer is ``silu(gate h) *
+    ``down [E, width, ff]``.  ``gated``: ``up [E, 2 ff, width]`` holds a gate and an up projection, and the inner layer is ``act(gate h) *
     (up h)``.  Forward only, CUDA only: dispatch into the block-padded expert-sorted layout, two grouped products (the
     activation in the epilogue of the first, or a gated activation between them), combine."""
     from . import lib
@@ -385,14 +385,15 @@ def add_expert_outputs(stream: torch.Tensor, h: torch.Tensor, routed: RoutedToke
 
     a = grouped_product(x_pad, up.to(h.dtype), tile_group, rows, not gated)
     if gated:
-        a = glu_of_rows(a, ff, ActivationFunctionEnum.silu)
+        a = glu_of_rows(a, ff, act)
     y = grouped_product(a, down.to(h.dtype), tile_group, rows, False)
     rc = _g["c"](y.data_ptr(), int(y.dtype == torch.float32), dest.data_ptr(), routed.w.data_ptr(), T, k, width, stream.data_ptr(), lib.stream_ptr())
     lib.check_rc(rc, "lvb_moe_combine")
     return stream
 
 
-def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torch.Tensor, down: torch.Tensor, *, gated: bool = False) -> torch.Tensor:
+def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torch.Tensor, down: torch.Tensor, *, gated: bool = False,
+                   act: GatedActivation = ActivationFunctionEnum.silu) -> torch.Tensor:
     """The sum :func:`add_expert_outputs` adds, as differentiable framework ops (training, and the CPU path): ``[T, width]`` fp32."""
     T, k = idx.shape
     keep = idx >= 0
@@ -400,7 +401,7 @@ def expert_outputs(h: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, up: torc
     x_pad = h.new_zeros(capacity, h.shape[1]).index_copy(0, dest, h.repeat_interleave(k, dim=0))
     a = grouped_linear(x_pad, up.to(h.dtype), tile_group, offsets)
     if gated:
-        a = gated_activation(a[:, :down.shape[2]], a[:, down.shape[2]:], ActivationFunctionEnum.silu)
+        a = gated_activation(a[:, :down.shape[2]], a[:, down.shape[2]:], act)
     else:
         a = torch.relu(a).square()
     y = grouped_linear(a, down.to(h.dtype), tile_group, offsets).index_select(0, dest).view(T, k, -1)

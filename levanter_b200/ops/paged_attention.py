@@ -308,22 +308,25 @@ def paged_attention_latent(q: torch.Tensor, kv_pages: torch.Tensor, rank: int, b
     return out
 
 
-def head_product(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, *, b_trans: bool) -> torch.Tensor:
+def head_product(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, *, b_trans: bool, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[t, h] = a[t, h] b[h]`` (``b [H, K, N]``) or ``a[t, h] b[h]^T`` (``b_trans``, ``b [H, N, K]``) for ``a [T, H, K]``, written into
-    ``out [T, H, N]``; all three may be strided views with packed last dimensions."""
+    ``out [T, H, N]``; all three may be strided views with packed last dimensions.  ``gate [T, H * N]``: the result is multiplied by its
+    sigmoid."""
     T, H, K = a.shape
     N = out.shape[2]
     kernel = (_use_kernel(a, b, out) and a.dtype == b.dtype == out.dtype == torch.bfloat16 and a.stride(2) == b.stride(2) == out.stride(2) == 1
               and not any(v % 8 for v in (N, K, a.stride(0), a.stride(1), b.stride(0), b.stride(1), out.stride(0), out.stride(1)))
-              and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0)
+              and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0
+              and (gate is None or (gate.dtype == a.dtype and gate.stride(1) == 1 and gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0)))
     if not kernel:
-        out.copy_(torch.matmul(a.transpose(0, 1), b.transpose(1, 2) if b_trans else b).transpose(0, 1))
+        y = torch.matmul(a.transpose(0, 1), b.transpose(1, 2) if b_trans else b).transpose(0, 1)
+        out.copy_(y if gate is None else _apply_gate(y.float(), gate))
         return out
     c = lib
     if "hp" not in _f:
-        _f["hp"] = lib.fn("lvb_head_product", [c.c_void_p] * 3 + [c.c_int] * 4 + [c.c_longlong] * 6 + [c.c_int, c.c_void_p])
-    rc = _f["hp"](a.data_ptr(), b.data_ptr(), out.data_ptr(), T, H, N, K, a.stride(0), a.stride(1), b.stride(1), b.stride(0), out.stride(0), out.stride(1),
-                  int(b_trans), lib.stream_ptr())
+        _f["hp"] = lib.fn("lvb_head_product", [c.c_void_p] * 4 + [c.c_int] * 4 + [c.c_longlong] * 7 + [c.c_int, c.c_void_p])
+    rc = _f["hp"](a.data_ptr(), b.data_ptr(), out.data_ptr(), lib.ptr(gate), T, H, N, K, a.stride(0), a.stride(1), b.stride(1), b.stride(0), out.stride(0),
+                  out.stride(1), 0 if gate is None else gate.stride(0), int(b_trans), lib.stream_ptr())
     lib.check_rc(rc, "lvb_head_product")
     return out
 

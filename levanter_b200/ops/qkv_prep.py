@@ -75,6 +75,14 @@ def prepare_qkv(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kv_pages: tor
     return qf.to(dt), k, v
 
 
+def _latent_fn():
+    if "l" not in _f:
+        c = lib
+        _f["l"] = lib.fn("lvb_latent_prep", [c.c_void_p] * 8 + [c.c_int] * 4 + [c.c_longlong] * 6 + [c.c_float, c.c_void_p, c.c_int, c.c_float, c.c_float,
+                                                                                                   c.c_int, c.c_int, c.c_void_p])
+    return _f["l"]
+
+
 def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv_pages: torch.Tensor, dests: torch.Tensor, pos: torch.Tensor,
                    rot: Optional[RotaryEmbeddings], q_rot: torch.Tensor, q_out: Optional[torch.Tensor] = None,
                    to_cache_only: bool = False) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
@@ -89,14 +97,10 @@ def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv
     assert (rot.rotary_dim if rot is not None else 0) == r, "the shared key part is rotated as a whole"
     if _kernel(down, norm_weight, kv_pages, q_rot, dst) and q_rot.dtype == dst.dtype == kv_pages.dtype == dt and down.stride(1) == 1 \
             and norm_weight.dtype in (torch.bfloat16, torch.float32) and q_rot.stride(2) == dst.stride(2) == 1:
-        c = lib
-        if "l" not in _f:
-            _f["l"] = lib.fn("lvb_latent_prep", [c.c_void_p] * 8 + [c.c_int] * 4 + [c.c_longlong] * 6 + [c.c_float, c.c_void_p, c.c_int, c.c_float, c.c_float,
-                                                                                                       c.c_int, c.c_int, c.c_void_p])
         latent = None if to_cache_only and rot is None else torch.empty(T, width, dtype=dt, device=down.device)
         d, p, w = _i32(dests), _i32(pos), norm_weight.contiguous()
         freq, dims, inter, pscale, mag = _rotation_args(rot, down.device)
-        rc = _f["l"](down.data_ptr(), w.data_ptr(), lib.ptr(latent), kv_pages.data_ptr(), q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), d.data_ptr(), T,
+        rc = _latent_fn()(down.data_ptr(), w.data_ptr(), lib.ptr(latent), kv_pages.data_ptr(), q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), d.data_ptr(), T,
                      q_rot.shape[1], rank, r, down.stride(0), q_rot.stride(0), q_rot.stride(1), dst.stride(0), dst.stride(1),
                      kv_pages.shape[0] * kv_pages.shape[1], float(eps), freq, inter, pscale, mag, int(dt == torch.float32), int(w.dtype == torch.float32),
                      lib.stream_ptr())
@@ -111,3 +115,33 @@ def prepare_latent(down: torch.Tensor, norm_weight: torch.Tensor, eps: float, kv
     if rot is not None:
         dst.copy_(rot(q_rot, pos))
     return latent, dst
+
+
+def rotate_queries(q_rot: torch.Tensor, pos: torch.Tensor, rot: RotaryEmbeddings, q_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The query half of :func:`prepare_latent`, for layers that read rows which another layer has cached: ``q_rot [T, H, r]`` rotated at ``pos``
+    into ``q_out`` (None: in place)."""
+    T, H, r = q_rot.shape
+    dst = q_rot if q_out is None else q_out
+    assert rot.rotary_dim == r
+    if _kernel(q_rot, dst) and q_rot.dtype == dst.dtype and q_rot.stride(2) == dst.stride(2) == 1:
+        p = _i32(pos)
+        freq, _, inter, pscale, mag = _rotation_args(rot, q_rot.device)
+        rc = _latent_fn()(0, 0, 0, 0, q_rot.data_ptr(), dst.data_ptr(), p.data_ptr(), 0, T, H, 0, r, 0, q_rot.stride(0), q_rot.stride(1), dst.stride(0),
+                          dst.stride(1), 0, 0.0, freq, inter, pscale, mag, int(q_rot.dtype == torch.float32), 0, lib.stream_ptr())
+        lib.check_rc(rc, "lvb_latent_prep")
+        return dst
+    dst.copy_(rot(q_rot, pos))
+    return dst
+
+
+def norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """RMS norm of ``x [T, width]``, a slice of wider rows (a compressed row on its way to the next projection) -> ``[T, width]`` packed."""
+    T, width = x.shape
+    if _kernel(x, weight) and x.stride(1) == 1 and weight.dtype in (torch.bfloat16, torch.float32):
+        y, w = torch.empty(T, width, dtype=x.dtype, device=x.device), weight.contiguous()
+        rc = _latent_fn()(x.data_ptr(), w.data_ptr(), y.data_ptr(), 0, 0, 0, 0, 0, T, 1, width, 0, x.stride(0), 0, 0, 0, 0, 0, float(eps), 0, 0, 1.0, 1.0,
+                          int(x.dtype == torch.float32), int(w.dtype == torch.float32), lib.stream_ptr())
+        lib.check_rc(rc, "lvb_latent_prep")
+        return y
+    f = x.float()
+    return (f * torch.rsqrt(f.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(x.dtype)

@@ -14,7 +14,7 @@ import torch
 from ..utils.activation import ActivationFunctionEnum
 from . import lib
 from .gemm import gemm, linear
-from .glu import gated_activation
+from .glu import ClampedGlu, GatedActivation, gated_activation
 
 _f = {}
 
@@ -24,8 +24,8 @@ def _kernels(*tensors) -> bool:
     return not torch.is_grad_enabled() and all(t.is_cuda for t in tensors) and lib.available()
 
 
-def embed_stream(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch.Tensor:
-    """``scale * weight[ids]`` in fp32."""
+def embed_stream(ids: torch.Tensor, weight: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``scale * weight[ids]`` in fp32.  ``out``: where to (serving; contiguous fp32 rows)."""
     if _kernels(ids, weight) and weight.dtype in (torch.float32, torch.bfloat16) and weight.is_contiguous():
         c = lib
         if "e" not in _f:
@@ -33,12 +33,13 @@ def embed_stream(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch
                                                   c.c_void_p, c.c_void_p])
         flat = ids.reshape(-1).to(torch.int32).contiguous()
         V, D = weight.shape
-        out = torch.empty(flat.numel(), D, dtype=torch.float32, device=weight.device)
+        out = torch.empty(flat.numel(), D, dtype=torch.float32, device=weight.device) if out is None else out
         rc = _f["e"](flat.data_ptr(), weight.data_ptr(), int(weight.dtype == torch.float32), out.data_ptr(), flat.numel(), D, V, float(scale),
                      lib.status_buffer().data_ptr(), lib.stream_ptr())
         lib.check_rc(rc, "lvb_embed_stream")
         return out.view(*ids.shape, D)
-    return torch.nn.functional.embedding(ids.long(), weight).float() * scale
+    x = torch.nn.functional.embedding(ids.long(), weight).float() * scale
+    return x if out is None else out.copy_(x.view_as(out)).view_as(x)
 
 
 def rms_norm_stream(x: torch.Tensor, weight: torch.Tensor, eps: float, *, w_offset: float = 0.0, out_dtype: Optional[torch.dtype] = None,
@@ -101,22 +102,23 @@ def add_norm_stream(x: torch.Tensor, y: torch.Tensor, w_post: torch.Tensor, w_ne
 _GLU_ANY = {ActivationFunctionEnum.gelu_new: 0, ActivationFunctionEnum.silu: 1, ActivationFunctionEnum.swish: 1}
 
 
-def glu_of_rows(y: torch.Tensor, cols: int, act: ActivationFunctionEnum, *, gate_logit: Optional[torch.Tensor] = None,
+def glu_of_rows(y: torch.Tensor, cols: int, act: GatedActivation, *, gate_logit: Optional[torch.Tensor] = None,
                 out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """``act(y[:, :cols]) * y[:, cols:2 * cols]`` of the joint product of a gate and an up projection, in ``out_dtype`` (default: ``y``'s).
     ``gate_logit [rows]``: every row is also multiplied by the sigmoid of its number."""
     gate, up = y[:, :cols], y[:, cols:2 * cols]
     dt = out_dtype or y.dtype
     plain = gate_logit is None and dt == y.dtype == torch.bfloat16 and cols % 8 == 0 and y.stride(0) % 8 == 0 and y.data_ptr() % 16 == 0
-    if act in _GLU_ANY and _kernels(y) and not plain \
+    clamped = isinstance(act, ClampedGlu)
+    if (clamped or (act in _GLU_ANY and not plain)) and _kernels(y) \
             and y.dtype in (torch.float32, torch.bfloat16) and dt in (y.dtype, torch.bfloat16) and y.stride(1) == 1 \
             and (gate_logit is None or gate_logit.dtype == torch.float32):
         c = lib
         if "g" not in _f:
-            _f["g"] = lib.fn("lvb_glu_any", [c.c_void_p] * 4 + [c.c_int] * 5 + [c.c_longlong] * 3 + [c.c_void_p])
+            _f["g"] = lib.fn("lvb_glu_any", [c.c_void_p] * 4 + [c.c_int, c.c_float] + [c.c_int] * 4 + [c.c_longlong] * 3 + [c.c_void_p])
         out = torch.empty(y.shape[0], cols, dtype=dt, device=y.device)
-        rc = _f["g"](gate.data_ptr(), up.data_ptr(), lib.ptr(gate_logit), out.data_ptr(), _GLU_ANY[act], int(y.dtype == torch.float32),
-                     int(dt == torch.float32), y.shape[0], cols, y.stride(0), y.stride(0), 0 if gate_logit is None else gate_logit.stride(0), lib.stream_ptr())
+        rc = _f["g"](gate.data_ptr(), up.data_ptr(), lib.ptr(gate_logit), out.data_ptr(), 2 if clamped else _GLU_ANY[act],
+                     act.limit if clamped else 0.0, int(y.dtype == torch.float32), int(dt == torch.float32), y.shape[0], cols, y.stride(0), y.stride(0), 0 if gate_logit is None else gate_logit.stride(0), lib.stream_ptr())
         lib.check_rc(rc, "lvb_glu_any")
         return out
     out = gated_activation(gate, up, act)
