@@ -44,10 +44,10 @@ def parse_args():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
-    ap.add_argument("--mode", default="train", choices=["train", "decode", "fedolorn", "zadepel", "zosipel"],
+    ap.add_argument("--mode", default="train", choices=["train", "decode", "fedolorn", "zadepel", "zosipel", "mumizen"],
                     help="train: the headline; decode: the inference engine serving Llama-3 8B, tensor parallel over the GPUs (a second metric: "
                          "prefill and decode tokens/s at 256 concurrent requests, prompts U[128, 2048], 256 greedy tokens, 16-token pages); "
-                         "fedolorn, zadepel, zosipel: prefill and decode throughput of that design beside the closest model at equal size, and its kernels "
+                         "fedolorn, zadepel, zosipel, mumizen: prefill and decode throughput of that design beside the closest model at equal size, and its kernels "
                          "beside the like kernels")
     ap.add_argument("--requests", type=int, default=256, help="decode mode: concurrent requests")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "torch_baseline"])
@@ -380,6 +380,22 @@ def main_zosipel(args):
     return 0
 
 
+def main_mumizen(args):
+    """Serving throughput of Mumizen beside Zadepel (dense) and Zosipel (mixtures of experts) at equal size, then its serving kernels beside the
+    like kernels of the closest models."""
+    from levanter_b200.inference import bench_mumizen
+
+    sampler = ClockSampler(_env()[2])
+    sampler.start()
+    runs = _serving_runs(("zadepel_8b", "mumizen_8b", "zosipel_moe", "mumizen_moe"), args.steps)
+    table = bench_mumizen.kernel_table()
+    best = max(r["decode_tokens_per_s"] for r in runs if r["model"] == "mumizen_8b")
+    print(json.dumps({"metric": "decode tokens/sec (inference engine, Mumizen at the size of Zadepel 8B)", "value": best, "unit": "tokens/s", "n_gpus": 1,
+                      "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic uniform-random prompts, random-init weights",
+                      "mode": "mumizen", "impl": "ours", "runs": runs, "clocks": sampler.stop(), **table}))
+    return 0
+
+
 def main_fedolorn(args):
     """Serving throughput of Fedolorn beside Llama-3 8B at equal size, and of its mixture-of-experts form; then every serving kernel beside
     the like kernel of the closest model."""
@@ -408,6 +424,8 @@ def main():
         return main_zadepel(args)
     if args.mode == "zosipel":
         return main_zosipel(args)
+    if args.mode == "mumizen":
+        return main_mumizen(args)
     if args.impl == "torch_baseline":
         return main_torch_baseline(args)
 

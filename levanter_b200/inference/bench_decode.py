@@ -42,6 +42,14 @@ MODELS = {
                          attention=dict(num_heads=4, num_kv_heads=2, head_dim=32, v_head_dim=64, attention_scale=0.18, sliding_window=96, soft_cap=20.0),
                          latent=dict(num_heads=4, head_dim=48, v_head_dim=32, kv_lora_rank=64, attention_scale=0.15),
                          moe=dict(num_experts=8, num_experts_per_tok=2, expert_groups=4, expert_groups_kept=2)),
+    # Mumizen at the size of zadepel_8b and, with mixtures, of zosipel_moe (as many layers as that has layer runs): a group of four layers is
+    # lightning, latent attention, retention, latent attention that reads the latents of the other
+    "mumizen_8b": dict(family="mumizen", hidden_dim=4096, num_layers=32, intermediate_dim=14336, vocab=128256),
+    "mumizen_moe": dict(family="mumizen", hidden_dim=4096, num_layers=16, intermediate_dim=1024, vocab=128256,
+                        moe=dict(num_experts=64, num_experts_per_tok=8, shared_intermediate_dim=2048)),
+    "tiny_mumizen": dict(family="mumizen", hidden_dim=256, num_layers=6, intermediate_dim=64, vocab=1024, linear=(4, 64),
+                         latent=dict(num_heads=4, head_dim=48, rotary_dim=16, v_head_dim=32, q_lora_rank=96, kv_lora_rank=64, attention_scale=0.125),
+                         moe=dict(num_experts=8, num_experts_per_tok=2, shared_intermediate_dim=96)),
     "tiny": dict(hidden_dim=256, intermediate_dim=512, num_layers=2, num_heads=4, num_kv_heads=2, vocab=1024),
 }
 
@@ -78,6 +86,19 @@ def model_config(m: dict, seq_len: int):
         start, stop, times = m["loop"] if m["num_layers"] >= m["loop"][1] else (0, 0, 0)
         return ZosipelConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], gradient_checkpointing=False, loop_start=start, loop_stop=stop, loop_times=times,
                              layers=tuple(layers[i % 4 == 2] for i in range(m["num_layers"])))
+    if family == "mumizen":
+        from ..layers.rotary import PartialYarnRotaryEmbeddingsConfig
+        from ..models.mumizen import MumizenConfig, MumizenLayerConfig
+
+        ff = dict(intermediate_dim=m["intermediate_dim"], **m.get("moe", {}))
+        heads, d = m.get("linear", (32, 128))
+        linear = dict(num_heads=heads, head_dim=d, v_head_dim=d, decay=tuple(1.0 - 2.0 ** (-3.0 - 5.0 * i / heads) for i in range(heads)), **ff)
+        rope = PartialYarnRotaryEmbeddingsConfig(theta=500000.0, factor=4.0, original_max_position_embeddings=2048)
+        latent = dict(mixer="latent_attention", rope=rope, **m.get("latent", dict(num_heads=32, head_dim=128, rotary_dim=64, v_head_dim=128, q_lora_rank=1536,
+                                                                                  kv_lora_rank=512, attention_scale=192 ** -0.5)), **ff)
+        group = [MumizenLayerConfig(mixer="lightning", **linear), MumizenLayerConfig(**latent), MumizenLayerConfig(mixer="retention", **linear), None]
+        layers = [group[i % 4] or MumizenLayerConfig(kv_from=i - 2, **latent) for i in range(m["num_layers"])]
+        return MumizenConfig(seq_len=seq_len, hidden_dim=m["hidden_dim"], norm_groups=8, gradient_checkpointing=False, layers=tuple(layers))
     from ..models.fedolorn import FedolornConfig, FedolornLayerConfig
 
     layer = FedolornLayerConfig(intermediate_dim=m["intermediate_dim"], **m.get("heads", {}), **m.get("moe", {}))

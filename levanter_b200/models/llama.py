@@ -184,7 +184,7 @@ class LlamaMlp(nn.Module):
 
     def add_to_stream(self, stream: torch.Tensor, x: torch.Tensor, batch_info=None) -> torch.Tensor:
         """``stream + mlp(x)`` on an fp32 stream, added in the epilogue of the last product."""
-        h = self._inner(x)
+        h = self._inner(x.reshape(-1, x.shape[-1])).view(*x.shape[:-1], -1)
         if type(self.down_proj) is Linear and self.down_proj.bias is None:
             return add_linear(stream, h, self.down_proj.weight)
         return stream + self.down_proj(h).float()
