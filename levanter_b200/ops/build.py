@@ -25,11 +25,13 @@ LIBNAME = "liblevanter_b200.so"
 # own, so that the first run in a fresh checkout compiles these sources and no others.
 SERVING_LIBNAME = "liblevanter_b200_serving.so"
 SERVING_SOURCES = ("attention_any", "depth_stream", "elementwise", "flash_attn_fwd2", "gated_scan", "gemm_bf16", "gemm_pair", "gemm_skinny",
-                   "linear_attention", "moe_experts", "page_table", "paged_attention", "paged_latent", "qkv_prep", "residual_stream", "sampler")
+                   "linear_attention", "linear_attention_umma", "moe_experts", "page_table", "paged_attention", "paged_latent", "qkv_prep",
+                   "residual_stream", "sampler")
 
 # Kernels whose results are 32-bit throughout (norms of an fp32 stream, router scores, rotary angles, recurrences, fp32 attention): no
 # fast-math exponentials, divisions or square roots.
-ACCURATE_SOURCES = ("attention_any", "depth_stream", "gated_scan", "linear_attention", "moe_experts", "qkv_prep", "residual_stream")
+ACCURATE_SOURCES = ("attention_any", "depth_stream", "gated_scan", "linear_attention", "linear_attention_umma", "moe_experts", "qkv_prep",
+                    "residual_stream")
 
 NVCC_FLAGS = [
     "-gencode",

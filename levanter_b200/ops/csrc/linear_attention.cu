@@ -4,45 +4,19 @@
 // The state, decays and everything added to the state are 32-bit; this file is built without fast-math.
 //
 // Decode rounds (and fp32, and sizes that are not multiples of 8) walk a sequence row by row with 32 columns of a head's state in
-// registers.  Prompts in bf16 are cut into pieces of chunks of 64 rows.  A first kernel sums up what every piece but a sequence's
-// last adds to the state, a second one turns these sums into the states that the pieces start from, and the third walks all pieces
-// at once on the tensor cores: with D the decays between the rows of a chunk,
+// registers.  Prompts in bf16 are cut into pieces of chunks.  A first kernel sums up what every piece but a sequence's last adds to the
+// state, a second one turns these sums into the states that the pieces start from, and the third walks all pieces at once on the
+// tensor cores: with D the decays between the rows of a chunk,
 //   O = decay^(i+1) (Q S) + ((Q K^T) o D) V,   S <- decay^n S + (K o decay^(n-1-j))^T V.
-// The fp32 state stays in accumulator registers; the products that read it (and the decayed keys that enter it) use two bf16 parts per
-// number, so that what is rounded to 16 bits is only what came in 16 bits, and the weights (Q K^T) o D as in the other attentions.
+// The fp32 state stays in accumulators; the products that read it, and the decayed factor that enters it, use two bf16 parts per number,
+// so that what is rounded to 16 bits is only what came in 16 bits, and the weights (Q K^T) o D as in the other attentions.
+// Keys of up to 128 run on tcgen05 (linear_attention_umma.cu); keys of up to 256, whose tiles leave no room for that, on warp-level MMAs
+// (below).
+#include "linear_attention.cuh"
 #include "row_groups.cuh"
 
 namespace lvb {
 namespace linattn {
-
-struct Params {
-  const void *q, *k, *v;   // rows of H * dk, H * dk, H * dv elements, row stride ld
-  void* out;               // [T, H * dv]
-  const float* decay;      // [H]
-  float* state;            // [slots, H, dk, dv]
-  const int *slot_ids, *kv_lens, *cu_q_lens, *num_seqs;
-  float* pieces;           // [work items, H, dk, dv]: what a piece adds to the state, then the state it starts from
-  long long ld;
-  int T, H, dk, dv, S, slots, piece;  // piece: rows of a piece, a multiple of the chunk
-  float key_scale;
-  int silu;                // q, k and v pass through silu first (row by row kernel only)
-};
-
-struct Sequence {
-  int r0, r1, slot;
-  bool from_state;
-};
-
-__device__ __forceinline__ int live_sequences(const Params& p) { return min(p.num_seqs[0], p.S); }
-
-// Rows and slot of sequence i.  False: nothing to do.
-__device__ __forceinline__ bool sequence(const Params& p, int i, Sequence& s) {
-  s.r0 = max(p.cu_q_lens[i], 0);
-  s.r1 = min(p.cu_q_lens[i + 1], p.T);
-  s.slot = p.slot_ids[i];
-  s.from_state = p.kv_lens[i] > s.r1 - s.r0;
-  return s.r1 > s.r0 && s.slot >= 0 && s.slot < p.slots;
-}
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -170,42 +144,6 @@ template <int kBytes>
 __device__ __forceinline__ uint32_t unit_at(int r, int u) {
   if constexpr (kBytes >= 128) return r * kBytes + ((u ^ (r & 7)) << 4);
   else return r * kBytes + ((u ^ ((r >> 1) & 3)) << 4);
-}
-
-// Two numbers as two bf16 parts each: hi + lo
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(a, b);
-  const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
-  lo = pack_bf16x2(a - h.x, b - h.y);
-}
-
-// Piece of work item w: sequence, number within the sequence and of how many.  A warp's lanes together.  False: there are only `of` items.
-__device__ __forceinline__ bool find_piece(const Params& p, int w, int& seq, int& c, int& of) {
-  const int lane = threadIdx.x & 31, n_seq = live_sequences(p);
-  int before = 0;
-  for (int base = 0; base < n_seq; base += 32) {
-    const int i = base + lane;
-    const int len = i < n_seq ? max(min(p.cu_q_lens[i + 1], p.T) - max(p.cu_q_lens[i], 0), 0) : 0;
-    const int n = (len + p.piece - 1) / p.piece;
-    int inc = n;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const int u = __shfl_up_sync(0xffffffffu, inc, o);
-      if (lane >= o) inc += u;
-    }
-    const bool mine = w >= before + inc - n && w < before + inc;
-    const unsigned found = __ballot_sync(0xffffffffu, mine);
-    if (found) {
-      const int src = __ffs(found) - 1;
-      seq = base + src;
-      of = __shfl_sync(0xffffffffu, n, src);
-      c = w - (before + __shfl_sync(0xffffffffu, inc, src) - of);
-      return true;
-    }
-    before += __shfl_sync(0xffffffffu, inc, 31);
-  }
-  of = before;
-  return false;
 }
 
 template <int kDK, int kDV>
@@ -480,6 +418,11 @@ __global__ void __launch_bounds__(256) carry_kernel(Params p) {
   }
 }
 
+void carry_states(const Params& p, cudaStream_t s) {
+  const long long head = static_cast<long long>(p.dk) * p.dv;
+  carry_kernel<<<dim3(static_cast<unsigned>((head / 4 + 255) / 256), p.H, p.S), 256, 0, s>>>(p);
+}
+
 template <int kDK, int kDV>
 int run_chunks(const Params& p, int items, cudaStream_t s) {
   using Tl = Tiles<kDK, kDV>;
@@ -489,8 +432,7 @@ int run_chunks(const Params& p, int items, cudaStream_t s) {
     return kErrCuda;
   if (p.pieces != nullptr) {
     chunk_kernel<kDK, kDV, true><<<grid, kChunkThreads, Tl::kStateAt, s>>>(p);
-    const long long head = static_cast<long long>(p.dk) * p.dv;
-    carry_kernel<<<dim3(static_cast<unsigned>((head / 4 + 255) / 256), p.H, p.S), 256, 0, s>>>(p);
+    carry_states(p, s);
   }
   chunk_kernel<kDK, kDV, false><<<grid, kChunkThreads, Tl::kSmem, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
@@ -576,11 +518,20 @@ extern "C" int lvb_linear_attention_plan(int T, int H, int dv, int S, int* piece
   using namespace lvb;
   using namespace lvb::linattn;
   if (T <= 0 || H <= 0 || dv <= 0 || S <= 0) return kErrBadArg;
-  // pieces as long as four per SM allow: a shorter piece is more work for the states in between
-  const long long cols = (dv + 63) / 64;
-  long long rows = static_cast<long long>(T) * H * cols / (4 * num_sms());
+  // waves of CTAs times the chunks that each walks (and some for its start); short pieces cost a pass over the states in between, at about
+  // half the work per chunk
+  const long long slices = static_cast<long long>(H) * ((dv + 63) / 64), sms = num_sms();
+  long long best = -1;
   int n = 256;
-  while (n < 4096 && n * 2 <= rows) n *= 2;
+  for (int rows = 256; rows <= 16384; rows *= 2) {
+    const long long count = (T + rows - 1) / rows, chunks = (rows < T ? rows : T) / 128 + 1;
+    const long long cost = 2 * ((count * slices + sms - 1) / sms) * (chunks + 3) + (count > 1 ? (((count - 1) * slices + sms - 1) / sms) * (chunks + 6) : 0);
+    if (best < 0 || cost < best) {
+      best = cost;
+      n = rows;
+    }
+    if (rows >= T) break;
+  }
   *piece = n;
   *items = T <= n ? 0 : (T + n - 1) / n + (S < T ? S : T);
   return kErrOk;
@@ -593,13 +544,14 @@ extern "C" int lvb_linear_attention_plan(int T, int H, int dv, int S, int* piece
 // multiples of 8, q, k, v 16-byte aligned; piece and pieces as lvb_linear_attention_plan says (pieces may be null when its items are 0).
 extern "C" int lvb_linear_attention(const void* q, const void* k, const void* v, void* out, const float* decay, float* state, const int* slot_ids,
                                     const int* kv_lens, const int* cu_q_lens, const int* num_seqs, float* pieces, int T, int H, int dk, int dv,
-                                    long long ld, int S, int slots, int piece, float key_scale, int silu, int is_f32, int chunked, void* stream) {
+                                    long long ld, int S, int slots, int piece, float key_scale, int silu, int is_f32, int chunked, int* status,
+                                    void* stream) {
   using namespace lvb;
   using namespace lvb::linattn;
   if (T <= 0) return kErrOk;
   if (H <= 0 || dk <= 0 || dv <= 0 || S <= 0 || slots <= 0) return kErrBadArg;
   if (H > 65535 || S >= 65535) return kErrTooLarge;
-  Params p{q, k, v, out, decay, state, slot_ids, kv_lens, cu_q_lens, num_seqs, pieces, ld, T, H, dk, dv, S, slots, piece, key_scale, silu};
+  Params p{q, k, v, out, decay, state, slot_ids, kv_lens, cu_q_lens, num_seqs, pieces, ld, T, H, dk, dv, S, slots, piece, key_scale, silu, status};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (!chunked) return is_f32 ? run_steps<float>(p, s) : run_steps<__nv_bfloat16>(p, s);
   if (is_f32 || silu || ((dk | dv | ld) & 7) || piece <= 0 || piece % kC != 0 ||
@@ -607,9 +559,7 @@ extern "C" int lvb_linear_attention(const void* q, const void* k, const void* v,
     return kErrBadArg;
   if (pieces == nullptr && T > piece) return kErrBadArg;
   const int items = (T + piece - 1) / piece + (S < T ? S : T);
-  if (dk <= 32) return run_chunks<32, 64>(p, items, s);
-  if (dk <= 64) return run_chunks<64, 64>(p, items, s);
-  if (dk <= 128) return run_chunks<128, 64>(p, items, s);
+  if (dk <= 128) return run_umma(p, items, s);
   if (dk <= 256) return run_chunks<256, 32>(p, items, s);
   return kErrTooLarge;
 }

@@ -66,7 +66,7 @@ def linear_attention_packed(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, d
             and all(t.stride(2) == 1 and t.stride(1) == t.shape[2] for t in (q, k, v)):
         c = lib
         if "l" not in _f:
-            _f["l"] = lib.fn("lvb_linear_attention", [c.c_void_p] * 11 + [c.c_int] * 4 + [c.c_longlong] + [c.c_int] * 3 + [c.c_float] + [c.c_int] * 3 + [c.c_void_p])
+            _f["l"] = lib.fn("lvb_linear_attention", [c.c_void_p] * 11 + [c.c_int] * 4 + [c.c_longlong] + [c.c_int] * 3 + [c.c_float] + [c.c_int] * 3 + [c.c_void_p] * 2)
             _f["plan"] = lib.fn("lvb_linear_attention_plan", [c.c_int] * 4 + [c.c_void_p] * 2, launches=0)
         i32 = lambda t: t.to(device=q.device, dtype=torch.int32).contiguous()  # noqa: E731
         slots, lens, cu, ns = i32(b.slot_ids), i32(b.seq_lens), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
@@ -85,7 +85,7 @@ def linear_attention_packed(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, d
         out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
         rc = _f["l"](q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), decay.data_ptr(), state.data_ptr(), slots.data_ptr(), lens.data_ptr(),
                      cu.data_ptr(), ns.data_ptr(), lib.ptr(pieces), T, H, d, dv, q.stride(0), S, state.shape[0], piece.value, float(key_scale),
-                     int(silu and not chunked), int(q.dtype == torch.float32), int(chunked), lib.stream_ptr())
+                     int(silu and not chunked), int(q.dtype == torch.float32), int(chunked), lib.status_buffer().data_ptr(), lib.stream_ptr())
         lib.check_rc(rc, "lvb_linear_attention")
         return out
     act = torch.nn.functional.silu if silu else (lambda t: t)
