@@ -20,6 +20,7 @@ def _batch(T, n_seq, S):
     cu = torch.full((S + 1,), T, dtype=torch.int32, device="cuda")
     cu[:n_seq + 1] = torch.arange(n_seq + 1, device="cuda") * L
     b.cu_q_lens, b.num_seqs, b.seq_lens = cu, torch.tensor(n_seq, device="cuda", dtype=torch.int32), torch.full((S,), L + 1, dtype=torch.int32, device="cuda")
+    b.longest = L
     return b
 
 
@@ -29,7 +30,7 @@ def recurrence(tb: Table):
     from ..ops.linear_attention import gated_norm, linear_attention_packed, silu_in_place
     from ..ops.norm import rms_norm
 
-    for T, n_seq, S, H, d in ((8192, 4, 16, 32, 128), (8192, 1, 16, 32, 128), (8192, 4, 16, 64, 64), (8192, 4, 16, 16, 256), (64, 64, 64, 32, 128), (64, 64, 64, 64, 64),
+    for T, n_seq, S, H, d in ((8192, 4, 16, 32, 128), (8192, 1, 16, 32, 128), (16384, 16, 16, 32, 128), (8192, 4, 16, 64, 64), (8192, 4, 16, 16, 256), (64, 64, 64, 32, 128), (64, 64, 64, 64, 64),
                               (8, 8, 8, 32, 128)):
         L, W = T // n_seq, H * d
         y = _randn(T, 4 * W)

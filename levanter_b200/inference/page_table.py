@@ -75,6 +75,9 @@ class PageBatchInfo:
     num_pages: int = 0
     """pages of the cache the destinations point into"""
 
+    longest: int = 0
+    """most tokens that a sequence has in the pass (0: not known): recurrent layers choose by it how they cut the work"""
+
     @property
     def num_slots(self) -> int:
         """Destinations outside ``[0, num_slots)`` are padding."""
@@ -90,7 +93,7 @@ class PageBatchInfo:
         mv = lambda t: t.to(device, non_blocking=non_blocking)  # noqa: E731
         return PageBatchInfo(mv(self.slot_ids), mv(self.page_indices), mv(self.seq_lens), mv(self.cu_q_lens), mv(self.num_seqs),
                              mv(self.new_token_dests), self.page_size,
-                             None if self.prefill_segment_ids is None else mv(self.prefill_segment_ids), self.num_pages)
+                             None if self.prefill_segment_ids is None else mv(self.prefill_segment_ids), self.num_pages, self.longest)
 
 
 @dataclass
@@ -178,7 +181,7 @@ class PageTable:
             num = _allocate_numpy(new, slots, pos, o_slot, o_pages, o_lens, o_cu, o_dest)
         info = PageBatchInfo(torch.from_numpy(o_slot), torch.from_numpy(o_pages), torch.from_numpy(o_lens), torch.from_numpy(o_cu),
                              torch.tensor(num, dtype=torch.int32), torch.from_numpy(o_dest), self.page_size,
-                             num_pages=self.num_pages)
+                             num_pages=self.num_pages, longest=int(np.diff(o_cu[:num + 1]).max()) if num > 0 else 0)
         return new, info
 
     # -- release ----------------------------------------------------------------------------------------------

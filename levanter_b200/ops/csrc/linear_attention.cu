@@ -512,28 +512,31 @@ __global__ void __launch_bounds__(256) silu_kernel(T* __restrict__ x, long long 
 }  // namespace linattn
 }  // namespace lvb
 
-// Rows of a piece of lvb_linear_attention's chunked form for T rows, and the work items that scratch [items, H, dk, dv] (fp32) is needed for when no
-// sequence can be longer than T: 0 when every sequence is one piece.
-extern "C" int lvb_linear_attention_plan(int T, int H, int dv, int S, int* piece, int* items) {
+// Rows of a piece of lvb_linear_attention's chunked form, and the work items that scratch [items, H, dk, dv] (fp32) is needed for: 0, and a piece of
+// at least T rows, when sequences are not to be cut.  longest: rows of the longest sequence (0: not known, or T); only the speed depends on it.
+extern "C" int lvb_linear_attention_plan(int T, int longest, int H, int dv, int S, int* piece, int* items) {
   using namespace lvb;
   using namespace lvb::linattn;
   if (T <= 0 || H <= 0 || dv <= 0 || S <= 0) return kErrBadArg;
-  // waves of CTAs times the chunks that each walks (and some for its start); short pieces cost a pass over the states in between, at about
-  // half the work per chunk
-  const long long slices = static_cast<long long>(H) * ((dv + 63) / 64), sms = num_sms();
+  if (longest <= 0 || longest > T) longest = T;
+  // rounds of the SMs times the chunks that each walks (and one for the start); cut sequences cost two more launches and a pass over what
+  // lies before their last pieces, at about half the work per chunk
+  const long long slices = static_cast<long long>(H) * ((dv + 63) / 64), sms = num_sms(), seqs = (T + longest - 1) / longest;
+  auto rounds = [&](long long pieces) { return (pieces * slices + sms - 1) / sms; };
   long long best = -1;
-  int n = 256;
-  for (int rows = 256; rows <= 16384; rows *= 2) {
-    const long long count = (T + rows - 1) / rows, chunks = (rows < T ? rows : T) / 128 + 1;
-    const long long cost = 2 * ((count * slices + sms - 1) / sms) * (chunks + 3) + (count > 1 ? (((count - 1) * slices + sms - 1) / sms) * (chunks + 6) : 0);
+  int n = 0;
+  for (int rows = 256;; rows *= 2) {
+    const bool whole = rows >= longest;
+    const long long per = whole ? 1 : (longest + rows - 1) / rows, chunks = ((whole ? longest : rows) + 127) / 128;
+    const long long cost = 2 * rounds(seqs * per) * (chunks + 1) + (whole ? 0 : rounds(seqs * (per - 1)) * (chunks + 2) + 24);
     if (best < 0 || cost < best) {
       best = cost;
-      n = rows;
+      n = whole ? 0 : rows;
     }
-    if (rows >= T) break;
+    if (whole) break;
   }
-  *piece = n;
-  *items = T <= n ? 0 : (T + n - 1) / n + (S < T ? S : T);
+  *piece = n > 0 ? n : (T + 127) / 128 * 128;
+  *items = n > 0 ? (T + n - 1) / n + (S < T ? S : T) : 0;
   return kErrOk;
 }
 

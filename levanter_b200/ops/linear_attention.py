@@ -52,12 +52,14 @@ def _chunked_ok(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> bool:
 
 
 def linear_attention_packed(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, batch_info, *,
-                            key_scale: float = 1.0, silu: bool = False, chunked: Optional[bool] = None) -> torch.Tensor:
+                            key_scale: float = 1.0, silu: bool = False, chunked: Optional[bool] = None,
+                            piece: Optional[int] = None) -> torch.Tensor:
     """``q, k [T, H, d]``, ``v [T, H, dv]`` (slices of the same packed rows) -> ``[T, H, dv]``; ``state [slots, H, d, dv]`` fp32, updated in place.
     ``key_scale``: factor on the keys.  ``silu``: q, k and v pass through it first (and may be overwritten).  A sequence whose first packed
     row is its position 0 starts from a zero state; rows of no sequence come out as zeros.  ``chunked``: by chunks on tensor cores (default:
     when sequences have many rows, in bf16, with sizes that are multiples of 8 and ``d`` up to 256), else row by row in fp32 arithmetic
-    (``d`` up to 512)."""
+    (``d`` up to 512).  ``piece``: rows (a multiple of 128) that the chunked form cuts longer sequences into, to walk the pieces at once
+    (default: what should be fastest)."""
     T, H, d = q.shape
     dv = v.shape[2]
     b = batch_info
@@ -67,24 +69,26 @@ def linear_attention_packed(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, d
         c = lib
         if "l" not in _f:
             _f["l"] = lib.fn("lvb_linear_attention", [c.c_void_p] * 11 + [c.c_int] * 4 + [c.c_longlong] + [c.c_int] * 3 + [c.c_float] + [c.c_int] * 3 + [c.c_void_p] * 2)
-            _f["plan"] = lib.fn("lvb_linear_attention_plan", [c.c_int] * 4 + [c.c_void_p] * 2, launches=0)
+            _f["plan"] = lib.fn("lvb_linear_attention_plan", [c.c_int] * 5 + [c.c_void_p] * 2, launches=0)
         i32 = lambda t: t.to(device=q.device, dtype=torch.int32).contiguous()  # noqa: E731
         slots, lens, cu, ns = i32(b.slot_ids), i32(b.seq_lens), i32(b.cu_q_lens), i32(b.num_seqs.reshape(1))
         S = slots.shape[0]
+        longest = getattr(b, "longest", 0)
         if chunked is None:
-            chunked = T > 4 * S
+            chunked = longest > 16 if longest > 0 else T > 4 * S
         chunked = chunked and _chunked_ok(q, k, v)
-        piece, items = ctypes.c_int(0), ctypes.c_int(0)
+        cut, items = ctypes.c_int(piece or 0), ctypes.c_int(-(-T // piece) + min(S, T) if piece else 0)
         pieces = None
         if chunked:
-            lib.check_rc(_f["plan"](T, H, dv, S, ctypes.addressof(piece), ctypes.addressof(items)), "lvb_linear_attention_plan")
+            if piece is None:
+                lib.check_rc(_f["plan"](T, longest, H, dv, S, ctypes.addressof(cut), ctypes.addressof(items)), "lvb_linear_attention_plan")
             if items.value:
                 pieces = torch.empty(items.value * H * d * dv, dtype=torch.float32, device=q.device)
             if silu:
                 silu_in_place(q, k, v)
         out = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
         rc = _f["l"](q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), decay.data_ptr(), state.data_ptr(), slots.data_ptr(), lens.data_ptr(),
-                     cu.data_ptr(), ns.data_ptr(), lib.ptr(pieces), T, H, d, dv, q.stride(0), S, state.shape[0], piece.value, float(key_scale),
+                     cu.data_ptr(), ns.data_ptr(), lib.ptr(pieces), T, H, d, dv, q.stride(0), S, state.shape[0], cut.value, float(key_scale),
                      int(silu and not chunked), int(q.dtype == torch.float32), int(chunked), lib.status_buffer().data_ptr(), lib.stream_ptr())
         lib.check_rc(rc, "lvb_linear_attention")
         return out

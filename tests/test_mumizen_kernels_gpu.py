@@ -98,20 +98,20 @@ def test_linear_attention(dtype, H, d, dv, decay, silu, scale):
     g = torch.tensor(decay, dtype=F32, device="cuda")
     state = torch.full((slots, H, d, dv), 3.0, device="cuda")
 
-    def run(batch, pad=3, chunked=None):
+    def run(batch, pad=3, chunked=None, piece=None):
         at = dict(seqs.at)
         b, _ = seqs.step(batch, pad)
         y = torch.cat([rows[i][at[i]:at[i] + m] for i, m in batch] + [torch.ones(pad, n + 8, dtype=dtype)]).cuda()
         with torch.no_grad():
-            o = linear_attention_packed(*split(y), g, state, b, key_scale=scale, silu=silu, chunked=chunked)
+            o = linear_attention_packed(*split(y), g, state, b, key_scale=scale, silu=silu, chunked=chunked, piece=piece)
         total = o.shape[0] - pad
         assert o.dtype == dtype and float(o[total:].float().abs().sum()) == 0.0
         _check_rows(o[:total], torch.cat([want[i][at[i]:at[i] + m] for i, m in batch]), dtype)
 
-    run([(0, 600), (1, 64), (2, 1), (3, 130)], chunked=True)
+    run([(0, 600), (1, 64), (2, 1), (3, 130)], chunked=True, piece=128)
     run([(0, 1), (1, 1), (2, 1), (3, 1)])
     run([(3, 2), (0, 1), (2, 66)], chunked=False)
-    run([(2, 2), (1, 300), (3, 63)], pad=70, chunked=True)
+    run([(2, 2), (1, 300), (3, 63)], pad=70, chunked=True, piece=256)
     run([(0, 3), (1, 1), (2, 1)], pad=0)
     for i in (0, 3):
         seqs.free(i)
@@ -135,13 +135,13 @@ def test_linear_attention_remembers_a_far_key():
     parts = lambda y: (t.unflatten(1, (H, -1)) for t in y.split([H * d, H * d, H * dv], dim=1))  # noqa: E731
     want = O.fixed_decay_attention(*parts(y.double()), decay)
     assert _rel(want[1199], k[5].double().mul(probe.double()).sum(-1, keepdim=True) * v[5].double()) < 0.6  # the key is what the answer is made of
-    for cuts in ([1200], [1024, 176], [6, 1018, 2, 173, 1], [1150] + [1] * 50):
+    for cuts, piece in (([1200], None), ([1200], 384), ([1024, 176], 128), ([6, 1018, 2, 173, 1], None), ([1150] + [1] * 50, 256)):
         seqs = _Sequences(1, page=16, pages=80, per_seq=80)
         state, outs, at = torch.zeros(1, H, d, dv, device="cuda"), [], 0
         for c in cuts:
             b, _ = seqs.step([(0, c)], 0)
             with torch.no_grad():
-                outs.append(linear_attention_packed(*parts(y[at:at + c].cuda()), torch.tensor(decay, device="cuda"), state, b))
+                outs.append(linear_attention_packed(*parts(y[at:at + c].cuda()), torch.tensor(decay, device="cuda"), state, b, piece=piece))
             at += c
         got = torch.cat(outs)
         for t in (70, 1024, 1030, 1199):
