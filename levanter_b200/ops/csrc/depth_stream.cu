@@ -28,25 +28,25 @@ struct Params {
   float eps;
 };
 
-template <int kN, int kVec, int kThreads>
-__global__ void __launch_bounds__(kThreads, kThreads <= 256 ? 3 : 1) depth_kernel(Params p) {
+template <int kN, int kVec, int kThreads, bool kShift>
+__global__ void __launch_bounds__(kThreads, kThreads <= 512 ? 3 : 1) depth_kernel(Params p) {
   using Row = rowg::Row<kN, kVec>;
   extern __shared__ float smem[];
   __shared__ int s_seq;
-  const int groups = p.dim / p.part, scratch = kN * blockDim.x + groups;
+  const typename Row::Groups groups(p.dim, p.part);
+  const int scratch = kN * blockDim.x + p.dim / p.part;
   float* s_coef = smem + 2 * scratch;
   for (int j = threadIdx.x; j < p.planes; j += blockDim.x) s_coef[j] = p.coef != nullptr ? rowg::ld1(p.coef, p.w_f32, j) : 1.f;
   const int r0 = blockIdx.x * p.per, r1 = min(r0 + p.per, p.T);
-  const bool shift = p.mu != nullptr;
-  if (threadIdx.x == 0) s_seq = -1;
-  __syncthreads();
   int n_seq = 0;
-  if (shift) {
+  if constexpr (kShift) {
+    if (threadIdx.x == 0) s_seq = -1;
+    __syncthreads();
     n_seq = min(p.num_seqs[0], p.S);
     for (int i = threadIdx.x; i < n_seq; i += blockDim.x)
       if (p.cu_q_lens[i] <= r0 && r0 < p.cu_q_lens[i + 1]) s_seq = i;
-    __syncthreads();
   }
+  __syncthreads();
   int turn = 0;
   // the normed row r; store: also its sum
   auto row_at = [&](int r, bool store, Row& x) {
@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(kThreads, kThreads <= 256 ? 3 : 1) depth_kerne
     for (int n = 0; n < kN; ++n)
 #pragma unroll
       for (int e = 0; e < kVec; ++e) x.a[n][e] = 0.f;
-#pragma unroll 4
+#pragma unroll 2
     for (int j = 0; j < p.planes; ++j) {
       const float c = s_coef[j];
 #pragma unroll
@@ -73,7 +73,7 @@ __global__ void __launch_bounds__(kThreads, kThreads <= 256 ? 3 : 1) depth_kerne
       for (int n = 0; n < kN; ++n)
         if (Row::column(n) < p.dim) rowg::st_unit<kVec>(p.out, 1, src + Row::column(n), x.a[n]);
     }
-    x.normalize(p.dim, p.part, p.eps, smem + turn * scratch);
+    x.normalize(groups, p.eps, smem + turn * scratch);
     turn ^= 1;
 #pragma unroll
     for (int n = 0; n < kN; ++n) {
@@ -85,73 +85,73 @@ __global__ void __launch_bounds__(kThreads, kThreads <= 256 ? 3 : 1) depth_kerne
     }
   };
   Row h;
-  if (!shift) {
+  if constexpr (!kShift) {
     for (int r = r0; r < r1; ++r) {
       row_at(r, true, h);
 #pragma unroll
       for (int n = 0; n < kN; ++n)
         if (Row::column(n) < p.dim) rowg::st_unit<kVec>(p.y, p.y_f32, static_cast<size_t>(r) * p.dim + Row::column(n), h.a[n]);
     }
-    return;
-  }
-  Row before;
-  auto clear = [&] {
+  } else {
+    Row before;
+    auto clear = [&] {
 #pragma unroll
-    for (int n = 0; n < kN; ++n)
+      for (int n = 0; n < kN; ++n)
 #pragma unroll
-      for (int e = 0; e < kVec; ++e) before.a[n][e] = 0.f;
-  };
-  auto leave = [&](float* at, const Row& x) {
+        for (int e = 0; e < kVec; ++e) before.a[n][e] = 0.f;
+    };
+    auto leave = [&](float* at, const Row& x) {
 #pragma unroll
-    for (int n = 0; n < kN; ++n)
-      if (Row::column(n) < p.dim) rowg::st_unit<kVec>(at, 1, Row::column(n), x.a[n]);
-  };
-  clear();
-  int seq = s_seq, first = 0, end = 0;
-  float* slot = nullptr;
-  auto enter = [&](int i) {  // rows [first, end) of sequence i, and its slot's row
-    first = p.cu_q_lens[i];
-    end = min(p.cu_q_lens[i + 1], p.T);
-    const int s = p.slot_ids[i];
-    slot = s >= 0 && s < p.slots ? p.state + static_cast<size_t>(s) * p.dim : nullptr;
-  };
-  if (seq >= 0) {
-    enter(seq);
-    if (first < r0) row_at(r0 - 1, false, before);
-  }
-  for (int r = r0; r < r1; ++r) {
-    while (seq >= 0 && r >= end) {
-      ++seq;
-      if (seq >= n_seq) seq = -1;  // padding from here on
-      else enter(seq);
+      for (int n = 0; n < kN; ++n)
+        if (Row::column(n) < p.dim) rowg::st_unit<kVec>(at, 1, Row::column(n), x.a[n]);
+    };
+    clear();
+    int seq = s_seq, first = 0, end = 0;
+    float* slot = nullptr;
+    auto enter = [&](int i) {  // rows [first, end) of sequence i, and its slot's row
+      first = p.cu_q_lens[i];
+      end = min(p.cu_q_lens[i + 1], p.T);
+      const int s = p.slot_ids[i];
+      slot = s >= 0 && s < p.slots ? p.state + static_cast<size_t>(s) * p.dim : nullptr;
+    };
+    if (seq >= 0) {
+      enter(seq);
+      if (first < r0) row_at(r0 - 1, false, before);
     }
-    if (seq < 0 || r == first) {
-      clear();
-      if (seq >= 0 && slot != nullptr && p.kv_lens[seq] > end - first) {
-#pragma unroll
-        for (int n = 0; n < kN; ++n)
-          if (Row::column(n) < p.dim) rowg::ld_unit<kVec>(slot, 1, Row::column(n), before.a[n]);
+    for (int r = r0; r < r1; ++r) {
+      while (seq >= 0 && r >= end) {
+        ++seq;
+        if (seq >= n_seq) seq = -1;  // padding from here on
+        else enter(seq);
       }
-    }
-    row_at(r, true, h);
+      if (seq < 0 || r == first) {
+        clear();
+        if (seq >= 0 && slot != nullptr && p.kv_lens[seq] > end - first) {
 #pragma unroll
-    for (int n = 0; n < kN; ++n) {
-      const int col = Row::column(n);
-      if (col >= p.dim) continue;
-      float m[kVec], v[kVec];
-      rowg::ld_unit<kVec>(p.mu, p.w_f32, col, m);
-#pragma unroll
-      for (int e = 0; e < kVec; ++e) {
-        v[e] = fmaf(before.a[n][e] - h.a[n][e], m[e], h.a[n][e]);
-        before.a[n][e] = h.a[n][e];
+          for (int n = 0; n < kN; ++n)
+            if (Row::column(n) < p.dim) rowg::ld_unit<kVec>(slot, 1, Row::column(n), before.a[n]);
+        }
       }
-      rowg::st_unit<kVec>(p.y, p.y_f32, static_cast<size_t>(r) * p.dim + col, v);
-    }
-    if (seq < 0 || first < r0 || slot == nullptr) continue;
-    if (r == end - 1) leave(slot, h);
-    else if (r == r1 - 1) {  // the sequence goes on beyond this CTA
-      row_at(end - 1, false, h);
-      leave(slot, h);
+      row_at(r, true, h);
+#pragma unroll
+      for (int n = 0; n < kN; ++n) {
+        const int col = Row::column(n);
+        if (col >= p.dim) continue;
+        float m[kVec], v[kVec];
+        rowg::ld_unit<kVec>(p.mu, p.w_f32, col, m);
+#pragma unroll
+        for (int e = 0; e < kVec; ++e) {
+          v[e] = fmaf(before.a[n][e] - h.a[n][e], m[e], h.a[n][e]);
+          before.a[n][e] = h.a[n][e];
+        }
+        rowg::st_unit<kVec>(p.y, p.y_f32, static_cast<size_t>(r) * p.dim + col, v);
+      }
+      if (seq < 0 || first < r0 || slot == nullptr) continue;
+      if (r == end - 1) leave(slot, h);
+      else if (r == r1 - 1) {  // the sequence goes on beyond this CTA
+        row_at(end - 1, false, h);
+        leave(slot, h);
+      }
     }
   }
 }
@@ -160,9 +160,9 @@ template <int kN, int kVec, int kThreads>
 int launch(const Params& p, int threads, cudaStream_t s) {
   const size_t smem = (2 * rowg::Row<kN, kVec>::scratch_floats(threads, p.dim / p.part) + p.planes) * 4;
   if (smem > 200 * 1024) return kErrTooLarge;
-  if (smem > 40 * 1024 && cudaFuncSetAttribute(depth_kernel<kN, kVec, kThreads>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
-    return kErrCuda;
-  depth_kernel<kN, kVec, kThreads><<<(p.T + p.per - 1) / p.per, threads, smem, s>>>(p);
+  auto kern = p.mu != nullptr ? depth_kernel<kN, kVec, kThreads, true> : depth_kernel<kN, kVec, kThreads, false>;
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return kErrCuda;
+  kern<<<(p.T + p.per - 1) / p.per, threads, smem, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
 }
 
@@ -189,8 +189,8 @@ extern "C" int lvb_depth_stream(const float* hist, long long plane, int planes, 
   const int mis = static_cast<int>((reinterpret_cast<uintptr_t>(hist) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(w) |
                                     reinterpret_cast<uintptr_t>(mu) | reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(y)) & 15);
   const int vec = (part & 3) == 0 && (plane & 3) == 0 && mis == 0 ? 4 : 1;
-  // rows per CTA: one wave of CTAs, and with a shift at least a few rows, since the one before the first is formed twice
-  int per = T / (num_sms() * 6);
+  // rows per CTA: with a shift about one wave of CTAs, and at least a few rows, since the one before the first is formed twice
+  int per = mu != nullptr ? T / (num_sms() * 6) : 1;
   if (mu != nullptr && per < 4) per = T / num_sms() < 4 ? T / num_sms() : 4;
   per = per < 1 ? 1 : per > 32 ? 32 : per;
   int n, threads;
@@ -198,8 +198,9 @@ extern "C" int lvb_depth_stream(const float* hist, long long plane, int planes, 
   Params p{hist, plane, planes, coef, out, rows, w, mu, w_f32, state, slot_ids, kv_lens, cu_q_lens, num_seqs, S, slots, y, y_f32, T, dim, part, per, eps};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (vec == 4) {
-    if (n == 16) return kErrTooLarge;
-    return n == 1 ? launch<1, 4, 1024>(p, threads, s) : threads <= 256 ? launch<4, 4, 256>(p, threads, s) : launch<4, 4, 1024>(p, threads, s);
+    if (n == 1) return threads <= 256 ? launch<1, 4, 256>(p, threads, s) : launch<1, 4, 1024>(p, threads, s);
+    return n == 2 ? launch<2, 4, 512>(p, threads, s) : n == 4 ? launch<4, 4, 1024>(p, threads, s) : kErrTooLarge;
   }
-  return n == 1 ? launch<1, 1, 1024>(p, threads, s) : n == 4 ? launch<4, 1, 1024>(p, threads, s) : launch<16, 1, 1024>(p, threads, s);
+  if (n == 1) return launch<1, 1, 1024>(p, threads, s);
+  return n == 2 ? launch<2, 1, 512>(p, threads, s) : n == 4 ? launch<4, 1, 1024>(p, threads, s) : launch<16, 1, 1024>(p, threads, s);
 }

@@ -460,26 +460,115 @@ gated_norm_kernel(const void* __restrict__ o, const void* __restrict__ gate, lon
   extern __shared__ float s_norm[];
   const size_t at = static_cast<size_t>(blockIdx.x) * dim;
   Row x;
+  float g[kN][kVec];
 #pragma unroll
   for (int n = 0; n < kN; ++n) {
 #pragma unroll
     for (int e = 0; e < kVec; ++e) x.a[n][e] = 0.f;
-    if (Row::column(n) < dim) rowg::ld_unit<kVec>(o, f32, at + Row::column(n), x.a[n]);
+    if (Row::column(n) >= dim) continue;
+    rowg::ld_unit<kVec>(o, f32, at + Row::column(n), x.a[n]);
+    rowg::ld_unit<kVec>(gate, f32, static_cast<size_t>(blockIdx.x) * ldg + Row::column(n), g[n]);
   }
-  x.normalize(dim, part, eps, s_norm);
+  x.normalize(typename Row::Groups(dim, part), eps, s_norm);
 #pragma unroll
   for (int n = 0; n < kN; ++n) {
     const int col = Row::column(n);
     if (col >= dim) continue;
-    float g[kVec], m[kVec];
-    rowg::ld_unit<kVec>(gate, f32, static_cast<size_t>(blockIdx.x) * ldg + col, g);
+    float m[kVec];
     if (w != nullptr) rowg::ld_unit<kVec>(w, w_f32, col, m);
 #pragma unroll
     for (int e = 0; e < kVec; ++e) {
-      const float s = 1.f / (1.f + expf(-g[e]));
-      x.a[n][e] *= (act == 0 ? g[e] * s : s) * (w != nullptr ? m[e] : 1.f);
+      // (a gate that multiplies 16-bit results needs no more than the fast forms)
+      const float s = f32 ? 1.f / (1.f + expf(-g[n][e])) : __fdividef(1.f, 1.f + __expf(-g[n][e]));
+      x.a[n][e] *= (act == 0 ? g[n][e] * s : s) * (w != nullptr ? m[e] : 1.f);
     }
     rowg::st_unit<kVec>(y, f32, at + col, x.a[n]);
+  }
+}
+
+// Eight consecutive bf16 numbers.
+struct Eight {
+  float v[8];
+  __device__ __forceinline__ void load(const void* p, long long i) {
+    const uint4 w = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p) + i);
+    const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[e]));
+      v[2 * e] = f.x;
+      v[2 * e + 1] = f.y;
+    }
+  }
+  __device__ __forceinline__ void store(void* p, long long i) const {
+    *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(p) + i) =
+        make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  }
+  __device__ __forceinline__ float squares() const {
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+    return s;
+  }
+  // times r, w and act(gate)
+  __device__ __forceinline__ void finish(float r, const Eight& gate, const void* w, int w_f32, int col, int act) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float s = __fdividef(1.f, 1.f + __expf(-gate.v[e]));
+      v[e] *= r * (act == 0 ? gate.v[e] * s : s) * (w != nullptr ? rowg::ld1(w, w_f32, col + e) : 1.f);
+    }
+  }
+};
+
+// gated_norm_kernel for bf16 rows and groups of 8, 16, .. 256 elements: `lanes` neighbouring lanes hold a group, and no warp waits for another.
+__global__ void __launch_bounds__(256)
+gated_norm_small_kernel(const void* __restrict__ o, const void* __restrict__ gate, long long ldg, const void* __restrict__ w, int w_f32,
+                        void* __restrict__ y, long long units, int per_row, int lanes, float eps, int act) {
+  const float inv = 1.f / static_cast<float>(lanes * 8);
+  const long long step = static_cast<long long>(gridDim.x) * 256;
+  for (long long base = static_cast<long long>(blockIdx.x) * 256; base < units; base += step) {  // whole warps: the sums are made together
+    const long long i = base + threadIdx.x;
+    const bool in = i < units;
+    const long long r = in ? i / per_row : 0;
+    const int col = in ? static_cast<int>(i - r * per_row) * 8 : 0;
+    Eight x, g;
+    x.load(o, in ? i * 8 : 0);
+    g.load(gate, r * ldg + col);
+    float ss = x.squares();
+    for (int m = 1; m < lanes; m <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    x.finish(1.f / sqrtf(ss * inv + eps), g, w, w_f32, col, act);
+    if (in) x.store(y, i * 8);
+  }
+}
+
+// The same for one group per row; a CTA per row, kU units of 8 per thread.
+template <int kU>
+__global__ void __launch_bounds__(512)
+gated_norm_row_kernel(const void* __restrict__ o, const void* __restrict__ gate, long long ldg, const void* __restrict__ w, int w_f32,
+                      void* __restrict__ y, int dim, float eps, int act) {
+  __shared__ float s_sum[16];
+  const long long row = blockIdx.x;
+  Eight x[kU], g[kU];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < kU; ++u) {
+    const int col = (threadIdx.x + u * blockDim.x) * 8;
+    if (col >= dim) continue;
+    x[u].load(o, row * dim + col);
+    g[u].load(gate, row * ldg + col);
+    ss += x[u].squares();
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) s_sum[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int i = 0; i < static_cast<int>(blockDim.x) / 32; ++i) ss += s_sum[i];
+  const float r = 1.f / sqrtf(ss / static_cast<float>(dim) + eps);
+#pragma unroll
+  for (int u = 0; u < kU; ++u) {
+    const int col = (threadIdx.x + u * blockDim.x) * 8;
+    if (col >= dim) continue;
+    x[u].finish(r, g[u], w, w_f32, col, act);
+    x[u].store(y, row * dim + col);
   }
 }
 
@@ -578,9 +667,24 @@ extern "C" int lvb_gated_norm(const void* o, const void* gate, long long ldg, co
   const int part = dim / groups;
   const uintptr_t mis = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y);
   const int vec = (part & 3) == 0 && (ldg & 3) == 0 && (mis & 15) == 0 ? 4 : 1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (!is_f32 && ((part | ldg) & 7) == 0 && (mis & 15) == 0) {
+    const int lanes = part / 8;
+    if (lanes <= 32 && (lanes & (lanes - 1)) == 0) {
+      const long long units = static_cast<long long>(T) * (dim / 8), cap = static_cast<long long>(num_sms()) * 32;
+      const long long blocks = (units + 255) / 256;
+      gated_norm_small_kernel<<<static_cast<int>(blocks < cap ? blocks : cap), 256, 0, s>>>(o, gate, ldg, w, w_f32, y, units, dim / 8, lanes, eps, act);
+      return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+    }
+    if (groups == 1 && dim <= 512 * 32) {
+      const int per = dim / 8 <= 512 ? 1 : dim / 8 <= 1024 ? 2 : 4, threads = ((dim / 8 + per - 1) / per + 31) / 32 * 32;
+      auto kern = per == 1 ? gated_norm_row_kernel<1> : per == 2 ? gated_norm_row_kernel<2> : gated_norm_row_kernel<4>;
+      kern<<<T, threads, 0, s>>>(o, gate, ldg, w, w_f32, y, dim, eps, act);
+      return cudaGetLastError() == cudaSuccess ? kErrOk : kErrCuda;
+    }
+  }
   int n, threads;
   if (!rowg::shape_for(dim, vec, T < 2 * num_sms(), n, threads)) return kErrTooLarge;
-  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto launch = [&](auto kern, size_t floats) {
     if (floats * 4 > 200 * 1024) return kErrTooLarge;
     if (floats * 4 > 40 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return kErrCuda;
@@ -589,10 +693,12 @@ extern "C" int lvb_gated_norm(const void* o, const void* gate, long long ldg, co
   };
   if (vec == 4) {
     if (n == 1) return launch(gated_norm_kernel<1, 4, 1024>, rowg::Row<1, 4>::scratch_floats(threads, groups));
+    if (n == 2) return launch(gated_norm_kernel<2, 4, 512>, rowg::Row<2, 4>::scratch_floats(threads, groups));
     if (n == 4) return launch(gated_norm_kernel<4, 4, 1024>, rowg::Row<4, 4>::scratch_floats(threads, groups));
     return kErrTooLarge;
   }
   if (n == 1) return launch(gated_norm_kernel<1, 1, 1024>, rowg::Row<1, 1>::scratch_floats(threads, groups));
+  if (n == 2) return launch(gated_norm_kernel<2, 1, 512>, rowg::Row<2, 1>::scratch_floats(threads, groups));
   if (n == 4) return launch(gated_norm_kernel<4, 1, 1024>, rowg::Row<4, 1>::scratch_floats(threads, groups));
   return launch(gated_norm_kernel<16, 1, 1024>, rowg::Row<16, 1>::scratch_floats(threads, groups));
 }

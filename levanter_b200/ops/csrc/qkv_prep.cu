@@ -332,6 +332,24 @@ __global__ void __launch_bounds__(kThreads) latent_norm_kernel(LatentParams p, i
     }
     return;
   }
+  if (p.vec_c) {  // the second read comes from L1
+    for (int c = lane * 8; c < p.rank; c += 256) {
+      float a[8];
+      Vec8<T>::load(down + c, a);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(a[j], a[j], ss);
+    }
+    const float r = scale(ss);
+    for (int c = lane * 8; c < p.rank; c += 256) {
+      float a[8];
+      Vec8<T>::load(down + c, a);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] *= r * weight(c + j);
+      if (latent != nullptr) Vec8<T>::store(latent + c, a);
+      if (cache != nullptr) Vec8<T>::store(cache + c, a);
+    }
+    return;
+  }
   for (int c = lane; c < p.rank; c += 32) {
     const float a = to_f<T>(down[c]);
     ss = fmaf(a, a, ss);

@@ -180,6 +180,27 @@ glu_kernel(const void* __restrict__ gate, const void* __restrict__ up, const flo
            int f32, long long total, int cols, long long ldg, long long ldu, long long ldr, int vec) {
   auto factor = [&](long long r) { return row_gate != nullptr ? 1.f / (1.f + expf(-row_gate[r * ldr])) : 1.f; };
   const long long step = static_cast<long long>(gridDim.x) * blockDim.x;
+  if constexpr (!kOutF32) {
+    if (vec == 8) {  // groups of 8 columns, bf16 throughout
+      const int per = cols / 8;
+      for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total / 8; i += step) {
+        const long long r = i / per, c = (i - r * per) * 8;
+        const uint4 g = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(gate) + r * ldg + c);
+        const uint4 u = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(up) + r * ldu + c);
+        const float f = factor(r);
+        const uint32_t gw[4] = {g.x, g.y, g.z, g.w}, uw[4] = {u.x, u.y, u.z, u.w};
+        uint32_t o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[e]));
+          const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[e]));
+          o[e] = pack_bf16x2(glu<true>(act, limit, a.x, b.x) * f, glu<true>(act, limit, a.y, b.y) * f);
+        }
+        reinterpret_cast<uint4*>(out)[i] = make_uint4(o[0], o[1], o[2], o[3]);
+      }
+      return;
+    }
+  }
   if (vec) {  // groups of 4 columns; cols is a multiple of 4
     const int per = cols / 4;
     for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total / 4; i += step) {
@@ -259,9 +280,9 @@ extern "C" int lvb_glu_any(const void* gate, const void* up, const float* row_ga
   using namespace lvb;
   if (rows <= 0 || cols <= 0 || act < 0 || act > 2 || (out_f32 && !in_f32)) return kErrBadArg;
   const uintptr_t mis = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out);
-  const int vec = ((cols | ldg | ldu) & 3) == 0 && (mis & 15) == 0;
+  const int vec = (mis & 15) != 0 ? 0 : !in_f32 && ((cols | ldg | ldu) & 7) == 0 ? 8 : ((cols | ldg | ldu) & 3) == 0 ? 4 : 0;
   const long long total = static_cast<long long>(rows) * cols, cap = static_cast<long long>(num_sms()) * 16;
-  long long blocks = (total / (vec ? 4 : 1) + 255) / 256;
+  long long blocks = (total / (vec ? vec : 1) + 255) / 256;
   if (blocks > cap) blocks = cap;
   auto kern = out_f32 ? stream32::glu_kernel<true> : stream32::glu_kernel<false>;
   kern<<<static_cast<int>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(gate, up, row_gate, out, act, limit, in_f32, total, cols, ldg, ldu, ldr,

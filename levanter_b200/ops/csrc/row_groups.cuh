@@ -46,9 +46,26 @@ struct Row {
 
   static __device__ __forceinline__ int column(int n) { return (threadIdx.x + n * blockDim.x) * kVec; }
 
+  // Where the groups lie, for all rows of a CTA.
+  struct Groups {
+    int dim, part, per;  // per: partial sums of a group
+    bool by_warp;        // the 32 units of a warp lie in one group: a partial sum per warp and n, else one per unit
+    int first[kN];       // by_warp: first partial sum of the group of unit n; else the number of its group
+
+    __device__ __forceinline__ Groups(int dim, int part) : dim(dim), part(part) {
+      by_warp = part == dim || part % (32 * kVec) == 0;
+      per = part == dim ? static_cast<int>(blockDim.x >> 5) * kN : by_warp ? part / (32 * kVec) : part / kVec;
+#pragma unroll
+      for (int n = 0; n < kN; ++n) {
+        const int g = part == dim || column(n) >= dim ? 0 : column(n) / part;
+        first[n] = by_warp ? g * per : g;
+      }
+    }
+  };
+
   // Multiplies every group by 1 / sqrt(mean of its squares + eps).  s: scratch of scratch_floats() floats, not in use by a slower warp (two
   // buffers in turn suffice).  Every thread of the CTA takes part.
-  __device__ __forceinline__ void normalize(int dim, int part, float eps, float* s) {
+  __device__ __forceinline__ void normalize(const Groups& g, float eps, float* s) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     float ss[kN];
 #pragma unroll
@@ -57,9 +74,8 @@ struct Row {
 #pragma unroll
       for (int e = 0; e < kVec; ++e) ss[n] = fmaf(a[n][e], a[n][e], ss[n]);
     }
-    const float inv = 1.f / static_cast<float>(part);
-    if (part == dim || part % (32 * kVec) == 0) {  // the 32 units of a warp lie in one group: a partial sum per warp and n
-      const int per = part == dim ? warps * kN : part / (32 * kVec);
+    const float inv = 1.f / static_cast<float>(g.part);
+    if (g.by_warp) {
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
         const float v = warp_sum(ss[n]);
@@ -67,37 +83,32 @@ struct Row {
       }
       __syncthreads();
       float r = 0.f;
-      int have = -1;
 #pragma unroll
       for (int n = 0; n < kN; ++n) {
-        const int g = part == dim ? 0 : column(n) / part;
-        if (column(n) < dim && g != have) {
+        if (n == 0 || g.first[n] != g.first[n - 1]) {
           float t = 0.f;
-          for (int i = 0; i < per; ++i) t += s[g * per + i];
+          for (int i = 0; i < g.per; ++i) t += s[g.first[n] + i];
           r = 1.f / sqrtf(t * inv + eps);
-          have = g;
         }
 #pragma unroll
         for (int e = 0; e < kVec; ++e) a[n][e] *= r;
       }
       return;
     }
-    const int per = part / kVec, groups = dim / part;
     float* s_r = s + kN * blockDim.x;
 #pragma unroll
     for (int n = 0; n < kN; ++n) s[threadIdx.x + n * blockDim.x] = ss[n];
     __syncthreads();
-    for (int g = warp; g < groups; g += warps) {
+    for (int j = warp; j < g.dim / g.part; j += warps) {
       float t = 0.f;
-      for (int i = lane; i < per; i += 32) t += s[g * per + i];
+      for (int i = lane; i < g.per; i += 32) t += s[j * g.per + i];
       t = warp_sum(t);
-      if (lane == 0) s_r[g] = 1.f / sqrtf(t * inv + eps);
+      if (lane == 0) s_r[j] = 1.f / sqrtf(t * inv + eps);
     }
     __syncthreads();
 #pragma unroll
     for (int n = 0; n < kN; ++n) {
-      if (column(n) >= dim) continue;
-      const float r = s_r[column(n) / part];
+      const float r = s_r[g.first[n]];
 #pragma unroll
       for (int e = 0; e < kVec; ++e) a[n][e] *= r;
     }
@@ -105,16 +116,15 @@ struct Row {
   static size_t scratch_floats(int threads, int groups) { return static_cast<size_t>(kN) * threads + groups; }
 };
 
-// Threads and units per thread for rows of `dim` elements; few_rows: the rows do not fill the GPU, so a row is spread over more threads.
-// False: too long.
+// Threads and units per thread (1, 2, 4 or 16) for rows of `dim` elements; few_rows: the rows do not fill the GPU, so a row is spread over
+// more threads.  False: too long.
 inline bool shape_for(int dim, int vec, bool few_rows, int& n, int& threads) {
   const int units = (dim + vec - 1) / vec;
-  const int choices[3] = {1, 4, 16};
-  for (int i = 0; i < 3; ++i) {
+  const int choices[4] = {1, 2, 4, 16}, most[4] = {few_rows ? 1024 : 256, 512, 1024, 1024};
+  for (int i = 0; i < 4; ++i) {
     n = choices[i];
     threads = ((units + n - 1) / n + 31) / 32 * 32;
-    if (threads <= (few_rows || n == 16 ? 1024 : 256)) return true;
-    if (n == 4 && threads <= 1024) return true;
+    if (threads <= most[i]) return true;
   }
   return false;
 }

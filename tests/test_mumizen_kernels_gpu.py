@@ -150,7 +150,8 @@ def test_linear_attention_remembers_a_far_key():
 
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("heads,dv,weighted,sigmoid", [(4, 64, True, True), (4, 64, False, False), (3, 10, False, False), (5, 9, True, True), (32, 128, True, True),
-                                                       (32, 128, False, False), (1, 1, False, True), (2, 2560, False, False)])
+                                                       (32, 128, False, False), (1, 1, False, True), (2, 2560, False, False), (5, 8, False, False), (3, 48, True, False),
+                                                       (3, 256, False, True), (40, 136, True, True), (90, 136, True, False), (3, 40, False, False)])
 def test_gated_norm(dtype, heads, dv, weighted, sigmoid):
     from levanter_b200.ops.linear_attention import gated_norm
 
